@@ -430,6 +430,115 @@ int tkv_skinny_gemm(const void* x, const void* w, float* partial, int m, int n, 
 int tkv_skinny_gemm_swiglu(const void* gate_up, const void* w, float* partial, int m, int n, int k, int dtype,
                            int32_t* status, tkv_stream_t stream);
 
+/* ---- decoders with recurrent layers and windowed differential attention -------------------------------------------
+ * Common conventions.  Tokens of a step are packed: request b owns rows cu_tokens[b] .. cu_tokens[b + 1) of every
+ * per-token array (cu_tokens NULL, where allowed: one token per request).  What a request keeps between steps lives in
+ * slot slots[b] of every state array; pos0[b] is the position of its first token of this step, and a request at position 0
+ * starts from the empty state whatever its slot holds.  dtype: TKV_BF16 or TKV_F32 (everything in fp32); statistics,
+ * decays, step sizes, angles, scores, the residual stream and recurrent state are fp32 in either case.  Small weight
+ * vectors (norms, biases, convolution taps) are fp32 arrays.  No counterpart in the reference.
+ */
+
+/* pos0[b] = lens[slots[b]]; lens[slots[b]] += tokens of request b in this step. */
+int tkv_batch_begin(int32_t* lens, const int32_t* slots, const int32_t* cu_tokens, int32_t* pos0, int batch,
+                    tkv_stream_t stream);
+
+/* stream_out[r, :] = table[ids[r], :] as fp32, copy_out (may be NULL) the same in the model type.  An id outside
+ * [0, vocab) yields zeros and TKV_DEV_BAD_INDEX. */
+int tkv_embed_stream(const int64_t* ids, const void* table, int64_t vocab, float* stream_out, void* copy_out, int rows, int width,
+                     int dtype, int32_t* status, tkv_stream_t stream);
+
+/* x[r, :] += mult * RMSNorm(y[r, :]) * (weight_offset + weight); copy_out (may be NULL) = x in the model type. */
+int tkv_postnorm_add(float* x, const void* y, const float* weight, void* copy_out, int rows, int width, float eps, float mult,
+                     float weight_offset, int dtype, tkv_stream_t stream);
+
+/* out[r, :] = RMSNorm(x[row_idx ? row_idx[r] : r, :]) * (weight_offset + weight). */
+int tkv_stream_norm(const float* x, const int32_t* row_idx, const float* weight, void* out, int rows, int width, float eps,
+                    float weight_offset, int dtype, tkv_stream_t stream);
+
+/* Group RMS norm with a SiLU gate: gate_first ? RMS(y * silu(z)) * weight : RMS(y) * weight * silu(z), every group of
+ * group_len elements over its own root mean square; weight may be NULL.  out is contiguous [rows, groups * group_len]. */
+int tkv_gated_norm(const void* y, int64_t y_stride, const void* z, int64_t z_stride, const float* weight, void* out, int rows,
+                   int groups, int group_len, float eps, int gate_first, int dtype, tkv_stream_t stream);
+
+/* u[i] = GELU(u[i]), tanh form, in place. */
+int tkv_gelu_tanh(void* u, int64_t n, int dtype, tkv_stream_t stream);
+
+/* Rotary positions on q [heads, dim] and k [heads, dim] (columns 0 and heads * dim of a projection row): the pair
+ * (i, i + rot_dims / 2) turns by position * f_i, freq_hi_lo[i] = {f_i rounded to fp32, the rest}; k is multiplied by k_scale
+ * afterwards.  out: contiguous [tokens, 2, heads, dim]. */
+int tkv_rotate_qk(const void* proj, int64_t row_stride, void* out, const int32_t* cu_tokens, const int32_t* pos0, int batch,
+                  int tokens, int heads, int dim, int rot_dims, const float* freq_hi_lo, float k_scale, int dtype,
+                  tkv_stream_t stream);
+
+/* Causal depthwise convolution (conv_w [channels, taps], last column the current token's) + bias + SiLU over columns
+ * 0 .. channels of the projection rows; inputs before the step come from ring [slots, taps, channels] (input of position p
+ * in row p mod taps), whose rows of the step's last inputs are then replaced.  out: contiguous [tokens, channels]. */
+int tkv_conv_silu(const void* proj, int64_t row_stride, void* ring, const float* conv_w, const float* conv_b, void* out,
+                  const int32_t* cu_tokens, const int32_t* slots, const int32_t* pos0, int batch, int max_tokens, int channels,
+                  int taps, int dtype, tkv_stream_t stream);
+
+/* dt[t, h] = softplus(dt_in[t, h] + dt_bias[h]), log_decay[t, h] = -exp(a_log[h]) * dt[t, h]. */
+int tkv_ssd_steps(const void* dt_in, int64_t row_stride, const float* dt_bias, const float* a_log, float* dt, float* log_decay,
+                  int tokens, int heads, int dtype, tkv_stream_t stream);
+
+/* One token per request of a retention layer.  proj row: q [heads, dim], k [heads, dim], v [heads, vdim], gate [heads, vdim].
+ * Rotates q and k as tkv_rotate_qk, S <- head_decay S + k v^T (state [slots, heads, dim, vdim] fp32), o = S^T q, and writes
+ * RMS(o) * silu(gate) per head to out [batch, heads, vdim]. */
+int tkv_retention_step(const void* proj, int64_t row_stride, float* state, const int32_t* slots, const int32_t* pos0,
+                       const float* head_decay, const float* freq_hi_lo, void* out, int batch, int heads, int dim, int vdim,
+                       int rot_dims, float k_scale, float eps, int dtype, tkv_stream_t stream);
+
+/* One token per request of a state-space (SSD) layer.  proj row: z [heads * vdim], x [heads * vdim], B [groups, n],
+ * C [groups, n], dt [heads].  Convolution (and ring) as tkv_conv_silu over x | B | C, dt and decay as tkv_ssd_steps,
+ * S <- a S + dt B x^T (state [slots, heads, n, vdim] fp32), out[b, h] = S^T C + skip[h] x. */
+int tkv_ssd_step(const void* proj, int64_t row_stride, void* ring, float* state, const int32_t* slots, const int32_t* pos0,
+                 const float* conv_w, const float* conv_b, const float* dt_bias, const float* a_log, const float* skip, void* out,
+                 int batch, int heads, int groups, int n, int vdim, int taps, int dtype, tkv_stream_t stream);
+
+/* Linear recurrence with one decay per head and token over a packed batch:
+ *   S_t = a_t S_(t-1) + k_t (s_t v_t)^T,  out_t = S_t^T q_t + skip v_t,
+ * head h using k/q group h / (heads / groups).  log_decay [tokens, heads] or, if NULL, a constant per head; v_scale
+ * [tokens, heads] or NULL (1); skip [heads] or NULL (0); state [slots, heads, n, vdim] fp32, read and written.
+ * tkv_linrec_scan runs token by token and takes every size (n <= 1760) and dtype; cu_tokens may be NULL.
+ * tkv_linrec_chunk is the tensor-core form for prompts: bf16, n <= 256, n, vdim and the strides multiples of 8, 16-byte
+ * aligned rows.  Its workspace (tkv_linrec_chunk_workspace_bytes; -1 = shape not supported, 0 = none) holds the states
+ * between the segments of long sequences. */
+int tkv_linrec_scan(const void* q, int64_t q_stride, const void* k, int64_t k_stride, const void* v, int64_t v_stride,
+                    const float* log_decay, const float* head_decay, const float* v_scale, const float* skip, void* out,
+                    float* state, const int32_t* slots, const int32_t* cu_tokens, const int32_t* pos0, int batch, int heads,
+                    int groups, int n, int vdim, int dtype, tkv_stream_t stream);
+int64_t tkv_linrec_chunk_workspace_bytes(int batch, int max_tokens, int heads, int n, int vdim, int dtype);
+int tkv_linrec_chunk(const void* q, int64_t q_stride, const void* k, int64_t k_stride, const void* v, int64_t v_stride,
+                     const float* log_decay, const float* head_log_decay, const float* v_scale, const float* skip, void* out,
+                     float* state, const int32_t* slots, const int32_t* cu_tokens, const int32_t* pos0, void* workspace,
+                     int64_t workspace_bytes, int batch, int max_tokens, int heads, int groups, int n, int vdim, int dtype,
+                     tkv_stream_t stream);
+
+/* Differential attention over a sliding window.  proj row: q [heads, 2, dim], k [kv_heads, 2, dim], v [kv_heads, vdim].
+ * tkv_diff_prep norms q and k per head and map (weights q_norm / k_norm [dim]) and stores them zero-padded to dp / pp
+ * elements (multiples of 64): q_out [tokens, heads, 2, dp]; k and v of position p in row p mod ring_rows of
+ * k_ring [slots, kv_heads, ring_rows, 2, dp] / v_ring [slots, kv_heads, ring_rows, pp] (ring_rows <= window, and
+ * >= min(window, tokens seen after the step)); and, for steps of several tokens, into the linear buffers
+ * k_lin [rows, kv_heads, 2, dp] / v_lin [rows, kv_heads, pp], where request b's part starts at row kv_start[b] with the
+ * min(pos0[b], window - 1) positions before the step (fetched from the ring; max_history bounds them over the batch).
+ * tkv_diff_prefill attends over the linear buffers, tkv_diff_decode (one token per request) over the ring; both write
+ * sigmoid(gate) (1 - diff) RMS(a1 - lambda a2) to out [tokens, heads, vdim], lambda read from device memory. */
+int tkv_diff_prep(const void* proj, int64_t row_stride, const float* q_norm, const float* k_norm, float eps, void* q_out,
+                  void* k_ring, void* v_ring, int ring_rows, void* k_lin, void* v_lin, const int32_t* kv_start,
+                  const int32_t* cu_tokens, const int32_t* slots, const int32_t* pos0, int batch, int tokens, int max_history,
+                  int heads, int kv_heads, int dim, int vdim, int dp, int pp, int window, int dtype, tkv_stream_t stream);
+int64_t tkv_diff_decode_workspace_bytes(int batch, int heads, int kv_heads, int ring_rows, int dp, int pp, int dtype);
+int tkv_diff_decode(const void* q, const void* k_ring, const void* v_ring, int ring_rows, const int32_t* slots,
+                    const int32_t* pos0, const float* lambda, float diff, float scale, float eps, const void* gate,
+                    int64_t gate_stride, void* out, void* workspace, int64_t workspace_bytes, int batch, int heads, int kv_heads,
+                    int dim, int vdim, int dp, int pp, int dtype, tkv_stream_t stream);
+int tkv_diff_prefill(const void* q, const void* k_lin, const void* v_lin, const int32_t* kv_start, int64_t kv_rows,
+                     const int32_t* cu_tokens, const int32_t* pos0, const float* lambda, float diff, float scale, float eps,
+                     const void* gate, int64_t gate_stride, void* out, int batch, int tokens, int max_tokens, int heads,
+                     int kv_heads, int dim, int vdim, int dp, int pp, int window, int dtype, int32_t* status,
+                     tkv_stream_t stream);
+
 /* Blocks until `stream` is idle, then returns *status (a TKV_DEV_* code) and clears it. */
 int tkv_read_status(int32_t* status, tkv_stream_t stream);
 

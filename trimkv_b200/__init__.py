@@ -9,6 +9,9 @@ from .attn import TRIMKV_ATTENTION_IMPLEMENTATIONS, get_attention_interface
 from .modeling_qwen3 import TrimKVQwen3Config, TrimKVQwen3ForCausalLM, TrimKVQwen3Model
 from .modeling_llama import TrimKVLlamaConfig, TrimKVLlamaForCausalLM, TrimKVLlamaModel
 from .modeling_phi3 import TrimKVPhi3Config, TrimKVPhi3ForCausalLM, TrimKVPhi3Model
+from .modeling_dafovik import DafovikConfig, DafovikForCausalLM, DafovikModel
+from .registry import load_model, model_class
+from .state_cache import HybridStateCache
 
 __all__ = [
     "TrimKVCache", "DynamicBudgetTrimKVCache", "BatchedDynamicBudgetTrimKVCache", "update_flatten_view",
@@ -16,4 +19,5 @@ __all__ = [
     "TrimKVQwen3Config", "TrimKVQwen3ForCausalLM", "TrimKVQwen3Model",
     "TrimKVLlamaConfig", "TrimKVLlamaForCausalLM", "TrimKVLlamaModel",
     "TrimKVPhi3Config", "TrimKVPhi3ForCausalLM", "TrimKVPhi3Model",
+    "DafovikConfig", "DafovikForCausalLM", "DafovikModel", "HybridStateCache", "load_model", "model_class",
 ]

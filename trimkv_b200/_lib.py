@@ -51,6 +51,24 @@ SIGNATURES = {
     "tkv_skinny_gemm_splits": (I, [I, I, I]),
     "tkv_skinny_gemm": (I, [P, P, P, I, I, I, I, P, P]),
     "tkv_skinny_gemm_swiglu": (I, [P, P, P, I, I, I, I, P, P]),
+    "tkv_batch_begin": (I, [P, P, P, P, I, P]),
+    "tkv_embed_stream": (I, [P, P, L, P, P, I, I, I, P, P]),
+    "tkv_postnorm_add": (I, [P, P, P, P, I, I, F, F, F, I, P]),
+    "tkv_stream_norm": (I, [P, P, P, P, I, I, F, F, I, P]),
+    "tkv_gated_norm": (I, [P, L, P, L, P, P, I, I, I, F, I, I, P]),
+    "tkv_gelu_tanh": (I, [P, L, I, P]),
+    "tkv_rotate_qk": (I, [P, L, P, P, P, I, I, I, I, I, P, F, I, P]),
+    "tkv_conv_silu": (I, [P, L, P, P, P, P, P, P, P, I, I, I, I, I, P]),
+    "tkv_ssd_steps": (I, [P, L, P, P, P, P, I, I, I, P]),
+    "tkv_retention_step": (I, [P, L, P, P, P, P, P, P, I, I, I, I, I, F, F, I, P]),
+    "tkv_ssd_step": (I, [P, L, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P]),
+    "tkv_linrec_scan": (I, [P, L, P, L, P, L, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, P]),
+    "tkv_linrec_chunk_workspace_bytes": (L, [I, I, I, I, I, I]),
+    "tkv_linrec_chunk": (I, [P, L, P, L, P, L, P, P, P, P, P, P, P, P, P, P, L, I, I, I, I, I, I, I, P]),
+    "tkv_diff_prep": (I, [P, L, P, P, F, P, P, P, I, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, P]),
+    "tkv_diff_decode_workspace_bytes": (L, [I, I, I, I, I, I, I]),
+    "tkv_diff_decode": (I, [P, P, P, I, P, P, P, F, F, F, P, L, P, P, L, I, I, I, I, I, I, I, I, P]),
+    "tkv_diff_prefill": (I, [P, P, P, P, L, P, P, P, F, F, F, P, L, P, I, I, I, I, I, I, I, I, I, I, I, P, P]),
     "tkv_read_status": (I, [P, P]),
 }
 

@@ -152,6 +152,14 @@ class TrimKVCache:
             self.n_seen_tokens[l] += num_tokens
             self._cache_len[l] += num_tokens
 
+    def graph_key(self):
+        """Identity of the storage a recorded decode step refers to."""
+        return (self._slab["k"].data_ptr(), self._cap, self._batch) if self._slab is not None else None
+
+    def fits(self, num_tokens: int = 1) -> bool:
+        """Whether ``num_tokens`` more tokens per segment fit the slabs as they are."""
+        return self._slab is not None and max(self._cache_len) + num_tokens <= self._cap
+
     def snapshot_counters(self):
         """The host-side counters that ``update`` / ``decode_prep`` / ``advance`` move, for ``restore_counters``: a CUDA
         graph capture of a decode step runs the host side of the step without running its kernels."""

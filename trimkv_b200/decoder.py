@@ -178,15 +178,12 @@ class GraphedForwardStep:
     EAGER_CALLS = 2
 
     def __init__(self, model, cache: TrimKVCache, use_graph: bool = True):
-        self.step = FusedDecodeStep(model, cache)
+        self.step = model._decode_step_cls()(model, cache)
         self.model, self.use_graph = model, use_graph
         dev = model.device
         self.ids = torch.zeros(cache._batch, 1, dtype=torch.int64, device=dev)
         self.pos = torch.zeros(1, dtype=torch.int64, device=dev)
         self.calls, self.graph, self.logits, self.key, self.launches_per_replay = 0, None, None, None, 0
-
-    def _slab_key(self, cache):
-        return (cache._slab["k"].data_ptr(), cache._cap, cache._batch) if cache._slab is not None else None
 
     def release_graph(self) -> None:
         if self.graph is not None:
@@ -198,8 +195,8 @@ class GraphedForwardStep:
         """input_ids [B,1], pos int64[1] (device) -> logits [B, vocab] (a tensor of the caller's own)."""
         self.ids.copy_(input_ids)
         self.pos.copy_(pos)
-        fits = cache._slab is not None and max(cache._cache_len) + 1 <= cache._cap
-        if self.graph is not None and (self.key != self._slab_key(cache) or not fits):
+        fits = cache.fits(1)
+        if self.graph is not None and (self.key != cache.graph_key() or not fits):
             self.release_graph()
             self.calls, cache.static_views = 0, False
         if (not self.use_graph or not fits or self.calls < self.EAGER_CALLS or torch.cuda.is_current_stream_capturing()):
@@ -215,7 +212,7 @@ class GraphedForwardStep:
             self.launches_per_replay = ops.launch_count - before
             ops.launch_count = before
             cache.restore_counters(snap)
-            self.key = self._slab_key(cache)
+            self.key = cache.graph_key()
         self.graph.replay()
         ops.launch_count += self.launches_per_replay
         cache.advance(1)
@@ -235,8 +232,10 @@ class GreedyDecoder:
         self.fused = None
         if head_shard_group is not None:
             self.fused = HeadShardedDecodeStep(model, cache, head_shard_group, fused_gather=fused_gather)
-        elif fused and FusedDecodeStep.supports(model) and model.lm_head.weight.dtype in (torch.bfloat16, torch.float16):
-            self.fused = FusedDecodeStep(model, cache, tc_gemm=tc_gemm, fused_down=fused_down)
+        elif fused and model._fused_decode_covers():
+            cls = model._decode_step_cls()
+            self.fused = cls(model, cache, tc_gemm=tc_gemm, fused_down=fused_down) if issubclass(cls, FusedDecodeStep) \
+                else cls(model, cache)
         dev = model.device
         self.batch = cache._batch
         self.ids = torch.zeros(self.batch, 1, dtype=torch.int64, device=dev)
@@ -294,6 +293,10 @@ class GreedyDecoder:
     def step(self, ids: Optional[torch.Tensor] = None, eager: bool = False) -> torch.Tensor:
         if ids is not None:
             self.ids.copy_(ids, non_blocking=True)
+        if self.graph is not None and not self.cache.fits(1):
+            self.release_graph()               # the step below makes room, which moves the arrays the graph refers to
+            self.cache.static_views = False
+            eager = True
         if self.use_graph and not eager:
             if self.graph is None:
                 self.capture()
@@ -304,6 +307,30 @@ class GreedyDecoder:
             self._forward()
         self.model.model.compress_after_forward(self.cache)     # the eviction check that ends the model's forward pass
         return self.next_ids
+
+
+class HybridDecodeStep:
+    """One-token step of a hybrid decoder (``modeling_dafovik``): its layers' one-token kernels around the library GEMMs.
+
+    Per layer with a recurrent mixer: one projection GEMM, the state step (rotation or convolution, state update, read-out
+    and, for retention, norm and gate in the same launch), the gated norm where the norm spans heads, the output GEMM, then
+    norm + residual add, up GEMM, GELU, down GEMM, norm + residual add; an attention layer has the norm-and-store kernel, the
+    split-KV kernel and the merge that also combines the maps.  Everything a step reads is on the device, so it can be
+    recorded in a CUDA graph."""
+
+    @staticmethod
+    def supports(model) -> bool:
+        return hasattr(model, "decode_step")
+
+    def __init__(self, model, cache):
+        self.model, self._cache = model, weakref.ref(cache)
+
+    def __call__(self, ids: torch.Tensor, pos: torch.Tensor) -> torch.Tensor:
+        """ids [B,1] int64 -> logits [B, vocab]; positions are counted per request on the device (``pos`` is not read)."""
+        cache = self._cache()
+        if cache is None:
+            raise RuntimeError("the cache this decode step was built for no longer exists")
+        return self.model.decode_step(ids.reshape(-1), cache)
 
 
 class HeadShardedDecodeStep(FusedDecodeStep):

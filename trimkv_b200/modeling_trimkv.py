@@ -386,6 +386,8 @@ class TrimKVModel(TrimKVPreTrainedModel):
 
 class TrimKVForCausalLM(TrimKVPreTrainedModel, GenerationMixin):
     model_cls = TrimKVModel
+    cache_cls = TrimKVCache                                   # what the one-token step of this family works on
+    decode_dtypes = (torch.bfloat16, torch.float16)           # and the weight types it runs in
     _tied_weights_keys = {"lm_head.weight": "model.embed_tokens.weight"}
 
     def __init__(self, config):
@@ -429,11 +431,11 @@ class TrimKVForCausalLM(TrimKVPreTrainedModel, GenerationMixin):
         if kwargs.get("output_attentions") or kwargs.get("output_hidden_states") or kwargs.get("labels") is not None:
             return None
         cache = past_key_values
-        if (not isinstance(cache, TrimKVCache) or cache.get_seq_length() == 0
+        if (not isinstance(cache, self.cache_cls) or cache.get_seq_length() == 0
                 or getattr(cache, "_batch", None) != input_ids.shape[0]):
             return None
-        from .decoder import FusedDecodeStep, GraphedForwardStep
-        if self.lm_head.weight.dtype not in (torch.bfloat16, torch.float16) or not FusedDecodeStep.supports(self):
+        from .decoder import GraphedForwardStep
+        if not self._fused_decode_covers():
             return None
         step = cache.__dict__.get("_fused_step")
         graph = self.config.fused_decode_step != "eager"
@@ -442,6 +444,14 @@ class TrimKVForCausalLM(TrimKVPreTrainedModel, GenerationMixin):
                 step.release_graph()
             step = cache.__dict__["_fused_step"] = GraphedForwardStep(self, cache, use_graph=graph)
         return step
+
+    def _decode_step_cls(self):
+        """The one-token step of this family (``decoder.py``)."""
+        from .decoder import FusedDecodeStep
+        return FusedDecodeStep
+
+    def _fused_decode_covers(self) -> bool:
+        return self.lm_head.weight.dtype in self.decode_dtypes and self._decode_step_cls().supports(self)
 
     def forward(self, input_ids=None, attention_mask=None, position_ids=None, past_key_values=None, inputs_embeds=None,
                 use_cache=None, cache_position=None, logits_to_keep=0, **kwargs):
@@ -477,7 +487,7 @@ class TrimKVForCausalLM(TrimKVPreTrainedModel, GenerationMixin):
             ids = inputs if inputs is not None else kwargs.pop("input_ids")
             return self.generate_greedy(ids, prefill_chunk_size=prefill_chunk_size, fused_decode=fused_decode,
                                         **{k: v for k, v in kwargs.items()
-                                           if k in ("max_new_tokens", "past_key_values", "eos_token_id")})
+                                           if k in ("max_new_tokens", "past_key_values", "eos_token_id", "attention_mask")})
         if kwargs.get("past_key_values") is None:
             ids = inputs if inputs is not None else kwargs.get("input_ids")
             kwargs["past_key_values"] = self.new_cache(ids.device if ids is not None else None)
@@ -485,7 +495,7 @@ class TrimKVForCausalLM(TrimKVPreTrainedModel, GenerationMixin):
 
     @torch.inference_mode()
     def generate_greedy(self, input_ids, max_new_tokens=16, past_key_values=None, eos_token_id=None,
-                        prefill_chunk_size=None, fused_decode=False):
+                        prefill_chunk_size=None, fused_decode=False, attention_mask=None):
         """Greedy decoding without the HF machinery; returns ``[B, prompt + new]`` token ids.
 
         ``fused_decode``: decode through ``decoder.GreedyDecoder`` (ten fused launches per layer, one CUDA graph per
@@ -496,23 +506,28 @@ class TrimKVForCausalLM(TrimKVPreTrainedModel, GenerationMixin):
         ``prefill_chunk_size``: feed the prompt in pieces of that many tokens, evicting after each piece (the model
         calls ``compress`` at the end of every forward), so that a prompt much longer than ``memory_size`` never has
         its whole K/V resident.  The eviction schedule, and with it the result, differs from the one-piece prompt pass
-        exactly as it would in the reference if it were fed the same pieces."""
+        exactly as it would in the reference if it were fed the same pieces.
+
+        ``attention_mask`` marks the padding of unequal prompts, on either side; only models that keep requests of unequal
+        length apart apply it (the TRIM-KV families attend over every cached row, as the reference does)."""
         if past_key_values is None:
             past_key_values = self.new_cache(input_ids.device)
-        if prefill_chunk_size:
-            for lo in range(0, input_ids.shape[1], prefill_chunk_size):
-                out = self(input_ids=input_ids[:, lo:lo + prefill_chunk_size], past_key_values=past_key_values,
-                           logits_to_keep=1)
-        else:
-            out = self(input_ids=input_ids, past_key_values=past_key_values, logits_to_keep=1)
+        piece = prefill_chunk_size or input_ids.shape[1]
+        last = None
+        for lo in range(0, input_ids.shape[1], piece):
+            mask = {} if attention_mask is None else {"attention_mask": attention_mask[:, lo:lo + piece]}
+            logits = self(input_ids=input_ids[:, lo:lo + piece], past_key_values=past_key_values, logits_to_keep=1, **mask).logits[:, -1]
+            if mask and last is not None:      # a request whose tokens ended in an earlier piece keeps its logits
+                logits = torch.where(mask["attention_mask"].bool().any(1, keepdim=True), logits, last)
+            last = logits
         tokens = [input_ids]
-        nxt = out.logits[:, -1].argmax(-1, keepdim=True)
+        nxt = last.argmax(-1, keepdim=True)
         done = torch.zeros_like(nxt, dtype=torch.bool)
         if fused_decode:
-            from .decoder import FusedDecodeStep, GreedyDecoder
-            if not (input_ids.is_cuda and FusedDecodeStep.supports(self)
-                    and self.lm_head.weight.dtype in (torch.bfloat16, torch.float16)):
-                raise NotImplementedError("fused_decode needs a CUDA model in bf16/f16 with head_dim 128, the 'rg' gate and SiLU")
+            from .decoder import GreedyDecoder
+            if not (input_ids.is_cuda and self._fused_decode_covers()):
+                raise NotImplementedError("fused_decode needs a CUDA model whose shape and dtype its decode step covers "
+                                          "(TRIM-KV families: bf16/f16, head_dim 128, the 'rg' gate and SiLU)")
             dec = GreedyDecoder(self, past_key_values, use_graph=True, fused=True)
             dec.ids.copy_(nxt)
             try:

@@ -419,3 +419,144 @@ def update_flatten_view(cache: torch.Tensor, state: torch.Tensor, headlens: torc
 
 
 update_flatten_view_triton = update_flatten_view  # the reference's name for the same operation
+
+
+# --------------------------------------------------------------------------------------------------------------------
+# Decoders with recurrent layers and windowed differential attention.  ``batch`` is a ``state_cache.StepBatch``: packed
+# tokens, ``cu`` (None in a one-token step), ``slots`` and ``pos0`` of the step's requests.
+
+def batch_begin(lens, slots, cu, pos0) -> None:
+    check(lib().tkv_batch_begin(lens.data_ptr(), slots.data_ptr(), _ptr(cu), pos0.data_ptr(), slots.shape[0], _stream(lens)),
+          "tkv_batch_begin")
+    _count(1)
+
+
+def embed_stream(ids, table, stream, copy, status=None) -> None:
+    check(lib().tkv_embed_stream(ids.data_ptr(), table.data_ptr(), table.shape[0], stream.data_ptr(), _ptr(copy), stream.shape[0],
+                                 stream.shape[1], dtype_code(table.dtype), _ptr(status), _stream(ids)), "tkv_embed_stream")
+    _count(1)
+
+
+def postnorm_add(stream, y, weight, copy, eps: float, mult: float, weight_offset: float) -> None:
+    """``stream += mult * RMSNorm(y) * (weight_offset + weight)`` (fp32, in place); ``copy`` (or None): the sum in y's type."""
+    check(lib().tkv_postnorm_add(stream.data_ptr(), y.data_ptr(), weight.data_ptr(), _ptr(copy), stream.shape[0], stream.shape[1],
+                                 float(eps), float(mult), float(weight_offset), dtype_code(y.dtype), _stream(stream)),
+          "tkv_postnorm_add")
+    _count(1)
+
+
+def stream_norm(stream, rows, weight, out, eps: float, weight_offset: float) -> None:
+    """RMS norm of the stream's rows (``rows`` int32, or None: all) into ``out``."""
+    check(lib().tkv_stream_norm(stream.data_ptr(), _ptr(rows), weight.data_ptr(), out.data_ptr(), out.shape[0], out.shape[1],
+                                float(eps), float(weight_offset), dtype_code(out.dtype), _stream(stream)), "tkv_stream_norm")
+    _count(1)
+
+
+def gated_norm(y, z, weight, out, groups: int, eps: float, gate_first: bool) -> None:
+    """Group RMS norm with a SiLU gate before (times ``weight``) or after it; ``z`` may be a column slice of a wider array."""
+    check(lib().tkv_gated_norm(y.data_ptr(), y.stride(0), z.data_ptr(), z.stride(0), _ptr(weight), out.data_ptr(), out.shape[0],
+                               groups, out.shape[1] // groups, float(eps), int(gate_first), dtype_code(out.dtype), _stream(y)),
+          "tkv_gated_norm")
+    _count(1)
+
+
+def gelu_tanh(u) -> None:
+    check(lib().tkv_gelu_tanh(u.data_ptr(), u.numel(), dtype_code(u.dtype), _stream(u)), "tkv_gelu_tanh")
+    _count(1)
+
+
+def rotate_qk(proj, out, batch, heads: int, dim: int, rot_dims: int, freq, k_scale: float) -> None:
+    check(lib().tkv_rotate_qk(proj.data_ptr(), proj.stride(0), out.data_ptr(), _ptr(batch.cu), batch.pos0.data_ptr(), batch.size,
+                              batch.tokens, heads, dim, rot_dims, freq.data_ptr(), float(k_scale), dtype_code(proj.dtype),
+                              _stream(proj)), "tkv_rotate_qk")
+    _count(1)
+
+
+def conv_silu(x, ring, weight, bias, out, batch) -> None:
+    """``x`` [tokens, channels] is a column slice of the projection; ``ring`` [slots, taps, channels]."""
+    check(lib().tkv_conv_silu(x.data_ptr(), x.stride(0), ring.data_ptr(), weight.data_ptr(), bias.data_ptr(), out.data_ptr(),
+                              batch.cu.data_ptr(), batch.slots.data_ptr(), batch.pos0.data_ptr(), batch.size, batch.max_tokens,
+                              x.shape[1], weight.shape[1], dtype_code(x.dtype), _stream(x)), "tkv_conv_silu")
+    _count(2)
+
+
+def ssd_steps(dt_in, dt_bias, a_log, dt, log_decay) -> None:
+    check(lib().tkv_ssd_steps(dt_in.data_ptr(), dt_in.stride(0), dt_bias.data_ptr(), a_log.data_ptr(), dt.data_ptr(),
+                              log_decay.data_ptr(), dt.shape[0], dt.shape[1], dtype_code(dt_in.dtype), _stream(dt)), "tkv_ssd_steps")
+    _count(1)
+
+
+def retention_step(proj, state, batch, decay, freq, out, dim: int, rot_dims: int, k_scale: float, eps: float) -> None:
+    heads, vdim = state.shape[1], state.shape[3]
+    check(lib().tkv_retention_step(proj.data_ptr(), proj.stride(0), state.data_ptr(), batch.slots.data_ptr(), batch.pos0.data_ptr(),
+                                   decay.data_ptr(), freq.data_ptr(), out.data_ptr(), batch.size, heads, dim, vdim, rot_dims,
+                                   float(k_scale), float(eps), dtype_code(proj.dtype), _stream(proj)), "tkv_retention_step")
+    _count(1)
+
+
+def ssd_step(proj, ring, state, batch, conv_w, conv_b, dt_bias, a_log, skip, out, groups: int) -> None:
+    heads, n, vdim = state.shape[1:]
+    check(lib().tkv_ssd_step(proj.data_ptr(), proj.stride(0), ring.data_ptr(), state.data_ptr(), batch.slots.data_ptr(),
+                             batch.pos0.data_ptr(), conv_w.data_ptr(), conv_b.data_ptr(), dt_bias.data_ptr(), a_log.data_ptr(),
+                             skip.data_ptr(), out.data_ptr(), batch.size, heads, groups, n, vdim, conv_w.shape[1],
+                             dtype_code(proj.dtype), _stream(proj)), "tkv_ssd_step")
+    _count(1)
+
+
+def linrec(q, k, v, state, batch, out, groups: int, log_decay=None, head_decay=None, head_log_decay=None, v_scale=None,
+           skip=None, force_scan: bool = False) -> None:
+    """Scalar-decay linear recurrence over the packed tokens of ``batch`` (see tkv_linrec_scan in the header): the chunked
+    tensor-core kernel where it covers the shape, the token-by-token scan otherwise.  ``state`` [slots, heads, n, p]."""
+    heads, n, p = state.shape[1:]
+    dt = dtype_code(out.dtype)
+    es = out.element_size()
+    need = lib().tkv_linrec_chunk_workspace_bytes(batch.size, batch.max_tokens, heads, n, p, dt)
+    rows_ok = all((t.stride(0) * es) % 16 == 0 and t.data_ptr() % 16 == 0 for t in (q, k, v, out))
+    if need >= 0 and rows_ok and batch.cu is not None and not force_scan and batch.size * heads <= 65535:
+        ws = torch.empty(need, dtype=torch.uint8, device=out.device) if need else None
+        check(lib().tkv_linrec_chunk(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0),
+                                     _ptr(log_decay), _ptr(head_log_decay), _ptr(v_scale), _ptr(skip), out.data_ptr(),
+                                     state.data_ptr(), batch.slots.data_ptr(), batch.cu.data_ptr(), batch.pos0.data_ptr(), _ptr(ws),
+                                     need, batch.size, batch.max_tokens, heads, groups, n, p, dt, _stream(out)), "tkv_linrec_chunk")
+        _count(3 if need else 1)
+        return
+    check(lib().tkv_linrec_scan(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), _ptr(log_decay),
+                                _ptr(head_decay), _ptr(v_scale), _ptr(skip), out.data_ptr(), state.data_ptr(),
+                                batch.slots.data_ptr(), _ptr(batch.cu), batch.pos0.data_ptr(), batch.size, heads, groups, n, p, dt,
+                                _stream(out)), "tkv_linrec_scan")
+    _count(1)
+
+
+def diff_attention(proj, gate, q_norm, k_norm, k_ring, v_ring, batch, lam, diff: float, scale: float, eps: float, out,
+                   heads: int, dim: int, vdim: int, window: int) -> None:
+    """Differential attention of a step (see tkv_diff_prep in the header).  ``k_ring`` [slots, kv_heads, rows, 2, dp],
+    ``v_ring`` [slots, kv_heads, rows, pp]; ``proj`` holds q | k | v per token, ``gate`` [tokens, heads]; ``out``
+    [tokens, heads * vdim]."""
+    _, kv_heads, rows, _, dp = k_ring.shape
+    pp = v_ring.shape[3]
+    dev, dt, T = proj.device, dtype_code(proj.dtype), batch.tokens
+    q = torch.empty(T, heads, 2, dp, dtype=proj.dtype, device=dev)
+    k_lin = v_lin = kv_start = None
+    hist = kv_rows = 0
+    if batch.cu is not None:
+        kv_start, kv_rows, hist = batch.window_plan(window)
+        k_lin = torch.empty(kv_rows, kv_heads, 2, dp, dtype=proj.dtype, device=dev)
+        v_lin = torch.empty(kv_rows, kv_heads, pp, dtype=proj.dtype, device=dev)
+    check(lib().tkv_diff_prep(proj.data_ptr(), proj.stride(0), q_norm.data_ptr(), k_norm.data_ptr(), float(eps), q.data_ptr(),
+                              k_ring.data_ptr(), v_ring.data_ptr(), rows, _ptr(k_lin), _ptr(v_lin), _ptr(kv_start), _ptr(batch.cu),
+                              batch.slots.data_ptr(), batch.pos0.data_ptr(), batch.size, T, hist, heads, kv_heads, dim, vdim, dp, pp,
+                              window, dt, _stream(proj)), "tkv_diff_prep")
+    if batch.cu is not None:
+        check(lib().tkv_diff_prefill(q.data_ptr(), k_lin.data_ptr(), v_lin.data_ptr(), kv_start.data_ptr(), kv_rows,
+                                     batch.cu.data_ptr(), batch.pos0.data_ptr(), lam.data_ptr(), float(diff), float(scale), float(eps),
+                                     gate.data_ptr(), gate.stride(0), out.data_ptr(), batch.size, T, batch.max_tokens, heads, kv_heads,
+                                     dim, vdim, dp, pp, window, dt, _ptr(batch.status), _stream(proj)), "tkv_diff_prefill")
+        _count(3 if hist else 2)
+        return
+    need = lib().tkv_diff_decode_workspace_bytes(batch.size, heads, kv_heads, rows, dp, pp, dt)
+    ws = torch.empty(need, dtype=torch.uint8, device=dev) if need else None
+    check(lib().tkv_diff_decode(q.data_ptr(), k_ring.data_ptr(), v_ring.data_ptr(), rows, batch.slots.data_ptr(),
+                                batch.pos0.data_ptr(), lam.data_ptr(), float(diff), float(scale), float(eps), gate.data_ptr(),
+                                gate.stride(0), out.data_ptr(), _ptr(ws), need, batch.size, heads, kv_heads, dim, vdim, dp, pp, dt,
+                                _stream(proj)), "tkv_diff_decode")
+    _count(3 if need else 2)
