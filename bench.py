@@ -352,10 +352,16 @@ def run_micro(args):
     append: one token per segment.
     steady: append every step, evict only the segments that reached M+B.
     generate: generate() of the model classes on --workload, HF loop against fused_decode=True (wall clock per token).
+    hybrid: the hybrid decoder (Dafovik: retention, state-space and windowed differential-attention layers) beside the Qwen3
+            model of equal width, depth and parameters: prompt pass, decoding, and every kernel against its roofline.
     multi : --q-tokens new tokens per request against M cached ones (a piece of a chunked prefill, multi-token
             decoding): the multi-token kernels beside the library attention, causal and with a length mask.
     Each timed launch works on data that was not touched by the previous one (buffers rotate; each is > L2).
     """
+    if args.micro == "hybrid":
+        for size in sorted(HYBRID_SIZES) if args.hybrid_size == "all" else [args.hybrid_size]:
+            run_hybrid(args, size)
+        return
     from trimkv_b200 import ops
     dev = torch.device("cuda", 0)
     torch.cuda.set_device(dev)
@@ -621,10 +627,258 @@ def run_micro(args):
     print(json.dumps(res))
 
 
+# Layer sizes of the hybrid microbenchmark.  `attn` is the Qwen3 side (GLU of 3 x ff); the hybrid's dense feed-forward gets
+# 1.5 x ff (equal parameters), its mixers heads of the same size and twice the width as state-space channels.
+HYBRID_SIZES = {
+    "1.7b": dict(width=2048, heads=16, kv_heads=8, ff=6144, layers=8, window=4096, batch=32, prompt=8192),
+    "8b": dict(width=4096, heads=32, kv_heads=8, ff=12288, layers=4, window=4096, batch=32, prompt=4096),
+    "tiny": dict(width=256, heads=2, kv_heads=1, ff=512, layers=4, window=128, batch=4, prompt=384),
+}
+
+
+def hybrid_config(z, vocab=32768):
+    w, h = z["width"], z["heads"]
+    ssd_heads = 2 * w // 64
+    kinds = {"retention": dict(heads=h, dim=128, vdim=128, rot=dict(base=1e6, dims=128), decay=[1 - 2.0 ** -(5 + 6 * i / h) for i in range(h)]),
+             "attention": dict(heads=h, kv_heads=z["kv_heads"], dim=64, vdim=128, mask=dict(size=z["window"]), scale=0.125, diff=0.5),
+             "mamba2": dict(heads=ssd_heads, vdim=64, state=128, groups=min(8, ssd_heads), conv=4, norm_groups=min(8, ssd_heads))}
+    order = ["retention", "attention", "mamba2", "mamba2"]
+    return dict(layers=[{"type": order[i % 4], "mixer": kinds[order[i % 4]], "mlp": {"kind": "dense", "ff": z["ff"] * 3 // 2}}
+                        for i in range(z["layers"])], norm={"eps": 1e-6}, residual_mult=0.5, vocab=vocab, width=w)
+
+
+def run_hybrid(args, size):
+    """One JSON line: the hybrid decoder at one size beside the Qwen3 model of the framework (same width, depth, head size
+    and parameters per layer, M = window), and its kernels one by one beside the like kernel of that model.  Device times;
+    every kernel is timed as a CUDA graph of launches over rotating operands that together exceed L2."""
+    from trimkv_b200 import DafovikConfig, DafovikForCausalLM, TrimKVCache, ops
+    from trimkv_b200.attn import _dense_causal
+    from trimkv_b200.decoder import GreedyDecoder
+    from trimkv_b200.state_cache import HybridStateCache, RecurrentState, WindowState
+    z = HYBRID_SIZES[size]
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    peak, peak_src = measured_peaks()
+    flops_peak = 1590.0
+    path = os.path.join(ROOT, "MEASURED_PEAKS.json")
+    if os.path.exists(path):
+        with open(path) as f:
+            flops_peak = json.load(f)["bf16_tflops"]
+    bf = torch.bfloat16
+    res = {"micro": "hybrid", "size": size, "config": z, "dtype": "bf16", "data": "synthetic", "peak_gbs": peak, "peak_tflops": flops_peak,
+           "peak_source": peak_src}
+    gen = torch.Generator(device=dev).manual_seed(0)
+    B, P = z["batch"], z["prompt"]
+
+    def events(fn, n):
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize(); e0.record()
+        for _ in range(n):
+            fn()
+        e1.record(); torch.cuda.synchronize()
+        return e0.elapsed_time(e1) / n
+
+    # ------------------------------------------------------------------------------------------------ whole models
+    if args.hybrid_part != "kernels":
+        torch.manual_seed(0)
+        with torch.device(dev):
+            hybrid = DafovikForCausalLM(DafovikConfig(**hybrid_config(z))).to(bf).eval()
+        wl = dict(hidden_size=z["width"], num_hidden_layers=z["layers"], num_attention_heads=z["heads"], num_key_value_heads=z["kv_heads"],
+                  head_dim=128, intermediate_size=z["ff"], vocab_size=32768, rope_theta=1e6, retention_gate_intermediate_size=128,
+                  retention_gate_bias_init=3.0, memory_size=z["window"], buffer_size=128)
+        qwen, _ = build_model(wl, dev)
+        with torch.inference_mode():
+            for name, model in (("hybrid", hybrid), ("qwen3", qwen)):
+                out = {"parameters": sum(p.numel() for p in model.parameters())}
+                for bsz, n in ((1, P), (max(1, B // 8), P)):
+                    ids = torch.randint(0, 32768, (bsz, n), generator=gen, device=dev)
+
+                    def prompt():
+                        cache = model.new_cache(dev, capacity_tokens=n) if name == "hybrid" else model.new_cache(dev)
+                        model(input_ids=ids, past_key_values=cache, logits_to_keep=1)
+                        return cache
+                    for _ in range(3):
+                        prompt()
+                    ms = events(prompt, 5)
+                    out[f"prefill_b{bsz}x{n}"] = {"ms": ms, "tok_per_s": bsz * n / (ms * 1e-3)}
+                for bsz in (B, 4 * B):
+                    cache = model.new_cache(dev, capacity_tokens=P + 512) if name == "hybrid" else TrimKVCache(
+                        device=dev, memory_size=z["window"], buffer_size=128, num_layers=z["layers"])
+                    n = min(P, z["window"] + 64)
+                    ids = torch.randint(0, 32768, (bsz, n), generator=gen, device=dev)
+                    if name == "hybrid":
+                        cache.open(bsz)
+                        for lo in range(0, bsz, 8):        # the prompt pass of a few requests at a time
+                            rows = list(range(lo, min(bsz, lo + 8)))
+                            model.forward_packed(ids[rows].reshape(-1), cache, [n] * len(rows), rows, [len(rows) * n - 1])
+                    elif bsz <= B:
+                        model(input_ids=ids, past_key_values=cache, logits_to_keep=1)
+                    else:
+                        continue
+                    dec = GreedyDecoder(model, cache)
+                    for _ in range(3):
+                        dec.step(eager=True)
+                    for _ in range(3):
+                        dec.step()
+                    ms = events(dec.step, 50)
+                    out[f"decode_b{bsz}_at_{n}"] = {"ms_per_step": ms, "tok_per_s": bsz / (ms * 1e-3)}
+                    cache.check_status()
+                    dec.close()
+                    del dec, cache
+                    torch.cuda.empty_cache()
+                res[name] = out
+        del hybrid, qwen, model
+        torch.cuda.empty_cache()
+
+    # ------------------------------------------------------------------------------------------------ single kernels
+    rows = {}
+
+    def kernel(name, calls, nbytes, flops=0.0, reps=8):
+        """calls: closures over distinct operands, launched in turn inside one CUDA graph."""
+        for c in calls:
+            c()
+        torch.cuda.synchronize()
+        graph = torch.cuda.CUDAGraph()
+        n = max(reps, len(calls))
+        with torch.cuda.graph(graph):
+            for i in range(n):
+                calls[i % len(calls)]()
+        for _ in range(3):
+            graph.replay()
+        ms = events(graph.replay, 5) / n
+        t_mem, t_math = nbytes / (peak * 1e9) * 1e3, flops / (flops_peak * 1e12) * 1e3
+        rows[name] = {"us": ms * 1e3, "gbs": nbytes / (ms * 1e-3) / 1e9, "tflops": flops / (ms * 1e-3) / 1e12,
+                      "bound": "tensor" if t_math > t_mem else "hbm", "frac_of_roofline": max(t_mem, t_math) / ms}
+        torch.cuda.synchronize()
+        graph.reset()
+        torch.cuda.empty_cache()
+
+    def rnd(*shape, dtype=bf, scale=1.0):
+        return torch.randn(*shape, generator=gen, device=dev, dtype=dtype) * scale
+
+    if args.hybrid_part != "models":
+        w, H, G, ff, W = z["width"], z["heads"], z["kv_heads"], z["ff"], z["window"]
+        bsz = max(1, B // 8)
+        T = bsz * P
+        with torch.inference_mode():
+            wf, wb = torch.zeros(w, device=dev), torch.ones(w, device=dev, dtype=bf)
+            x32, y, c16 = rnd(T, w, dtype=torch.float32), rnd(T, w), torch.empty(T, w, dtype=bf, device=dev)
+            kernel("prompt: postnorm_add", [lambda: ops.postnorm_add(x32, y, wf, c16, 1e-6, 0.5, 1.0)], T * w * 12)
+            r16 = rnd(T, w)
+            kernel("prompt: add_rmsnorm (qwen3)", [lambda: ops.add_rmsnorm(r16, y, wb, c16, 1e-6)], T * w * 8)
+            ids = torch.randint(0, 32768, (T,), generator=gen, device=dev)
+            table = rnd(32768, w)
+            kernel("prompt: embed_stream", [lambda: ops.embed_stream(ids, table, x32, c16)], T * w * 8)
+            del table, r16
+            u = rnd(T, ff * 3 // 2)
+            kernel("prompt: gelu_tanh", [lambda: ops.gelu_tanh(u)], u.numel() * 4)
+            del u
+            gu, act = rnd(T, 2 * ff), torch.empty(T, ff, dtype=bf, device=dev)
+            kernel("prompt: silu_mul (qwen3)", [lambda: ops.silu_mul(gu, act)], T * ff * 6)
+            del gu, act, x32, y, c16
+
+            def batch_for(layer, bsz, n, start=0):
+                cache = HybridStateCache([layer], dev, bf, capacity_tokens=start + n + 8)
+                cache.open(bsz)
+                if start:
+                    cache._lens[cache._rows] = start
+                    for s in cache._rows:
+                        cache._len[s] = start
+                return cache, cache.begin([n] * bsz if n > 1 else None)
+            # retention
+            D, V = 128, 128
+            hd, hv = H * D, H * V
+            cache, b = batch_for(RecurrentState(H, D, V), bsz, P)
+            proj, qk, yy, oo = rnd(T, 2 * hd + 2 * hv), torch.empty(T, 2 * hd, dtype=bf, device=dev), torch.empty(T, hv, dtype=bf, device=dev), torch.empty(T, hv, dtype=bf, device=dev)
+            from trimkv_b200.mixers import RetentionMixer
+            mix = RetentionMixer(8, H, D, V, [1 - 2.0 ** -(5 + 6 * i / H) for i in range(H)], D, 1e6, 1e-6)
+            freq, dec_, ldec = mix._freq(dev), mix._decay(dev, False), mix._decay(dev, True)
+            kernel("prompt: rotate_qk", [lambda: ops.rotate_qk(proj, qk, b, H, D, D, freq, D ** -0.5)], T * 2 * hd * 4)
+            fl = T * H * (2.0 * 32 * (D + V) + 4.0 * D * V)      # chunks of 64: causal half of the intra-chunk block, state in and out
+            kernel("prompt: linrec_chunk (retention)", [lambda: ops.linrec(qk[:, :hd], qk[:, hd:], proj[:, 2 * hd:2 * hd + hv], cache.arrays(0)["state"], b, yy, H, head_decay=dec_, head_log_decay=ldec)],
+                   T * (2 * hd + 2 * hv) * 2, fl)
+            kernel("prompt: gated_norm (retention)", [lambda: ops.gated_norm(yy, proj[:, 2 * hd + hv:], None, oo, H, 1e-6, False)], T * hv * 6)
+            del proj, qk, yy, oo, cache
+            # state space
+            S_H, S_P, S_N, S_G = 2 * w // 64, 64, 128, min(8, 2 * w // 64)
+            inner, ch = S_H * S_P, S_H * S_P + 2 * S_G * S_N
+            cache, b = batch_for(RecurrentState(S_H, S_N, S_P, 4, ch), bsz, P)
+            proj, xbc = rnd(T, inner + ch + S_H), torch.empty(T, ch, dtype=bf, device=dev)
+            cw, cb, hb = rnd(ch, 4, dtype=torch.float32), rnd(ch, dtype=torch.float32), torch.zeros(S_H, device=dev)
+            dt, ld = torch.empty(T, S_H, device=dev), torch.empty(T, S_H, device=dev)
+            yy, oo, nw = torch.empty(T, inner, dtype=bf, device=dev), torch.empty(T, inner, dtype=bf, device=dev), torch.ones(inner, device=dev)
+            kernel("prompt: conv_silu", [lambda: ops.conv_silu(proj[:, inner:inner + ch], cache.arrays(0)["conv"], cw, cb, xbc, b)], T * ch * 4)
+            kernel("prompt: ssd_steps", [lambda: ops.ssd_steps(proj[:, inner + ch:], hb, hb, dt, ld)], T * S_H * 10)
+            fl = T * S_H * (2.0 * 32 * (S_N + S_P) + 4.0 * S_N * S_P)
+            kernel("prompt: linrec_chunk (state space)", [lambda: ops.linrec(xbc[:, inner + S_G * S_N:], xbc[:, inner:inner + S_G * S_N], xbc[:, :inner], cache.arrays(0)["state"], b, yy, S_G, log_decay=ld, v_scale=dt, skip=hb)],
+                   T * (ch + inner) * 2 + T * S_H * 8, fl)
+            kernel("prompt: gated_norm (state space)", [lambda: ops.gated_norm(yy, proj[:, :inner], nw, oo, S_G, 1e-6, True)], T * inner * 6)
+            del proj, xbc, yy, oo, cache
+            # attention: prompt pass
+            D = 64
+            cols = 2 * (H + G) * D + G * V
+            lam, qn = torch.full((1,), 0.4, device=dev), torch.ones(D, device=dev)
+            cache, b = batch_for(WindowState(G, 64, 128, W), bsz, P)
+            proj, gate, oo = rnd(T, cols + H), rnd(T, H), torch.empty(T, H * V, dtype=bf, device=dev)
+            keys = sum(min(i + 1, W) for i in range(P)) * bsz
+
+            def whole():
+                ops.diff_attention(proj, gate, qn, qn, cache.arrays(0)["k"], cache.arrays(0)["v"], b, lam, 0.5, 0.125, 1e-6, oo, H, D, V, W)
+            kernel("prompt: diff_prep + diff_prefill", [whole], T * (2 * cols + 2 * H * V), keys * H * 2.0 * 2 * (D + V))
+            q4 = rnd(bsz, P, H, 128)
+            k4, v4 = rnd(bsz, G, P, 128), rnd(bsz, G, P, 128)
+            o4 = torch.empty_like(q4)
+            causal = bsz * P * (P + 1) / 2 * H * 4.0 * 128
+            kernel("prompt: prefill_attn (qwen3, own kernel)", [lambda: ops.prefill_attn(q4, k4, v4, None, P, o4, G, 0.09, P)], T * (2 * H + 2 * G) * 256, causal)
+            kernel("prompt: library attention (qwen3)", [lambda: _dense_causal(q4.transpose(1, 2), k4, v4, 0.09)], T * (2 * H + 2 * G) * 256, causal)
+            del proj, gate, oo, q4, k4, v4, o4, cache
+            # one token per request
+            for bsz in (B, 4 * B):
+                D = 128
+                cache, b = batch_for(RecurrentState(H, D, V), bsz, 1, start=P)
+                state = cache.arrays(0)["state"]
+                n = max(1, -(-300_000_000 // (state.numel() * 4)))
+                states, proj = [torch.zeros_like(state) for _ in range(n)], rnd(bsz, 2 * hd + 2 * hv)
+                out = torch.empty(bsz, hv, dtype=bf, device=dev)
+                kernel(f"decode b{bsz}: retention_step", [lambda s=s: ops.retention_step(proj, s, b, dec_, freq, out, D, D, D ** -0.5, 1e-6) for s in states],
+                       bsz * H * D * V * 8)
+                del states, state, cache
+                cache, b = batch_for(RecurrentState(S_H, S_N, S_P, 4, ch), bsz, 1, start=P)
+                state, ring = cache.arrays(0)["state"], cache.arrays(0)["conv"]
+                ring.zero_()
+                n = max(1, -(-300_000_000 // (state.numel() * 4)))
+                states, proj = [torch.zeros_like(state) for _ in range(n)], rnd(bsz, inner + ch + S_H)
+                out = torch.empty(bsz, inner, dtype=bf, device=dev)
+                kernel(f"decode b{bsz}: ssd_step", [lambda s=s: ops.ssd_step(proj, ring, s, b, cw, cb, hb, hb, hb, out, S_G) for s in states],
+                       bsz * S_H * S_N * S_P * 8)
+                del states, state, cache
+                D = 64
+                cache, b = batch_for(WindowState(G, 64, 128, W), bsz, 1, start=W)
+                n = max(1, -(-300_000_000 // (cache.arrays(0)["k"].numel() * 4)))
+                rings = [(rnd(*cache.arrays(0)["k"].shape), rnd(*cache.arrays(0)["v"].shape)) for _ in range(n)]
+                proj, gate, out = rnd(bsz, cols + H), rnd(bsz, H), torch.empty(bsz, H * V, dtype=bf, device=dev)
+                kernel(f"decode b{bsz}: diff_prep + diff_decode", [lambda r=r: ops.diff_attention(proj, gate, qn, qn, r[0], r[1], b, lam, 0.5, 0.125, 1e-6, out, H, D, V, W) for r in rings],
+                       bsz * G * W * (2 * D + V) * 2)
+                del cache, rings
+                q3 = rnd(bsz, H, 128)
+                n = max(1, -(-300_000_000 // (bsz * G * W * 512)))
+                kv = [(rnd(bsz * G * W, 128), rnd(bsz * G * W, 128)) for _ in range(n)]
+                o3, lens = torch.empty_like(q3), torch.full((bsz * G,), W, dtype=torch.int32, device=dev)
+                ws = torch.empty(ops.decode_attn_workspace_bytes(bsz, H, G, 128, W), dtype=torch.uint8, device=dev)
+                kernel(f"decode b{bsz}: decode_attn (qwen3)", [lambda k=k, v=v: ops.decode_attn(q3, k, v, lens, None, W, o3, ws, G, 0.09, W) for k, v in kv],
+                       bsz * G * W * 512)
+                del kv
+        res["kernels"] = rows
+    print(json.dumps(res))
+
+
 def parse_args(argv=None):
     ap = argparse.ArgumentParser()
-    ap.add_argument("--micro", default=None, choices=["evict", "attn", "append", "steady", "multi", "prefill", "generate"],
+    ap.add_argument("--micro", default=None, choices=["evict", "attn", "append", "steady", "multi", "prefill", "generate", "hybrid"],
                     help="run one kernel microbenchmark instead of the decode benchmark")
+    ap.add_argument("--hybrid-size", default="1.7b", choices=sorted(HYBRID_SIZES) + ["all"], help="hybrid microbenchmark: layer sizes")
+    ap.add_argument("--hybrid-part", default="all", choices=["all", "models", "kernels"],
+                    help="hybrid microbenchmark: whole models, single kernels, or both")
     ap.add_argument("--attn-shape", default="config4", choices=["config4", "config2"])
     ap.add_argument("--M", type=int, default=4096)
     ap.add_argument("--nseg", type=int, default=2048)
