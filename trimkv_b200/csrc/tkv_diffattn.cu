@@ -20,8 +20,11 @@ namespace tkv {
 
 constexpr int kPrepThreads = 128;
 
-// Warp per (token, vector): vectors are the 2 * heads query maps, the 2 * kv_heads key maps and the kv_heads values.
-template <typename T>
+// kVecLanes lanes per (token, vector): vectors are the 2 * heads query maps, the 2 * kv_heads key maps and the kv_heads
+// values.  V: elements per access (8: dim, vdim and the row stride are multiples of 8).
+constexpr int kVecLanes = 8;
+
+template <typename T, int V>
 __global__ void __launch_bounds__(kPrepThreads) diff_prep_kernel(const T* proj, int64_t row_stride, const float* q_norm,
                                                                 const float* k_norm, float eps, T* q_out, T* k_ring, T* v_ring,
                                                                 int ring_rows, T* k_lin, T* v_lin, const int32_t* kv_start,
@@ -30,47 +33,66 @@ __global__ void __launch_bounds__(kPrepThreads) diff_prep_kernel(const T* proj, 
                                                                 int dp, int pp, int window) {
   grid_dependency_wait();
   grid_launch_dependents();
-  const int lane = threadIdx.x & 31;
+  const int lane = threadIdx.x & (kVecLanes - 1);
   const int vecs = 2 * heads + 3 * kv_heads;
-  const int64_t item = (int64_t)blockIdx.x * (kPrepThreads / 32) + (threadIdx.x >> 5);
-  if (item >= (int64_t)tokens * vecs) return;
+  const int64_t items = (int64_t)tokens * vecs;
+  const int64_t item_rt = (int64_t)blockIdx.x * (kPrepThreads / kVecLanes) + threadIdx.x / kVecLanes;
+  const bool live = item_rt < items;                     // the rest of a warp takes part in its shuffles
+  const int64_t item = live ? item_rt : items - 1;
   const int t = (int)(item / vecs), u = (int)(item - (int64_t)t * vecs);
+  const bool is_q = u < 2 * heads, is_k = !is_q && u < 2 * (heads + kv_heads);
   const T* row = proj + (int64_t)t * row_stride;
-  auto normed = [&](const T* src, const float* w, T* d0, T* d1) {
-    float ss = 0.f;
-    for (int i = lane; i < dim; i += 32) { const float x = to_f32<T>(src[i]); ss += x * x; }
-    const float r = 1.0f / sqrtf(warp_add(ss) / (float)dim + eps);
-    for (int i = lane; i < dp; i += 32) {
-      const T x = from_f32<T>(i < dim ? to_f32<T>(src[i]) * r * w[i] : 0.f);
-      if (d0 != nullptr) d0[i] = x;
-      if (d1 != nullptr) d1[i] = x;
+  T *d0 = nullptr, *d1 = nullptr;                        // where the vector goes: q, or ring and linear buffer
+  const T* src;
+  if (is_q) {
+    d0 = q_out + ((int64_t)t * 2 * heads + u) * dp;
+    src = row + (int64_t)u * dim;
+  } else {
+    const int b = owner_of(cu, batch, t);
+    const int i = cu != nullptr ? t - cu[b] : 0, n = cu != nullptr ? cu[b + 1] - cu[b] : 1;
+    const int p0 = pos0[b], slot = slots[b], rr = (p0 + i) % ring_rows;
+    const bool to_ring = i >= n - ring_rows;             // later tokens of the same step own the other rows
+    const int64_t lin = k_lin != nullptr ? (int64_t)kv_start[b] + min(p0, window - 1) + i : 0;
+    if (is_k) {
+      const int km = u - 2 * heads, g = km >> 1, m = km & 1;
+      if (to_ring) d0 = k_ring + ((((int64_t)slot * kv_heads + g) * ring_rows + rr) * 2 + m) * dp;
+      if (k_lin != nullptr) d1 = k_lin + ((lin * kv_heads + g) * 2 + m) * dp;
+      src = row + (int64_t)2 * heads * dim + (int64_t)km * dim;
+    } else {
+      const int g = u - 2 * (heads + kv_heads);
+      if (to_ring) d0 = v_ring + (((int64_t)slot * kv_heads + g) * ring_rows + rr) * pp;
+      if (v_lin != nullptr) d1 = v_lin + (lin * kv_heads + g) * pp;
+      src = row + (int64_t)2 * (heads + kv_heads) * dim + (int64_t)g * vdim;
     }
-  };
-  if (u < 2 * heads) {
-    normed(row + (int64_t)u * dim, q_norm, q_out + ((int64_t)t * 2 * heads + u) * dp, nullptr);
-    return;
   }
-  const int b = owner_of(cu, batch, t);
-  const int i = cu != nullptr ? t - cu[b] : 0, n = cu != nullptr ? cu[b + 1] - cu[b] : 1;
-  const int p0 = pos0[b], slot = slots[b];
-  const int rr = (p0 + i) % ring_rows;
-  const bool to_ring = i >= n - ring_rows;               // later tokens of the same step own the other rows
-  const int64_t lin = k_lin != nullptr ? (int64_t)kv_start[b] + min(p0, window - 1) + i : 0;
-  if (u < 2 * heads + 2 * kv_heads) {
-    const int km = u - 2 * heads, g = km >> 1, m = km & 1;
-    T* d0 = to_ring ? k_ring + ((((int64_t)slot * kv_heads + g) * ring_rows + rr) * 2 + m) * dp : nullptr;
-    T* d1 = k_lin != nullptr ? k_lin + ((lin * kv_heads + g) * 2 + m) * dp : nullptr;
-    normed(row + (int64_t)2 * heads * dim + (int64_t)km * dim, k_norm, d0, d1);
-    return;
-  }
-  const int g = u - 2 * heads - 2 * kv_heads;
-  const T* src = row + (int64_t)2 * (heads + kv_heads) * dim + (int64_t)g * vdim;
-  T* d0 = to_ring ? v_ring + (((int64_t)slot * kv_heads + g) * ring_rows + rr) * pp : nullptr;
-  T* d1 = v_lin != nullptr ? v_lin + (lin * kv_heads + g) * pp : nullptr;
-  for (int j = lane; j < pp; j += 32) {
-    const T x = j < vdim ? src[j] : from_f32<T>(0.f);
-    if (d0 != nullptr) d0[j] = x;
-    if (d1 != nullptr) d1[j] = x;
+  const int len = is_q || is_k ? dim : vdim, padded = is_q || is_k ? dp : pp;
+  const float* w = is_q ? q_norm : k_norm;
+  float ss = 0.f;
+  if (is_q || is_k)
+    for (int i = lane * V; i < len; i += kVecLanes * V) {
+      float x[V];
+      load_vec<V>(src + i, x);
+#pragma unroll
+      for (int e = 0; e < V; ++e) ss += x[e] * x[e];
+    }
+#pragma unroll
+  for (int o = kVecLanes / 2; o >= 1; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  if (!live) return;
+  const float r = 1.0f / sqrtf(ss / (float)dim + eps);
+  for (int i = lane * V; i < padded; i += kVecLanes * V) {
+    float x[V];
+    if (i < len) {
+      load_vec<V>(src + i, x);
+      if (is_q || is_k) {
+#pragma unroll
+        for (int e = 0; e < V; ++e) x[e] *= r * w[i + e];
+      }
+    } else {
+#pragma unroll
+      for (int e = 0; e < V; ++e) x[e] = 0.f;
+    }
+    if (d0 != nullptr) store_vec<V>(d0 + i, x);
+    if (d1 != nullptr) store_vec<V>(d1 + i, x);
   }
 }
 
@@ -191,12 +213,19 @@ __global__ void __launch_bounds__(kAnyThreads) diff_attn_any_kernel(DiffAttnPara
 }
 
 // ---------------------------------------------------------------------------------------------------- split-KV decode
-// CTA = (256 ring rows, (request, kv head), 8 query heads), four warps, each 16 rows at a time straight from global
+// CTA = (a chunk of ring rows, (request, kv head), 8 query heads), four warps, each 16 rows at a time straight from global
 // memory into mma.sync fragments (HBM-bound: no shared-memory staging).  MMA rows 0..7 are the first maps of up to eight
 // query heads, rows 8..15 their second maps, so one P.V product serves both maps.  The contraction index of a product
 // may be permuted as long as both operands agree, so a thread loads 16 contiguous bytes of a key (or of a value row) and
 // uses its words as the fragments of two MMA steps.
-constexpr int kDecChunk = 256, kDecWarps = 4;
+constexpr int kDecWarps = 4;
+
+// Ring rows per CTA: long chunks (their start and their merge cost what a few hundred rows do) as long as they fill the GPU.
+static int dec_chunk(int64_t segments, int ring_rows) {
+  for (int c = 1024; c > 256; c /= 2)
+    if (segments * ((ring_rows + c - 1) / c) >= 148 * 6) return c;
+  return 256;
+}
 
 __device__ __forceinline__ void mma16816(float* d, const uint32_t a0, const uint32_t a1, const uint32_t a2, const uint32_t a3,
                                          const uint32_t b0, const uint32_t b1) {
@@ -211,7 +240,7 @@ __device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
 }
 
 template <int KG /* dp / 32 */, int VG /* pp / 64 */>
-__global__ void __launch_bounds__(kDecWarps * 32) diff_decode_kernel(DiffAttnParams p) {
+__global__ void __launch_bounds__(kDecWarps * 32, KG == 2 ? 3 : 2) diff_decode_kernel(DiffAttnParams p) {
   constexpr int DP = KG * 32, PP = VG * 64;
   __shared__ float sm_o[kDecWarps][16][PP];
   __shared__ float sm_ml[kDecWarps][16][2];
@@ -221,7 +250,7 @@ __global__ void __launch_bounds__(kDecWarps * 32) diff_decode_kernel(DiffAttnPar
   const int chunk = blockIdx.x, seg = blockIdx.y, qg = blockIdx.z;
   const int b = seg / p.kv_heads, g = seg - b * p.kv_heads, hpg = p.heads / p.kv_heads;
   const int len = min(p.pos0[b] + 1, p.ring_rows);
-  const int t0 = chunk * kDecChunk, t1 = min(len, t0 + kDecChunk);
+  const int t0 = chunk * p.chunk, t1 = min(len, t0 + p.chunk);
   if (t0 >= len) return;
   const int nq = min(8, hpg - qg * 8);                    // query heads of this CTA
   const int64_t row0 = ((int64_t)p.slots[b] * p.kv_heads + g) * p.ring_rows;
@@ -248,9 +277,8 @@ __global__ void __launch_bounds__(kDecWarps * 32) diff_decode_kernel(DiffAttnPar
         for (int d = 0; d < KG; ++d) kf[n8][m][d] = ld16_stream(K + ((int64_t)row * 2 + m) * DP + d * 32 + c * 8);
     }
   };
-  const int first = t0 + warp * 16;
-  if (first < t1) load_k(first);
-  for (int t = first; t < t1; t += kDecWarps * 16) {
+  for (int t = t0 + warp * 16; t < t1; t += kDecWarps * 16) {
+    load_k(t);
     uint4 vf[4][VG];
 #pragma unroll
     for (int k = 0; k < 4; ++k) {
@@ -269,8 +297,6 @@ __global__ void __launch_bounds__(kDecWarps * 32) diff_decode_kernel(DiffAttnPar
         mma16816(s[n8], 0u, qf[1][d].x, 0u, qf[1][d].y, kf[n8][1][d].x, kf[n8][1][d].y);
         mma16816(s[n8], 0u, qf[1][d].z, 0u, qf[1][d].w, kf[n8][1][d].z, kf[n8][1][d].w);
       }
-    const int tn = t + kDecWarps * 16;
-    if (tn < t1) load_k(tn);
     float top[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int n8 = 0; n8 < 2; ++n8)
@@ -320,6 +346,7 @@ __global__ void __launch_bounds__(kDecWarps * 32) diff_decode_kernel(DiffAttnPar
     l[m] += __shfl_xor_sync(0xffffffffu, l[m], 2);
     if (c == 0) { sm_ml[warp][m * 8 + r][0] = mx[m]; sm_ml[warp][m * 8 + r][1] = l[m]; }
   }
+  if (r < nq)
 #pragma unroll
   for (int v = 0; v < VG; ++v)
 #pragma unroll
@@ -353,7 +380,7 @@ __global__ void __launch_bounds__(kAnyThreads) diff_merge_kernel(DiffAttnParams 
   grid_dependency_wait();
   grid_launch_dependents();
   const int b = blockIdx.x / p.heads, h = blockIdx.x - b * p.heads, hpg = p.heads / p.kv_heads, g = h / hpg, hh = h - g * hpg;
-  const int len = min(p.pos0[b] + 1, p.ring_rows), used = (len + kDecChunk - 1) / kDecChunk;
+  const int len = min(p.pos0[b] + 1, p.ring_rows), used = (len + p.chunk - 1) / p.chunk;
   const int64_t part = (((int64_t)b * p.kv_heads + g) * qgroups + (hh >> 3)) * nchunks;
   const int tid = threadIdx.x;
   float a[2][2] = {}, sum[2] = {0.f, 0.f};
@@ -421,7 +448,8 @@ extern "C" int tkv_diff_prep(const void* proj, int64_t row_stride, const float* 
   if (batch == 0 || tokens == 0) return TKV_OK;
   if (batch > 65535) return fail(TKV_ERR_UNSUPPORTED, "tkv_diff_prep: batch=%d", batch);
   const int64_t items = (int64_t)tokens * (2 * heads + 3 * kv_heads);
-  const int64_t grid = (items + kPrepThreads / 32 - 1) / (kPrepThreads / 32);
+  const int64_t grid = (items + kPrepThreads / kVecLanes - 1) / (kPrepThreads / kVecLanes);
+  const bool vec = dim % 8 == 0 && vdim % 8 == 0 && (row_stride * elem_size(dtype)) % 16 == 0 && aligned16(proj);
   if (grid > INT32_MAX) return fail(TKV_ERR_UNSUPPORTED, "tkv_diff_prep: %lld blocks", (long long)grid);
   TKV_WITH_TYPE(dtype, T, {
     if (k_lin != nullptr && max_history > 0) {            // before the new tokens overwrite the ring rows it reads
@@ -433,7 +461,7 @@ extern "C" int tkv_diff_prep(const void* proj, int64_t row_stride, const float* 
         if (e != cudaSuccess) return fail(TKV_ERR_LAUNCH, "tkv_diff_prep: %s", cudaGetErrorString(e));
       }
     }
-    cudaError_t e = launch_pdl(diff_prep_kernel<T>, dim3((unsigned)grid), dim3(kPrepThreads), 0, (cudaStream_t)stream, (const T*)proj, row_stride,
+    cudaError_t e = launch_pdl(vec ? diff_prep_kernel<T, 8> : diff_prep_kernel<T, 1>, dim3((unsigned)grid), dim3(kPrepThreads), 0, (cudaStream_t)stream, (const T*)proj, row_stride,
                                q_norm, k_norm, eps, (T*)q_out, (T*)k_ring, (T*)v_ring, ring_rows, (T*)k_lin, (T*)v_lin, kv_start, cu_tokens,
                                slots, pos0, batch, tokens, heads, kv_heads, dim, vdim, dp, pp, window);
     if (e != cudaSuccess) return fail(TKV_ERR_LAUNCH, "tkv_diff_prep: %s", cudaGetErrorString(e));
@@ -443,7 +471,8 @@ extern "C" int tkv_diff_prep(const void* proj, int64_t row_stride, const float* 
 
 extern "C" int64_t tkv_diff_decode_workspace_bytes(int batch, int heads, int kv_heads, int ring_rows, int dp, int pp, int dtype) {
   if (!fast_shape(dp, pp, dtype) || batch <= 0 || kv_heads <= 0 || heads < kv_heads || ring_rows <= 0) return 0;
-  const int64_t chunks = (ring_rows + kDecChunk - 1) / kDecChunk, qg = (heads / kv_heads + 7) / 8;
+  const int chunk = dec_chunk((int64_t)batch * kv_heads, ring_rows);
+  const int64_t chunks = (ring_rows + chunk - 1) / chunk, qg = (heads / kv_heads + 7) / 8;
   return (int64_t)batch * kv_heads * qg * chunks * 16 * (pp + 2) * (int64_t)sizeof(float);
 }
 
@@ -465,7 +494,8 @@ extern "C" int tkv_diff_decode(const void* q, const void* k_ring, const void* v_
   if (!aligned16(q) || !aligned16(k_ring) || !aligned16(v_ring)) return fail(TKV_ERR_ARG, "tkv_diff_decode: pointers must be 16-byte aligned");
   const int64_t need = tkv_diff_decode_workspace_bytes(batch, heads, kv_heads, ring_rows, dp, pp, dtype);
   if (!workspace || workspace_bytes < need) return fail(TKV_ERR_ARG, "tkv_diff_decode: workspace of %lld bytes, %lld needed", (long long)workspace_bytes, (long long)need);
-  const int chunks = (ring_rows + kDecChunk - 1) / kDecChunk, qg = (heads / kv_heads + 7) / 8;
+  p.chunk = dec_chunk((int64_t)batch * kv_heads, ring_rows);
+  const int chunks = (ring_rows + p.chunk - 1) / p.chunk, qg = (heads / kv_heads + 7) / 8;
   if ((int64_t)batch * kv_heads > 65535 || qg > 65535) return fail(TKV_ERR_UNSUPPORTED, "tkv_diff_decode: batch * kv_heads = %lld", (long long)batch * kv_heads);
   p.part_o = (float*)workspace;
   p.part_ml = p.part_o + (int64_t)batch * kv_heads * qg * chunks * 16 * pp;

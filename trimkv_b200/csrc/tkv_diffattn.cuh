@@ -13,7 +13,7 @@ struct DiffAttnParams {
   const void* gate; int64_t gate_stride;                  // [tokens, heads] within a wider row
   void* out;                                              // [tokens, heads, vdim]
   float* part_o; float* part_ml;                          // split-KV partials
-  int batch, tokens, heads, kv_heads, dim, vdim, dp, pp, window;
+  int batch, tokens, heads, kv_heads, dim, vdim, dp, pp, window, chunk;
   int32_t* status;
 };
 

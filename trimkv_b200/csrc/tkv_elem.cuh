@@ -77,6 +77,18 @@ __device__ __forceinline__ float sigmoid_f32(float x) { return 1.0f / (1.0f + ex
 __device__ __forceinline__ float silu_f32(float x) { return x / (1.0f + expf(-x)); }
 __device__ __forceinline__ float softplus_f32(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 
+// SiLU and GELU of values that are then used in the model type: full precision for fp32 models, the hardware's exponential
+// and division (errors far below a 16-bit rounding) for 16-bit ones.
+template <typename T> __device__ __forceinline__ float silu_act(float x) {
+  if constexpr (sizeof(T) == 4) return silu_f32(x);
+  else return __fdividef(x, 1.0f + __expf(fminf(-x, 80.f)));
+}
+template <typename T> __device__ __forceinline__ float gelu_tanh_act(float z) {
+  const float u = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+  if constexpr (sizeof(T) == 4) return 0.5f * z * (1.0f + tanhf(u));
+  else return __fdividef(z, 1.0f + __expf(fminf(-2.0f * u, 80.f)));      // (1 + tanh u) / 2 = 1 / (1 + e^(-2u))
+}
+
 // Request that owns packed row t: largest b with cu[b] <= t (cu == nullptr: one row per request).
 __device__ __forceinline__ int owner_of(const int32_t* cu, int batch, int t) {
   if (cu == nullptr) return t;

@@ -72,7 +72,7 @@ __global__ void __launch_bounds__(kRotThreads) rotate_qk_kernel(const T* proj, i
   }
 }
 
-constexpr int kConvThreads = 128, kConvStrip = 16;
+constexpr int kConvThreads = 128, kConvStrip = 32;
 
 // grid: (channel blocks, strips of kConvStrip tokens, requests).  kTaps = 0: any number of taps, inputs re-read per tap.
 template <typename T, int V, int kTaps>
@@ -119,7 +119,7 @@ __global__ void __launch_bounds__(kConvThreads) conv_silu_kernel(const T* proj, 
         acc[e] = bs[e];
 #pragma unroll
         for (int k = kT - 1; k >= 0; --k) acc[e] = fmaf(wt[k][e], win[k][e], acc[e]);
-        acc[e] = silu_f32(acc[e]);
+        acc[e] = silu_act<T>(acc[e]);
       }
       store_vec<V>(out + (int64_t)(t0 + i) * channels + ch, acc);
     }
@@ -135,7 +135,7 @@ __global__ void __launch_bounds__(kConvThreads) conv_silu_kernel(const T* proj, 
         for (int e = 0; e < V; ++e) acc[e] = fmaf(w[(int64_t)(ch + e) * taps + taps - 1 - k], v[e], acc[e]);
       }
 #pragma unroll
-      for (int e = 0; e < V; ++e) acc[e] = silu_f32(acc[e]);
+      for (int e = 0; e < V; ++e) acc[e] = silu_act<T>(acc[e]);
       store_vec<V>(out + (int64_t)(t0 + i) * channels + ch, acc);
     }
   }
@@ -172,75 +172,86 @@ __global__ void __launch_bounds__(256) ssd_steps_kernel(const T* dt_in, int64_t 
 constexpr int kStepThreads = 256;
 
 // S <- decay S + k v^T and o = S^T q for one head: S [n, p] fp32 in global memory, k / q [n], v [p], o [p] in shared
-// memory.  Threads cover columns in vectors of V and rows in an interleaved fashion; `red` holds kStepThreads * V floats.
-// All threads of the CTA call it; k, q, v must be visible (a barrier before), o is visible on return.
-template <int V>
-__device__ __forceinline__ void state_step(float* S, int n, int p, float decay, bool fresh, const float* k, const float* q,
-                                           const float* v, float* o, float* red) {
-  constexpr int U = 8;
-  const int nc = p / V, cb = min(nc, kStepThreads), rg = kStepThreads / cb;
-  const int r = threadIdx.x / cb, c0 = threadIdx.x - r * cb;
-  const bool active = r < rg;
-  for (int cbase = 0; cbase < nc; cbase += cb) {
-    const int c = cbase + c0;
-    float acc[V];
+// memory.  Threads cover columns in vectors of V and rows in an interleaved fashion.  The first rows are requested by
+// `prefetch` before the step's k, q, v are known, so that their latency overlaps the producers' work.
+template <int V> struct StateStep {
+  static constexpr int U = 8;
+  float* S; int n, p, nc, cb, rg, r, c0; bool fresh;
+  float s[U][V];
+
+  __device__ __forceinline__ void load(int row, int c) {
 #pragma unroll
-    for (int e = 0; e < V; ++e) acc[e] = 0.f;
-    if (active && c < nc) {
-      float vv[V];
-#pragma unroll
-      for (int e = 0; e < V; ++e) vv[e] = v[c * V + e];
-      for (int row = r; row < n; row += rg * U) {
-        float s[U][V];
-#pragma unroll
-        for (int u = 0; u < U; ++u) {
-          const int rr = row + u * rg;
-          if (rr < n && !fresh) {
-            if constexpr (V == 4) {
-              const float4 x = *reinterpret_cast<const float4*>(S + (int64_t)rr * p + c * V);
-              s[u][0] = x.x; s[u][1] = x.y; s[u][2] = x.z; s[u][3] = x.w;
-            } else {
-              s[u][0] = S[(int64_t)rr * p + c];
-            }
-          } else {
-#pragma unroll
-            for (int e = 0; e < V; ++e) s[u][e] = 0.f;
-          }
+    for (int u = 0; u < U; ++u) {
+      const int rr = row + u * rg;
+      if (rr < n && !fresh) {
+        if constexpr (V == 4) {
+          const float4 x = *reinterpret_cast<const float4*>(S + (int64_t)rr * p + c * V);
+          s[u][0] = x.x; s[u][1] = x.y; s[u][2] = x.z; s[u][3] = x.w;
+        } else {
+          s[u][0] = S[(int64_t)rr * p + c];
         }
+      } else {
 #pragma unroll
-        for (int u = 0; u < U; ++u) {
-          const int rr = row + u * rg;
-          if (rr < n) {
-            const float kk = k[rr], qq = q[rr];
+        for (int e = 0; e < V; ++e) s[u][e] = 0.f;
+      }
+    }
+  }
+  __device__ __forceinline__ void prefetch(float* S_, int n_, int p_, bool fresh_) {
+    S = S_; n = n_; p = p_; fresh = fresh_;
+    nc = p / V; cb = min(nc, kStepThreads); rg = kStepThreads / cb;
+    r = threadIdx.x / cb; c0 = threadIdx.x - r * cb;
+    if (r < rg) load(r, c0);
+  }
+  // All threads of the CTA call it; k, q, v must be visible (a barrier before), o is visible on return.  red holds
+  // kStepThreads * V floats.
+  __device__ __forceinline__ void run(float decay, const float* k, const float* q, const float* v, float* o, float* red) {
+    const bool active = r < rg;
+    for (int cbase = 0; cbase < nc; cbase += cb) {
+      const int c = cbase + c0;
+      float acc[V];
 #pragma unroll
-            for (int e = 0; e < V; ++e) {
-              s[u][e] = fmaf(decay, s[u][e], kk * vv[e]);
-              acc[e] = fmaf(qq, s[u][e], acc[e]);
+      for (int e = 0; e < V; ++e) acc[e] = 0.f;
+      if (active && c < nc) {
+        float vv[V];
+#pragma unroll
+        for (int e = 0; e < V; ++e) vv[e] = v[c * V + e];
+        for (int row = r; row < n; row += rg * U) {
+          if (row != r || cbase != 0) load(row, c);
+#pragma unroll
+          for (int u = 0; u < U; ++u) {
+            const int rr = row + u * rg;
+            if (rr < n) {
+              const float kk = k[rr], qq = q[rr];
+#pragma unroll
+              for (int e = 0; e < V; ++e) {
+                s[u][e] = fmaf(decay, s[u][e], kk * vv[e]);
+                acc[e] = fmaf(qq, s[u][e], acc[e]);
+              }
+              if constexpr (V == 4)
+                *reinterpret_cast<float4*>(S + (int64_t)rr * p + c * V) = make_float4(s[u][0], s[u][1], s[u][2], s[u][3]);
+              else
+                S[(int64_t)rr * p + c] = s[u][0];
             }
-            if constexpr (V == 4)
-              *reinterpret_cast<float4*>(S + (int64_t)rr * p + c * V) = make_float4(s[u][0], s[u][1], s[u][2], s[u][3]);
-            else
-              S[(int64_t)rr * p + c] = s[u][0];
           }
         }
       }
-    }
-    if (active) {
+      if (active) {
 #pragma unroll
-      for (int e = 0; e < V; ++e) red[(r * cb + c0) * V + e] = acc[e];
+        for (int e = 0; e < V; ++e) red[(r * cb + c0) * V + e] = acc[e];
+      }
+      __syncthreads();
+      for (int i = threadIdx.x; i < cb * V && cbase * V + i < p; i += kStepThreads) {
+        float a = 0.f;
+        for (int g = 0; g < rg; ++g) a += red[g * cb * V + i];
+        o[cbase * V + i] = a;
+      }
+      __syncthreads();
     }
-    __syncthreads();
-    for (int i = threadIdx.x; i < cb * V && cbase * V + i < p; i += kStepThreads) {
-      float a = 0.f;
-      for (int g = 0; g < rg; ++g) a += red[g * cb * V + i];
-      o[cbase * V + i] = a;
-    }
-    __syncthreads();
   }
-}
+};
 
 // One CTA per (request, head).  proj row: q [heads, dim], k [heads, dim], v [heads, vdim], gate [heads, vdim].
-template <typename T>
+template <typename T, int V>
 __global__ void __launch_bounds__(kStepThreads) retention_step_kernel(const T* proj, int64_t row_stride, float* state,
                                                                      const int32_t* slots, const int32_t* pos0, const float* decay,
                                                                      const float2* freq, T* out, int heads, int dim, int vdim,
@@ -252,6 +263,8 @@ __global__ void __launch_bounds__(kStepThreads) retention_step_kernel(const T* p
   grid_launch_dependents();
   const int b = blockIdx.x / heads, h = blockIdx.x - b * heads;
   const int pos = pos0[b];
+  StateStep<V> step;
+  step.prefetch(state + ((int64_t)slots[b] * heads + h) * dim * vdim, dim, vdim, pos == 0);
   const T* row = proj + (int64_t)b * row_stride;
   const T *qg = row + (int64_t)h * dim, *kg = row + (int64_t)(heads + h) * dim;
   const T* vg = row + (int64_t)2 * heads * dim + (int64_t)h * vdim;
@@ -272,20 +285,18 @@ __global__ void __launch_bounds__(kStepThreads) retention_step_kernel(const T* p
   }
   for (int i = threadIdx.x; i < vdim; i += kStepThreads) v[i] = to_f32<T>(vg[i]);
   __syncthreads();
-  float* S = state + ((int64_t)slots[b] * heads + h) * dim * vdim;
-  if (vdim % 4 == 0) state_step<4>(S, dim, vdim, decay[h], pos == 0, k, q, v, o, red);
-  else state_step<1>(S, dim, vdim, decay[h], pos == 0, k, q, v, o, red);
+  step.run(decay[h], k, q, v, o, red);
   float ss = 0.f;
   for (int i = threadIdx.x; i < vdim; i += kStepThreads) ss += o[i] * o[i];
   const float rstd = 1.0f / sqrtf(block_add<kStepThreads>(ss, wred) / (float)vdim + eps);
   T* dst = out + ((int64_t)b * heads + h) * vdim;
-  for (int i = threadIdx.x; i < vdim; i += kStepThreads) dst[i] = from_f32<T>(o[i] * rstd * silu_f32(to_f32<T>(gg[i])));
+  for (int i = threadIdx.x; i < vdim; i += kStepThreads) dst[i] = from_f32<T>(o[i] * rstd * silu_act<T>(to_f32<T>(gg[i])));
 }
 
 // One CTA per (request, head).  proj row: z [inner], x [inner], B [groups, n], C [groups, n], dt [heads]; the ring holds
 // the last `taps` inputs of x | B | C.  This step's inputs go to ring row pos mod taps, which holds an input that no
 // longer counts, so heads of a group may read the other rows while one of them writes.
-template <typename T>
+template <typename T, int V>
 __global__ void __launch_bounds__(kStepThreads) ssd_step_kernel(const T* proj, int64_t row_stride, T* ring, float* state,
                                                                const int32_t* slots, const int32_t* pos0, const float* conv_w,
                                                                const float* conv_b, const float* dt_bias, const float* a_log,
@@ -298,6 +309,8 @@ __global__ void __launch_bounds__(kStepThreads) ssd_step_kernel(const T* proj, i
   const int b = blockIdx.x / heads, h = blockIdx.x - b * heads;
   const int hpg = heads / groups, g = h / hpg;
   const int pos = pos0[b], slot = slots[b], inner = heads * vdim, channels = inner + 2 * groups * n;
+  StateStep<V> step;
+  step.prefetch(state + ((int64_t)slot * heads + h) * n * vdim, n, vdim, pos == 0);
   const T* cur = proj + (int64_t)b * row_stride + inner;
   T* rg = ring + (int64_t)slot * taps * channels;
   const float dt = softplus_f32(to_f32<T>(cur[channels + h]) + dt_bias[h]);
@@ -305,20 +318,27 @@ __global__ void __launch_bounds__(kStepThreads) ssd_step_kernel(const T* proj, i
   for (int i = threadIdx.x; i < vdim + 2 * n; i += kStepThreads) {
     const int ch = i < vdim ? h * vdim + i : (i < vdim + n ? inner + g * n + (i - vdim) : inner + (groups + g) * n + (i - vdim - n));
     float acc = conv_b[ch];
-    for (int d = taps - 1; d > 0; --d)
-      if (pos - d >= 0) acc = fmaf(conv_w[(int64_t)ch * taps + taps - 1 - d], to_f32<T>(rg[(int64_t)((pos - d) % taps) * channels + ch]), acc);
     const T in = cur[ch];
+    if (taps == 4) {                                       // the usual number: every load is requested before the first use
+      const float4 w = *reinterpret_cast<const float4*>(conv_w + (int64_t)ch * 4);
+      const int r0 = pos & 3;
+      const float x3 = pos >= 3 ? to_f32<T>(rg[(int64_t)((r0 + 1) & 3) * channels + ch]) : 0.f;
+      const float x2 = pos >= 2 ? to_f32<T>(rg[(int64_t)((r0 + 2) & 3) * channels + ch]) : 0.f;
+      const float x1 = pos >= 1 ? to_f32<T>(rg[(int64_t)((r0 + 3) & 3) * channels + ch]) : 0.f;
+      acc = fmaf(w.z, x1, fmaf(w.y, x2, fmaf(w.x, x3, acc)));
+    } else {
+      for (int d = taps - 1; d > 0; --d)
+        if (pos - d >= 0) acc = fmaf(conv_w[(int64_t)ch * taps + taps - 1 - d], to_f32<T>(rg[(int64_t)((pos - d) % taps) * channels + ch]), acc);
+    }
     acc = fmaf(conv_w[(int64_t)ch * taps + taps - 1], to_f32<T>(in), acc);
     if (i < vdim || h == g * hpg) rg[(int64_t)(pos % taps) * channels + ch] = in;
-    const float y = round_as<T>(silu_f32(acc));
+    const float y = round_as<T>(silu_act<T>(acc));
     if (i < vdim) { x[i] = y; v[i] = dt * y; }
     else if (i < vdim + n) k[i - vdim] = y;
     else q[i - vdim - n] = y;
   }
   __syncthreads();
-  float* S = state + ((int64_t)slot * heads + h) * n * vdim;
-  if (vdim % 4 == 0) state_step<4>(S, n, vdim, decay, pos == 0, k, q, v, o, red);
-  else state_step<1>(S, n, vdim, decay, pos == 0, k, q, v, o, red);
+  step.run(decay, k, q, v, o, red);
   T* dst = out + (int64_t)b * inner + (int64_t)h * vdim;
   for (int i = threadIdx.x; i < vdim; i += kStepThreads) dst[i] = from_f32<T>(fmaf(skip[h], x[i], o[i]));
 }
@@ -426,7 +446,7 @@ extern "C" int tkv_conv_silu(const void* proj, int64_t row_stride, void* ring, c
   if (batch < 0 || max_tokens < 0 || channels <= 0 || taps <= 0 || row_stride < channels) return fail(TKV_ERR_ARG, "tkv_conv_silu: bad sizes");
   if (batch == 0 || max_tokens == 0) return TKV_OK;
   const int64_t strips = ((int64_t)max_tokens + kConvStrip - 1) / kConvStrip;
-  if (batch > 65535 || strips > 65535) return fail(TKV_ERR_UNSUPPORTED, "tkv_conv_silu: batch=%d max_tokens=%d (at most 65535 requests of 1048560 tokens)", batch, max_tokens);
+  if (batch > 65535 || strips > 65535) return fail(TKV_ERR_UNSUPPORTED, "tkv_conv_silu: batch=%d max_tokens=%d (at most 65535 requests of 2097120 tokens)", batch, max_tokens);
   const int64_t es = elem_size(dtype);
   const bool vec = channels % 8 == 0 && (row_stride * es) % 16 == 0 && aligned16(proj) && aligned16(out) && aligned16(ring);
   const int per = kConvThreads * (vec ? 8 : 1);
@@ -477,8 +497,9 @@ extern "C" int tkv_retention_step(const void* proj, int64_t row_stride, float* s
   if (batch == 0) return TKV_OK;
   const size_t smem = ((size_t)2 * dim + 2 * vdim + kStepThreads * 4) * sizeof(float);
   TKV_WITH_TYPE(dtype, T, {
-    if (!allow_smem(retention_step_kernel<T>, smem)) return fail(TKV_ERR_UNSUPPORTED, "tkv_retention_step: dim=%d vdim=%d", dim, vdim);
-    TKV_CHECK_LAUNCH(launch_pdl(retention_step_kernel<T>, dim3((unsigned)(batch * heads)), dim3(kStepThreads), smem, (cudaStream_t)stream,
+    auto kern = vdim % 4 == 0 ? retention_step_kernel<T, 4> : retention_step_kernel<T, 1>;
+    if (!allow_smem(kern, smem)) return fail(TKV_ERR_UNSUPPORTED, "tkv_retention_step: dim=%d vdim=%d", dim, vdim);
+    TKV_CHECK_LAUNCH(launch_pdl(kern, dim3((unsigned)(batch * heads)), dim3(kStepThreads), smem, (cudaStream_t)stream,
                                 (const T*)proj, row_stride, state, slots, pos0, head_decay, (const float2*)freq_hi_lo, (T*)out, heads, dim,
                                 vdim, rot_dims, k_scale, eps), "tkv_retention_step");
   });
@@ -498,8 +519,9 @@ extern "C" int tkv_ssd_step(const void* proj, int64_t row_stride, void* ring, fl
   if (batch == 0) return TKV_OK;
   const size_t smem = ((size_t)2 * n + 3 * vdim + kStepThreads * 4) * sizeof(float);
   TKV_WITH_TYPE(dtype, T, {
-    if (!allow_smem(ssd_step_kernel<T>, smem)) return fail(TKV_ERR_UNSUPPORTED, "tkv_ssd_step: n=%d vdim=%d", n, vdim);
-    TKV_CHECK_LAUNCH(launch_pdl(ssd_step_kernel<T>, dim3((unsigned)(batch * heads)), dim3(kStepThreads), smem, (cudaStream_t)stream,
+    auto kern = vdim % 4 == 0 ? ssd_step_kernel<T, 4> : ssd_step_kernel<T, 1>;
+    if (!allow_smem(kern, smem)) return fail(TKV_ERR_UNSUPPORTED, "tkv_ssd_step: n=%d vdim=%d", n, vdim);
+    TKV_CHECK_LAUNCH(launch_pdl(kern, dim3((unsigned)(batch * heads)), dim3(kStepThreads), smem, (cudaStream_t)stream,
                                 (const T*)proj, row_stride, (T*)ring, state, slots, pos0, conv_w, conv_b, dt_bias, a_log, skip, (T*)out,
                                 heads, groups, n, vdim, taps), "tkv_ssd_step");
   });

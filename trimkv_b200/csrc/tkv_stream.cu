@@ -116,15 +116,17 @@ __global__ void __launch_bounds__(kRowThreads) stream_norm_kernel(const float* x
   }
 }
 
-// One warp per (row, group) of `len` elements.  gate_first: RMS(y * silu(z)) * w, else RMS(y) * w * silu(z).
-template <typename T, int V>
+// kLanes lanes per (row, group) of `len` elements.  gate_first: RMS(y * silu(z)) * w, else RMS(y) * w * silu(z).
+template <typename T, int V, int kLanes>
 __global__ void __launch_bounds__(kRowThreads) gated_norm_kernel(const T* y, int64_t y_stride, const T* z, int64_t z_stride,
                                                                 const float* w, T* out, int rows, int groups, int len,
                                                                 float eps, int gate_first) {
-  constexpr int kKeep = V == 8 ? 2 : 4;          // vectors per lane held in registers (512 elements per group)
-  const int lane = threadIdx.x & 31;
-  const int64_t item = (int64_t)blockIdx.x * (kRowThreads / 32) + (threadIdx.x >> 5);
-  if (item >= (int64_t)rows * groups) return;
+  constexpr int kKeep = V == 8 ? 2 : 4;          // vectors per lane held in registers
+  const int lane = threadIdx.x & (kLanes - 1);
+  const int64_t items = (int64_t)rows * groups;
+  const int64_t item_rt = (int64_t)blockIdx.x * (kRowThreads / kLanes) + threadIdx.x / kLanes;
+  const bool live = item_rt < items;             // the rest of a warp takes part in its shuffles
+  const int64_t item = live ? item_rt : items - 1;
   grid_dependency_wait();
   grid_launch_dependents();
   const int64_t row = item / groups;
@@ -134,29 +136,33 @@ __global__ void __launch_bounds__(kRowThreads) gated_norm_kernel(const T* y, int
   T* o = out + (row * groups + grp) * (int64_t)len;
   const int nvec = len / V;
   float a[kKeep][V], g[kKeep][V], ss = 0.f;
-  auto load = [&](int i, float* av, float* gv) {
-    load_vec<V>(yr + (int64_t)i * V, av);
-    load_vec<V>(zr + (int64_t)i * V, gv);
+  auto gate = [&](float* av, float* gv) {
 #pragma unroll
     for (int e = 0; e < V; ++e) {
-      gv[e] = silu_f32(gv[e]);
+      gv[e] = silu_act<T>(gv[e]);
       if (gate_first) av[e] *= gv[e];
+      ss += av[e] * av[e];
     }
   };
 #pragma unroll
   for (int j = 0; j < kKeep; ++j)
-    if (lane + 32 * j < nvec) {
-      load(lane + 32 * j, a[j], g[j]);
-#pragma unroll
-      for (int e = 0; e < V; ++e) ss += a[j][e] * a[j][e];
+    if (lane + kLanes * j < nvec) {
+      load_vec<V>(yr + (int64_t)(lane + kLanes * j) * V, a[j]);
+      load_vec<V>(zr + (int64_t)(lane + kLanes * j) * V, g[j]);
     }
-  for (int i = lane + 32 * kKeep; i < nvec; i += 32) {
-    float av[V], gv[V];
-    load(i, av, gv);
 #pragma unroll
-    for (int e = 0; e < V; ++e) ss += av[e] * av[e];
+  for (int j = 0; j < kKeep; ++j)
+    if (lane + kLanes * j < nvec) gate(a[j], g[j]);
+  for (int i = lane + kLanes * kKeep; i < nvec; i += kLanes) {
+    float av[V], gv[V];
+    load_vec<V>(yr + (int64_t)i * V, av);
+    load_vec<V>(zr + (int64_t)i * V, gv);
+    gate(av, gv);
   }
-  const float rstd = 1.0f / sqrtf(warp_add(ss) / (float)len + eps);
+#pragma unroll
+  for (int d = kLanes / 2; d >= 1; d >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, d);
+  const float rstd = 1.0f / sqrtf(ss / (float)len + eps);
+  if (!live) return;
   auto finish = [&](int i, float* av, const float* gv) {
     float wv[V];
     if (w != nullptr) load_vec<V>(w + (int64_t)grp * len + (int64_t)i * V, wv);
@@ -170,17 +176,18 @@ __global__ void __launch_bounds__(kRowThreads) gated_norm_kernel(const T* y, int
   };
 #pragma unroll
   for (int j = 0; j < kKeep; ++j)
-    if (lane + 32 * j < nvec) finish(lane + 32 * j, a[j], g[j]);
-  for (int i = lane + 32 * kKeep; i < nvec; i += 32) {
+    if (lane + kLanes * j < nvec) finish(lane + kLanes * j, a[j], g[j]);
+  for (int i = lane + kLanes * kKeep; i < nvec; i += kLanes) {
     float av[V], gv[V];
-    load(i, av, gv);
+    load_vec<V>(yr + (int64_t)i * V, av);
+    load_vec<V>(zr + (int64_t)i * V, gv);
+    const float keep = ss;
+    gate(av, gv);
+    ss = keep;
     finish(i, av, gv);
   }
 }
 
-__device__ __forceinline__ float gelu_tanh_f32(float z) {
-  return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-}
 template <typename T, int V>
 __global__ void __launch_bounds__(kRowThreads) gelu_tanh_kernel(T* u, int64_t n) {
   grid_dependency_wait();
@@ -190,7 +197,7 @@ __global__ void __launch_bounds__(kRowThreads) gelu_tanh_kernel(T* u, int64_t n)
     float a[V];
     load_vec<V>(u + i * V, a);
 #pragma unroll
-    for (int e = 0; e < V; ++e) a[e] = gelu_tanh_f32(a[e]);
+    for (int e = 0; e < V; ++e) a[e] = gelu_tanh_act<T>(a[e]);
     store_vec<V>(u + i * V, a);
   }
 }
@@ -268,15 +275,18 @@ extern "C" int tkv_gated_norm(const void* y, int64_t y_stride, const void* z, in
   const int64_t width = (int64_t)groups * group_len;
   if (y_stride < width || z_stride < width) return fail(TKV_ERR_ARG, "tkv_gated_norm: row strides shorter than a row");
   if (rows == 0) return TKV_OK;
-  const int64_t grid = ((int64_t)rows * groups + kRowThreads / 32 - 1) / (kRowThreads / 32);
-  int rc = rows_grid("tkv_gated_norm", grid);
-  if (rc != TKV_OK) return rc;
   const int64_t es = elem_size(dtype);
   const bool vec = group_len % 8 == 0 && (y_stride * es) % 16 == 0 && (z_stride * es) % 16 == 0 && aligned16(y) && aligned16(z) &&
                    aligned16(out) && (!weight || aligned16(weight));
+  const int lanes = !vec || group_len > 256 ? 32 : group_len > 128 ? 16 : 8;
+  const int64_t grid = ((int64_t)rows * groups + kRowThreads / lanes - 1) / (kRowThreads / lanes);
+  int rc = rows_grid("tkv_gated_norm", grid);
+  if (rc != TKV_OK) return rc;
   TKV_WITH_TYPE(dtype, T, {
-    TKV_LAUNCH_V(vec, gated_norm_kernel, grid, kRowThreads, (const T*)y, y_stride, (const T*)z, z_stride, weight, (T*)out, rows, groups,
-                 group_len, eps, gate_first);
+    auto k = !vec ? gated_norm_kernel<T, 1, 32> : lanes == 8 ? gated_norm_kernel<T, 8, 8> : lanes == 16 ? gated_norm_kernel<T, 8, 16> : gated_norm_kernel<T, 8, 32>;
+    cudaError_t e = launch_pdl(k, dim3((unsigned)grid), dim3(kRowThreads), 0, (cudaStream_t)stream, (const T*)y, y_stride, (const T*)z,
+                               z_stride, weight, (T*)out, rows, groups, group_len, eps, gate_first);
+    if (e != cudaSuccess) return fail(TKV_ERR_LAUNCH, "tkv_gated_norm: %s", cudaGetErrorString(e));
   });
   return check_launch("tkv_gated_norm");
 }
