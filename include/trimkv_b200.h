@@ -502,18 +502,19 @@ int tkv_ssd_step(const void* proj, int64_t row_stride, void* ring, float* state,
  * [tokens, heads] or NULL (1); skip [heads] or NULL (0); state [slots, heads, n, vdim] fp32, read and written.
  * tkv_linrec_scan runs token by token and takes every size (n <= 1760) and dtype; cu_tokens may be NULL.
  * tkv_linrec_chunk is the tensor-core form for prompts: bf16, n <= 256, n, vdim and the strides multiples of 8, 16-byte
- * aligned rows.  Its workspace (tkv_linrec_chunk_workspace_bytes; -1 = shape not supported, 0 = none) holds the states
+ * aligned rows (64 < n <= 128 and prompts of at least 128 tokens: tcgen05; else mma.sync).  tokens: rows of the packed arrays.
+ * Its workspace (tkv_linrec_chunk_workspace_bytes; -1 = shape not supported, 0 = none) holds the states
  * between the segments of long sequences. */
 int tkv_linrec_scan(const void* q, int64_t q_stride, const void* k, int64_t k_stride, const void* v, int64_t v_stride,
                     const float* log_decay, const float* head_decay, const float* v_scale, const float* skip, void* out,
                     float* state, const int32_t* slots, const int32_t* cu_tokens, const int32_t* pos0, int batch, int heads,
                     int groups, int n, int vdim, int dtype, tkv_stream_t stream);
-int64_t tkv_linrec_chunk_workspace_bytes(int batch, int max_tokens, int heads, int n, int vdim, int dtype);
+int64_t tkv_linrec_chunk_workspace_bytes(int batch, int max_tokens, int tokens, int heads, int n, int vdim, int dtype);
 int tkv_linrec_chunk(const void* q, int64_t q_stride, const void* k, int64_t k_stride, const void* v, int64_t v_stride,
                      const float* log_decay, const float* head_log_decay, const float* v_scale, const float* skip, void* out,
                      float* state, const int32_t* slots, const int32_t* cu_tokens, const int32_t* pos0, void* workspace,
-                     int64_t workspace_bytes, int batch, int max_tokens, int heads, int groups, int n, int vdim, int dtype,
-                     tkv_stream_t stream);
+                     int64_t workspace_bytes, int batch, int max_tokens, int tokens, int heads, int groups, int n, int vdim,
+                     int dtype, int32_t* status, tkv_stream_t stream);
 
 /* Differential attention over a sliding window.  proj row: q [heads, 2, dim], k [kv_heads, 2, dim], v [kv_heads, vdim].
  * tkv_diff_prep norms q and k per head and map (weights q_norm / k_norm [dim]) and stores them zero-padded to dp / pp

@@ -175,16 +175,16 @@ def _oracle_recurrence(q, k, v, logd, scale, skip, lens):
 
 
 @pytest.mark.parametrize("dtype,scan", [(F32, True), (BF16, True), (BF16, False)])
-@pytest.mark.parametrize("heads,groups,n,p", [(2, 1, 64, 64), (4, 2, 48, 32), (2, 2, 128, 128), (1, 1, 8, 136), (2, 1, 200, 72), (6, 3, 16, 8)])
+@pytest.mark.parametrize("heads,groups,n,p", [(2, 1, 64, 64), (4, 2, 48, 32), (2, 2, 128, 128), (1, 1, 8, 136), (2, 1, 200, 72), (6, 3, 16, 8), (2, 1, 72, 72), (4, 2, 128, 64)])
 def test_recurrence_ragged_and_in_portions(dtype, scan, heads, groups, n, p):
     from trimkv_b200 import ops
     from trimkv_b200.state_cache import RecurrentState
     rng = np.random.default_rng(n * p)
-    lens = [131, 64, 2, 1]
-    q, k, v, logd, scale, skip = _recurrence_case(rng, lens, heads, groups, n, p, dtype, far=(3, 129))
+    lens = [300, 64, 2, 1]
+    q, k, v, logd, scale, skip = _recurrence_case(rng, lens, heads, groups, n, p, dtype, far=(3, 298))
     want, states = _oracle_recurrence(q, k, v, logd, scale, skip, lens)
     start = np.cumsum([0] + lens)
-    for sizes in ([1000], [2, 63, 65], [64]):
+    for sizes in ([1000], [2, 63, 65], [64], [129, 140]):
         c = cache_of(RecurrentState(heads, n, p), dtype=dtype)
         c.open(len(lens))
         c.arrays(0)["state"].fill_(float("nan"))
@@ -205,13 +205,14 @@ def test_recurrence_ragged_and_in_portions(dtype, scan, heads, groups, n, p):
             assert rel_rms(c.arrays(0)["state"][c._rows[r]], S) < 3e-5, (sizes, r)
 
 
-def test_recurrence_cut_into_segments():
+@pytest.mark.parametrize("n,p", [(32, 40), (128, 64), (96, 136), (200, 64)])
+def test_recurrence_cut_into_segments(n, p):
     """Few heads and a long sequence: segments run side by side and start from the chained states."""
     from trimkv_b200 import _lib, ops
     from trimkv_b200.state_cache import RecurrentState
     rng = np.random.default_rng(5)
-    lens, heads, n, p = [1500, 70, 777], 2, 32, 40
-    assert _lib.lib().tkv_linrec_chunk_workspace_bytes(3, 1500, heads, n, p, 0) > 0
+    lens, heads = [1500, 70, 777], 2
+    assert _lib.lib().tkv_linrec_chunk_workspace_bytes(3, 1500, sum(lens), heads, n, p, 0) > 0
     q, k, v, logd, scale, skip = _recurrence_case(rng, lens, heads, 1, n, p, BF16, far=(1, 1499))
     want, states = _oracle_recurrence(q, k, v, logd, scale, skip, lens)
     c = cache_of(RecurrentState(heads, n, p), dtype=BF16)

@@ -283,8 +283,8 @@ def test_argument_errors_are_reported_without_a_gpu():
     assert lib.tkv_rotate_qk(one, 64, one, None, one, 1, 1, 2, 8, 7, one, 1.0, 0, None) == -1       # odd rotary dims
     assert lib.tkv_conv_silu(one, 4, one, one, one, one, one, one, one, 1, 1, 8, 4, 0, None) == -1
     assert lib.tkv_linrec_scan(one, 8, one, 8, one, 8, None, None, None, None, one, one, one, None, one, 1, 1, 1, 8, 8, 0, None) == -1
-    assert lib.tkv_linrec_chunk_workspace_bytes(1, 64, 2, 12, 8, 0) == -1 and lib.tkv_linrec_chunk_workspace_bytes(1, 64, 2, 16, 8, 2) == -1
-    assert lib.tkv_linrec_chunk_workspace_bytes(4, 64, 64, 64, 64, 0) == 0 and lib.tkv_linrec_chunk_workspace_bytes(1, 4096, 2, 64, 64, 0) > 0
+    assert lib.tkv_linrec_chunk_workspace_bytes(1, 64, 64, 2, 12, 8, 0) == -1 and lib.tkv_linrec_chunk_workspace_bytes(1, 64, 64, 2, 16, 8, 2) == -1
+    assert lib.tkv_linrec_chunk_workspace_bytes(4, 64, 256, 64, 64, 64, 0) == 0 and lib.tkv_linrec_chunk_workspace_bytes(1, 4096, 4096, 2, 64, 64, 0) > 0
     assert lib.tkv_diff_decode_workspace_bytes(2, 4, 2, 300, 192, 64, 0) == 0
     assert lib.tkv_diff_decode(one, one, one, 9, one, one, one, 0.1, 1.0, 1e-6, one, 4, one, None, 0, 1, 4, 3, 8, 8, 64, 64, 0, None) == -1
     assert lib.tkv_diff_decode(one, one, one, 9, one, one, one, 0.1, 1.0, 1e-6, one, 4, one, None, 0, 1, 4, 2, 8, 8, 64, 64, 0, None) == -1

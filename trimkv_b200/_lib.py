@@ -63,8 +63,8 @@ SIGNATURES = {
     "tkv_retention_step": (I, [P, L, P, P, P, P, P, P, I, I, I, I, I, F, F, I, P]),
     "tkv_ssd_step": (I, [P, L, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P]),
     "tkv_linrec_scan": (I, [P, L, P, L, P, L, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, P]),
-    "tkv_linrec_chunk_workspace_bytes": (L, [I, I, I, I, I, I]),
-    "tkv_linrec_chunk": (I, [P, L, P, L, P, L, P, P, P, P, P, P, P, P, P, P, L, I, I, I, I, I, I, I, P]),
+    "tkv_linrec_chunk_workspace_bytes": (L, [I, I, I, I, I, I, I]),
+    "tkv_linrec_chunk": (I, [P, L, P, L, P, L, P, P, P, P, P, P, P, P, P, P, L, I, I, I, I, I, I, I, I, P, P]),
     "tkv_diff_prep": (I, [P, L, P, P, F, P, P, P, I, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, P]),
     "tkv_diff_decode_workspace_bytes": (L, [I, I, I, I, I, I, I]),
     "tkv_diff_decode": (I, [P, P, P, I, P, P, P, F, F, F, P, L, P, P, L, I, I, I, I, I, I, I, I, P]),

@@ -338,6 +338,20 @@ int make_map_2d(CUtensorMap* map, const void* base, int64_t cols, int64_t rows, 
   return TKV_OK;
 }
 
+int make_map_3d_bf16(CUtensorMap* map, const void* base, int64_t inner, int64_t mid, int64_t outer, int64_t outer_stride, int box_inner,
+                     int box_outer) {
+  EncodeTiledFn fn = encode_fn();
+  if (fn == nullptr) return fail(TKV_ERR_LAUNCH, "cuTensorMapEncodeTiled is not available");
+  const cuuint64_t dims[3] = {(cuuint64_t)inner, (cuuint64_t)mid, (cuuint64_t)outer};
+  const cuuint64_t strides[2] = {(cuuint64_t)inner * 2, (cuuint64_t)outer_stride * 2};
+  const cuuint32_t box[3] = {(cuuint32_t)box_inner, 1, (cuuint32_t)box_outer};
+  const cuuint32_t estr[3] = {1, 1, 1};
+  CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                  CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (r != CUDA_SUCCESS) return fail(TKV_ERR_LAUNCH, "cuTensorMapEncodeTiled failed with %d", (int)r);
+  return TKV_OK;
+}
+
 int attn_tc_chunk_tokens() { return kTcChunk; }
 
 template <int kDtype, int kG, bool kMulti = false>

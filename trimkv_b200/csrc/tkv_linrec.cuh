@@ -21,4 +21,18 @@ struct LinrecParams {
   int batch, heads, groups, n, p;
 };
 
+// A long sequence cut into segments that run side by side: a first pass computes every segment's own state, a small kernel
+// chains them, the main pass starts each segment from its true state.
+struct LinrecSegs {
+  int count, tokens;                                      // segments per request, tokens per segment
+  float* start;                                           // [batch, heads, count, n, p]
+  float* log_sum;                                         // [batch, heads, count], log2
+};
+
+int launch_linrec_chain(const LinrecParams& a, const LinrecSegs& sg, cudaStream_t st);
+// The tcgen05 form (tkv_linrec_tc.cu): shapes it takes, and its segments.
+bool linrec_tc_shape(int n, int p, int max_tokens, int64_t tokens);
+LinrecSegs linrec_tc_segments(int batch, int max_tokens, int heads, int p);
+int launch_linrec_tc(const LinrecParams& a, const LinrecSegs& sg, int64_t tokens, int32_t* status, cudaStream_t st);
+
 }  // namespace tkv

@@ -46,12 +46,6 @@ __device__ __forceinline__ void lc_split(float a, float b, uint32_t* hi, uint32_
   *lo = *reinterpret_cast<const uint32_t*>(&l);
 }
 
-struct LinrecSegs {
-  int count, chunks;                                      // segments per request, chunks per segment
-  float* start;                                           // [batch, heads, count, n, p]
-  float* log_sum;                                         // [batch, heads, count], log2
-};
-
 template <int NP, int kWarps> struct LcSmem {
   static constexpr int PT = kWarps * 16, QS = NP + 8, VS = PT + 8, PS = kCk + 8;
   __nv_bfloat16 q[2][kCk * QS], k[2][kCk * QS], v[2][kCk * VS];
@@ -74,7 +68,7 @@ __global__ void __launch_bounds__(kWarps * 32) linrec_chunk_kernel(LinrecParams 
   const int pt = item % ptiles, bh = item / ptiles, b = bh / a.heads, h = bh - b * a.heads, g = h / (a.heads / a.groups);
   const int tok0 = a.cu[b], ntok = a.cu[b + 1] - tok0;
   const int nchunks_all = (ntok + kCk - 1) / kCk;
-  const int c0 = seg * sg.chunks, c1 = min(nchunks_all, c0 + sg.chunks);
+  const int per = sg.tokens / kCk, c0 = seg * per, c1 = min(nchunks_all, c0 + per);
   if (c0 >= c1) return;
   if (kStateOnly && c1 == nchunks_all) return;            // nobody starts from the end of the last segment
   const int pbase = pt * PT, p0 = warp * 16;              // this CTA's columns, this warp's columns within them
@@ -303,7 +297,7 @@ __global__ void __launch_bounds__(256) linrec_chain_kernel(LinrecParams a, Linre
   const int bh = blockIdx.y, b = bh / a.heads, h = bh - b * a.heads;
   const int64_t np = (int64_t)a.n * a.p, i = (int64_t)blockIdx.x * 256 + threadIdx.x;
   if (i >= np) return;
-  const int nchunks = (a.cu[b + 1] - a.cu[b] + kCk - 1) / kCk, used = (nchunks + sg.chunks - 1) / sg.chunks;
+  const int used = (a.cu[b + 1] - a.cu[b] + sg.tokens - 1) / sg.tokens;
   float run = a.pos0[b] == 0 ? 0.f : a.state[((int64_t)a.slots[b] * a.heads + h) * np + i];
   float* at = sg.start + (int64_t)bh * sg.count * np + i;
   for (int k = 0; k < used; ++k) {
@@ -325,9 +319,16 @@ static LinrecSegs plan_segments(int batch, int max_tokens, int heads, int n, int
     if (segs > chunks / 4) segs = chunks / 4;
   }
   LinrecSegs s = {};
-  s.chunks = (chunks + segs - 1) / segs;
-  s.count = s.chunks > 0 ? (chunks + s.chunks - 1) / s.chunks : 1;
+  const int per = segs > 0 ? (chunks + segs - 1) / segs : 1;
+  s.tokens = per * kCk;
+  s.count = per > 0 ? (chunks + per - 1) / per : 1;
   return s;
+}
+
+int launch_linrec_chain(const LinrecParams& a, const LinrecSegs& sg, cudaStream_t st) {
+  cudaError_t e = launch_pdl(linrec_chain_kernel, dim3((unsigned)(((int64_t)a.n * a.p + 255) / 256), a.batch * a.heads), dim3(256), 0, st, a, sg);
+  if (e != cudaSuccess) return fail(TKV_ERR_LAUNCH, "tkv_linrec_chunk: %s", cudaGetErrorString(e));
+  return TKV_OK;
 }
 
 template <int NP, int kWarps>
@@ -345,8 +346,10 @@ static int launch_chunk(const LinrecParams& a, const LinrecSegs& sg, cudaStream_
   cudaError_t e = cudaSuccess;
   if (sg.count > 1) {
     e = launch_pdl(linrec_chunk_kernel<NP, kWarps, true>, dim3((unsigned)(per_seg * sg.count)), dim3(kWarps * 32), (size_t)kBytes, st, a, sg);
-    if (e == cudaSuccess)
-      e = launch_pdl(linrec_chain_kernel, dim3((unsigned)(((int64_t)a.n * a.p + 255) / 256), a.batch * a.heads), dim3(256), 0, st, a, sg);
+    if (e == cudaSuccess) {
+      int rc = launch_linrec_chain(a, sg, st);
+      if (rc != TKV_OK) return rc;
+    }
   }
   if (e == cudaSuccess)
     e = launch_pdl(linrec_chunk_kernel<NP, kWarps, false>, dim3((unsigned)(per_seg * sg.count)), dim3(kWarps * 32), (size_t)kBytes, st, a, sg);
@@ -358,20 +361,26 @@ static int launch_chunk(const LinrecParams& a, const LinrecSegs& sg, cudaStream_
 
 using namespace tkv;
 
-extern "C" int64_t tkv_linrec_chunk_workspace_bytes(int batch, int max_tokens, int heads, int n, int vdim, int dtype) {
+namespace tkv {
+static LinrecSegs plan(int batch, int max_tokens, int64_t tokens, int heads, int n, int vdim) {
+  return linrec_tc_shape(n, vdim, max_tokens, tokens) ? linrec_tc_segments(batch, max_tokens, heads, vdim) : plan_segments(batch, max_tokens, heads, n, vdim);
+}
+}  // namespace tkv
+
+extern "C" int64_t tkv_linrec_chunk_workspace_bytes(int batch, int max_tokens, int tokens, int heads, int n, int vdim, int dtype) {
   if (dtype != TKV_BF16 || !chunk_shape(n, vdim) || batch <= 0 || heads <= 0 || n <= 0 || vdim <= 0 || max_tokens <= 0) return -1;
-  const LinrecSegs s = plan_segments(batch, max_tokens, heads, n, vdim);
+  const LinrecSegs s = plan(batch, max_tokens, tokens, heads, n, vdim);
   return s.count > 1 ? (int64_t)batch * heads * s.count * ((int64_t)n * vdim + 1) * (int64_t)sizeof(float) : 0;
 }
 
 extern "C" int tkv_linrec_chunk(const void* q, int64_t q_stride, const void* k, int64_t k_stride, const void* v, int64_t v_stride,
                                 const float* log_decay, const float* head_log_decay, const float* v_scale, const float* skip,
                                 void* out, float* state, const int32_t* slots, const int32_t* cu_tokens, const int32_t* pos0,
-                                void* workspace, int64_t workspace_bytes, int batch, int max_tokens, int heads, int groups, int n,
-                                int vdim, int dtype, tkv_stream_t stream) {
+                                void* workspace, int64_t workspace_bytes, int batch, int max_tokens, int tokens, int heads,
+                                int groups, int n, int vdim, int dtype, int32_t* status, tkv_stream_t stream) {
   if (!q || !k || !v || (!log_decay && !head_log_decay) || !out || !state || !slots || !cu_tokens || !pos0)
     return fail(TKV_ERR_ARG, "tkv_linrec_chunk: NULL pointer argument");
-  if (batch < 0 || max_tokens < 0 || heads <= 0 || groups <= 0 || heads % groups || n <= 0 || vdim <= 0 ||
+  if (batch < 0 || max_tokens < 0 || tokens < max_tokens || heads <= 0 || groups <= 0 || heads % groups || n <= 0 || vdim <= 0 ||
       q_stride < (int64_t)groups * n || k_stride < (int64_t)groups * n || v_stride < (int64_t)heads * vdim)
     return fail(TKV_ERR_ARG, "tkv_linrec_chunk: bad sizes");
   if (dtype != TKV_BF16 || !chunk_shape(n, vdim))
@@ -380,15 +389,16 @@ extern "C" int tkv_linrec_chunk(const void* q, int64_t q_stride, const void* k, 
     return fail(TKV_ERR_ARG, "tkv_linrec_chunk: rows must start on 16-byte boundaries");
   if (batch == 0 || max_tokens == 0) return TKV_OK;
   if ((int64_t)batch * heads > 65535) return fail(TKV_ERR_UNSUPPORTED, "tkv_linrec_chunk: batch * heads = %lld", (long long)batch * heads);
-  const int64_t need = tkv_linrec_chunk_workspace_bytes(batch, max_tokens, heads, n, vdim, dtype);
+  const int64_t need = tkv_linrec_chunk_workspace_bytes(batch, max_tokens, tokens, heads, n, vdim, dtype);
   if (need > 0 && (!workspace || workspace_bytes < need))
     return fail(TKV_ERR_ARG, "tkv_linrec_chunk: workspace of %lld bytes, %lld needed", (long long)workspace_bytes, (long long)need);
   LinrecParams a = {q, q_stride, k, k_stride, v, v_stride, log_decay, nullptr, head_log_decay, v_scale, skip, out, state, slots,
                     cu_tokens, pos0, batch, heads, groups, n, vdim};
-  LinrecSegs s = plan_segments(batch, max_tokens, heads, n, vdim);
+  LinrecSegs s = plan(batch, max_tokens, tokens, heads, n, vdim);
   s.start = (float*)workspace;
   s.log_sum = s.start + (s.count > 1 ? (int64_t)batch * heads * s.count * n * vdim : 0);
   cudaStream_t st = (cudaStream_t)stream;
+  if (linrec_tc_shape(n, vdim, max_tokens, tokens)) return launch_linrec_tc(a, s, tokens, status, st);
   if (n <= 64) return vdim > 64 ? launch_chunk<64, 8>(a, s, st) : launch_chunk<64, 4>(a, s, st);
   if (n <= 128) return vdim > 64 ? launch_chunk<128, 8>(a, s, st) : launch_chunk<128, 4>(a, s, st);
   return launch_chunk<256, 4>(a, s, st);

@@ -50,6 +50,11 @@ __device__ __forceinline__ void tma_load_2d(void* smem_dst, const CUtensorMap* m
       "cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];"
       ::"r"(smem_u32(smem_dst)), "l"(map), "r"(smem_u32(bar)), "r"(x), "r"(y) : "memory");
 }
+__device__ __forceinline__ void tma_load_3d(void* smem_dst, const CUtensorMap* map, uint64_t* bar, int x, int y, int z) {
+  asm volatile(
+      "cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];"
+      ::"r"(smem_u32(smem_dst)), "l"(map), "r"(smem_u32(bar)), "r"(x), "r"(y), "r"(z) : "memory");
+}
 // 2^x for x <= 0 (softmax weights): the hardware approximation, results below the normal range flushed to zero.
 __device__ __forceinline__ float exp2_weight(float x) {
   float y;
@@ -112,5 +117,9 @@ __device__ __forceinline__ void tmem_ld32(uint32_t taddr, float* v) {
 
 // Encodes a 2-D tiled tensor map over a row-major [rows, cols] matrix of 16-bit elements (128-byte swizzle).
 int make_map_2d(CUtensorMap* map, const void* base, int64_t cols, int64_t rows, int box_cols, int box_rows, int dtype);
+// 3-D map over bf16 [outer][mid][inner] with element strides inner_len between mids and outer_stride between outers; the box
+// is one mid wide, so columns beyond inner_len read as zeros instead of the next mid's.
+int make_map_3d_bf16(CUtensorMap* map, const void* base, int64_t inner, int64_t mid, int64_t outer, int64_t outer_stride, int box_inner,
+                     int box_outer);
 
 }  // namespace tkv

@@ -510,14 +510,15 @@ def linrec(q, k, v, state, batch, out, groups: int, log_decay=None, head_decay=N
     heads, n, p = state.shape[1:]
     dt = dtype_code(out.dtype)
     es = out.element_size()
-    need = lib().tkv_linrec_chunk_workspace_bytes(batch.size, batch.max_tokens, heads, n, p, dt)
+    need = lib().tkv_linrec_chunk_workspace_bytes(batch.size, batch.max_tokens, batch.tokens, heads, n, p, dt)
     rows_ok = all((t.stride(0) * es) % 16 == 0 and t.data_ptr() % 16 == 0 for t in (q, k, v, out))
     if need >= 0 and rows_ok and batch.cu is not None and not force_scan and batch.size * heads <= 65535:
         ws = torch.empty(need, dtype=torch.uint8, device=out.device) if need else None
         check(lib().tkv_linrec_chunk(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0),
                                      _ptr(log_decay), _ptr(head_log_decay), _ptr(v_scale), _ptr(skip), out.data_ptr(),
                                      state.data_ptr(), batch.slots.data_ptr(), batch.cu.data_ptr(), batch.pos0.data_ptr(), _ptr(ws),
-                                     need, batch.size, batch.max_tokens, heads, groups, n, p, dt, _stream(out)), "tkv_linrec_chunk")
+                                     need, batch.size, batch.max_tokens, batch.tokens, heads, groups, n, p, dt, _ptr(batch.status),
+                                     _stream(out)), "tkv_linrec_chunk")
         _count(3 if need else 1)
         return
     check(lib().tkv_linrec_scan(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), _ptr(log_decay),
