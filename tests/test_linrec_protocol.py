@@ -25,8 +25,8 @@ class Sim:
     def __init__(self, nchunks, state_only, partial, rng):
         self.n, self.so, self.partial, self.rng = nchunks, state_only, partial, rng
         two = 2
-        self.bar = {k: Bar(1) for k in ("qk", "v0", "v1", "l0", "l1", "s0", "s1", "o1", "st", "o2")}
-        self.bar.update({k: Bar(two) for k in ("sfree0", "sfree1", "sp", "wv", "p", "e", "clr")})
+        self.bar = {k: Bar(1) for k in ("qk0", "qk1", "v0", "v1", "l0", "l1", "s", "o1", "st", "o2")}
+        self.bar.update({k: Bar(two) for k in ("sfree", "sp", "wv", "p", "e", "clr")})
         self.buf = {}                                               # resource -> chunk it holds
         self.busy = {}                                              # resource -> products reading it
         self.queues = {"main": [], "o2": [], "tma": []}
@@ -69,31 +69,35 @@ class Sim:
         self.bar[bar].arrive()
 
     # ---- roles
+    def load_qk(self, i):
+        self.copy([f"K{i & 1}"] if self.so else [f"Q{i & 1}", f"K{i & 1}"], i, f"qk{i & 1}")
+
     def main(self):
-        qk = ["K"] if self.so else ["Q", "K"]
-        self.copy(qk, 0, "qk")
+        self.load_qk(0)
+        if self.n > 1:
+            self.load_qk(1)
         for i in range(self.n):
-            yield from self.wait("qk", i)
+            yield from self.wait(f"qk{i & 1}", i >> 1)
             if i == self.n - 1 and self.partial:
                 yield from self.wait("clr", 0)
-            if not self.so and i >= 2:
-                yield from self.wait(f"sfree{i & 1}", (i - 2) >> 1)
             if not self.so:
-                self.product("main", ["Q", "K"], f"S{i & 1}", i, f"s{i & 1}")
+                if i > 0:
+                    yield from self.wait("sfree", i - 1)
+                self.product("main", [f"Q{i & 1}", f"K{i & 1}"], "S", i, "s")
+                yield
+            if i > 0 and i + 1 < self.n:
+                yield from self.wait("st", i - 1)
+                if not self.so:
+                    yield from self.wait("o1", i - 1)
+                self.load_qk(i + 1)
                 yield
             yield from self.wait("sp", i)
             if not self.so:
-                self.product("main", ["Q", "SP"], f"O1{i & 1}", i, "o1")
+                self.product("main", [f"Q{i & 1}", "SP"], f"O1{i & 1}", i, "o1")
                 yield
             yield from self.wait("wv", i)
-            self.product("main", ["K", "WV"], "ST", i, "st")
+            self.product("main", [f"K{i & 1}", "WV"], "ST", i, "st")
             yield
-            if i + 1 < self.n:
-                yield from self.wait("st", i)
-                if not self.so:
-                    yield from self.wait("o1", i)
-                self.copy(qk, i + 1, "qk")
-                yield
 
     def copy_v(self):
         self.copy(["V0"], 0, "v0")
@@ -126,16 +130,17 @@ class Sim:
             return
         for i in range(self.n):
             yield from self.wait(f"l{i & 1}", i >> 1)
-            yield from self.wait(f"s{i & 1}", i >> 1)
+            yield from self.wait("s", i)
             if i > 0:
                 yield from self.wait("o2", i - 1)
-            for _ in range(2):
-                self.read(f"S{i & 1}", i)
+            for c2 in range(2):
+                self.read("S", i)
+                if c2 == 1:
+                    self.bar["sfree"].arrive()
+                    yield
                 self.read(f"L{i & 1}", i)
                 self.write("P", i)
                 yield
-            self.bar[f"sfree{i & 1}"].arrive()
-            yield
             self.bar["p"].arrive()
             yield
 
@@ -146,9 +151,9 @@ class Sim:
             if not self.so:
                 yield from self.wait("o1", i - 1)
         if i == self.n - 1 and self.partial:
-            yield from self.wait("qk", i)
+            yield from self.wait(f"qk{i & 1}", i >> 1)
             yield from self.wait(f"v{i & 1}", i >> 1)
-            self.write("K", i)
+            self.write(f"K{i & 1}", i)
             self.write(f"V{i & 1}", i)
             yield
             self.bar["clr"].arrive()

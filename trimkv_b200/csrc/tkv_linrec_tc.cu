@@ -4,7 +4,8 @@
 // One CTA walks the chunks of one (request, head, 64 columns of v, segment).  Per chunk, D in TMEM:
 //   S  [128 tok x 128 tok] = Q . K^T                     A = Q, B = K as TMA wrote them (K-major)
 //   O1 [128 tok x 64]      = Q . S_prev                  B = the state before the chunk, high and low bf16 part (MN-major)
-//   O2 [128 tok x 64]      = P . V                       A = P, the weighted scores, high and low part; B = V (MN-major)
+//   O2 [128 tok x 64]      = P . V                       A = P, the weighted scores, high and low part, read from TMEM;
+//                                                        B = V (MN-major)
 //   ST [128 n x 64]        = e^{L_end} ST + K^T . (w V)  A = K read MN-major, B = weighted values, high and low part
 // The state stays in TMEM as the accumulator of its own update; once per chunk its rows pass through registers to be scaled
 // and to be written as the operand of O1.  fp32 factors of a product enter as two bf16 parts, so nothing that recurs is
@@ -15,8 +16,8 @@
 //   warps 8-15  pass the state through registers, weight the values, and write the output; they run the state side one
 //               chunk ahead of the output side, so the chain ST -> operand -> ST never waits for scores;
 //   warp 16     copies of Q and K, products S, O1, ST;   warp 17  running log decays;   warp 18  copies of V, product O2.
-// S and O1 have two TMEM buffers, V two stages; Q and K are refetched (from L2, where a prefetch has put them) as soon as the
-// products that read them have completed.  A barrier is waited for in every phase by each of its waiters, or its next phase
+// O1 has two TMEM buffers; Q and K, and V, have two stages.  With M = 128 rows and N = 64 columns a product reads more operand
+// bytes than shared memory delivers in the time of its multiplications, which is why P goes through TMEM.  A barrier is waited for in every phase by each of its waiters, or its next phase
 // depends on the waiter, so that a parity never stands for two phases.  Every wait is bounded; on expiry the CTA records
 // TKV_DEV_TIMEOUT, drains its copies, frees its TMEM and returns.
 #include <cuda.h>
@@ -28,11 +29,11 @@ namespace tkv {
 constexpr int kLtC = 128, kLtP = 64;                       // tokens per chunk, value columns per CTA
 constexpr int kLtRows = 256, kLtThreads = 2 * kLtRows + 96;   // threads of one row role; all
 constexpr int kLtHalf = 16384;                             // 128 rows x 64 bf16
-constexpr int kLtS = 0, kLtO1 = 256, kLtO2 = 384, kLtST = 448, kLtCols = 512;   // S and O1: two buffers
+constexpr int kLtS = 0, kLtPm = 128, kLtO1 = 256, kLtO2 = 384, kLtST = 448, kLtCols = 512;   // P: high | low; O1: two buffers
 
 struct LtSmem {
   float2 lv[2][kLtC];                                      // running log2 decay and value scale; by chunk parity
-  uint64_t bar_qk, bar_v[2], bar_l[2], bar_s[2], bar_sfree[2], bar_sp, bar_o1, bar_wv, bar_st, bar_p, bar_o2, bar_e, bar_clr;
+  uint64_t bar_qk[2], bar_v[2], bar_l[2], bar_s, bar_sfree, bar_sp, bar_o1, bar_wv, bar_st, bar_p, bar_o2, bar_e, bar_clr;
   uint32_t tmem_base;
   int abort_flag;
 };
@@ -83,8 +84,20 @@ __device__ __forceinline__ void lt_split(float a, float b, uint32_t* hi, uint32_
   *lo = *reinterpret_cast<const uint32_t*>(&l);
 }
 
-__device__ __forceinline__ void lt_prefetch_3d(const CUtensorMap* map, int x, int y, int z) {
-  asm volatile("cp.async.bulk.prefetch.tensor.3d.L2.global [%0, {%1, %2, %3}];" ::"l"(map), "r"(x), "r"(y), "r"(z) : "memory");
+__device__ __forceinline__ void lt_st16(uint32_t taddr, const uint32_t* v) {   // without waiting
+  asm volatile(
+      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};"
+      ::"r"(taddr), "r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]), "r"(v[4]), "r"(v[5]), "r"(v[6]), "r"(v[7]), "r"(v[8]), "r"(v[9]),
+        "r"(v[10]), "r"(v[11]), "r"(v[12]), "r"(v[13]), "r"(v[14]), "r"(v[15])
+      : "memory");
+}
+// D += A . B with A in TMEM: lane = row, one 32-bit column holds two consecutive elements of a row.
+__device__ __forceinline__ void lt_umma_ts(uint32_t d_tmem, uint32_t a_tmem, uint64_t b_desc, uint32_t idesc, uint32_t accum) {
+  asm volatile(
+      "{\n\t.reg .pred p;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, {%5, %5, %5, %5}, p;\n\t}"
+      ::"r"(d_tmem), "r"(a_tmem), "l"(b_desc), "r"(idesc), "r"(accum), "r"(0u) : "memory");
 }
 
 template <bool kStateOnly>
@@ -110,46 +123,36 @@ linrec_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constan
   const int last_rows = t_end - t_first - (nchunks - 1) * kLtC;    // live tokens of the last chunk
   const int pbase = pt * kLtP;
 
-  uint8_t* q_s = base;                                     // two 64-column halves
-  uint8_t* k_s = q_s + 2 * kLtHalf;
-  uint8_t* v_s = k_s + 2 * kLtHalf;                        // two stages
+  uint8_t* q_s = base;                                     // two stages of two 64-column halves
+  uint8_t* k_s = q_s + 4 * kLtHalf;
+  uint8_t* v_s = k_s + 4 * kLtHalf;                        // two stages
   uint8_t* wv_s = v_s + 2 * kLtHalf;                       // high, low
   uint8_t* sp_s = wv_s + 2 * kLtHalf;                      // high, low
-  uint8_t* p_s = sp_s + 2 * kLtHalf;                       // high (two halves), low (two halves)
-  LtSmem* sm = reinterpret_cast<LtSmem*>(p_s + 4 * kLtHalf);
+  LtSmem* sm = reinterpret_cast<LtSmem*>(sp_s + 2 * kLtHalf);
   volatile int* abort_flag = &sm->abort_flag;
 
   int issued = 0;                                          // of this thread's copies (a copy thread)
   const int row_first = tok0 + t_first;
   auto load_qk = [&](int i) {
-    mbar_expect_tx(&sm->bar_qk, (kStateOnly ? 2 : 4) * kLtHalf);
-    const int row = row_first + i * kLtC;
+    uint64_t* bar = &sm->bar_qk[i & 1];
+    mbar_expect_tx(bar, (kStateOnly ? 2 : 4) * kLtHalf);
 #pragma unroll
     for (int hh = 0; hh < 2; ++hh) {
-      if (!kStateOnly) tma_load_3d(q_s + hh * kLtHalf, &map_q, &sm->bar_qk, hh * 64, g, row);
-      tma_load_3d(k_s + hh * kLtHalf, &map_k, &sm->bar_qk, hh * 64, g, row);
-    }
-    if (i + 1 < nchunks) {
-#pragma unroll
-      for (int hh = 0; hh < 2; ++hh) {
-        if (!kStateOnly) lt_prefetch_3d(&map_q, hh * 64, g, row + kLtC);
-        lt_prefetch_3d(&map_k, hh * 64, g, row + kLtC);
-      }
+      const int at = (2 * (i & 1) + hh) * kLtHalf;
+      if (!kStateOnly) tma_load_3d(q_s + at, &map_q, bar, hh * 64, g, row_first + i * kLtC);
+      tma_load_3d(k_s + at, &map_k, bar, hh * 64, g, row_first + i * kLtC);
     }
     ++issued;
   };
   auto load_v = [&](int i) {
     mbar_expect_tx(&sm->bar_v[i & 1], kLtHalf);
     tma_load_3d(v_s + (i & 1) * kLtHalf, &map_v, &sm->bar_v[i & 1], pbase, h, row_first + i * kLtC);
-    if (i + 1 < nchunks) lt_prefetch_3d(&map_v, pbase, h, row_first + (i + 1) * kLtC);
     ++issued;
   };
   constexpr int kCopyQK = 2 * kLtRows, kCopyV = 2 * kLtRows + 64;   // the two copy threads
   if (tid == kCopyQK) {
-    mbar_init(&sm->bar_qk, 1);
-    for (int i = 0; i < 2; ++i) {
-      mbar_init(&sm->bar_v[i], 1); mbar_init(&sm->bar_l[i], 32); mbar_init(&sm->bar_s[i], 1); mbar_init(&sm->bar_sfree[i], kLtRows);
-    }
+    for (int i = 0; i < 2; ++i) { mbar_init(&sm->bar_qk[i], 1); mbar_init(&sm->bar_v[i], 1); mbar_init(&sm->bar_l[i], 32); }
+    mbar_init(&sm->bar_s, 1); mbar_init(&sm->bar_sfree, kLtRows);
     mbar_init(&sm->bar_o1, 1); mbar_init(&sm->bar_st, 1); mbar_init(&sm->bar_o2, 1);
     mbar_init(&sm->bar_sp, kLtRows); mbar_init(&sm->bar_wv, kLtRows); mbar_init(&sm->bar_p, kLtRows); mbar_init(&sm->bar_e, kLtRows);
     mbar_init(&sm->bar_clr, kLtRows);
@@ -182,19 +185,27 @@ linrec_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constan
     // ------------------------------------------------------------------------------------ Q, K; S, O1, ST (one lane)
     if (lane == 0) {
       const uint32_t id_s = lt_idesc(128, 0, 0), id_o = lt_idesc(kLtP, 0, 1), id_st = lt_idesc(kLtP, 1, 1);
-      const uint32_t qa = smem_u32(q_s), ka = smem_u32(k_s), sp = smem_u32(sp_s), wv = smem_u32(wv_s);
+      const uint32_t sp = smem_u32(sp_s), wv = smem_u32(wv_s);
       load_qk(0);
+      if (nchunks > 1) load_qk(1);
       for (int i = 0; i < nchunks; ++i) {
         const int ph = i & 1;
-        alive = mbar_wait_or_abort(&sm->bar_qk, ph, abort_flag);
+        const uint32_t qa = smem_u32(q_s + 2 * ph * kLtHalf), ka = smem_u32(k_s + 2 * ph * kLtHalf);
+        alive = mbar_wait_or_abort(&sm->bar_qk[ph], (i >> 1) & 1, abort_flag);
         if (alive && i == nchunks - 1 && last_rows < kLtC) alive = mbar_wait_or_abort(&sm->bar_clr, 0, abort_flag);
-        if (alive && !kStateOnly && i >= 2) alive = mbar_wait_or_abort(&sm->bar_sfree[ph], ((i - 2) >> 1) & 1, abort_flag);
+        if (alive && !kStateOnly && i > 0) alive = mbar_wait_or_abort(&sm->bar_sfree, (i - 1) & 1, abort_flag);
         if (!alive) break;
         tc_fence_after();
         if (!kStateOnly) {
 #pragma unroll
-          for (int k = 0; k < 8; ++k) umma(tmem + kLtS + 128 * ph, kmaj(qa, k), kmaj(ka, k), id_s, k > 0);
-          umma_commit(&sm->bar_s[ph]);
+          for (int k = 0; k < 8; ++k) umma(tmem + kLtS, kmaj(qa, k), kmaj(ka, k), id_s, k > 0);
+          umma_commit(&sm->bar_s);
+        }
+        if (i > 0 && i + 1 < nchunks) {                    // the other stage is free once the products of chunk i - 1 have completed
+          alive = mbar_wait_or_abort(&sm->bar_st, (i - 1) & 1, abort_flag);
+          if (alive && !kStateOnly) alive = mbar_wait_or_abort(&sm->bar_o1, (i - 1) & 1, abort_flag);
+          if (!alive) break;
+          load_qk(i + 1);
         }
         alive = mbar_wait_or_abort(&sm->bar_sp, ph, abort_flag);   // the state is scaled and its operand written; O1 of i - 2 is read
         if (!alive) break;
@@ -214,19 +225,13 @@ linrec_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constan
 #pragma unroll
           for (int k = 0; k < 8; ++k) umma(tmem + kLtST, mnmaj(ka, k), mnmaj(wv + part * kLtHalf, k), id_st, 1);
         umma_commit(&sm->bar_st);
-        if (i + 1 < nchunks) {                             // Q and K are free once their products (S among them) have completed
-          alive = mbar_wait_or_abort(&sm->bar_st, ph, abort_flag);
-          if (alive && !kStateOnly) alive = mbar_wait_or_abort(&sm->bar_o1, ph, abort_flag);
-          if (!alive) break;
-          load_qk(i + 1);
-        }
       }
     }
     __syncwarp();
   } else if (warp == 18) {
     // ------------------------------------------------------------------------------------ V; O2 (one lane)
     if (lane == 0) {
-      const uint32_t id_o = lt_idesc(kLtP, 0, 1), pa = smem_u32(p_s);
+      const uint32_t id_o = lt_idesc(kLtP, 0, 1);
       load_v(0);
       if (nchunks > 1) load_v(1);
       for (int i = 0; i < nchunks; ++i) {
@@ -245,7 +250,7 @@ linrec_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constan
 #pragma unroll
         for (int part = 0; part < 2; ++part)
 #pragma unroll
-          for (int k = 0; k < 8; ++k) umma(tmem + kLtO2, kmaj(pa + part * 2 * kLtHalf, k), mnmaj(va, k), id_o, part > 0 || k > 0);
+          for (int k = 0; k < 8; ++k) lt_umma_ts(tmem + kLtO2, tmem + kLtPm + part * 64 + k * 8, mnmaj(va, k), id_o, part > 0 || k > 0);
         umma_commit(&sm->bar_o2);
       }
     }
@@ -288,11 +293,9 @@ linrec_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constan
     // ------------------------------------------------------------------------------------ scores -> P: 64 columns of a row
     if (!kStateOnly) {
       const int j0 = half * 64, r0 = row & ~31;            // rows r0 .. r0 + 31 of this warp
-      uint8_t* p_hi = p_s + half * kLtHalf;
-      uint8_t* p_lo = p_hi + 2 * kLtHalf;
       for (int i = 0; i < nchunks; ++i) {
         const float2* lv = sm->lv[i & 1];
-        alive = sync_on(&sm->bar_l[i & 1], i >> 1) && sync_on(&sm->bar_s[i & 1], i >> 1);
+        alive = sync_on(&sm->bar_l[i & 1], i >> 1) && sync_on(&sm->bar_s, i);
         if (alive && i > 0) alive = sync_on(&sm->bar_o2, i - 1);   // P of the previous chunk has been read
         if (!alive) break;
         tc_fence_after();
@@ -300,37 +303,34 @@ linrec_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constan
 #pragma unroll
         for (int c2 = 0; c2 < 2; ++c2) {
           const int jb = j0 + c2 * 32;
-          if (jb > r0 + 31) {                              // all of it in the future (warp-uniform)
-#pragma unroll
-            for (int c = 0; c < 4; ++c) {
-              const uint32_t at = lt_swz(row, c2 * 4 + c);
-              st16(p_hi + at, make_uint4(0, 0, 0, 0));
-              st16(p_lo + at, make_uint4(0, 0, 0, 0));
-            }
-            continue;
+          const bool future = jb > r0 + 31;                // all of it (warp-uniform)
+          uint32_t sv[32], hi[16], lo[16];
+          if (!future) {
+            lt_ld32_nowait(lanes + kLtS + jb, sv);
+            lt_wait_ld();
           }
-          uint32_t sv[32];
-          lt_ld32_nowait(lanes + kLtS + 128 * (i & 1) + jb, sv);
-          lt_wait_ld();
+          if (c2 == 1) {
+            tc_fence_before();
+            lt_arrive(&sm->bar_sfree);
+          }
+          if (future) {
 #pragma unroll
-          for (int c = 0; c < 4; ++c) {
-            uint32_t hi[4], lo[4];
+            for (int e = 0; e < 16; ++e) hi[e] = lo[e] = 0;
+          } else {
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-              const int j = jb + c * 8 + 2 * e;
+            for (int e = 0; e < 16; ++e) {
+              const int j = jb + 2 * e;
               const float4 w = *reinterpret_cast<const float4*>(&lv[j]);   // two tokens: log decay, scale
-              const float x = j <= row ? __uint_as_float(sv[c * 8 + 2 * e]) * exp2_weight(l_row - w.x) * w.y : 0.f;
-              const float y = j + 1 <= row ? __uint_as_float(sv[c * 8 + 2 * e + 1]) * exp2_weight(l_row - w.z) * w.w : 0.f;
+              const float x = j <= row ? __uint_as_float(sv[2 * e]) * exp2_weight(l_row - w.x) * w.y : 0.f;
+              const float y = j + 1 <= row ? __uint_as_float(sv[2 * e + 1]) * exp2_weight(l_row - w.z) * w.w : 0.f;
               lt_split(x, y, &hi[e], &lo[e]);
             }
-            const uint32_t at = lt_swz(row, c2 * 4 + c);
-            st16(p_hi + at, make_uint4(hi[0], hi[1], hi[2], hi[3]));
-            st16(p_lo + at, make_uint4(lo[0], lo[1], lo[2], lo[3]));
           }
+          lt_st16(lanes + kLtPm + jb / 2, hi);
+          lt_st16(lanes + kLtPm + 64 + jb / 2, lo);
         }
-        fence_async_smem();
+        asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
         tc_fence_before();
-        lt_arrive(&sm->bar_sfree[i & 1]);
         lt_arrive(&sm->bar_p);
       }
     }
@@ -360,10 +360,10 @@ linrec_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constan
       if (!kStateOnly && i > 0 && !sync_on(&sm->bar_o1, i - 1)) return false;   // the operand of the previous chunk has been read
       tc_fence_after();
       if (i == nchunks - 1 && last_rows < kLtC) {          // tokens beyond the end belong to another request: they read as zeros
-        if (!sync_on(&sm->bar_qk, i) || !sync_on(&sm->bar_v[i & 1], i >> 1)) return false;
+        if (!sync_on(&sm->bar_qk[i & 1], i >> 1) || !sync_on(&sm->bar_v[i & 1], i >> 1)) return false;
         if (row >= last_rows) {
 #pragma unroll
-          for (int c = 0; c < 8; ++c) st16(k_s + half * kLtHalf + row * 128 + c * 16, make_uint4(0, 0, 0, 0));
+          for (int c = 0; c < 8; ++c) st16(k_s + (2 * (i & 1) + half) * kLtHalf + row * 128 + c * 16, make_uint4(0, 0, 0, 0));
 #pragma unroll
           for (int c = 0; c < 4; ++c) st16(v_t + row * 128 + half * 64 + c * 16, make_uint4(0, 0, 0, 0));
         }
@@ -468,9 +468,8 @@ linrec_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constan
   __syncthreads();
   // An aborting CTA drains the copies it started before its shared memory is released.
   if (*abort_flag != 0) {
-    if (tid == kCopyQK && issued > 0) mbar_wait(&sm->bar_qk, (issued - 1) & 1);
-    if (tid == kCopyV)
-      for (int i = max(0, issued - 2); i < issued; ++i) mbar_wait(&sm->bar_v[i & 1], (i >> 1) & 1);
+    if (tid == kCopyQK || tid == kCopyV)
+      for (int i = max(0, issued - 2); i < issued; ++i) mbar_wait(tid == kCopyQK ? &sm->bar_qk[i & 1] : &sm->bar_v[i & 1], (i >> 1) & 1);
   }
   __syncthreads();
   if (warp == 16) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(kLtCols));
