@@ -25,11 +25,11 @@ class Sim:
     def __init__(self, nchunks, state_only, partial, rng):
         self.n, self.so, self.partial, self.rng = nchunks, state_only, partial, rng
         two = 2
-        self.bar = {k: Bar(1) for k in ("qk0", "qk1", "v0", "v1", "l0", "l1", "s", "o1", "st", "o2")}
-        self.bar.update({k: Bar(two) for k in ("sfree", "sp", "wv", "p", "e", "clr")})
+        self.bar = {k: Bar(1) for k in ("qk", "v0", "v1", "l0", "l1", "s", "o1", "st", "o2")}
+        self.bar.update({k: Bar(two) for k in ("sp", "wv", "p", "clr")})
         self.buf = {}                                               # resource -> chunk it holds
         self.busy = {}                                              # resource -> products reading it
-        self.queues = {"main": [], "o2": [], "tma": []}
+        self.queues = {"main": [], "tma": []}
 
     # ---- primitives
     def wait(self, name, phase):
@@ -70,130 +70,97 @@ class Sim:
 
     # ---- roles
     def load_qk(self, i):
-        self.copy([f"K{i & 1}"] if self.so else [f"Q{i & 1}", f"K{i & 1}"], i, f"qk{i & 1}")
+        self.copy(["K"] if self.so else ["Q", "K"], i, "qk")
 
-    def main(self):
+    def load_v(self, i):
+        self.copy([f"V{i & 1}"], i, f"v{i & 1}")
+
+    def control(self):
         self.load_qk(0)
-        if self.n > 1:
-            self.load_qk(1)
+        self.load_v(0)
         for i in range(self.n):
-            yield from self.wait(f"qk{i & 1}", i >> 1)
+            yield from self.wait("qk", i)
             if i == self.n - 1 and self.partial:
                 yield from self.wait("clr", 0)
             if not self.so:
-                if i > 0:
-                    yield from self.wait("sfree", i - 1)
-                self.product("main", [f"Q{i & 1}", f"K{i & 1}"], "S", i, "s")
-                yield
-            if i > 0 and i + 1 < self.n:
-                yield from self.wait("st", i - 1)
-                if not self.so:
-                    yield from self.wait("o1", i - 1)
-                self.load_qk(i + 1)
+                self.product("main", ["Q", "K"], "S", i, "s")
                 yield
             yield from self.wait("sp", i)
+            if i + 1 < self.n:
+                self.load_v(i + 1)
             if not self.so:
-                self.product("main", [f"Q{i & 1}", "SP"], f"O1{i & 1}", i, "o1")
+                self.product("main", ["Q", "SP"], "O1", i, "o1")
                 yield
             yield from self.wait("wv", i)
-            self.product("main", [f"K{i & 1}", "WV"], "ST", i, "st")
+            self.product("main", ["K", "WV"], "ST", i, "st")
             yield
-
-    def copy_v(self):
-        self.copy(["V0"], 0, "v0")
-        if self.n > 1:
-            self.copy(["V1"], 1, "v1")
-        for i in range(self.n):
-            if i > 0 and (not self.so or i + 1 < self.n):
-                yield from self.wait("e", i - 1)
-                if i + 1 < self.n:
-                    self.copy([f"V{(i + 1) & 1}"], i + 1, f"v{(i + 1) & 1}")
+            if i + 1 < self.n:
+                yield from self.wait("st", i)
+                if not self.so:
+                    yield from self.wait("o1", i)
+                self.load_qk(i + 1)
                 yield
-            if self.so:
-                continue
-            yield from self.wait("p", i)
-            yield from self.wait(f"v{i & 1}", i >> 1)
-            self.product("o2", ["P", f"V{i & 1}"], "O2", i, "o2")
-            yield
+            if not self.so:
+                yield from self.wait("p", i)
+                self.product("main", ["P", f"V{i & 1}"], "O2", i, "o2")
+                yield
 
     def scan(self):
         for i in range(self.n):
-            if i >= 2:
-                yield from self.wait("e", i - 2)
+            if i >= 1:
+                yield from self.wait("sp", i - 1)
             self.write(f"L{i & 1}", i)
             yield
             self.bar[f"l{i & 1}"].arrive()
             yield
 
-    def scores(self, me):
-        if self.so:
-            return
+    def rows(self):
         for i in range(self.n):
+            if i == self.n - 1 and self.partial:
+                yield from self.wait("qk", i)
+                yield from self.wait(f"v{i & 1}", i >> 1)
+                self.write("K", i)
+                self.write(f"V{i & 1}", i)
+                yield
+                self.bar["clr"].arrive()
+                yield
             yield from self.wait(f"l{i & 1}", i >> 1)
-            yield from self.wait("s", i)
             if i > 0:
-                yield from self.wait("o2", i - 1)
-            for c2 in range(2):
+                yield from self.wait("st", i - 1)
+                self.read("ST", i - 1)
+            self.read(f"L{i & 1}", i)
+            if not self.so:
+                self.write("SP", i)
+                yield
+            self.bar["sp"].arrive()
+            yield
+            yield from self.wait(f"v{i & 1}", i >> 1)
+            self.read(f"V{i & 1}", i)
+            self.read(f"L{i & 1}", i)
+            self.write("WV", i)
+            yield
+            self.bar["wv"].arrive()
+            yield
+            if self.so:
+                continue
+            yield from self.wait("s", i)
+            for _ in range(2):
                 self.read("S", i)
-                if c2 == 1:
-                    self.bar["sfree"].arrive()
-                    yield
                 self.read(f"L{i & 1}", i)
                 self.write("P", i)
                 yield
             self.bar["p"].arrive()
             yield
-
-    def state_side(self, i):
-        yield from self.wait(f"l{i & 1}", i >> 1)
-        if i > 0:
-            yield from self.wait("st", i - 1)
-            if not self.so:
-                yield from self.wait("o1", i - 1)
-        if i == self.n - 1 and self.partial:
-            yield from self.wait(f"qk{i & 1}", i >> 1)
-            yield from self.wait(f"v{i & 1}", i >> 1)
-            self.write(f"K{i & 1}", i)
-            self.write(f"V{i & 1}", i)
-            yield
-            self.bar["clr"].arrive()
-            yield
-        self.read(f"L{i & 1}", i)
-        if not self.so:
-            self.write("SP", i)
-            yield
-        self.bar["sp"].arrive()
-        yield
-        yield from self.wait(f"v{i & 1}", i >> 1)
-        self.read(f"V{i & 1}", i)
-        self.read(f"L{i & 1}", i)
-        self.write("WV", i)
-        yield
-        self.bar["wv"].arrive()
-        yield
-
-    def rows(self, me):
-        yield from self.state_side(0)
-        for i in range(self.n):
-            if i + 1 < self.n:
-                yield from self.state_side(i + 1)
-            elif not self.so:
-                yield from self.wait("o1", i)
-            if self.so:
-                self.bar["e"].arrive()
-                yield
-                continue
+            yield from self.wait("o1", i)
             yield from self.wait("o2", i)
-            for res in (f"O1{i & 1}", "O2", f"V{i & 1}", f"L{i & 1}"):
+            for res in ("O1", "O2", f"V{i & 1}", f"L{i & 1}"):
                 self.read(res, i)
                 yield
-            self.bar["e"].arrive()
-            yield
         yield from self.wait("st", self.n - 1)
         self.read("ST", self.n - 1)
 
     def run(self):
-        agents = [self.main(), self.copy_v(), self.scan(), self.scores(0), self.scores(1), self.rows(0), self.rows(1)]
+        agents = [self.control(), self.scan(), self.rows(), self.rows()]
         speed = [self.rng.choice([1, 1, 4, 30]) for _ in agents]
         blocked = {}
         while agents:
@@ -224,10 +191,10 @@ def test_hand_offs_hold_under_random_interleavings(nchunks, state_only):
 
 
 def test_the_simulation_notices_a_missing_wait():
-    """With the wait for the operand of the previous read-out taken out of the model, some interleaving overwrites it."""
+    """With the wait for the previous state update taken out of the model, some interleaving overwrites what it reads."""
     class Broken(Sim):
         def wait(self, name, phase):
-            if name == "o1":
+            if name == "st":
                 return
             yield from super().wait(name, phase)
     with pytest.raises(AssertionError):

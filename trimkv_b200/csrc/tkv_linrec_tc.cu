@@ -3,23 +3,18 @@
 //
 // One CTA walks the chunks of one (request, head, 64 columns of v, segment).  Per chunk, D in TMEM:
 //   S  [128 tok x 128 tok] = Q . K^T                     A = Q, B = K as TMA wrote them (K-major)
-//   O1 [128 tok x 64]      = Q . S_prev                  B = the state before the chunk, high and low bf16 part (MN-major)
-//   O2 [128 tok x 64]      = P . V                       A = P, the weighted scores, high and low part, read from TMEM;
-//                                                        B = V (MN-major)
-//   ST [128 n x 64]        = e^{L_end} ST + K^T . (w V)  A = K read MN-major, B = weighted values, high and low part
-// The state stays in TMEM as the accumulator of its own update; once per chunk its rows pass through registers to be scaled
+//   O1 [128 tok x 2 x 64]  = Q . [S_prev high | low]     B = the state before the chunk as two bf16 parts (MN-major)
+//   O2 [128 tok x 64]      = P . V                       A = P, the weighted scores, high and low part; B = V (MN-major)
+//   ST [128 n x 2 x 64]    = e^{L_end} ST + K^T . [w V high | low]   A = K read MN-major, B = weighted values as two parts
+// A product with few columns costs what reading its 128 rows costs, so the two parts of a B operand go side by side into one
+// product of 128 columns and are added when they are read.  The state stays in TMEM as the accumulator of its own update; once per chunk its rows pass through registers to be scaled
 // and to be written as the operand of O1.  fp32 factors of a product enter as two bf16 parts, so nothing that recurs is
 // rounded to 16 bits.
 //
-// Roles.  TMEM lane = token, or state row; a row is shared by two threads, one per column half.
-//   warps 0-7   weight the scores: S -> P;
-//   warps 8-15  pass the state through registers, weight the values, and write the output; they run the state side one
-//               chunk ahead of the output side, so the chain ST -> operand -> ST never waits for scores;
-//   warp 16     copies of Q and K, products S, O1, ST;   warp 17  running log decays;   warp 18  copies of V, product O2.
-// O1 has two TMEM buffers; Q and K, and V, have two stages.  With M = 128 rows and N = 64 columns a product reads more operand
-// bytes than shared memory delivers in the time of its multiplications, which is why P goes through TMEM.  A barrier is waited for in every phase by each of its waiters, or its next phase
-// depends on the waiter, so that a parity never stands for two phases.  Every wait is bounded; on expiry the CTA records
-// TKV_DEV_TIMEOUT, drains its copies, frees its TMEM and returns.
+// Roles: warps 0-7 hold rows (TMEM lane = token, or state row; two threads per row, one per column half); warp 8 issues TMA
+// copies and MMAs (one lane); warp 9 computes the running log decays of the next chunk.  Q and K are refetched as soon as
+// the products that read them have completed, under the weighting of the scores; V has two stages.  Every wait is bounded;
+// on expiry the CTA records TKV_DEV_TIMEOUT, drains its copies, frees its TMEM and returns.
 #include <cuda.h>
 #include "tkv_linrec.cuh"
 #include "tkv_tc.cuh"
@@ -27,13 +22,13 @@
 namespace tkv {
 
 constexpr int kLtC = 128, kLtP = 64;                       // tokens per chunk, value columns per CTA
-constexpr int kLtRows = 256, kLtThreads = 2 * kLtRows + 96;   // threads of one row role; all
+constexpr int kLtRows = 256, kLtThreads = kLtRows + 64;
 constexpr int kLtHalf = 16384;                             // 128 rows x 64 bf16
-constexpr int kLtS = 0, kLtPm = 128, kLtO1 = 256, kLtO2 = 384, kLtST = 448, kLtCols = 512;   // P: high | low; O1: two buffers
+constexpr int kLtS = 0, kLtO1 = 128, kLtO2 = 256, kLtST = 320, kLtCols = 512;   // O1, ST: high | low
 
 struct LtSmem {
   float2 lv[2][kLtC];                                      // running log2 decay and value scale; by chunk parity
-  uint64_t bar_qk[2], bar_v[2], bar_l[2], bar_s, bar_sfree, bar_sp, bar_o1, bar_wv, bar_st, bar_p, bar_o2, bar_e, bar_clr;
+  uint64_t bar_qk, bar_v[2], bar_l[2], bar_s, bar_sp, bar_o1, bar_wv, bar_st, bar_p, bar_o2, bar_clr;
   uint32_t tmem_base;
   int abort_flag;
 };
@@ -84,22 +79,6 @@ __device__ __forceinline__ void lt_split(float a, float b, uint32_t* hi, uint32_
   *lo = *reinterpret_cast<const uint32_t*>(&l);
 }
 
-__device__ __forceinline__ void lt_st16(uint32_t taddr, const uint32_t* v) {   // without waiting
-  asm volatile(
-      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};"
-      ::"r"(taddr), "r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]), "r"(v[4]), "r"(v[5]), "r"(v[6]), "r"(v[7]), "r"(v[8]), "r"(v[9]),
-        "r"(v[10]), "r"(v[11]), "r"(v[12]), "r"(v[13]), "r"(v[14]), "r"(v[15])
-      : "memory");
-}
-// D += A . B with A in TMEM: lane = row, one 32-bit column holds two consecutive elements of a row.
-__device__ __forceinline__ void lt_umma_ts(uint32_t d_tmem, uint32_t a_tmem, uint64_t b_desc, uint32_t idesc, uint32_t accum) {
-  asm volatile(
-      "{\n\t.reg .pred p;\n\t"
-      "setp.ne.b32 p, %4, 0;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, {%5, %5, %5, %5}, p;\n\t}"
-      ::"r"(d_tmem), "r"(a_tmem), "l"(b_desc), "r"(idesc), "r"(accum), "r"(0u) : "memory");
-}
-
 template <bool kStateOnly>
 __global__ void __launch_bounds__(kLtThreads, 1)
 linrec_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
@@ -123,44 +102,43 @@ linrec_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constan
   const int last_rows = t_end - t_first - (nchunks - 1) * kLtC;    // live tokens of the last chunk
   const int pbase = pt * kLtP;
 
-  uint8_t* q_s = base;                                     // two stages of two 64-column halves
-  uint8_t* k_s = q_s + 4 * kLtHalf;
-  uint8_t* v_s = k_s + 4 * kLtHalf;                        // two stages
+  uint8_t* q_s = base;                                     // two 64-column halves
+  uint8_t* k_s = q_s + 2 * kLtHalf;
+  uint8_t* v_s = k_s + 2 * kLtHalf;                        // two stages
   uint8_t* wv_s = v_s + 2 * kLtHalf;                       // high, low
   uint8_t* sp_s = wv_s + 2 * kLtHalf;                      // high, low
-  LtSmem* sm = reinterpret_cast<LtSmem*>(sp_s + 2 * kLtHalf);
+  uint8_t* p_s = sp_s + 2 * kLtHalf;                       // high (two halves), low (two halves)
+  LtSmem* sm = reinterpret_cast<LtSmem*>(p_s + 4 * kLtHalf);
   volatile int* abort_flag = &sm->abort_flag;
 
-  int issued = 0;                                          // of this thread's copies (a copy thread)
-  const int row_first = tok0 + t_first;
+  int qk_issued = 0, v_issued = 0;
   auto load_qk = [&](int i) {
-    uint64_t* bar = &sm->bar_qk[i & 1];
-    mbar_expect_tx(bar, (kStateOnly ? 2 : 4) * kLtHalf);
+    mbar_expect_tx(&sm->bar_qk, (kStateOnly ? 2 : 4) * kLtHalf);
+    const int row = tok0 + t_first + i * kLtC;
 #pragma unroll
     for (int hh = 0; hh < 2; ++hh) {
-      const int at = (2 * (i & 1) + hh) * kLtHalf;
-      if (!kStateOnly) tma_load_3d(q_s + at, &map_q, bar, hh * 64, g, row_first + i * kLtC);
-      tma_load_3d(k_s + at, &map_k, bar, hh * 64, g, row_first + i * kLtC);
+      if (!kStateOnly) tma_load_3d(q_s + hh * kLtHalf, &map_q, &sm->bar_qk, hh * 64, g, row);
+      tma_load_3d(k_s + hh * kLtHalf, &map_k, &sm->bar_qk, hh * 64, g, row);
     }
-    ++issued;
+    ++qk_issued;
   };
   auto load_v = [&](int i) {
     mbar_expect_tx(&sm->bar_v[i & 1], kLtHalf);
-    tma_load_3d(v_s + (i & 1) * kLtHalf, &map_v, &sm->bar_v[i & 1], pbase, h, row_first + i * kLtC);
-    ++issued;
+    tma_load_3d(v_s + (i & 1) * kLtHalf, &map_v, &sm->bar_v[i & 1], pbase, h, tok0 + t_first + i * kLtC);
+    ++v_issued;
   };
-  constexpr int kCopyQK = 2 * kLtRows, kCopyV = 2 * kLtRows + 64;   // the two copy threads
-  if (tid == kCopyQK) {
-    for (int i = 0; i < 2; ++i) { mbar_init(&sm->bar_qk[i], 1); mbar_init(&sm->bar_v[i], 1); mbar_init(&sm->bar_l[i], 32); }
-    mbar_init(&sm->bar_s, 1); mbar_init(&sm->bar_sfree, kLtRows);
-    mbar_init(&sm->bar_o1, 1); mbar_init(&sm->bar_st, 1); mbar_init(&sm->bar_o2, 1);
-    mbar_init(&sm->bar_sp, kLtRows); mbar_init(&sm->bar_wv, kLtRows); mbar_init(&sm->bar_p, kLtRows); mbar_init(&sm->bar_e, kLtRows);
-    mbar_init(&sm->bar_clr, kLtRows);
+  if (tid == kLtRows) {
+    mbar_init(&sm->bar_qk, 1);
+    for (int i = 0; i < 2; ++i) { mbar_init(&sm->bar_v[i], 1); mbar_init(&sm->bar_l[i], 32); }
+    mbar_init(&sm->bar_s, 1); mbar_init(&sm->bar_o1, 1); mbar_init(&sm->bar_st, 1); mbar_init(&sm->bar_o2, 1);
+    mbar_init(&sm->bar_sp, kLtRows); mbar_init(&sm->bar_wv, kLtRows); mbar_init(&sm->bar_p, kLtRows); mbar_init(&sm->bar_clr, kLtRows);
     sm->abort_flag = 0;
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    load_qk(0);
+    load_v(0);
   }
   __syncwarp();
-  if (warp == 16) {
+  if (warp == 8) {
     asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&sm->tmem_base)), "r"(kLtCols));
     asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::);
   }
@@ -170,92 +148,65 @@ linrec_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constan
   const uint32_t tmem = sm->tmem_base;
   const int64_t np = (int64_t)a.n * a.p;
   float* const final_state = a.state + ((int64_t)a.slots[b] * a.heads + h) * np;
-  // operand descriptors: K-major, step k covers 16 columns; MN-major over 128 rows, step k covers 16 rows
-  auto kmaj = [&](uint32_t at, int k) { return make_desc(at + (k >> 2) * kLtHalf + (k & 3) * 32, 16, 1024, 2); };
-  auto mnmaj = [&](uint32_t at, int k) { return make_desc(at + k * 2048, kLtHalf, 1024, 2); };
-  const int row = tid & 127, half = (tid >> 7) & 1;        // of a row thread
-  const uint32_t lanes = tmem + ((uint32_t)((warp & 3) * 32) << 16);
-  auto sync_on = [&](uint64_t* bar, int parity) {          // a whole warp
-    const bool ok = mbar_wait_or_abort(bar, parity & 1, abort_flag);
-    return (bool)__all_sync(0xffffffffu, ok);
-  };
-  bool alive = true;
 
-  if (warp == 16) {
-    // ------------------------------------------------------------------------------------ Q, K; S, O1, ST (one lane)
+  if (warp == 8) {
+    // ------------------------------------------------------------------------------------ TMA + MMA issue (one lane)
     if (lane == 0) {
-      const uint32_t id_s = lt_idesc(128, 0, 0), id_o = lt_idesc(kLtP, 0, 1), id_st = lt_idesc(kLtP, 1, 1);
-      const uint32_t sp = smem_u32(sp_s), wv = smem_u32(wv_s);
-      load_qk(0);
-      if (nchunks > 1) load_qk(1);
-      for (int i = 0; i < nchunks; ++i) {
+      const uint32_t id_s = lt_idesc(128, 0, 0), id_o1 = lt_idesc(2 * kLtP, 0, 1), id_o2 = lt_idesc(kLtP, 0, 1), id_st = lt_idesc(2 * kLtP, 1, 1);
+      const uint32_t qa = smem_u32(q_s), ka = smem_u32(k_s);
+      // K-major operand: step k covers 16 columns; MN-major operand of 128 rows: step k covers 16 rows.
+      auto kmaj = [&](uint32_t at, int k) { return make_desc(at + (k >> 2) * kLtHalf + (k & 3) * 32, 16, 1024, 2); };
+      auto mnmaj = [&](uint32_t at, int k) { return make_desc(at + k * 2048, kLtHalf, 1024, 2); };
+      bool ok = true;
+      for (int i = 0; i < nchunks && ok; ++i) {
         const int ph = i & 1;
-        const uint32_t qa = smem_u32(q_s + 2 * ph * kLtHalf), ka = smem_u32(k_s + 2 * ph * kLtHalf);
-        alive = mbar_wait_or_abort(&sm->bar_qk[ph], (i >> 1) & 1, abort_flag);
-        if (alive && i == nchunks - 1 && last_rows < kLtC) alive = mbar_wait_or_abort(&sm->bar_clr, 0, abort_flag);
-        if (alive && !kStateOnly && i > 0) alive = mbar_wait_or_abort(&sm->bar_sfree, (i - 1) & 1, abort_flag);
-        if (!alive) break;
+        ok = mbar_wait_or_abort(&sm->bar_qk, ph, abort_flag);
+        if (ok && i == nchunks - 1 && last_rows < kLtC) ok = mbar_wait_or_abort(&sm->bar_clr, 0, abort_flag);
+        if (!ok) break;
         tc_fence_after();
         if (!kStateOnly) {
 #pragma unroll
           for (int k = 0; k < 8; ++k) umma(tmem + kLtS, kmaj(qa, k), kmaj(ka, k), id_s, k > 0);
           umma_commit(&sm->bar_s);
         }
-        if (i > 0 && i + 1 < nchunks) {                    // the other stage is free once the products of chunk i - 1 have completed
-          alive = mbar_wait_or_abort(&sm->bar_st, (i - 1) & 1, abort_flag);
-          if (alive && !kStateOnly) alive = mbar_wait_or_abort(&sm->bar_o1, (i - 1) & 1, abort_flag);
-          if (!alive) break;
-          load_qk(i + 1);
-        }
-        alive = mbar_wait_or_abort(&sm->bar_sp, ph, abort_flag);   // the state is scaled and its operand written; O1 of i - 2 is read
-        if (!alive) break;
+        ok = mbar_wait_or_abort(&sm->bar_sp, ph, abort_flag);      // the state is scaled, its operand written, chunk i - 1 finished
+        if (!ok) break;
         tc_fence_after();
+        if (i + 1 < nchunks) load_v(i + 1);
         if (!kStateOnly) {
+          const uint32_t sp = smem_u32(sp_s);
+#pragma unroll
+          for (int k = 0; k < 8; ++k) umma(tmem + kLtO1, kmaj(qa, k), mnmaj(sp, k), id_o1, k > 0);
+          umma_commit(&sm->bar_o1);
+        }
+        ok = mbar_wait_or_abort(&sm->bar_wv, ph, abort_flag);
+        if (!ok) break;
+        tc_fence_after();
+        const uint32_t wv = smem_u32(wv_s);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) umma(tmem + kLtST, mnmaj(ka, k), mnmaj(wv, k), id_st, 1);
+        umma_commit(&sm->bar_st);
+        if (i + 1 < nchunks) {                             // Q and K are free once these products have completed
+          ok = mbar_wait_or_abort(&sm->bar_st, ph, abort_flag);
+          if (ok && !kStateOnly) ok = mbar_wait_or_abort(&sm->bar_o1, ph, abort_flag);
+          if (ok) load_qk(i + 1);
+        }
+        if (!kStateOnly && ok) {
+          ok = mbar_wait_or_abort(&sm->bar_p, ph, abort_flag);
+          if (!ok) break;
+          tc_fence_after();
+          const uint32_t pa = smem_u32(p_s), va = smem_u32(v_s + (i & 1) * kLtHalf);   // V has arrived: wV was made of it
 #pragma unroll
           for (int part = 0; part < 2; ++part)
 #pragma unroll
-            for (int k = 0; k < 8; ++k) umma(tmem + kLtO1 + 64 * ph, kmaj(qa, k), mnmaj(sp + part * kLtHalf, k), id_o, part > 0 || k > 0);
-          umma_commit(&sm->bar_o1);
+            for (int k = 0; k < 8; ++k) umma(tmem + kLtO2, kmaj(pa + part * 2 * kLtHalf, k), mnmaj(va, k), id_o2, part > 0 || k > 0);
+          umma_commit(&sm->bar_o2);
         }
-        alive = mbar_wait_or_abort(&sm->bar_wv, ph, abort_flag);
-        if (!alive) break;
-        tc_fence_after();
-#pragma unroll
-        for (int part = 0; part < 2; ++part)
-#pragma unroll
-          for (int k = 0; k < 8; ++k) umma(tmem + kLtST, mnmaj(ka, k), mnmaj(wv + part * kLtHalf, k), id_st, 1);
-        umma_commit(&sm->bar_st);
       }
+      if (!ok && *abort_flag == 0) { *abort_flag = 1; report(status, TKV_DEV_TIMEOUT); }
     }
     __syncwarp();
-  } else if (warp == 18) {
-    // ------------------------------------------------------------------------------------ V; O2 (one lane)
-    if (lane == 0) {
-      const uint32_t id_o = lt_idesc(kLtP, 0, 1);
-      load_v(0);
-      if (nchunks > 1) load_v(1);
-      for (int i = 0; i < nchunks; ++i) {
-        // Chunk i - 1 is out: its V stage and O2 are free.  (Without outputs the last phases go unwatched: nothing holds them back.)
-        if (i > 0 && (!kStateOnly || i + 1 < nchunks)) {
-          alive = mbar_wait_or_abort(&sm->bar_e, (i - 1) & 1, abort_flag);
-          if (!alive) break;
-          if (i + 1 < nchunks) load_v(i + 1);
-        }
-        if (kStateOnly) continue;
-        alive = mbar_wait_or_abort(&sm->bar_p, i & 1, abort_flag);
-        if (alive) alive = mbar_wait_or_abort(&sm->bar_v[i & 1], (i >> 1) & 1, abort_flag);
-        if (!alive) break;
-        tc_fence_after();
-        const uint32_t va = smem_u32(v_s + (i & 1) * kLtHalf);
-#pragma unroll
-        for (int part = 0; part < 2; ++part)
-#pragma unroll
-          for (int k = 0; k < 8; ++k) lt_umma_ts(tmem + kLtO2, tmem + kLtPm + part * 64 + k * 8, mnmaj(va, k), id_o, part > 0 || k > 0);
-        umma_commit(&sm->bar_o2);
-      }
-    }
-    __syncwarp();
-  } else if (warp == 17) {
+  } else if (warp == 9) {
     // ------------------------------------------------------------------------------------ running log decays, 4 tokens a lane
     float d[4], s[4], seg_log = 0.f;
     auto fetch = [&](int i) {
@@ -269,7 +220,8 @@ linrec_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constan
       }
     };
     fetch(0);
-    for (int i = 0; i < nchunks; ++i) {
+    bool ok = true;
+    for (int i = 0; i < nchunks && ok; ++i) {
       d[1] += d[0]; d[2] += d[1]; d[3] += d[2];
       float sum = d[3];
 #pragma unroll
@@ -278,9 +230,11 @@ linrec_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constan
         if (lane >= o) sum += y;
       }
       const float before = sum - d[3];
-      // The buffer last served chunk i - 2 (chunk i - 1 is only finished once lv of chunk i is there: one phase at a time)
-      if (i >= 2) alive = sync_on(&sm->bar_e, i - 2);
-      if (!alive) break;
+      if (i >= 1) {                                        // chunk i - 2, which used this buffer last, is finished
+        ok = mbar_wait_or_abort(&sm->bar_sp, (i - 1) & 1, abort_flag);
+        ok = __all_sync(0xffffffffu, ok);
+        if (!ok) break;
+      }
       constexpr float kLog2e = 1.4426950408889634f;
 #pragma unroll
       for (int e = 0; e < 4; ++e) sm->lv[i & 1][4 * lane + e] = make_float2((before + d[e]) * kLog2e, s[e]);
@@ -288,55 +242,17 @@ linrec_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constan
       lt_arrive(&sm->bar_l[i & 1]);
       if (i + 1 < nchunks) fetch(i + 1);
     }
-    if (kStateOnly && alive && lane == 0 && pt == 0) sg.log_sum[(int64_t)bh * sg.count + seg] = seg_log;
-  } else if (warp < 8) {
-    // ------------------------------------------------------------------------------------ scores -> P: 64 columns of a row
-    if (!kStateOnly) {
-      const int j0 = half * 64, r0 = row & ~31;            // rows r0 .. r0 + 31 of this warp
-      for (int i = 0; i < nchunks; ++i) {
-        const float2* lv = sm->lv[i & 1];
-        alive = sync_on(&sm->bar_l[i & 1], i >> 1) && sync_on(&sm->bar_s, i);
-        if (alive && i > 0) alive = sync_on(&sm->bar_o2, i - 1);   // P of the previous chunk has been read
-        if (!alive) break;
-        tc_fence_after();
-        const float l_row = lv[row].x;
-#pragma unroll
-        for (int c2 = 0; c2 < 2; ++c2) {
-          const int jb = j0 + c2 * 32;
-          const bool future = jb > r0 + 31;                // all of it (warp-uniform)
-          uint32_t sv[32], hi[16], lo[16];
-          if (!future) {
-            lt_ld32_nowait(lanes + kLtS + jb, sv);
-            lt_wait_ld();
-          }
-          if (c2 == 1) {
-            tc_fence_before();
-            lt_arrive(&sm->bar_sfree);
-          }
-          if (future) {
-#pragma unroll
-            for (int e = 0; e < 16; ++e) hi[e] = lo[e] = 0;
-          } else {
-#pragma unroll
-            for (int e = 0; e < 16; ++e) {
-              const int j = jb + 2 * e;
-              const float4 w = *reinterpret_cast<const float4*>(&lv[j]);   // two tokens: log decay, scale
-              const float x = j <= row ? __uint_as_float(sv[2 * e]) * exp2_weight(l_row - w.x) * w.y : 0.f;
-              const float y = j + 1 <= row ? __uint_as_float(sv[2 * e + 1]) * exp2_weight(l_row - w.z) * w.w : 0.f;
-              lt_split(x, y, &hi[e], &lo[e]);
-            }
-          }
-          lt_st16(lanes + kLtPm + jb / 2, hi);
-          lt_st16(lanes + kLtPm + 64 + jb / 2, lo);
-        }
-        asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
-        tc_fence_before();
-        lt_arrive(&sm->bar_p);
-      }
-    }
+    if (!ok && lane == 0 && *abort_flag == 0) { *abort_flag = 1; report(status, TKV_DEV_TIMEOUT); }
+    if (kStateOnly && ok && lane == 0 && pt == 0) sg.log_sum[(int64_t)bh * sg.count + seg] = seg_log;
   } else {
-    // ------------------------------------------------------------------------------------ state, values, output: 32 columns of a row
+    // ------------------------------------------------------------------------------------ rows
+    const int row = tid & 127, half = tid >> 7;
+    const uint32_t lanes = tmem + ((uint32_t)((warp & 3) * 32) << 16);
     const uint32_t st_at = lanes + kLtST + half * 32;
+    auto sync_on = [&](uint64_t* bar, int parity) {
+      const bool ok = mbar_wait_or_abort(bar, parity & 1, abort_flag);
+      return (bool)__all_sync(0xffffffffu, ok);
+    };
     {                                                      // the state before the first chunk
       const float* S = kStateOnly ? nullptr : sg.count > 1 ? sg.start + ((int64_t)bh * sg.count + seg) * np : a.pos0[b] == 0 ? nullptr : final_state;
       float s[32];
@@ -348,32 +264,45 @@ linrec_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constan
         s[c] = x.x; s[c + 1] = x.y; s[c + 2] = x.z; s[c + 3] = x.w;
       }
       lt_st32(st_at, s);
+#pragma unroll
+      for (int c = 0; c < 32; ++c) s[c] = 0.f;
+      lt_st32(st_at + kLtP, s);
     }
     const float skip = a.skip != nullptr ? a.skip[h] : 0.f;
-
-    // State side of chunk i: the state before it becomes the operand of O1 and is scaled for its update; weighted values.
-    auto state_side = [&](int i) -> bool {
-      const float2* lv = sm->lv[i & 1];
+    bool alive = true;
+    for (int i = 0; i < nchunks; ++i) {
+      const int ph = i & 1;
+      const float2* lv = sm->lv[ph];
       uint8_t* v_t = v_s + (i & 1) * kLtHalf;
-      if (!sync_on(&sm->bar_l[i & 1], i >> 1)) return false;
-      if (i > 0 && !sync_on(&sm->bar_st, i - 1)) return false;
-      if (!kStateOnly && i > 0 && !sync_on(&sm->bar_o1, i - 1)) return false;   // the operand of the previous chunk has been read
-      tc_fence_after();
-      if (i == nchunks - 1 && last_rows < kLtC) {          // tokens beyond the end belong to another request: they read as zeros
-        if (!sync_on(&sm->bar_qk[i & 1], i >> 1) || !sync_on(&sm->bar_v[i & 1], i >> 1)) return false;
+      // ---- tokens beyond the request's end belong to another request: their keys and values read as zeros
+      if (i == nchunks - 1 && last_rows < kLtC) {
+        alive = sync_on(&sm->bar_qk, ph) && sync_on(&sm->bar_v[i & 1], i >> 1);
+        if (!alive) break;
         if (row >= last_rows) {
 #pragma unroll
-          for (int c = 0; c < 8; ++c) st16(k_s + (2 * (i & 1) + half) * kLtHalf + row * 128 + c * 16, make_uint4(0, 0, 0, 0));
+          for (int c = 0; c < 8; ++c) st16(k_s + half * kLtHalf + row * 128 + c * 16, make_uint4(0, 0, 0, 0));
 #pragma unroll
           for (int c = 0; c < 4; ++c) st16(v_t + row * 128 + half * 64 + c * 16, make_uint4(0, 0, 0, 0));
         }
         fence_async_smem();
         lt_arrive(&sm->bar_clr);
       }
+      // ---- the state before this chunk: operand of the read-out, then scaled for its update
+      alive = sync_on(&sm->bar_l[i & 1], i >> 1);
+      if (alive && i > 0) alive = sync_on(&sm->bar_st, i - 1);
+      if (!alive) break;
+      tc_fence_after();
       const float lend = lv[kLtC - 1].x;
       {
         float s[32];
-        tmem_ld32(st_at, s);
+        {
+          uint32_t x[32], y[32];
+          lt_ld32_nowait(st_at, x);
+          lt_ld32_nowait(st_at + kLtP, y);
+          lt_wait_ld();
+#pragma unroll
+          for (int c = 0; c < 32; ++c) s[c] = __uint_as_float(x[c]) + __uint_as_float(y[c]);
+        }
         if (!kStateOnly) {
 #pragma unroll
           for (int c = 0; c < 4; ++c) {
@@ -389,12 +318,17 @@ linrec_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constan
 #pragma unroll
         for (int c = 0; c < 32; ++c) s[c] *= ec;
         lt_st32(st_at, s);
+#pragma unroll
+        for (int c = 0; c < 32; ++c) s[c] = 0.f;
+        lt_st32(st_at + kLtP, s);
       }
       fence_async_smem();
       tc_fence_before();
       lt_arrive(&sm->bar_sp);
-      if (!sync_on(&sm->bar_v[i & 1], i >> 1)) return false;
-      const float w_row = exp2_weight(lend - lv[row].x) * lv[row].y;
+      // ---- weighted values
+      alive = sync_on(&sm->bar_v[i & 1], i >> 1);
+      if (!alive) break;
+      const float l_row = lv[row].x, w_row = exp2_weight(lend - l_row) * lv[row].y;
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
         const uint32_t at = lt_swz(row, half * 4 + c);
@@ -408,51 +342,87 @@ linrec_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constan
       }
       fence_async_smem();
       lt_arrive(&sm->bar_wv);
-      return true;
-    };
-
-    alive = state_side(0);
-    for (int i = 0; i < nchunks && alive; ++i) {
-      if (i + 1 < nchunks) alive = state_side(i + 1);
-      else if (!kStateOnly) alive = sync_on(&sm->bar_o1, i);
-      if (kStateOnly) {
-        if (alive) lt_arrive(&sm->bar_e);
-        continue;
-      }
-      if (alive) alive = sync_on(&sm->bar_o2, i);
+      if (kStateOnly) continue;
+      // ---- weighted scores: this thread's 64 columns of its row
+      alive = sync_on(&sm->bar_s, ph);
       if (!alive) break;
       tc_fence_after();
-      uint32_t o1[32], o2[32];
-      lt_ld32_nowait(lanes + kLtO1 + 64 * (i & 1) + half * 32, o1);
-      lt_ld32_nowait(lanes + kLtO2 + half * 32, o2);
-      lt_wait_ld();
-      const float er = exp2_weight(sm->lv[i & 1][row].x);
-      const uint8_t* v_t = v_s + (i & 1) * kLtHalf;
-      const int t = t_first + i * kLtC + row;
-      __nv_bfloat16* dst = (__nv_bfloat16*)a.out + ((int64_t)(tok0 + t) * a.heads + h) * a.p + pbase + half * 32;
+      const int j0 = half * 64, r0 = row & ~31;            // rows r0 .. r0 + 31 of this warp
+      uint8_t* p_hi = p_s + half * kLtHalf;
+      uint8_t* p_lo = p_hi + 2 * kLtHalf;
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        const uint4 x = ld16(v_t + lt_swz(row, half * 4 + c));
-        const uint32_t xs[4] = {x.x, x.y, x.z, x.w};
-        uint32_t w[4];
+      for (int c2 = 0; c2 < 2; ++c2) {
+        const int jb = j0 + c2 * 32;
+        if (jb > r0 + 31) {                                // all of it in the future (warp-uniform)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int at = c * 8 + 2 * e;
-          const float u = fmaf(er, __uint_as_float(o1[at]), __uint_as_float(o2[at])) + skip * __uint_as_float(xs[e] << 16);
-          const float v = fmaf(er, __uint_as_float(o1[at + 1]), __uint_as_float(o2[at + 1])) + skip * __uint_as_float(xs[e] & 0xffff0000u);
-          const __nv_bfloat162 pr = __floats2bfloat162_rn(u, v);
-          w[e] = *reinterpret_cast<const uint32_t*>(&pr);
+          for (int c = 0; c < 4; ++c) {
+            const uint32_t at = lt_swz(row, c2 * 4 + c);
+            st16(p_hi + at, make_uint4(0, 0, 0, 0));
+            st16(p_lo + at, make_uint4(0, 0, 0, 0));
+          }
+          continue;
         }
-        if (t < t_end && pbase + half * 32 + c * 8 < a.p) st16(dst + c * 8, make_uint4(w[0], w[1], w[2], w[3]));
+        uint32_t sv[32];
+        lt_ld32_nowait(lanes + kLtS + jb, sv);
+        lt_wait_ld();
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          uint32_t hi[4], lo[4];
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int j = jb + c * 8 + 2 * e;
+            const float4 w = *reinterpret_cast<const float4*>(&lv[j]);     // two tokens: log decay, scale
+            const float x = j <= row ? __uint_as_float(sv[c * 8 + 2 * e]) * exp2_weight(l_row - w.x) * w.y : 0.f;
+            const float y = j + 1 <= row ? __uint_as_float(sv[c * 8 + 2 * e + 1]) * exp2_weight(l_row - w.z) * w.w : 0.f;
+            lt_split(x, y, &hi[e], &lo[e]);
+          }
+          const uint32_t at = lt_swz(row, c2 * 4 + c);
+          st16(p_hi + at, make_uint4(hi[0], hi[1], hi[2], hi[3]));
+          st16(p_lo + at, make_uint4(lo[0], lo[1], lo[2], lo[3]));
+        }
+      }
+      fence_async_smem();
+      tc_fence_before();
+      lt_arrive(&sm->bar_p);
+      // ---- output
+      alive = sync_on(&sm->bar_o1, ph) && sync_on(&sm->bar_o2, ph);
+      if (!alive) break;
+      tc_fence_after();
+      {
+        uint32_t o1[32], o2[32], o3[32];
+        lt_ld32_nowait(lanes + kLtO1 + half * 32, o1);
+        lt_ld32_nowait(lanes + kLtO1 + kLtP + half * 32, o3);
+        lt_ld32_nowait(lanes + kLtO2 + half * 32, o2);
+        lt_wait_ld();
+        const float er = exp2_weight(l_row);
+        const int t = t_first + i * kLtC + row;
+        __nv_bfloat16* dst = (__nv_bfloat16*)a.out + ((int64_t)(tok0 + t) * a.heads + h) * a.p + pbase + half * 32;
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          const uint4 x = ld16(v_t + lt_swz(row, half * 4 + c));
+          const uint32_t xs[4] = {x.x, x.y, x.z, x.w};
+          uint32_t w[4];
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int at = c * 8 + 2 * e;
+            const float u = fmaf(er, __uint_as_float(o1[at]) + __uint_as_float(o3[at]), __uint_as_float(o2[at])) + skip * __uint_as_float(xs[e] << 16);
+            const float v = fmaf(er, __uint_as_float(o1[at + 1]) + __uint_as_float(o3[at + 1]), __uint_as_float(o2[at + 1])) + skip * __uint_as_float(xs[e] & 0xffff0000u);
+            const __nv_bfloat162 pr = __floats2bfloat162_rn(u, v);
+            w[e] = *reinterpret_cast<const uint32_t*>(&pr);
+          }
+          if (t < t_end && pbase + half * 32 + c * 8 < a.p) st16(dst + c * 8, make_uint4(w[0], w[1], w[2], w[3]));
+        }
       }
       tc_fence_before();
-      lt_arrive(&sm->bar_e);
     }
     if (alive) alive = sync_on(&sm->bar_st, nchunks - 1);
     if (alive) {
       tc_fence_after();
-      float s[32];
+      float s[32], lo[32];
       tmem_ld32(st_at, s);
+      tmem_ld32(st_at + kLtP, lo);
+#pragma unroll
+      for (int c = 0; c < 32; ++c) s[c] += lo[c];
       float* dst = kStateOnly ? sg.start + ((int64_t)bh * sg.count + seg) * np : (t_end == ntok ? final_state : nullptr);
       if (dst != nullptr && row < a.n) {
 #pragma unroll
@@ -461,18 +431,19 @@ linrec_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constan
           if (p < a.p) *reinterpret_cast<float4*>(dst + (int64_t)row * a.p + p) = make_float4(s[c], s[c + 1], s[c + 2], s[c + 3]);
         }
       }
+    } else if (lane == 0 && *abort_flag == 0) {
+      *abort_flag = 1; report(status, TKV_DEV_TIMEOUT);
     }
   }
-  if (!alive && *abort_flag == 0) { *abort_flag = 1; report(status, TKV_DEV_TIMEOUT); }
   tc_fence_before();
   __syncthreads();
   // An aborting CTA drains the copies it started before its shared memory is released.
-  if (*abort_flag != 0) {
-    if (tid == kCopyQK || tid == kCopyV)
-      for (int i = max(0, issued - 2); i < issued; ++i) mbar_wait(tid == kCopyQK ? &sm->bar_qk[i & 1] : &sm->bar_v[i & 1], (i >> 1) & 1);
+  if (tid == kLtRows && *abort_flag != 0) {
+    if (qk_issued > 0) mbar_wait(&sm->bar_qk, (qk_issued - 1) & 1);
+    for (int i = max(0, v_issued - 2); i < v_issued; ++i) mbar_wait(&sm->bar_v[i & 1], (i >> 1) & 1);
   }
   __syncthreads();
-  if (warp == 16) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(kLtCols));
+  if (warp == 8) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(kLtCols));
 }
 
 bool linrec_tc_shape(int n, int p, int max_tokens, int64_t tokens) {
