@@ -104,3 +104,16 @@ def test_every_microbenchmark_runs_and_prints_a_line(argv, capsys):
     assert d["micro"] == argv[1]
     times = [v for k, v in d.items() if k in ("avg_ms", "avg_ms_per_step", "query_resident_ms")]
     assert times and all(t > 0 for t in times)
+
+
+@pytest.mark.gpu
+def test_hybrid_microbenchmark_runs_and_prints_a_line(capsys):
+    sys.path.insert(0, ROOT)
+    import bench
+    bench.run_micro(bench.parse_args(["--micro", "hybrid", "--hybrid-size", "tiny"]))
+    lines = [l for l in capsys.readouterr().out.splitlines() if l.startswith("{")]
+    assert len(lines) == 1
+    d = json.loads(lines[0])
+    for model in ("hybrid", "qwen3"):
+        assert any(k.startswith("prefill") for k in d[model]) and any(k.startswith("decode") for k in d[model])
+    assert d["kernels"] and all(k["us"] > 0 for k in d["kernels"].values())

@@ -297,7 +297,7 @@ __global__ void __launch_bounds__(kStepThreads) retention_step_kernel(const T* p
 // the last `taps` inputs of x | B | C.  This step's inputs go to ring row pos mod taps, which holds an input that no
 // longer counts, so heads of a group may read the other rows while one of them writes.
 template <typename T, int V>
-__global__ void __launch_bounds__(kStepThreads) ssd_step_kernel(const T* proj, int64_t row_stride, T* ring, float* state,
+__global__ void __launch_bounds__(kStepThreads, 4) ssd_step_kernel(const T* proj, int64_t row_stride, T* ring, float* state,
                                                                const int32_t* slots, const int32_t* pos0, const float* conv_w,
                                                                const float* conv_b, const float* dt_bias, const float* a_log,
                                                                const float* skip, T* out, int heads, int groups, int n, int vdim,
@@ -315,32 +315,48 @@ __global__ void __launch_bounds__(kStepThreads) ssd_step_kernel(const T* proj, i
   T* rg = ring + (int64_t)slot * taps * channels;
   const float dt = softplus_f32(to_f32<T>(cur[channels + h]) + dt_bias[h]);
   const float decay = expf(-expf(a_log[h]) * dt);
-  for (int i = threadIdx.x; i < vdim + 2 * n; i += kStepThreads) {
-    const int ch = i < vdim ? h * vdim + i : (i < vdim + n ? inner + g * n + (i - vdim) : inner + (groups + g) * n + (i - vdim - n));
-    float acc = conv_b[ch];
-    const T in = cur[ch];
-    if (taps == 4) {                                       // the usual number: every load is requested before the first use
-      const float4 w = *reinterpret_cast<const float4*>(conv_w + (int64_t)ch * 4);
-      const int r0 = pos & 3;
-      const float x3 = pos >= 3 ? to_f32<T>(rg[(int64_t)((r0 + 1) & 3) * channels + ch]) : 0.f;
-      const float x2 = pos >= 2 ? to_f32<T>(rg[(int64_t)((r0 + 2) & 3) * channels + ch]) : 0.f;
-      const float x1 = pos >= 1 ? to_f32<T>(rg[(int64_t)((r0 + 3) & 3) * channels + ch]) : 0.f;
-      acc = fmaf(w.z, x1, fmaf(w.y, x2, fmaf(w.x, x3, acc)));
-    } else {
-      for (int d = taps - 1; d > 0; --d)
-        if (pos - d >= 0) acc = fmaf(conv_w[(int64_t)ch * taps + taps - 1 - d], to_f32<T>(rg[(int64_t)((pos - d) % taps) * channels + ch]), acc);
+  const float sk = skip[h];
+  // Two channels per thread and pass, every load requested before the first use.
+  for (int base = threadIdx.x; base < vdim + 2 * n; base += 2 * kStepThreads) {
+    float acc[2];
+    T in[2];
+    int chs[2];
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int i = base + u * kStepThreads;
+      if (i >= vdim + 2 * n) continue;
+      const int ch = i < vdim ? h * vdim + i : (i < vdim + n ? inner + g * n + (i - vdim) : inner + (groups + g) * n + (i - vdim - n));
+      chs[u] = ch;
+      acc[u] = conv_b[ch];
+      in[u] = cur[ch];
+      if (taps == 4) {                                     // the usual number
+        const float4 w = *reinterpret_cast<const float4*>(conv_w + (int64_t)ch * 4);
+        const int r0 = pos & 3;
+        const float x3 = pos >= 3 ? to_f32<T>(rg[(int64_t)((r0 + 1) & 3) * channels + ch]) : 0.f;
+        const float x2 = pos >= 2 ? to_f32<T>(rg[(int64_t)((r0 + 2) & 3) * channels + ch]) : 0.f;
+        const float x1 = pos >= 1 ? to_f32<T>(rg[(int64_t)((r0 + 3) & 3) * channels + ch]) : 0.f;
+        acc[u] = fmaf(w.w, to_f32<T>(in[u]), fmaf(w.z, x1, fmaf(w.y, x2, fmaf(w.x, x3, acc[u]))));
+      } else {
+        for (int d = taps - 1; d > 0; --d)
+          if (pos - d >= 0) acc[u] = fmaf(conv_w[(int64_t)ch * taps + taps - 1 - d], to_f32<T>(rg[(int64_t)((pos - d) % taps) * channels + ch]), acc[u]);
+        acc[u] = fmaf(conv_w[(int64_t)ch * taps + taps - 1], to_f32<T>(in[u]), acc[u]);
+      }
     }
-    acc = fmaf(conv_w[(int64_t)ch * taps + taps - 1], to_f32<T>(in), acc);
-    if (i < vdim || h == g * hpg) rg[(int64_t)(pos % taps) * channels + ch] = in;
-    const float y = round_as<T>(silu_act<T>(acc));
-    if (i < vdim) { x[i] = y; v[i] = dt * y; }
-    else if (i < vdim + n) k[i - vdim] = y;
-    else q[i - vdim - n] = y;
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int i = base + u * kStepThreads;
+      if (i >= vdim + 2 * n) continue;
+      if (i < vdim || h == g * hpg) rg[(int64_t)(pos % taps) * channels + chs[u]] = in[u];
+      const float y = round_as<T>(silu_act<T>(acc[u]));
+      if (i < vdim) { x[i] = y; v[i] = dt * y; }
+      else if (i < vdim + n) k[i - vdim] = y;
+      else q[i - vdim - n] = y;
+    }
   }
   __syncthreads();
   step.run(decay, k, q, v, o, red);
   T* dst = out + (int64_t)b * inner + (int64_t)h * vdim;
-  for (int i = threadIdx.x; i < vdim; i += kStepThreads) dst[i] = from_f32<T>(fmaf(skip[h], x[i], o[i]));
+  for (int i = threadIdx.x; i < vdim; i += kStepThreads) dst[i] = from_f32<T>(fmaf(sk, x[i], o[i]));
 }
 
 // ---------------------------------------------------------------------------------------------- scan, token by token
