@@ -4,6 +4,7 @@ import io
 import json
 import os
 import sys
+from concurrent.futures import ThreadPoolExecutor
 
 import numpy as np
 import pytest
@@ -272,7 +273,7 @@ def test_trace_needs_requests_of_unequal_length():
 
 
 # ------------------------------------------------------------------------------------------------ entry points
-def test_argument_errors_are_reported_without_a_gpu():
+def _argument_errors():
     from trimkv_b200 import _lib, build
     build.build()
     lib = _lib.lib()
@@ -290,3 +291,9 @@ def test_argument_errors_are_reported_without_a_gpu():
     assert lib.tkv_diff_decode(one, one, one, 9, one, one, one, 0.1, 1.0, 1e-6, one, 4, one, None, 0, 1, 4, 2, 8, 8, 64, 64, 0, None) == -1
     assert b"workspace" in lib.tkv_last_error()
     assert lib.tkv_batch_begin(one, None, None, one, 1, None) == -1
+
+
+def test_argument_errors_are_reported_without_a_gpu():
+    # in a thread of its own: the library's last error is kept per thread, and another test looks at the main thread's
+    with ThreadPoolExecutor(1) as pool:
+        pool.submit(_argument_errors).result()
