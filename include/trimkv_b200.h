@@ -430,7 +430,7 @@ int tkv_skinny_gemm(const void* x, const void* w, float* partial, int m, int n, 
 int tkv_skinny_gemm_swiglu(const void* gate_up, const void* w, float* partial, int m, int n, int k, int dtype,
                            int32_t* status, tkv_stream_t stream);
 
-/* ---- decoders with recurrent layers and windowed differential attention -------------------------------------------
+/* ---- decoders with recurrent layers, windowed attention and experts -------------------------------------------
  * Common conventions.  Tokens of a step are packed: request b owns rows cu_tokens[b] .. cu_tokens[b + 1) of every
  * per-token array (cu_tokens NULL, where allowed: one token per request).  What a request keeps between steps lives in
  * slot slots[b] of every state array; pos0[b] is the position of its first token of this step, and a request at position 0
@@ -443,23 +443,36 @@ int tkv_skinny_gemm_swiglu(const void* gate_up, const void* w, float* partial, i
 int tkv_batch_begin(int32_t* lens, const int32_t* slots, const int32_t* cu_tokens, int32_t* pos0, int batch,
                     tkv_stream_t stream);
 
-/* stream_out[r, :] = table[ids[r], :] as fp32, copy_out (may be NULL) the same in the model type.  An id outside
+/* stream_out[r, :] = scale * table[ids[r], :] in fp32, copy_out (may be NULL) the same in the model type.  An id outside
  * [0, vocab) yields zeros and TKV_DEV_BAD_INDEX. */
 int tkv_embed_stream(const int64_t* ids, const void* table, int64_t vocab, float* stream_out, void* copy_out, int rows, int width,
-                     int dtype, int32_t* status, tkv_stream_t stream);
+                     float scale, int dtype, int32_t* status, tkv_stream_t stream);
 
 /* x[r, :] += mult * RMSNorm(y[r, :]) * (weight_offset + weight); copy_out (may be NULL) = x in the model type. */
 int tkv_postnorm_add(float* x, const void* y, const float* weight, void* copy_out, int rows, int width, float eps, float mult,
                      float weight_offset, int dtype, tkv_stream_t stream);
 
-/* out[r, :] = RMSNorm(x[row_idx ? row_idx[r] : r, :]) * (weight_offset + weight). */
-int tkv_stream_norm(const float* x, const int32_t* row_idx, const float* weight, void* out, int rows, int width, float eps,
-                    float weight_offset, int dtype, tkv_stream_t stream);
+/* x[r, :] = RMS(alpha x[r, :] + sigmoid(gate[r, :] + gate_bias) * y[r, :]) * weight, each of `groups` equal consecutive parts of
+ * the row over its own root mean square; copy_out (may be NULL) = x in the model type.  gate NULL: no gate.  place / choice_w
+ * [rows, top] (place may be NULL): y[r, :] is the sum over the row's choices of choice_w * y[place, :], place < 0 standing for x
+ * itself (an expert that returns its input). */
+int tkv_gated_sum_norm(float* x, const void* y, const int32_t* place, const float* choice_w, int top, const void* gate,
+                       int64_t gate_stride, const float* gate_bias, const float* weight, void* copy_out, int rows, int width,
+                       int groups, float eps, float alpha, int dtype, tkv_stream_t stream);
+
+/* out[r, :] = RMSNorm(x[row_idx ? row_idx[r] : r, :]) * (weight_offset + weight), each of `groups` equal parts over its own root
+ * mean square. */
+int tkv_stream_norm(const float* x, const int32_t* row_idx, const float* weight, void* out, int rows, int width, int groups,
+                    float eps, float weight_offset, int dtype, tkv_stream_t stream);
 
 /* Group RMS norm with a SiLU gate: gate_first ? RMS(y * silu(z)) * weight : RMS(y) * weight * silu(z), every group of
- * group_len elements over its own root mean square; weight may be NULL.  out is contiguous [rows, groups * group_len]. */
-int tkv_gated_norm(const void* y, int64_t y_stride, const void* z, int64_t z_stride, const float* weight, void* out, int rows,
-                   int groups, int group_len, float eps, int gate_first, int dtype, tkv_stream_t stream);
+ * group_len elements over its own root mean square; z may be NULL (no gate); weight may be NULL, has one element per channel
+ * or (weight_shared) group_len elements for all groups.  out is contiguous [rows, groups * group_len]. */
+int tkv_gated_norm(const void* y, int64_t y_stride, const void* z, int64_t z_stride, const float* weight, int weight_shared,
+                   void* out, int rows, int groups, int group_len, float eps, int gate_first, int dtype, tkv_stream_t stream);
+
+/* out[r, j] = SiLU(u[r, j]) * u[r, ff + j]; rows of u are u_stride elements apart. */
+int tkv_swiglu(const void* u, int64_t u_stride, void* out, int rows, int ff, int dtype, tkv_stream_t stream);
 
 /* u[i] = GELU(u[i]), tanh form, in place. */
 int tkv_gelu_tanh(void* u, int64_t n, int dtype, tkv_stream_t stream);
@@ -539,6 +552,68 @@ int tkv_diff_prefill(const void* q, const void* k_lin, const void* v_lin, const 
                      const void* gate, int64_t gate_stride, void* out, int batch, int tokens, int max_tokens, int heads,
                      int kv_heads, int dim, int vdim, int dp, int pp, int window, int dtype, int32_t* status,
                      tkv_stream_t stream);
+
+/* Channel-decay recurrence in which the forget gate also writes.  q, f [.., heads * n] and v [.., heads * vdim] are columns of
+ * projection rows row_stride elements apart; per head
+ *   f_t = lower + (1 - lower) sigmoid(f + f_bias),  S_t = diag(f_t) S_(t-1) + (1 - f_t) v_t^T,  o_t = S_t^T silu(q_t)
+ * with f_bias, lower [heads * n] and state [slots, heads, n, vdim] fp32, read and written.
+ * tkv_chanrec_step: one token per request, writes RMS(o) * norm_w [vdim] per head.  tkv_chanrec_scan: token by token, every size
+ * (n <= 1400) and dtype, writes o; cu_tokens may be NULL.  tkv_chanrec_chunk: the tensor-core form for prompts, writes o: bf16,
+ * n <= 256, n, vdim and row_stride multiples of 8, 16-byte aligned rows.  Its workspace (tkv_chanrec_chunk_workspace_bytes; -1 =
+ * shape not supported, 0 = none) holds the states between the segments of long sequences. */
+int tkv_chanrec_step(const void* q, const void* f, const void* v, int64_t row_stride, const float* f_bias, const float* lower,
+                     const float* norm_w, float eps, void* out, float* state, const int32_t* slots, const int32_t* pos0, int batch,
+                     int heads, int n, int vdim, int dtype, tkv_stream_t stream);
+int tkv_chanrec_scan(const void* q, const void* f, const void* v, int64_t row_stride, const float* f_bias, const float* lower,
+                     void* out, float* state, const int32_t* slots, const int32_t* cu_tokens, const int32_t* pos0, int batch,
+                     int heads, int n, int vdim, int dtype, tkv_stream_t stream);
+
+/* Rotary positions in place on elements offset .. offset + rot_dims of every head of head_len elements: the pair (2i, 2i + 1)
+ * turns by position * f_i, freq_hi_lo[i] = {f_i rounded to fp32, the rest}. */
+int tkv_rotate_pairs(void* x, int64_t row_stride, const int32_t* cu_tokens, const int32_t* pos0, int batch, int tokens, int heads,
+                     int head_len, int offset, int rot_dims, const float* freq_hi_lo, int dtype, tkv_stream_t stream);
+
+/* Latent attention over a sliding window: keys and values of all heads are linear maps of one latent per position, plus a
+ * rotated key part that the heads share.  A position is one row of lw = pad64(kv_rank) + pad64(rot_dim) elements: the normed
+ * latent and the rotated part, each zero-padded to a multiple of 64.
+ * tkv_latent_prep: u row [q_rank | kv_rank | rot_dim | ..]; cq [tokens, q_rank] = RMSNorm of the first part with q_norm; latent
+ * (normed with kv_norm) and rotated key part (pairs as tkv_rotate_pairs) of position p go to row p mod ring_rows of ring
+ * [slots, ring_rows, lw] (ring_rows <= window, >= min(window, tokens seen after the step)) and, for steps of several tokens, to
+ * lin [rows, lw], request b's part starting at row kv_start[b] with the min(pos0[b], window - 1) positions before the step
+ * (fetched from the ring; max_history bounds them over the batch).
+ * tkv_latent_prefill: q [tokens, heads, dim + rot_dim] with its last rot_dim rotated, kv row (of every row of lin)
+ * [heads * dim keys | heads * vdim values], out [tokens, heads * vdim] = softmax((q k + q_rot k_rot) scale) v.
+ * tkv_latent_decode: one token per request against the ring, in the latent space: q_abs [.., kv_rank] = W_uk^T q per head, q_rot
+ * [.., rot_dim] not yet rotated (already rotated where the workspace size is -1), out [.., kv_rank] = softmax-weighted latents;
+ * strides in elements between tokens and heads.  Workspace: tkv_latent_decode_workspace_bytes (-1: none, the form for every
+ * size and dtype; the fast one takes bf16, kv_rank <= 512, rot_dim <= 128). */
+int tkv_latent_prep(const void* u, int64_t u_stride, const float* q_norm, const float* kv_norm, float eps, int q_rank, int kv_rank,
+                    int rot_dim, int rot_dims, const float* freq_hi_lo, void* cq, void* ring, int ring_rows, void* lin,
+                    const int32_t* kv_start, const int32_t* cu_tokens, const int32_t* slots, const int32_t* pos0, int batch,
+                    int tokens, int max_history, int window, int dtype, tkv_stream_t stream);
+int tkv_latent_prefill(const void* q, int64_t q_stride, const void* kv, int64_t kv_stride, const void* lin, const int32_t* kv_start,
+                       int64_t kv_rows, const int32_t* cu_tokens, const int32_t* pos0, float scale, void* out, int batch, int tokens,
+                       int max_tokens, int heads, int dim, int rot_dim, int vdim, int kv_rank, int window, int dtype,
+                       int32_t* status, tkv_stream_t stream);
+int64_t tkv_latent_decode_workspace_bytes(int batch, int heads, int kv_rank, int rot_dim, int ring_rows, int dtype);
+int tkv_latent_decode(const void* q_abs, int64_t qa_token, int64_t qa_head, const void* q_rot, int64_t qr_token, int64_t qr_head,
+                      const float* freq_hi_lo, const void* ring, int ring_rows, const int32_t* slots, const int32_t* pos0, float scale,
+                      void* out, int64_t out_token, int64_t out_head, void* workspace, int64_t workspace_bytes, int batch, int heads,
+                      int kv_rank, int rot_dim, int rot_dims, int dtype, tkv_stream_t stream);
+
+/* Mixture of experts.  experts counts all experts; the last `identity` of them return their input and own no rows.
+ * tkv_moe_route: logits [tokens, experts] fp32 (rows logit_stride apart) -> scores s = softmax(logits); the `top` experts with the
+ * largest s + correction among the `keep` of `groups` equal consecutive groups whose best s + correction is largest; weight
+ * [tokens, top] = s / (sum of the chosen s + 1e-20) * scale; choice [tokens, top].  place [tokens, top]: the choice's row when all
+ * choices are ordered by expert (-1: identity expert), src [tokens * top]: token of a row, offsets [experts - identity + 1]: first
+ * row of every expert.  counts [experts]: zeros on entry (may be NULL for at most 128 tokens).  top <= 64, experts <= 1024.
+ * tkv_moe_gemm: out[r, :] = act(a[src ? src[r] : r, :] . w[e]^T), r in expert e's rows; w [experts, n, k]; act 0 none, 1 GELU
+ * (erf); max_rows: host bound on the number of rows; a_rows: rows of a; experts here: those that own rows. */
+int tkv_moe_route(const float* logits, int64_t logit_stride, const float* correction, int tokens, int experts, int identity, int top,
+                  int groups, int keep, float scale, float* weight, int32_t* choice, int32_t* place, int32_t* src, int32_t* counts,
+                  int32_t* offsets, tkv_stream_t stream);
+int tkv_moe_gemm(const void* a, int64_t a_stride, int64_t a_rows, const int32_t* src, const void* w, const int32_t* offsets,
+                 void* out, int64_t max_rows, int experts, int n, int k, int act, int dtype, int32_t* status, tkv_stream_t stream);
 
 /* Blocks until `stream` is idle, then returns *status (a TKV_DEV_* code) and clears it. */
 int tkv_read_status(int32_t* status, tkv_stream_t stream);

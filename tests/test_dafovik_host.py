@@ -278,9 +278,9 @@ def _argument_errors():
     build.build()
     lib = _lib.lib()
     one = 16                                                            # a non-NULL, aligned address that is never used
-    assert lib.tkv_embed_stream(None, one, 4, one, None, 1, 8, 0, None, None) == -1
+    assert lib.tkv_embed_stream(None, one, 4, one, None, 1, 8, 1.0, 0, None, None) == -1
     assert lib.tkv_postnorm_add(one, one, one, None, 1, 8, 1e-6, 1.0, 1.0, 1, None) == -2           # f16
-    assert lib.tkv_gated_norm(one, 4, one, 8, None, one, 1, 1, 8, 1e-6, 0, 0, None) == -1           # stride below a row
+    assert lib.tkv_gated_norm(one, 4, one, 8, None, 0, one, 1, 1, 8, 1e-6, 0, 0, None) == -1           # stride below a row
     assert lib.tkv_rotate_qk(one, 64, one, None, one, 1, 1, 2, 8, 7, one, 1.0, 0, None) == -1       # odd rotary dims
     assert lib.tkv_conv_silu(one, 4, one, one, one, one, one, one, one, 1, 1, 8, 4, 0, None) == -1
     assert lib.tkv_linrec_scan(one, 8, one, 8, one, 8, None, None, None, None, one, one, one, None, one, 1, 1, 1, 8, 8, 0, None) == -1

@@ -10,6 +10,7 @@ from .modeling_qwen3 import TrimKVQwen3Config, TrimKVQwen3ForCausalLM, TrimKVQwe
 from .modeling_llama import TrimKVLlamaConfig, TrimKVLlamaForCausalLM, TrimKVLlamaModel
 from .modeling_phi3 import TrimKVPhi3Config, TrimKVPhi3ForCausalLM, TrimKVPhi3Model
 from .modeling_dafovik import DafovikConfig, DafovikForCausalLM, DafovikModel
+from .modeling_lonulix import LonulixConfig, LonulixForCausalLM, LonulixModel
 from .registry import load_model, model_class
 from .state_cache import HybridStateCache
 
@@ -19,5 +20,6 @@ __all__ = [
     "TrimKVQwen3Config", "TrimKVQwen3ForCausalLM", "TrimKVQwen3Model",
     "TrimKVLlamaConfig", "TrimKVLlamaForCausalLM", "TrimKVLlamaModel",
     "TrimKVPhi3Config", "TrimKVPhi3ForCausalLM", "TrimKVPhi3Model",
-    "DafovikConfig", "DafovikForCausalLM", "DafovikModel", "HybridStateCache", "load_model", "model_class",
+    "DafovikConfig", "DafovikForCausalLM", "DafovikModel", "LonulixConfig", "LonulixForCausalLM", "LonulixModel",
+    "HybridStateCache", "load_model", "model_class",
 ]

@@ -52,10 +52,12 @@ SIGNATURES = {
     "tkv_skinny_gemm": (I, [P, P, P, I, I, I, I, P, P]),
     "tkv_skinny_gemm_swiglu": (I, [P, P, P, I, I, I, I, P, P]),
     "tkv_batch_begin": (I, [P, P, P, P, I, P]),
-    "tkv_embed_stream": (I, [P, P, L, P, P, I, I, I, P, P]),
+    "tkv_embed_stream": (I, [P, P, L, P, P, I, I, F, I, P, P]),
     "tkv_postnorm_add": (I, [P, P, P, P, I, I, F, F, F, I, P]),
-    "tkv_stream_norm": (I, [P, P, P, P, I, I, F, F, I, P]),
-    "tkv_gated_norm": (I, [P, L, P, L, P, P, I, I, I, F, I, I, P]),
+    "tkv_gated_sum_norm": (I, [P, P, P, P, I, P, L, P, P, P, I, I, I, F, F, I, P]),
+    "tkv_stream_norm": (I, [P, P, P, P, I, I, I, F, F, I, P]),
+    "tkv_gated_norm": (I, [P, L, P, L, P, I, P, I, I, I, F, I, I, P]),
+    "tkv_swiglu": (I, [P, L, P, I, I, I, P]),
     "tkv_gelu_tanh": (I, [P, L, I, P]),
     "tkv_rotate_qk": (I, [P, L, P, P, P, I, I, I, I, I, P, F, I, P]),
     "tkv_conv_silu": (I, [P, L, P, P, P, P, P, P, P, I, I, I, I, I, P]),
@@ -69,6 +71,15 @@ SIGNATURES = {
     "tkv_diff_decode_workspace_bytes": (L, [I, I, I, I, I, I, I]),
     "tkv_diff_decode": (I, [P, P, P, I, P, P, P, F, F, F, P, L, P, P, L, I, I, I, I, I, I, I, I, P]),
     "tkv_diff_prefill": (I, [P, P, P, P, L, P, P, P, F, F, F, P, L, P, I, I, I, I, I, I, I, I, I, I, I, P, P]),
+    "tkv_chanrec_step": (I, [P, P, P, L, P, P, P, F, P, P, P, P, I, I, I, I, I, P]),
+    "tkv_chanrec_scan": (I, [P, P, P, L, P, P, P, P, P, P, P, I, I, I, I, I, P]),
+    "tkv_rotate_pairs": (I, [P, L, P, P, I, I, I, I, I, I, P, I, P]),
+    "tkv_latent_prep": (I, [P, L, P, P, F, I, I, I, I, P, P, P, I, P, P, P, P, P, I, I, I, I, I, P]),
+    "tkv_latent_prefill": (I, [P, L, P, L, P, P, L, P, P, F, P, I, I, I, I, I, I, I, I, I, I, P, P]),
+    "tkv_latent_decode_workspace_bytes": (L, [I, I, I, I, I, I]),
+    "tkv_latent_decode": (I, [P, L, L, P, L, L, P, P, I, P, P, F, P, L, L, P, L, I, I, I, I, I, I, P]),
+    "tkv_moe_route": (I, [P, L, P, I, I, I, I, I, I, F, P, P, P, P, P, P, P]),
+    "tkv_moe_gemm": (I, [P, L, L, P, P, P, P, L, I, I, I, I, I, P, P]),
     "tkv_read_status": (I, [P, P]),
 }
 

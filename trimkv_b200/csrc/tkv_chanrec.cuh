@@ -1,0 +1,34 @@
+// Linear recurrences with one decay per state row (channel of q) and token, in which the forget gate also writes:
+//   f = lower + (1 - lower) sigmoid(z_f + bias),  S_t = diag(f_t) S_(t-1) + (1 - f_t) v_t^T,  o_t = S_t^T silu(z_q).
+// The gate, its complement and the state are fp32 whatever the type of the projections z_q, z_f, v.
+#pragma once
+#include "tkv_elem.cuh"
+
+namespace tkv {
+
+struct ChanrecParams {
+  const void* q; const void* f; const void* v;        // [tokens, heads * n], same, [tokens, heads * p]: columns of projection rows
+  int64_t row_stride;                                 // of all three, in elements
+  const float* f_bias; const float* lower;            // [heads * n]
+  void* out;                                          // [tokens, heads * p], model type
+  float* state;                                       // [slots, heads, n, p] fp32
+  const int32_t* slots; const int32_t* cu; const int32_t* pos0;
+  int batch, heads, n, p;
+};
+
+// f and 1 - f, each to fp32 accuracy (1 - f is (1 - lower) sigmoid(-x), not a difference).
+__device__ __forceinline__ void forget_gate(float x, float lower, float* f, float* k) {
+  const float e = expf(-fabsf(x)), r = 1.0f / (1.0f + e);
+  const float big = r, small = e * r;                 // sigmoid(|x|), sigmoid(-|x|)
+  *f = fmaf(1.0f - lower, x >= 0.f ? big : small, lower);
+  *k = (1.0f - lower) * (x >= 0.f ? small : big);
+}
+
+// A long sequence cut into segments that run side by side (see LinrecSegs), with a decay per state row.
+struct ChanrecSegs {
+  int count, tokens;                                  // segments per request, tokens per segment
+  float* start;                                       // [batch, heads, count, n, p]
+  float* decay;                                       // [batch, heads, count, n]: product of f over the segment
+};
+
+}  // namespace tkv

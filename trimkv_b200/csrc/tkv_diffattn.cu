@@ -14,6 +14,7 @@
 // type and its merge, and a kernel for every size in fp32 arithmetic.  The prompt kernel on tcgen05 is in
 // tkv_diffattn_tc.cu.
 #include "tkv_diffattn.cuh"
+#include "tkv_ring.cuh"
 #include "tkv_tc.cuh"
 
 namespace tkv {
@@ -94,26 +95,6 @@ __global__ void __launch_bounds__(kPrepThreads) diff_prep_kernel(const T* proj, 
     if (d0 != nullptr) store_vec<V>(d0 + i, x);
     if (d1 != nullptr) store_vec<V>(d1 + i, x);
   }
-}
-
-// The positions before a request's step that its window still reaches, from the ring into the linear buffers.  One warp
-// per (history row, kv head); grid.y = request.
-template <typename T>
-__global__ void __launch_bounds__(kPrepThreads) ring_fetch_kernel(const T* k_ring, const T* v_ring, int ring_rows, T* k_lin, T* v_lin,
-                                                                 const int32_t* kv_start, const int32_t* slots,
-                                                                 const int32_t* pos0, int kv_heads, int dp, int pp, int window) {
-  grid_dependency_wait();
-  grid_launch_dependents();
-  const int lane = threadIdx.x & 31, b = blockIdx.y;
-  const int hist = min(pos0[b], window - 1);
-  const int item = blockIdx.x * (kPrepThreads / 32) + (threadIdx.x >> 5);
-  const int r = item / kv_heads, g = item - r * kv_heads;
-  if (r >= hist) return;
-  const int64_t src = ((int64_t)slots[b] * kv_heads + g) * ring_rows + (pos0[b] - hist + r) % ring_rows;
-  const int64_t dst = ((int64_t)kv_start[b] + r) * kv_heads + g;
-  constexpr int kPer = 16 / (int)sizeof(T);
-  for (int i = lane * kPer; i < 2 * dp; i += 32 * kPer) st16(k_lin + dst * 2 * dp + i, ld16(k_ring + src * 2 * dp + i));
-  for (int i = lane * kPer; i < pp; i += 32 * kPer) st16(v_lin + dst * pp + i, ld16(v_ring + src * pp + i));
 }
 
 // ------------------------------------------------------------------------------------------------ any size, fp32 arithmetic
@@ -454,10 +435,10 @@ extern "C" int tkv_diff_prep(const void* proj, int64_t row_stride, const float* 
   TKV_WITH_TYPE(dtype, T, {
     if (k_lin != nullptr && max_history > 0) {            // before the new tokens overwrite the ring rows it reads
       const int hist = max_history < window - 1 ? max_history : window - 1;
-      const dim3 fgrid((unsigned)(((int64_t)hist * kv_heads + kPrepThreads / 32 - 1) / (kPrepThreads / 32)), batch);
+      const dim3 fgrid((unsigned)(((int64_t)hist * kv_heads + kFetchThreads / 32 - 1) / (kFetchThreads / 32)), batch);
       if (fgrid.x > 0) {
-        cudaError_t e = launch_pdl(ring_fetch_kernel<T>, fgrid, dim3(kPrepThreads), 0, (cudaStream_t)stream, (const T*)k_ring, (const T*)v_ring,
-                                   ring_rows, (T*)k_lin, (T*)v_lin, kv_start, slots, pos0, kv_heads, dp, pp, window);
+        cudaError_t e = launch_pdl(ring_fetch_kernel<T>, fgrid, dim3(kFetchThreads), 0, (cudaStream_t)stream, (const T*)k_ring, (const T*)v_ring,
+                                   ring_rows, (T*)k_lin, (T*)v_lin, kv_start, slots, pos0, kv_heads, 2 * dp, pp, window);
         if (e != cudaSuccess) return fail(TKV_ERR_LAUNCH, "tkv_diff_prep: %s", cudaGetErrorString(e));
       }
     }

@@ -89,6 +89,18 @@ template <typename T> __device__ __forceinline__ float gelu_tanh_act(float z) {
   else return __fdividef(z, 1.0f + __expf(fminf(-2.0f * u, 80.f)));      // (1 + tanh u) / 2 = 1 / (1 + e^(-2u))
 }
 
+// sin and cos of pos * (f_hi + f_lo): the fp32 product's rounding error and the frequency's low part are carried as a
+// first-order correction, so that the angle keeps its accuracy at large positions.
+__device__ __forceinline__ void turn(int pos, float f_hi, float f_lo, float* s, float* c) {
+  const float p = (float)pos;
+  const float a = p * f_hi;
+  const float e = fmaf(p, f_hi, -a) + p * f_lo;
+  float s0, c0;
+  sincosf(a, &s0, &c0);
+  *s = fmaf(c0, e, s0);
+  *c = fmaf(-s0, e, c0);
+}
+
 // Request that owns packed row t: largest b with cu[b] <= t (cu == nullptr: one row per request).
 __device__ __forceinline__ int owner_of(const int32_t* cu, int batch, int t) {
   if (cu == nullptr) return t;

@@ -11,20 +11,9 @@
 // A request whose start position is 0 starts from the zero state whatever its slot held before.  The state is fp32 and
 // is read and written once per step; its 8 n p bytes per head are what a decode step costs.
 #include "tkv_linrec.cuh"
+#include "tkv_state_step.cuh"
 
 namespace tkv {
-
-// sin and cos of pos * (f_hi + f_lo): the fp32 product's rounding error and the frequency's low part are carried as a
-// first-order correction, so that the angle keeps its accuracy at large positions.
-__device__ __forceinline__ void turn(int pos, float f_hi, float f_lo, float* s, float* c) {
-  const float p = (float)pos;
-  const float a = p * f_hi;
-  const float e = fmaf(p, f_hi, -a) + p * f_lo;
-  float s0, c0;
-  sincosf(a, &s0, &c0);
-  *s = fmaf(c0, e, s0);
-  *c = fmaf(-s0, e, c0);
-}
 
 constexpr int kRotThreads = 128;
 
@@ -168,88 +157,6 @@ __global__ void __launch_bounds__(256) ssd_steps_kernel(const T* dt_in, int64_t 
   log_decay[i] = -expf(a_log[h]) * d;
 }
 
-// ---------------------------------------------------------------------------------------------- one-token state update
-constexpr int kStepThreads = 256;
-
-// S <- decay S + k v^T and o = S^T q for one head: S [n, p] fp32 in global memory, k / q [n], v [p], o [p] in shared
-// memory.  Threads cover columns in vectors of V and rows in an interleaved fashion.  The first rows are requested by
-// `prefetch` before the step's k, q, v are known, so that their latency overlaps the producers' work.
-template <int V> struct StateStep {
-  static constexpr int U = 8;
-  float* S; int n, p, nc, cb, rg, r, c0; bool fresh;
-  float s[U][V];
-
-  __device__ __forceinline__ void load(int row, int c) {
-#pragma unroll
-    for (int u = 0; u < U; ++u) {
-      const int rr = row + u * rg;
-      if (rr < n && !fresh) {
-        if constexpr (V == 4) {
-          const float4 x = *reinterpret_cast<const float4*>(S + (int64_t)rr * p + c * V);
-          s[u][0] = x.x; s[u][1] = x.y; s[u][2] = x.z; s[u][3] = x.w;
-        } else {
-          s[u][0] = S[(int64_t)rr * p + c];
-        }
-      } else {
-#pragma unroll
-        for (int e = 0; e < V; ++e) s[u][e] = 0.f;
-      }
-    }
-  }
-  __device__ __forceinline__ void prefetch(float* S_, int n_, int p_, bool fresh_) {
-    S = S_; n = n_; p = p_; fresh = fresh_;
-    nc = p / V; cb = min(nc, kStepThreads); rg = kStepThreads / cb;
-    r = threadIdx.x / cb; c0 = threadIdx.x - r * cb;
-    if (r < rg) load(r, c0);
-  }
-  // All threads of the CTA call it; k, q, v must be visible (a barrier before), o is visible on return.  red holds
-  // kStepThreads * V floats.
-  __device__ __forceinline__ void run(float decay, const float* k, const float* q, const float* v, float* o, float* red) {
-    const bool active = r < rg;
-    for (int cbase = 0; cbase < nc; cbase += cb) {
-      const int c = cbase + c0;
-      float acc[V];
-#pragma unroll
-      for (int e = 0; e < V; ++e) acc[e] = 0.f;
-      if (active && c < nc) {
-        float vv[V];
-#pragma unroll
-        for (int e = 0; e < V; ++e) vv[e] = v[c * V + e];
-        for (int row = r; row < n; row += rg * U) {
-          if (row != r || cbase != 0) load(row, c);
-#pragma unroll
-          for (int u = 0; u < U; ++u) {
-            const int rr = row + u * rg;
-            if (rr < n) {
-              const float kk = k[rr], qq = q[rr];
-#pragma unroll
-              for (int e = 0; e < V; ++e) {
-                s[u][e] = fmaf(decay, s[u][e], kk * vv[e]);
-                acc[e] = fmaf(qq, s[u][e], acc[e]);
-              }
-              if constexpr (V == 4)
-                *reinterpret_cast<float4*>(S + (int64_t)rr * p + c * V) = make_float4(s[u][0], s[u][1], s[u][2], s[u][3]);
-              else
-                S[(int64_t)rr * p + c] = s[u][0];
-            }
-          }
-        }
-      }
-      if (active) {
-#pragma unroll
-        for (int e = 0; e < V; ++e) red[(r * cb + c0) * V + e] = acc[e];
-      }
-      __syncthreads();
-      for (int i = threadIdx.x; i < cb * V && cbase * V + i < p; i += kStepThreads) {
-        float a = 0.f;
-        for (int g = 0; g < rg; ++g) a += red[g * cb * V + i];
-        o[cbase * V + i] = a;
-      }
-      __syncthreads();
-    }
-  }
-};
-
 // One CTA per (request, head).  proj row: q [heads, dim], k [heads, dim], v [heads, vdim], gate [heads, vdim].
 template <typename T, int V>
 __global__ void __launch_bounds__(kStepThreads) retention_step_kernel(const T* proj, int64_t row_stride, float* state,
@@ -285,7 +192,8 @@ __global__ void __launch_bounds__(kStepThreads) retention_step_kernel(const T* p
   }
   for (int i = threadIdx.x; i < vdim; i += kStepThreads) v[i] = to_f32<T>(vg[i]);
   __syncthreads();
-  step.run(decay[h], k, q, v, o, red);
+  const float a = decay[h];
+  step.run([a](int) { return a; }, k, q, v, o, red);
   float ss = 0.f;
   for (int i = threadIdx.x; i < vdim; i += kStepThreads) ss += o[i] * o[i];
   const float rstd = 1.0f / sqrtf(block_add<kStepThreads>(ss, wred) / (float)vdim + eps);
@@ -354,7 +262,7 @@ __global__ void __launch_bounds__(kStepThreads, 4) ssd_step_kernel(const T* proj
     }
   }
   __syncthreads();
-  step.run(decay, k, q, v, o, red);
+  step.run([decay](int) { return decay; }, k, q, v, o, red);
   T* dst = out + (int64_t)b * inner + (int64_t)h * vdim;
   for (int i = threadIdx.x; i < vdim; i += kStepThreads) dst[i] = from_f32<T>(fmaf(sk, x[i], o[i]));
 }
@@ -491,15 +399,6 @@ extern "C" int tkv_ssd_steps(const void* dt_in, int64_t row_stride, const float*
   });
   return check_launch("tkv_ssd_steps");
 }
-
-namespace tkv {
-// Raises a kernel's dynamic shared memory limit (once per kernel and size); false if the size is out of reach.
-template <typename K> static bool allow_smem(K kernel, size_t bytes) {
-  if (bytes <= 48 * 1024) return true;
-  if (bytes > 220 * 1024) return false;
-  return cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) == cudaSuccess;
-}
-}  // namespace tkv
 
 extern "C" int tkv_retention_step(const void* proj, int64_t row_stride, float* state, const int32_t* slots, const int32_t* pos0,
                                   const float* head_decay, const float* freq_hi_lo, void* out, int batch, int heads, int dim,

@@ -310,7 +310,7 @@ class GreedyDecoder:
 
 
 class HybridDecodeStep:
-    """One-token step of a hybrid decoder (``modeling_dafovik``): its layers' one-token kernels around the library GEMMs.
+    """One-token step of a hybrid decoder (``modeling_hybrid``): its layers' one-token kernels around the library GEMMs.
 
     Per layer with a recurrent mixer: one projection GEMM, the state step (rotation or convolution, state update, read-out
     and, for retention, norm and gate in the same launch), the gated norm where the norm spans heads, the output GEMM, then

@@ -1,4 +1,5 @@
-"""Token mixers of hybrid decoders: retention, state-space duality (Mamba-2) and windowed differential attention.
+"""Token mixers of hybrid decoders: retention, state-space duality (Mamba-2), HGRN2, windowed differential attention and
+windowed latent attention.
 
 A mixer reads the packed tokens of a step, keeps its requests' state in ``HybridStateCache`` slots and runs the CUDA
 kernels: one fused projection, the mixing kernels (a chunked or windowed form for steps of several tokens, a one-token form
@@ -15,7 +16,7 @@ import torch.nn.functional as F
 from torch import nn
 
 from . import ops
-from .state_cache import RecurrentState, StepBatch, WindowState
+from .state_cache import LatentState, RecurrentState, StepBatch, WindowState
 
 
 def _stamp(p: torch.Tensor):
@@ -63,8 +64,28 @@ class FusedProjection(nn.Module):
         return F.linear(x, self.weight)
 
 
+def rotary_frequencies(base: float, dims: int) -> torch.Tensor:
+    """``base^(-2i/dims)`` for the pairs i, each as a high and a low fp32 part ``[dims / 2, 2]``."""
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    f = base ** (-2.0 * i / max(dims, 1))
+    hi = f.float()
+    return torch.stack([hi, (f - hi.double()).float()], dim=1).contiguous()
+
+
 class Mixer(nn.Module):
-    """``state()`` describes what a request keeps; ``checkpoint()`` maps the names a checkpoint uses to parameters."""
+    """``state()`` describes what a request keeps; ``checkpoint()`` maps the names a checkpoint uses to parameters.
+
+    Mixers built with ``gate_rows`` compute that many rows of a gate of the same input in their fused projection:
+    ``gate_part()`` is its weight, and ``forward`` returns ``(result, gate logits)``."""
+
+    gate_rows = 0
+
+    def gate_part(self) -> torch.Tensor:
+        return self.proj.part("gate_rows")
+
+    def _gate(self, u: torch.Tensor) -> torch.Tensor:
+        lo, hi = self.proj.offsets["gate_rows"]
+        return u[:, lo:hi]
 
     def state(self):
         raise NotImplementedError
@@ -112,12 +133,7 @@ class RetentionMixer(Mixer):
         nn.init.normal_(self.o, mean=0.0, std=std)
 
     def _freq(self, device):
-        def make():
-            i = torch.arange(self.rot_dims // 2, dtype=torch.float64)
-            f = self.rot_base ** (-2.0 * i / max(self.rot_dims, 1))
-            hi = f.float()
-            return torch.stack([hi, (f - hi.double()).float()], dim=1).contiguous()
-        return self._constant("freq", device, make)
+        return self._constant("freq", device, lambda: rotary_frequencies(self.rot_base, self.rot_dims))
 
     def _decay(self, device, log: bool):
         return self._constant(("decay", log), device, lambda: (
@@ -251,6 +267,108 @@ class DifferentialAttentionMixer(Mixer):
         return F.linear(out, self.o)
 
 
+class HGRN2Mixer(Mixer):
+    """Linear attention whose forget gate, one per head and channel and bounded from below, also decides what is written."""
+
+    def __init__(self, width: int, heads: int, dim: int, vdim: int, eps: float, gate_rows: int = 0):
+        super().__init__()
+        self.heads, self.dim, self.vdim, self.eps, self.gate_rows = heads, dim, vdim, eps, gate_rows
+        self.proj = FusedProjection(width, {"q": heads * dim, "f": heads * dim, "v": heads * vdim, "gate_rows": gate_rows})
+        self.f_bias = nn.Parameter(torch.zeros(heads * dim))
+        self.lower = nn.Parameter(torch.zeros(heads * dim))
+        self.norm = nn.Parameter(torch.ones(vdim))
+        self.o = nn.Parameter(torch.zeros(width, heads * vdim))
+
+    def state(self):
+        return RecurrentState(self.heads, self.dim, self.vdim)
+
+    def checkpoint(self):
+        return {**{n: self.proj.part(n) for n in ("q", "f", "v")}, "f.b": self.f_bias, "lower": self.lower, "norm": self.norm, "o": self.o}
+
+    def reset_parameters(self, std):
+        self.proj.reset_parameters(std)
+        nn.init.normal_(self.o, mean=0.0, std=std)
+        nn.init.ones_(self.norm)
+        with torch.no_grad():
+            self.f_bias.uniform_(0.0, 4.0)
+            self.lower.uniform_(0.0, 0.5)
+
+    def forward(self, x, batch, data):
+        h, n, p = self.heads, self.dim, self.vdim
+        u = self.proj(x)
+        q, f, v = (u[:, lo:hi] for lo, hi in (self.proj.offsets[k] for k in ("q", "f", "v")))
+        bias, lower, norm = (as_f32(self, k) for k in ("f_bias", "lower", "norm"))
+        out = torch.empty(x.shape[0], h * p, dtype=x.dtype, device=x.device)
+        if batch.cu is None:
+            ops.chanrec_step(q, f, v, bias, lower, norm, data["state"], batch, out, self.eps)
+        else:
+            y = torch.empty_like(out)
+            ops.chanrec(q, f, v, bias, lower, data["state"], batch, y)
+            ops.gated_norm(y, None, norm, out, h, self.eps)
+        y = F.linear(out, self.o)
+        return (y, self._gate(u)) if self.gate_rows else y
+
+
+class LatentAttentionMixer(Mixer):
+    """Softmax attention inside a sliding window whose keys and values come from one normed latent per position; a rotated key
+    part is shared by the heads.  A request keeps the latent and the rotated part only.
+
+    Steps of several tokens expand the latents to every head's keys and values; one-token steps take the queries into the
+    latent space instead (``W_uk`` on the query, ``W_uv`` on the weighted latents)."""
+
+    def __init__(self, width: int, heads: int, dim: int, rot_dim: int, vdim: int, q_rank: int, kv_rank: int, window: int,
+                 scale: float, rot_dims: int, rot_base: float, eps: float, gate_rows: int = 0):
+        super().__init__()
+        if rot_dims % 2 or rot_dims > rot_dim:
+            raise ValueError(f"rotary dims {rot_dims} of a part of {rot_dim}")
+        self.heads, self.dim, self.rot_dim, self.vdim, self.kv_rank = heads, dim, rot_dim, vdim, kv_rank
+        self.window, self.scale, self.eps, self.gate_rows = window, float(scale), eps, gate_rows
+        self.rot_dims, self.rot_base = rot_dims, float(rot_base)
+        self.proj = FusedProjection(width, {"dq": q_rank, "dkv": kv_rank + rot_dim, "gate_rows": gate_rows})
+        self.q_norm, self.kv_norm = nn.Parameter(torch.ones(q_rank)), nn.Parameter(torch.ones(kv_rank))
+        self.uq = nn.Parameter(torch.zeros(heads * (dim + rot_dim), q_rank))
+        self.ukv = FusedProjection(kv_rank, {"uk": heads * dim, "uv": heads * vdim})
+        self.o = nn.Parameter(torch.zeros(width, heads * vdim))
+
+    def state(self):
+        return LatentState(-(-self.kv_rank // 64) * 64 + -(-self.rot_dim // 64) * 64, self.window)
+
+    def checkpoint(self):
+        return {"dq": self.proj.part("dq"), "dq.norm": self.q_norm, "uq": self.uq, "dkv": self.proj.part("dkv"),
+                "dkv.norm": self.kv_norm, "uk": self.ukv.part("uk"), "uv": self.ukv.part("uv"), "o": self.o}
+
+    def reset_parameters(self, std):
+        self.proj.reset_parameters(std)
+        self.ukv.reset_parameters(std)
+        for w in (self.uq, self.o):
+            nn.init.normal_(w, mean=0.0, std=std)
+        for w in (self.q_norm, self.kv_norm):
+            nn.init.ones_(w)
+
+    def _freq(self, device):
+        return self._constant("freq", device, lambda: rotary_frequencies(self.rot_base, self.rot_dims))
+
+    def forward(self, x, batch, data):
+        h, d, r, p, rank, T = self.heads, self.dim, self.rot_dim, self.vdim, self.kv_rank, x.shape[0]
+        u, freq = self.proj(x), self._freq(x.device)
+        cq, lin = ops.latent_prep(u, as_f32(self, "q_norm"), as_f32(self, "kv_norm"), self.eps, r, self.rot_dims, freq, data["latent"],
+                                  batch, self.window)
+        q = F.linear(cq, self.uq)
+        out = torch.empty(T, h * p, dtype=x.dtype, device=x.device)
+        if batch.cu is None:
+            q3 = q.view(T, h, d + r)
+            q_abs = torch.bmm(q3[:, :, :d].transpose(0, 1), self.ukv.part("uk").view(h, d, rank))
+            o_lat = torch.empty_like(q_abs)
+            ops.latent_decode(q_abs.transpose(0, 1), q3, r, freq, data["latent"], batch, self.scale, o_lat.transpose(0, 1), self.rot_dims)
+            torch.bmm(o_lat, self.ukv.part("uv").view(h, p, rank).transpose(1, 2), out=out.view(T, h, p).transpose(0, 1))
+        else:
+            ops.rotate_pairs(q, batch, h, d + r, d, self.rot_dims, freq)
+            kv = self.ukv(lin[:, :rank])
+            ops.latent_prefill(q, kv, lin, batch, self.scale, out, h, d, r, p, rank, self.window)
+        y = F.linear(out, self.o)
+        return (y, self._gate(u)) if self.gate_rows else y
+
+
 class GeluMLP(nn.Module):
     """Dense feed-forward with the tanh form of GELU."""
 
@@ -272,4 +390,5 @@ class GeluMLP(nn.Module):
         return F.linear(u, self.down)
 
 
-__all__ = ["DifferentialAttentionMixer", "FusedProjection", "GeluMLP", "Mixer", "RetentionMixer", "SSDMixer", "as_f32"]
+__all__ = ["DifferentialAttentionMixer", "FusedProjection", "GeluMLP", "HGRN2Mixer", "LatentAttentionMixer", "Mixer",
+           "RetentionMixer", "SSDMixer", "as_f32", "rotary_frequencies"]

@@ -2,29 +2,19 @@
 
 The order of layers, each layer's mixer and all its sizes come from the configuration.  A sublayer reads the residual
 stream itself and only its output is normed:  x <- x + m norm1(mixer(x)),  x <- x + m norm2(mlp(x)),  with RMS norms whose
-weights are stored around zero.  The stream is fp32 whatever the model type; the products read its copy in the model type.
-
-One forward serves prompts, portions of prompts and decoding: the tokens of a step's requests are packed (no padding is
-computed) and every layer takes its state from ``HybridStateCache``.  bf16 models run the tensor-core kernels, fp32 models
-the fp32 forms of the same kernels.  ``generate`` (HF), ``generate_greedy``, ``GreedyDecoder`` and the graph-replayed
-one-token step are those of the other families.
+weights are stored around zero.  Everything else is that of the hybrid decoders (``modeling_hybrid``).
 """
 from __future__ import annotations
 
-import json
-import os
-from typing import Dict, List, Optional, Sequence
+from typing import List, Optional
 
 import torch
-import torch.nn.functional as F
 from torch import nn
-from transformers import PretrainedConfig
-from transformers.modeling_outputs import BaseModelOutputWithPast, CausalLMOutputWithPast
 
 from . import ops
-from .mixers import DifferentialAttentionMixer, FusedProjection, GeluMLP, Mixer, RetentionMixer, SSDMixer, as_f32
-from .modeling_trimkv import TrimKVForCausalLM, TrimKVPreTrainedModel
-from .state_cache import HybridStateCache, StepBatch
+from .mixers import DifferentialAttentionMixer, GeluMLP, Mixer, RetentionMixer, SSDMixer, as_f32
+from .modeling_hybrid import HybridConfig, HybridForCausalLM, HybridModel, StreamNorm
+from .state_cache import StepBatch
 
 
 def _retention(width, m, eps):
@@ -43,49 +33,19 @@ def _attention(width, m, eps):
 MIXERS = {"retention": _retention, "mamba2": _mamba2, "attention": _attention}
 
 
-class DafovikConfig(PretrainedConfig):
-    """``layers``: one entry per layer with ``type`` (a key of ``MIXERS``), ``mixer`` (its sizes and constants) and ``mlp``
-    ({"kind": "dense", "ff": n} or None); ``norm.eps``, ``residual_mult``, ``vocab``, ``width``."""
+class DafovikConfig(HybridConfig):
+    """``mlp``: {"kind": "dense", "ff": n} or None; ``residual_mult`` beside the entries of ``HybridConfig``."""
 
     model_type = "dafovik"
+    architecture = "Dafovik"
+    mixers = MIXERS
+    feed_forwards = {"dense": GeluMLP}
+    checkpoint_keys = ("layers", "norm", "residual_mult", "vocab", "width")
 
     def __init__(self, layers: Optional[List[dict]] = None, norm: Optional[dict] = None, residual_mult: float = 1.0,
                  vocab: int = 256, width: int = 64, **kwargs):
-        self.layers = list(layers or [])
-        self.norm = dict(norm or {"eps": 1e-6})
-        self.residual_mult, self.vocab, self.width = float(residual_mult), int(vocab), int(width)
-        for i, layer in enumerate(self.layers):
-            if layer["type"] not in MIXERS:
-                raise ValueError(f"layer {i}: unknown mixer {layer['type']!r} (known: {sorted(MIXERS)})")
-            mlp = layer.get("mlp")
-            if mlp is not None and mlp.get("kind", "dense") != "dense":
-                raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r} (known: 'dense' or null)")
-        # the names the rest of the framework and HF generation read
-        self.vocab_size, self.hidden_size, self.num_hidden_layers = self.vocab, self.width, len(self.layers)
-        self.initializer_range = kwargs.pop("initializer_range", 0.02)
-        self.fused_decode_step = kwargs.pop("fused_decode_step", False)
-        self.compress_memory = False                     # nothing of this design's state is ever evicted
-        kwargs.pop("architecture", None)
-        kwargs.setdefault("tie_word_embeddings", False)
-        super().__init__(**kwargs)
-
-    @classmethod
-    def from_pretrained(cls, path, **kwargs):
-        file = os.path.join(path, "config.json") if os.path.isdir(path) else path
-        with open(file) as f:
-            return cls(**{**json.load(f), **kwargs})
-
-    def checkpoint_dict(self) -> dict:
-        return {"architecture": "Dafovik", "layers": self.layers, "norm": self.norm, "residual_mult": self.residual_mult,
-                "vocab": self.vocab, "width": self.width}
-
-
-class CentredNorm(nn.Module):
-    """Weight of an RMS norm stored around zero (the kernels add the one)."""
-
-    def __init__(self, width: int):
-        super().__init__()
-        self.weight = nn.Parameter(torch.zeros(width))
+        self.residual_mult = float(residual_mult)
+        super().__init__(layers, norm, vocab, width, **kwargs)
 
 
 class DafovikLayer(nn.Module):
@@ -94,9 +54,15 @@ class DafovikLayer(nn.Module):
         spec = config.layers[idx]
         self.eps, self.mult = float(config.norm["eps"]), config.residual_mult
         self.mix: Mixer = MIXERS[spec["type"]](config.width, spec["mixer"], self.eps)
-        self.norm1 = CentredNorm(config.width)
+        self.norm1 = StreamNorm(config.width, centre=0.0)
         self.mlp = GeluMLP(config.width, spec["mlp"]["ff"]) if spec.get("mlp") is not None else None
-        self.norm2 = CentredNorm(config.width) if self.mlp is not None else None
+        self.norm2 = StreamNorm(config.width, centre=0.0) if self.mlp is not None else None
+
+    def checkpoint(self):
+        out = {"norm1": self.norm1.weight, **{f"mix.{k}": v for k, v in self.mix.checkpoint().items()}}
+        if self.mlp is not None:
+            out.update({"norm2": self.norm2.weight, **{f"mlp.{k}": v for k, v in self.mlp.checkpoint().items()}})
+        return out
 
     def forward(self, stream: torch.Tensor, copy: Optional[torch.Tensor], batch: StepBatch, data: dict) -> None:
         """Updates the fp32 stream and its copy in the model type (None: the stream is in the model type) in place."""
@@ -106,210 +72,17 @@ class DafovikLayer(nn.Module):
             ops.postnorm_add(stream, self.mlp(x), as_f32(self.norm2, "weight"), copy, self.eps, self.mult, 1.0)
 
 
-class DafovikPreTrainedModel(TrimKVPreTrainedModel):
+class DafovikModel(HybridModel):
     config_class = DafovikConfig
     _no_split_modules = ["DafovikLayer"]
-
-    def _init_weights(self, module):
-        std = self.config.initializer_range
-        if isinstance(module, (Mixer, GeluMLP)):
-            module.reset_parameters(std)
-        elif isinstance(module, CentredNorm):
-            nn.init.zeros_(module.weight)
-        elif not isinstance(module, FusedProjection):     # its mixer fills it
-            super()._init_weights(module)
-
-    @classmethod
-    def from_pretrained(cls, pretrained_model_name_or_path, *, dtype=None, torch_dtype=None, device=None, device_map=None, **kwargs):
-        """``config.json`` and ``model.safetensors`` of a local folder.  Every tensor the configuration calls for must be there
-        in the right shape, and nothing else."""
-        path = pretrained_model_name_or_path
-        if not os.path.isdir(path):
-            raise ValueError(f"Path {path} does not exist.")
-        config = DafovikConfig.from_pretrained(path, **kwargs)
-        dtype = dtype or torch_dtype or torch.bfloat16
-        if isinstance(dtype, str):
-            dtype = getattr(torch, dtype)
-        if dtype not in (torch.bfloat16, torch.float32):
-            raise ValueError(f"dtype {dtype}: this design runs in bfloat16 or float32")
-        device = torch.device(device if device is not None else (device_map if isinstance(device_map, (str, torch.device)) else "cpu"))
-        with torch.device("meta"):
-            model = cls(config)
-        model = model.to(dtype).to_empty(device=device)
-        model.load_checkpoint(os.path.join(path, "model.safetensors"))
-        return model.eval()
+    layer_cls = DafovikLayer
+    norm_centre = 0.0
 
 
-class DafovikModel(DafovikPreTrainedModel):
-    def __init__(self, config: DafovikConfig):
-        super().__init__(config)
-        self.embed_tokens = nn.Embedding(config.vocab, config.width)
-        self.layers = nn.ModuleList([DafovikLayer(config, i) for i in range(len(config.layers))])
-        self.norm = CentredNorm(config.width)
-        self.post_init()
-
-    def get_input_embeddings(self):
-        return self.embed_tokens
-
-    def set_input_embeddings(self, value):
-        self.embed_tokens = value
-
-    def step(self, ids: torch.Tensor, batch: StepBatch, cache: HybridStateCache, layers_out: Optional[list] = None) -> torch.Tensor:
-        """Packed token ids ``[tokens]`` of a begun step -> the fp32 residual stream ``[tokens, width]``."""
-        w = self.embed_tokens.weight
-        stream = torch.empty(batch.tokens, w.shape[1], dtype=torch.float32, device=w.device)
-        copy = None if w.dtype == torch.float32 else torch.empty(batch.tokens, w.shape[1], dtype=w.dtype, device=w.device)
-        ops.embed_stream(ids, w, stream, copy, batch.status)
-        for i, layer in enumerate(self.layers):
-            layer(stream, copy, batch, cache.arrays(i))
-            if layers_out is not None:
-                layers_out.append(stream.clone())
-        return stream
-
-    def final_norm(self, stream: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
-        """The normed stream in the model type, of all rows or of those named by ``rows`` (int32)."""
-        w = self.embed_tokens.weight
-        out = torch.empty(stream.shape[0] if rows is None else rows.shape[0], w.shape[1], dtype=w.dtype, device=w.device)
-        ops.stream_norm(stream, rows, as_f32(self.norm, "weight"), out, self.config.norm["eps"], 1.0)
-        return out
-
-    def compress_after_forward(self, past_key_values) -> None:
-        """Windows and states are bounded by construction: nothing to evict at the end of a step."""
-
-    def forward(self, input_ids=None, attention_mask=None, past_key_values: Optional[HybridStateCache] = None, **_unused):
-        return BaseModelOutputWithPast(last_hidden_state=None, past_key_values=past_key_values)
-
-
-class DafovikForCausalLM(DafovikPreTrainedModel, TrimKVForCausalLM):
+class DafovikForCausalLM(HybridForCausalLM):
+    config_class = DafovikConfig
+    _no_split_modules = ["DafovikLayer"]
     model_cls = DafovikModel
-    cache_cls = HybridStateCache
-    decode_dtypes = (torch.bfloat16, torch.float32)
-    _tied_weights_keys = {}
-
-    # ------------------------------------------------------------------ checkpoints
-    def checkpoint_tensors(self) -> Dict[str, torch.Tensor]:
-        """The names a checkpoint uses -> the parameters (or the parts of fused ones) they fill."""
-        m = self.model
-        out = {"embed": m.embed_tokens.weight, "final.norm": m.norm.weight, "head": self.lm_head.weight}
-        for i, layer in enumerate(m.layers):
-            out[f"l{i}.norm1"] = layer.norm1.weight
-            out.update({f"l{i}.mix.{k}": v for k, v in layer.mix.checkpoint().items()})
-            if layer.mlp is not None:
-                out[f"l{i}.norm2"] = layer.norm2.weight
-                out.update({f"l{i}.mlp.{k}": v for k, v in layer.mlp.checkpoint().items()})
-        return out
-
-    @torch.no_grad()
-    def load_checkpoint(self, file: str) -> None:
-        from safetensors import safe_open
-        want = self.checkpoint_tensors()
-        for p in self.parameters():                       # the padding rows of fused projections are not in a checkpoint
-            p.zero_()
-        with safe_open(file, framework="pt") as f:
-            have = set(f.keys())
-            if have != set(want):
-                raise ValueError(f"{file}: missing tensors {sorted(set(want) - have)}, unexpected tensors {sorted(have - set(want))}")
-            for name, param in want.items():
-                t = f.get_tensor(name)
-                if t.shape != param.shape:
-                    raise ValueError(f"{file}: {name} has shape {tuple(t.shape)}, the configuration says {tuple(param.shape)}")
-                param.copy_(t)
-
-    def save_checkpoint(self, path: str) -> None:
-        """``config.json`` and ``model.safetensors`` (bfloat16) as ``from_pretrained`` reads them."""
-        from safetensors.torch import save_file
-        os.makedirs(path, exist_ok=True)
-        with open(os.path.join(path, "config.json"), "w") as f:
-            json.dump(self.config.checkpoint_dict(), f, indent=1)
-        save_file({k: v.detach().to(torch.bfloat16).cpu().contiguous().clone() for k, v in self.checkpoint_tensors().items()},
-                  os.path.join(path, "model.safetensors"))
-
-    # ------------------------------------------------------------------ steps
-    def new_cache(self, device=None, capacity_tokens: int = 0) -> HybridStateCache:
-        return HybridStateCache([layer.mix.state() for layer in self.model.layers], device or self.device,
-                                self.lm_head.weight.dtype, capacity_tokens)
-
-    def head(self, normed: torch.Tensor) -> torch.Tensor:
-        """Logits in fp32."""
-        w = self.lm_head.weight
-        return F.linear(normed, w) if w.dtype == torch.float32 else torch.mm(normed, w.t(), out_dtype=torch.float32)
-
-    @torch.no_grad()
-    def forward_packed(self, ids: torch.Tensor, cache: HybridStateCache, lengths: Optional[Sequence[int]],
-                       rows: Optional[Sequence[int]] = None, want: Optional[Sequence[int]] = None,
-                       layers_out: Optional[list] = None) -> torch.Tensor:
-        """One step of any requests of the batch: packed ids ``[sum(lengths)]`` -> fp32 logits ``[wanted, vocab]``.
-        ``lengths`` None: one token per request.  ``want``: packed places (None: every token)."""
-        if not ids.is_cuda:
-            raise ops._lib.TrimKVNativeError("this model runs on CUDA tensors only (no CPU path)")
-        batch = cache.begin(lengths, rows)
-        if ids.shape[0] != batch.tokens:
-            raise ValueError(f"{ids.shape[0]} token ids for {batch.tokens} tokens")
-        stream = self.model.step(ids, batch, cache, layers_out)
-        at = None
-        if want is not None:
-            if len(want) == 0:
-                return stream.new_empty(0, self.config.vocab)
-            at = torch.tensor(list(want), dtype=torch.int32).to(ids.device, non_blocking=True)
-        return self.head(self.model.final_norm(stream, at))
-
-    def decode_step(self, ids: torch.Tensor, cache: HybridStateCache) -> torch.Tensor:
-        """One token of every request of the batch, ids ``[B]`` on the device -> fp32 logits ``[B, vocab]``.  Recordable in a
-        CUDA graph once it has run on this batch."""
-        stream = self.model.step(ids, cache.begin(None), cache)
-        return self.head(self.model.final_norm(stream))
-
-    def forward(self, input_ids=None, attention_mask=None, position_ids=None, past_key_values=None, inputs_embeds=None,
-                use_cache=None, cache_position=None, logits_to_keep=0, **kwargs):
-        """HF call form.  ``attention_mask`` ``[B, >= S]`` marks the padding of unequal prompts, on either side; positions are
-        counted per request.  ``logits_to_keep=1``: every request's last token; 0: all places (zeros at padding)."""
-        if input_ids is None or inputs_embeds is not None:
-            raise ValueError("this model takes input_ids")
-        cache = past_key_values if past_key_values is not None else self.new_cache(input_ids.device)
-        bsz, width = input_ids.shape
-        if cache._batch == 0:
-            cache.open(bsz)
-        if cache._batch != bsz:
-            raise ValueError(f"{bsz} rows for a cache of {cache._batch} requests")
-        step = self._fused_step_for(input_ids, cache, inputs_embeds, kwargs)
-        if step is not None:
-            logits = step(cache, input_ids, torch.zeros(1, dtype=torch.int64, device=input_ids.device))
-            return CausalLMOutputWithPast(logits=logits[:, None, :], past_key_values=cache)
-        if width == 1:
-            logits = self.forward_packed(input_ids.reshape(-1), cache, None)
-            return CausalLMOutputWithPast(logits=logits[:, None, :], past_key_values=cache)
-        live = None
-        if attention_mask is not None and attention_mask.dim() == 2:
-            live = attention_mask[:, -width:].bool()
-            if bool(live.all()):
-                live = None
-        lengths = [width] * bsz if live is None else live.sum(1).tolist()
-        rows = [b for b in range(bsz) if lengths[b] > 0]  # a portion that is padding only for some requests
-        ids = input_ids.reshape(-1) if live is None else input_ids[live]
-        counts = [lengths[b] for b in rows]
-        if logits_to_keep == 1:
-            ends, at = [], -1
-            for n in counts:
-                at += n
-                ends.append(at)
-            got = self.forward_packed(ids, cache, counts, rows, ends)
-            logits = got if len(rows) == bsz else got.new_zeros(bsz, got.shape[1]).index_copy_(0, torch.tensor(rows, device=got.device), got)
-            return CausalLMOutputWithPast(logits=logits[:, None, :], past_key_values=cache)
-        got = self.forward_packed(ids, cache, counts, rows)
-        if live is None:
-            logits = got.view(bsz, width, -1)
-        else:
-            logits = got.new_zeros(bsz, width, got.shape[1])
-            logits[live] = got
-        if not isinstance(logits_to_keep, int):
-            logits = logits[:, logits_to_keep]
-        elif logits_to_keep:
-            logits = logits[:, -logits_to_keep:]
-        return CausalLMOutputWithPast(logits=logits, past_key_values=cache)
-
-    def _decode_step_cls(self):
-        from .decoder import HybridDecodeStep
-        return HybridDecodeStep
 
 
 __all__ = ["DafovikConfig", "DafovikForCausalLM", "DafovikModel"]

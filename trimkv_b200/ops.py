@@ -422,7 +422,7 @@ update_flatten_view_triton = update_flatten_view  # the reference's name for the
 
 
 # --------------------------------------------------------------------------------------------------------------------
-# Decoders with recurrent layers and windowed differential attention.  ``batch`` is a ``state_cache.StepBatch``: packed
+# Decoders with recurrent layers, windowed attention and experts.  ``batch`` is a ``state_cache.StepBatch``: packed
 # tokens, ``cu`` (None in a one-token step), ``slots`` and ``pos0`` of the step's requests.
 
 def batch_begin(lens, slots, cu, pos0) -> None:
@@ -431,9 +431,9 @@ def batch_begin(lens, slots, cu, pos0) -> None:
     _count(1)
 
 
-def embed_stream(ids, table, stream, copy, status=None) -> None:
+def embed_stream(ids, table, stream, copy, status=None, scale: float = 1.0) -> None:
     check(lib().tkv_embed_stream(ids.data_ptr(), table.data_ptr(), table.shape[0], stream.data_ptr(), _ptr(copy), stream.shape[0],
-                                 stream.shape[1], dtype_code(table.dtype), _ptr(status), _stream(ids)), "tkv_embed_stream")
+                                 stream.shape[1], float(scale), dtype_code(table.dtype), _ptr(status), _stream(ids)), "tkv_embed_stream")
     _count(1)
 
 
@@ -445,18 +445,39 @@ def postnorm_add(stream, y, weight, copy, eps: float, mult: float, weight_offset
     _count(1)
 
 
-def stream_norm(stream, rows, weight, out, eps: float, weight_offset: float) -> None:
-    """RMS norm of the stream's rows (``rows`` int32, or None: all) into ``out``."""
-    check(lib().tkv_stream_norm(stream.data_ptr(), _ptr(rows), weight.data_ptr(), out.data_ptr(), out.shape[0], out.shape[1],
+def gated_sum_norm(stream, y, weight, copy, groups: int, eps: float, alpha: float, gate=None, gate_bias=None, place=None,
+                   choice_weight=None) -> None:
+    """``stream = GroupRMSNorm(alpha * stream + sigmoid(gate + gate_bias) * y) * weight`` (fp32, in place); ``copy`` (or None):
+    the result in y's type.  ``place`` / ``choice_weight`` ``[rows, top]``: y holds expert rows to be gathered and added up
+    (place -1: the stream itself)."""
+    check(lib().tkv_gated_sum_norm(stream.data_ptr(), y.data_ptr(), _ptr(place), _ptr(choice_weight), 0 if place is None else place.shape[1],
+                                   _ptr(gate), 0 if gate is None else gate.stride(0), _ptr(gate_bias), weight.data_ptr(), _ptr(copy),
+                                   stream.shape[0], stream.shape[1], groups, float(eps), float(alpha), dtype_code(y.dtype),
+                                   _stream(stream)), "tkv_gated_sum_norm")
+    _count(1)
+
+
+def stream_norm(stream, rows, weight, out, eps: float, weight_offset: float, groups: int = 1) -> None:
+    """RMS norm of the stream's rows (``rows`` int32, or None: all) into ``out``, in ``groups`` equal parts."""
+    check(lib().tkv_stream_norm(stream.data_ptr(), _ptr(rows), weight.data_ptr(), out.data_ptr(), out.shape[0], out.shape[1], groups,
                                 float(eps), float(weight_offset), dtype_code(out.dtype), _stream(stream)), "tkv_stream_norm")
     _count(1)
 
 
-def gated_norm(y, z, weight, out, groups: int, eps: float, gate_first: bool) -> None:
-    """Group RMS norm with a SiLU gate before (times ``weight``) or after it; ``z`` may be a column slice of a wider array."""
-    check(lib().tkv_gated_norm(y.data_ptr(), y.stride(0), z.data_ptr(), z.stride(0), _ptr(weight), out.data_ptr(), out.shape[0],
-                               groups, out.shape[1] // groups, float(eps), int(gate_first), dtype_code(out.dtype), _stream(y)),
-          "tkv_gated_norm")
+def gated_norm(y, z, weight, out, groups: int, eps: float, gate_first: bool = False) -> None:
+    """Group RMS norm with a SiLU gate before (times ``weight``) or after it; ``z`` may be None (no gate) or a column slice of a
+    wider array; a ``weight`` of one group's length serves all groups."""
+    shared = weight is not None and weight.numel() * groups == out.shape[1] and groups > 1
+    check(lib().tkv_gated_norm(y.data_ptr(), y.stride(0), _ptr(z), 0 if z is None else z.stride(0), _ptr(weight), int(shared),
+                               out.data_ptr(), out.shape[0], groups, out.shape[1] // groups, float(eps), int(gate_first),
+                               dtype_code(out.dtype), _stream(y)), "tkv_gated_norm")
+    _count(1)
+
+
+def swiglu(u, out) -> None:
+    """``out = SiLU(u[:, :ff]) * u[:, ff:2 ff]``, ``ff`` the width of ``out``; u may have further columns."""
+    check(lib().tkv_swiglu(u.data_ptr(), u.stride(0), out.data_ptr(), out.shape[0], out.shape[1], dtype_code(out.dtype), _stream(u)),
+          "tkv_swiglu")
     _count(1)
 
 
@@ -561,3 +582,99 @@ def diff_attention(proj, gate, q_norm, k_norm, k_ring, v_ring, batch, lam, diff:
                                 gate.stride(0), out.data_ptr(), _ptr(ws), need, batch.size, heads, kv_heads, dim, vdim, dp, pp, dt,
                                 _stream(proj)), "tkv_diff_decode")
     _count(3 if need else 2)
+
+
+# ---- channel-decay recurrence
+def chanrec_step(q, f, v, f_bias, lower, norm, state, batch, out, eps: float) -> None:
+    """One token per request; ``q``, ``f``, ``v`` are column slices of one projection, ``out`` is normed per head."""
+    _, heads, n, p = state.shape
+    check(lib().tkv_chanrec_step(q.data_ptr(), f.data_ptr(), v.data_ptr(), q.stride(0), f_bias.data_ptr(), lower.data_ptr(), norm.data_ptr(),
+                                 float(eps), out.data_ptr(), state.data_ptr(), batch.slots.data_ptr(), batch.pos0.data_ptr(), batch.size,
+                                 heads, n, p, dtype_code(out.dtype), _stream(out)), "tkv_chanrec_step")
+    _count(1)
+
+
+def chanrec(q, f, v, f_bias, lower, state, batch, out, force_scan: bool = False) -> None:
+    """The recurrence over the packed tokens of ``batch`` (see tkv_chanrec_scan in the header)."""
+    _, heads, n, p = state.shape
+    check(lib().tkv_chanrec_scan(q.data_ptr(), f.data_ptr(), v.data_ptr(), q.stride(0), f_bias.data_ptr(), lower.data_ptr(), out.data_ptr(),
+                                 state.data_ptr(), batch.slots.data_ptr(), _ptr(batch.cu), batch.pos0.data_ptr(), batch.size, heads, n, p,
+                                 dtype_code(out.dtype), _stream(out)), "tkv_chanrec_scan")
+    _count(1)
+
+
+# ---- latent attention
+def rotate_pairs(x, batch, heads: int, head_len: int, offset: int, rot_dims: int, freq) -> None:
+    """Rotary positions (pairs of neighbours) in place on a part of every head; ``x`` [tokens, >= heads * head_len]."""
+    check(lib().tkv_rotate_pairs(x.data_ptr(), x.stride(0), _ptr(batch.cu), batch.pos0.data_ptr(), batch.size, batch.tokens, heads,
+                                 head_len, offset, rot_dims, freq.data_ptr(), dtype_code(x.dtype), _stream(x)), "tkv_rotate_pairs")
+    _count(1)
+
+
+def latent_prep(u, q_norm, kv_norm, eps: float, rot_dim: int, rot_dims: int, freq, ring, batch, window: int):
+    """Query latent ``[tokens, q_rank]`` and (steps of several tokens) the linear buffer ``[rows, lw]`` of a step; stores the
+    latents of its tokens in ``ring`` [slots, rows, lw]."""
+    q_rank, kv_rank = q_norm.shape[0], kv_norm.shape[0]
+    cq = torch.empty(batch.tokens, q_rank, dtype=u.dtype, device=u.device)
+    lin = kv_start = None
+    hist = 0
+    if batch.cu is not None:
+        kv_start, rows, hist = batch.window_plan(window)
+        lin = torch.empty(rows, ring.shape[2], dtype=u.dtype, device=u.device)
+    check(lib().tkv_latent_prep(u.data_ptr(), u.stride(0), q_norm.data_ptr(), kv_norm.data_ptr(), float(eps), q_rank, kv_rank, rot_dim,
+                                rot_dims, freq.data_ptr(), cq.data_ptr(), ring.data_ptr(), ring.shape[1], _ptr(lin), _ptr(kv_start),
+                                _ptr(batch.cu), batch.slots.data_ptr(), batch.pos0.data_ptr(), batch.size, batch.tokens, hist, window,
+                                dtype_code(u.dtype), _stream(u)), "tkv_latent_prep")
+    _count(2 if hist else 1)
+    return cq, lin
+
+
+def latent_prefill(q, kv, lin, batch, scale: float, out, heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int, window: int) -> None:
+    """``q`` [tokens, heads * (dim + rot_dim)] rotated, ``kv`` [rows, >= heads * (dim + vdim)] keys and values of ``lin``'s rows."""
+    kv_start, rows, _ = batch.window_plan(window)
+    check(lib().tkv_latent_prefill(q.data_ptr(), q.stride(0), kv.data_ptr(), kv.stride(0), lin.data_ptr(), kv_start.data_ptr(), rows,
+                                   batch.cu.data_ptr(), batch.pos0.data_ptr(), float(scale), out.data_ptr(), batch.size, batch.tokens,
+                                   batch.max_tokens, heads, dim, rot_dim, vdim, kv_rank, window, dtype_code(q.dtype), _ptr(batch.status),
+                                   _stream(q)), "tkv_latent_prefill")
+    _count(1)
+
+
+def latent_decode(q_abs, q, rot_dim: int, freq, ring, batch, scale: float, out, rot_dims: int) -> None:
+    """One token per request: ``q_abs`` [B, heads, kv_rank], ``q`` [B, heads, dim + rot_dim] whose last part is not yet rotated
+    (it is rotated in place where the form for every size runs), ``out`` [B, heads, kv_rank]; ``q_abs`` and ``out`` with any
+    token and head strides."""
+    bsz, heads, rank = q_abs.shape
+    dt, q_rot = dtype_code(q_abs.dtype), q[:, :, q.shape[2] - rot_dim:]
+    need = lib().tkv_latent_decode_workspace_bytes(bsz, heads, rank, rot_dim, ring.shape[1], dt)
+    if need < 0 and rot_dims:
+        rotate_pairs(q.view(bsz, -1), batch, heads, q.shape[2], q.shape[2] - rot_dim, rot_dims, freq)
+    ws = torch.empty(need, dtype=torch.uint8, device=out.device) if need > 0 else None
+    check(lib().tkv_latent_decode(q_abs.data_ptr(), q_abs.stride(0), q_abs.stride(1), q_rot.data_ptr(), q_rot.stride(0), q_rot.stride(1),
+                                  freq.data_ptr(), ring.data_ptr(), ring.shape[1], batch.slots.data_ptr(), batch.pos0.data_ptr(),
+                                  float(scale), out.data_ptr(), out.stride(0), out.stride(1), _ptr(ws), max(need, 0), bsz, heads, rank,
+                                  rot_dim, rot_dims, dt, _stream(out)), "tkv_latent_decode")
+    _count(2 if need > 0 else 1)
+
+
+# ---- mixture of experts
+def moe_route(logits, correction, identity: int, top: int, groups: int, keep: int, scale: float):
+    """``(place [T, top], weight [T, top], src [T * top], offsets)`` of fp32 router logits (see tkv_moe_route in the header)."""
+    T, E = logits.shape
+    dev = logits.device
+    ints = torch.empty(3 * T * top + E - identity + 1, dtype=torch.int32, device=dev)
+    place, choice, src, offsets = ints[:T * top].view(T, top), ints[T * top:2 * T * top], ints[2 * T * top:3 * T * top], ints[3 * T * top:]
+    weight = torch.empty(T, top, dtype=torch.float32, device=dev)
+    counts = torch.zeros(E, dtype=torch.int32, device=dev) if T > 128 else None
+    check(lib().tkv_moe_route(logits.data_ptr(), logits.stride(0), correction.data_ptr(), T, E, identity, top, groups, keep, float(scale),
+                              weight.data_ptr(), choice.data_ptr(), place.data_ptr(), src.data_ptr(), _ptr(counts), offsets.data_ptr(),
+                              _stream(logits)), "tkv_moe_route")
+    _count(2 if T > 128 else 1)
+    return place, weight, src, offsets
+
+
+def moe_gemm(a, w, offsets, out, src=None, act: str = "none", status=None) -> None:
+    """Grouped product: ``out[r] = act(a[src[r] or r] @ w[e].T)`` for the rows r of expert e; ``w`` [experts, n, k]."""
+    check(lib().tkv_moe_gemm(a.data_ptr(), a.stride(0), a.shape[0], _ptr(src), w.data_ptr(), offsets.data_ptr(), out.data_ptr(), out.shape[0],
+                             w.shape[0], w.shape[1], w.shape[2], {"none": 0, "gelu": 1}[act], dtype_code(a.dtype), _ptr(status),
+                             _stream(a)), "tkv_moe_gemm")
+    _count(1)

@@ -8,11 +8,13 @@ import torch
 
 from .modeling_dafovik import DafovikForCausalLM
 from .modeling_llama import TrimKVLlamaForCausalLM
+from .modeling_lonulix import LonulixForCausalLM
 from .modeling_phi3 import TrimKVPhi3ForCausalLM
 from .modeling_qwen3 import TrimKVQwen3ForCausalLM
 
 MODEL_CLASSES = {
     "Dafovik": DafovikForCausalLM, "dafovik": DafovikForCausalLM, "DafovikForCausalLM": DafovikForCausalLM,
+    "Lonulix": LonulixForCausalLM, "lonulix": LonulixForCausalLM, "LonulixForCausalLM": LonulixForCausalLM,
     "TrimKVQwen3ForCausalLM": TrimKVQwen3ForCausalLM, "Qwen3ForCausalLM": TrimKVQwen3ForCausalLM, "qwen3": TrimKVQwen3ForCausalLM,
     "TrimKVLlamaForCausalLM": TrimKVLlamaForCausalLM, "LlamaForCausalLM": TrimKVLlamaForCausalLM, "llama": TrimKVLlamaForCausalLM,
     "TrimKVPhi3ForCausalLM": TrimKVPhi3ForCausalLM, "Phi3ForCausalLM": TrimKVPhi3ForCausalLM, "phi3": TrimKVPhi3ForCausalLM,

@@ -6,7 +6,8 @@ past.  A request owns one *slot*, the same in every layer's arrays:
   * ``RecurrentState``: fp32 state ``[slots, heads, n, p]`` and, where the layer has a short convolution, a ring of its last
     ``taps`` inputs ``[slots, taps, channels]`` (input of position p in row p mod taps);
   * ``WindowState``: keys and values of the last ``window`` positions, ``[slots, kv_heads, rows, ...]`` with position p in row
-    p mod rows; rows grow with the sequences up to the window and then stay.
+    p mod rows; rows grow with the sequences up to the window and then stay;
+  * ``LatentState``: the same for latent attention, one row per position that all heads share, ``[slots, rows, ...]``.
 
 Nothing is cleared when a slot is given back and taken again: every kernel starts a request at position 0 from the empty
 state.  Lengths may differ between the requests of a batch; tokens of a step are packed (``StepBatch``), so no kernel sees
@@ -30,6 +31,14 @@ class RecurrentState:
     p: int
     conv_taps: int = 0
     conv_channels: int = 0
+    window = 0
+
+    def arrays(self, rows: int, dtype):
+        """name -> (shape of a slot, type, axis of the ring rows or None)"""
+        out = {"state": ((self.heads, self.n, self.p), torch.float32, None)}
+        if self.conv_taps:
+            out["conv"] = ((self.conv_taps, self.conv_channels), dtype, None)
+        return out
 
 
 @dataclass(frozen=True)
@@ -39,6 +48,18 @@ class WindowState:
     pp: int          # padded value size
     window: int
     maps: int = 2
+
+    def arrays(self, rows: int, dtype):
+        return {"k": ((self.kv_heads, rows, self.maps, self.dp), dtype, 1), "v": ((self.kv_heads, rows, self.pp), dtype, 1)}
+
+
+@dataclass(frozen=True)
+class LatentState:
+    row: int         # elements of a position: padded latent and padded rotated key part
+    window: int
+
+    def arrays(self, rows: int, dtype):
+        return {"latent": ((rows, self.row), dtype, 0)}
 
 
 @dataclass
@@ -148,7 +169,7 @@ class HybridStateCache:
     def get_cache_length(self, layer_idx: int = 0) -> int:
         """Positions a layer holds something of: its window's rows, or 0 for a layer whose past is a state."""
         st = self.layers[layer_idx]
-        return min(self.get_seq_length(), st.window) if isinstance(st, WindowState) else 0
+        return min(self.get_seq_length(), st.window)
 
     def get_mask_sizes(self, cache_position, layer_idx: int = 0):
         n = cache_position if isinstance(cache_position, int) else cache_position.shape[0]
@@ -226,12 +247,12 @@ class HybridStateCache:
         cap = max(tokens, 2 * self._cap)
         before, self._cap = self._cap, cap
         for st, data in zip(self.layers, self._data):
-            if isinstance(st, WindowState) and data and min(st.window, cap) > min(st.window, before):
+            if data and min(st.window, cap) > min(st.window, before):
                 # no sequence has wrapped yet (rows < window), so a position keeps its row
-                for name in ("k", "v"):
+                for name, (shape, dtype, axis) in st.arrays(min(st.window, cap), self.dtype).items():
                     old = data[name]
-                    new = old.new_empty(*old.shape[:2], min(st.window, cap), *old.shape[3:])
-                    new[:, :, :old.shape[2]] = old
+                    new = torch.empty(self._nslots, *shape, dtype=dtype, device=self.device)
+                    new.narrow(axis + 1, 0, old.shape[axis + 1]).copy_(old)
                     data[name] = new
                 self._generation += 1
 
@@ -247,14 +268,8 @@ class HybridStateCache:
         if self._status is None:
             self._status = ops.new_status(self.device)
         for st, data in zip(self.layers, self._data):
-            if isinstance(st, WindowState):
-                rows = min(st.window, self._cap)
-                data["k"] = grown(data.get("k"), st.kv_heads, rows, st.maps, st.dp, dtype=self.dtype)
-                data["v"] = grown(data.get("v"), st.kv_heads, rows, st.pp, dtype=self.dtype)
-            else:
-                data["state"] = grown(data.get("state"), st.heads, st.n, st.p, dtype=torch.float32)
-                if st.conv_taps:
-                    data["conv"] = grown(data.get("conv"), st.conv_taps, st.conv_channels, dtype=self.dtype)
+            for name, (shape, dtype, _) in st.arrays(min(st.window, self._cap), self.dtype).items():
+                data[name] = grown(data.get(name), *shape, dtype=dtype)
         lens = torch.zeros(nslots, dtype=torch.int32, device=self.device)
         if self._lens is not None:
             lens[:self._nslots] = self._lens
@@ -264,4 +279,4 @@ class HybridStateCache:
         self._generation += 1
 
 
-__all__ = ["HybridStateCache", "RecurrentState", "StepBatch", "WindowState"]
+__all__ = ["HybridStateCache", "LatentState", "RecurrentState", "StepBatch", "WindowState"]
