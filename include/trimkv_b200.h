@@ -568,6 +568,11 @@ int tkv_chanrec_scan(const void* q, const void* f, const void* v, int64_t row_st
                      void* out, float* state, const int32_t* slots, const int32_t* cu_tokens, const int32_t* pos0, int batch,
                      int heads, int n, int vdim, int dtype, tkv_stream_t stream);
 
+int64_t tkv_chanrec_chunk_workspace_bytes(int batch, int max_tokens, int heads, int n, int vdim, int dtype);
+int tkv_chanrec_chunk(const void* q, const void* f, const void* v, int64_t row_stride, const float* f_bias, const float* lower,
+                      void* out, float* state, const int32_t* slots, const int32_t* cu_tokens, const int32_t* pos0, void* workspace,
+                      int64_t workspace_bytes, int batch, int max_tokens, int heads, int n, int vdim, int dtype, tkv_stream_t stream);
+
 /* Rotary positions in place on elements offset .. offset + rot_dims of every head of head_len elements: the pair (2i, 2i + 1)
  * turns by position * f_i, freq_hi_lo[i] = {f_i rounded to fp32, the rest}. */
 int tkv_rotate_pairs(void* x, int64_t row_stride, const int32_t* cu_tokens, const int32_t* pos0, int batch, int tokens, int heads,

@@ -338,6 +338,19 @@ int make_map_2d(CUtensorMap* map, const void* base, int64_t cols, int64_t rows, 
   return TKV_OK;
 }
 
+int make_map_rows(CUtensorMap* map, const void* base, int64_t cols, int64_t rows, int64_t row_stride, int box_cols, int box_rows) {
+  EncodeTiledFn fn = encode_fn();
+  if (fn == nullptr) return fail(TKV_ERR_LAUNCH, "cuTensorMapEncodeTiled is not available");
+  const cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
+  const cuuint64_t strides[1] = {(cuuint64_t)row_stride * 2};
+  const cuuint32_t box[2] = {(cuuint32_t)box_cols, (cuuint32_t)box_rows};
+  const cuuint32_t estr[2] = {1, 1};
+  CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                  CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (r != CUDA_SUCCESS) return fail(TKV_ERR_LAUNCH, "cuTensorMapEncodeTiled failed with %d", (int)r);
+  return TKV_OK;
+}
+
 int make_map_3d_bf16(CUtensorMap* map, const void* base, int64_t inner, int64_t mid, int64_t outer, int64_t outer_stride, int box_inner,
                      int box_outer) {
   EncodeTiledFn fn = encode_fn();

@@ -1,0 +1,430 @@
+// Chunked form of the channel-decay recurrence (tkv_chanrec.cuh) for prompts, 16-bit operands with fp32 state.
+//
+// A block of 16 tokens, with P_i the product of the forget gates of its tokens up to i (per state row), S the state before it:
+//   a_ij = (q_i P_i) . (k_j / P_j)           j <= i, k = 1 - f
+//   o_i  = S^T (q_i P_i) + sum_j a_ij v_j
+//   S   <- diag(P_16) (S + sum_j (k_j / P_j) v_j^T) .
+// The scaled vectors q P and k / P are fp32 and enter the 16-bit products as a high and a low part, as do the state and a; v is
+// 16-bit exactly.  Where the product of a row falls below kFloor within a block (gates near zero), 1 / P could leave the range of
+// fp32: such a chunk is walked token by token instead, in the same registers.
+//
+// One CTA walks chunks of 32 tokens (two blocks) of one (request, head, block of 16 * kWarps value columns, segment of the
+// sequence).  The state never leaves registers: a warp owns 16 columns of v and holds S^T [16 x n] as fp32 MMA accumulators, whose
+// layout is also the A-operand layout of the read-out.  Per chunk: gates and scaled vectors of all channels (a thread walks a
+// channel of a block), the two 16 x 16 blocks a, then every warp its own columns without further barriers.
+// Where (request, head, column) blocks alone do not fill the GPU, the sequence is cut into segments: a first pass computes
+// every segment's own state, a small kernel chains them, and the main pass starts each segment from its true state.
+#include "tkv_chanrec.cuh"
+#include "tkv_tc.cuh"
+
+namespace tkv {
+
+constexpr int kCrTokens = 32, kCrBlock = 16;
+constexpr float kFloor = 1e-24f;
+
+__device__ __forceinline__ void cr_mma(float* d, const uint32_t* a, uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void cr_ldm(uint32_t* r, const __nv_bfloat16* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)) : "memory");
+}
+__device__ __forceinline__ void cr_ldmt(uint32_t* r, const __nv_bfloat16* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)) : "memory");
+}
+__device__ __forceinline__ void cr_cp16(void* dst, const void* src, bool live) {
+  const int bytes = live ? 16 : 0;                        // 0: the 16 bytes are zero-filled
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(bytes) : "memory");
+}
+// x = hi + lo in bf16, two values at a time.
+__device__ __forceinline__ void cr_split(float a, float b, uint32_t* hi, uint32_t* lo) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+  *hi = *reinterpret_cast<const uint32_t*>(&h);
+  const __nv_bfloat162 l = __floats2bfloat162_rn(a - __uint_as_float(*hi << 16), b - __uint_as_float(*hi & 0xffff0000u));
+  *lo = *reinterpret_cast<const uint32_t*>(&l);
+}
+// sigmoid(x) and sigmoid(-x), each to a few units in the last place of fp32.
+__device__ __forceinline__ void cr_sigmoid(float x, float* pos, float* neg) {
+  const float e = exp2_weight(fabsf(x) * -1.4426950408889634f), r = __frcp_rn(1.0f + e);
+  const float small = e * r;
+  *pos = x >= 0.f ? r : small;
+  *neg = x >= 0.f ? small : r;
+}
+
+template <int NP, int kWarps> struct CrSmem {
+  static constexpr int PT = kWarps * 16, QS = NP + 8, VS = PT + 8, PS = kCrBlock + 8;
+  __nv_bfloat16 zq[2][kCrTokens * QS], zf[2][kCrTokens * QS], v[2][kCrTokens * VS];
+  __nv_bfloat16 q_hi[kCrTokens * QS], q_lo[kCrTokens * QS], k_hi[kCrTokens * QS], k_lo[kCrTokens * QS];
+  __nv_bfloat16 a_hi[2][kCrBlock * PS], a_lo[2][kCrBlock * PS];
+  float end[2][NP];                                       // product of the gates of a block
+  float gate[2][3][NP];                                   // q, f, k of one token (token-by-token path)
+};
+
+template <int NP, int kWarps, bool kStateOnly>
+__global__ void __launch_bounds__(kWarps * 32, NP == 256 ? 1 : kWarps == 8 ? 2 : 3) chanrec_chunk_kernel(ChanrecParams a, ChanrecSegs sg) {
+  using Sm = CrSmem<NP, kWarps>;
+  constexpr int PT = Sm::PT, QS = Sm::QS, VS = Sm::VS, PS = Sm::PS, kThreads = kWarps * 32;
+  extern __shared__ __align__(16) uint8_t raw[];
+  Sm& sm = *reinterpret_cast<Sm*>(raw);
+  grid_dependency_wait();
+  grid_launch_dependents();
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gr = lane >> 2, gc = lane & 3;
+  const int ptiles = (a.p + PT - 1) / PT;
+  const int per_seg = a.batch * a.heads * ptiles;
+  const int seg = blockIdx.x / per_seg, item = blockIdx.x - seg * per_seg;
+  const int pt = item % ptiles, bh = item / ptiles, b = bh / a.heads, h = bh - b * a.heads;
+  const int tok0 = a.cu[b], ntok = a.cu[b + 1] - tok0;
+  const int nchunks = (ntok + kCrTokens - 1) / kCrTokens;
+  const int per = sg.tokens / kCrTokens, c0 = seg * per, c1 = min(nchunks, c0 + per);
+  if (c0 >= c1) return;
+  if (kStateOnly && c1 == nchunks) return;                // nobody starts from the end of the last segment
+  const int pbase = pt * PT, p0 = warp * 16;              // this CTA's columns, this warp's columns within them
+  const __nv_bfloat16* Q = (const __nv_bfloat16*)a.q + (int64_t)tok0 * a.row_stride + (int64_t)h * a.n;
+  const __nv_bfloat16* F = (const __nv_bfloat16*)a.f + (int64_t)tok0 * a.row_stride + (int64_t)h * a.n;
+  const __nv_bfloat16* V = (const __nv_bfloat16*)a.v + (int64_t)tok0 * a.row_stride + (int64_t)h * a.p + pbase;
+  const float *bias = a.f_bias + (int64_t)h * a.n, *lower = a.lower + (int64_t)h * a.n;
+
+  auto fetch = [&](int chunk) {
+    const int st = chunk & 1, t0 = chunk * kCrTokens;
+    for (int i = tid; i < kCrTokens * (NP / 8); i += kThreads) {
+      const int r = i / (NP / 8), c = (i - r * (NP / 8)) * 8;
+      const bool live = t0 + r < ntok && c < a.n;
+      const int64_t at = live ? (int64_t)(t0 + r) * a.row_stride + c : 0;
+      if (!kStateOnly) cr_cp16(&sm.zq[st][r * QS + c], Q + at, live);
+      cr_cp16(&sm.zf[st][r * QS + c], F + at, live);
+    }
+    for (int i = tid; i < kCrTokens * (PT / 8); i += kThreads) {
+      const int r = i / (PT / 8), c = (i - r * (PT / 8)) * 8;
+      const bool live = t0 + r < ntok && pbase + c < a.p;
+      cr_cp16(&sm.v[st][r * VS + c], V + (live ? (int64_t)(t0 + r) * a.row_stride + c : 0), live);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  // f and k = 1 - f of a channel; a token or channel that does not exist leaves the state as it is
+  auto gate = [&](float z, float lo, bool live, float* f, float* k) {
+    float pos, neg;
+    cr_sigmoid(z, &pos, &neg);
+    *f = live ? fmaf(1.0f - lo, pos, lo) : 1.0f;
+    *k = live ? (1.0f - lo) * neg : 0.0f;
+  };
+  auto query = [&](float z) {
+    float pos, neg;
+    cr_sigmoid(z, &pos, &neg);
+    return z * pos;
+  };
+
+  // ---- state: S^T rows p0 + gr (+ 8), columns 8 nt + 2 gc (+ 1)
+  float s[NP / 8][4];
+  const int pc0 = pbase + p0 + gr, pc1 = pc0 + 8;
+  const int64_t np = (int64_t)a.n * a.p;
+  float* const final_state = a.state + ((int64_t)a.slots[b] * a.heads + h) * np;
+  {
+    const float* S = kStateOnly ? nullptr : sg.count > 1 ? sg.start + ((int64_t)bh * sg.count + seg) * np : a.pos0[b] == 0 ? nullptr : final_state;
+#pragma unroll
+    for (int nt = 0; nt < NP / 8; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int n = nt * 8 + 2 * gc + (e & 1), p = e < 2 ? pc0 : pc1;
+        s[nt][e] = (S != nullptr && n < a.n && p < a.p) ? S[(int64_t)n * a.p + p] : 0.f;
+      }
+  }
+  constexpr int kOwn = (NP + kThreads - 1) / kThreads;
+  float seg_decay[kOwn];                                  // of channels tid, tid + kThreads, ..
+#pragma unroll
+  for (int i = 0; i < kOwn; ++i) seg_decay[i] = 1.0f;
+
+  fetch(c0);
+  for (int chunk = c0; chunk < c1; ++chunk) {
+    const int st = chunk & 1, t0 = chunk * kCrTokens;
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                                       // this chunk is here; everyone is done with the last one
+    if (chunk + 1 < c1) fetch(chunk + 1);
+    // ---- gates and scaled vectors: a thread walks one channel of one block
+    bool tiny = false;
+    for (int i = tid; i < 2 * NP; i += kThreads) {
+      const int blk = i / NP, c = i - blk * NP;
+      const bool ch = c < a.n;
+      const float bi = ch ? bias[c] : 0.f, lo = ch ? lower[c] : 0.f;
+      float P = 1.0f;
+#pragma unroll
+      for (int j = 0; j < kCrBlock; ++j) {
+        const int r = blk * kCrBlock + j;
+        float f, k;
+        gate(__bfloat162float(sm.zf[st][r * QS + c]) + bi, lo, ch && t0 + r < ntok, &f, &k);
+        P *= f;
+        const float ks = __fdividef(k, P);
+        const __nv_bfloat16 kh = __float2bfloat16_rn(ks);
+        sm.k_hi[r * QS + c] = kh;
+        sm.k_lo[r * QS + c] = __float2bfloat16_rn(ks - __bfloat162float(kh));
+        if (!kStateOnly) {
+          const float qs = query(__bfloat162float(sm.zq[st][r * QS + c])) * P;
+          const __nv_bfloat16 qh = __float2bfloat16_rn(qs);
+          sm.q_hi[r * QS + c] = qh;
+          sm.q_lo[r * QS + c] = __float2bfloat16_rn(qs - __bfloat162float(qh));
+        }
+      }
+      sm.end[blk][c] = P;
+      tiny |= P < kFloor;
+    }
+    const bool walk = __syncthreads_or(tiny);
+#pragma unroll
+    for (int i = 0; i < kOwn; ++i) {
+      const int c = tid + i * kThreads;
+      if (c < NP) seg_decay[i] *= sm.end[0][c] * sm.end[1][c];
+    }
+    __nv_bfloat16* v_s = sm.v[st];
+    if (!walk) {
+      if (!kStateOnly) {
+        // ---- the blocks a: warps 0 .. 3 take (block, 8 columns)
+        if (warp < 4) {
+          const int blk = warp >> 1, jt = warp & 1;
+          float sc[3][4] = {};
+#pragma unroll 4
+          for (int kk = 0; kk < NP / 16; ++kk) {
+            uint32_t ah[4], al[4];
+            cr_ldm(ah, sm.q_hi + (blk * 16 + (lane & 15)) * QS + kk * 16 + (lane >> 4) * 8);
+            cr_ldm(al, sm.q_lo + (blk * 16 + (lane & 15)) * QS + kk * 16 + (lane >> 4) * 8);
+            const int at = (blk * 16 + jt * 8 + gr) * QS + kk * 16 + 2 * gc;
+            const uint32_t* kh = reinterpret_cast<const uint32_t*>(sm.k_hi + at);
+            const uint32_t* kl = reinterpret_cast<const uint32_t*>(sm.k_lo + at);
+            cr_mma(sc[0], ah, kh[0], kh[4]);
+            cr_mma(sc[1], ah, kl[0], kl[4]);
+            cr_mma(sc[2], al, kh[0], kh[4]);
+          }
+          const int j = jt * 8 + 2 * gc;
+#pragma unroll
+          for (int e = 0; e < 4; e += 2) {
+            const int i = gr + (e >> 1) * 8;
+            uint32_t hi, lo;
+            cr_split(j <= i ? sc[0][e] + sc[1][e] + sc[2][e] : 0.f, j + 1 <= i ? sc[0][e + 1] + sc[1][e + 1] + sc[2][e + 1] : 0.f, &hi, &lo);
+            *reinterpret_cast<uint32_t*>(sm.a_hi[blk] + i * PS + j) = hi;
+            *reinterpret_cast<uint32_t*>(sm.a_lo[blk] + i * PS + j) = lo;
+          }
+        }
+        __syncthreads();
+      }
+#pragma unroll
+      for (int blk = 0; blk < 2; ++blk) {
+        uint32_t vf[4];                                    // V^T of this warp's columns, as an A fragment
+        cr_ldmt(vf, v_s + (blk * 16 + ((lane >> 4) & 1) * 8 + (lane & 7)) * VS + p0 + ((lane >> 3) & 1) * 8);
+        if (!kStateOnly) {
+          float o[2][4] = {}, o2[2][4] = {};
+          const int qrow = (blk * 16 + ((lane >> 4) & 1) * 8 + (lane & 7)) * QS + ((lane >> 3) & 1) * 8;
+#pragma unroll
+          for (int kk = 0; kk < NP / 16; ++kk) {
+            uint32_t hi[4], lo[4], bh_[4], bl_[4];
+            cr_split(s[2 * kk][0], s[2 * kk][1], &hi[0], &lo[0]);
+            cr_split(s[2 * kk][2], s[2 * kk][3], &hi[1], &lo[1]);
+            cr_split(s[2 * kk + 1][0], s[2 * kk + 1][1], &hi[2], &lo[2]);
+            cr_split(s[2 * kk + 1][2], s[2 * kk + 1][3], &hi[3], &lo[3]);
+            cr_ldm(bh_, sm.q_hi + qrow + kk * 16);
+            cr_ldm(bl_, sm.q_lo + qrow + kk * 16);
+            cr_mma(o[0], hi, bh_[0], bh_[1]);
+            cr_mma(o[1], hi, bh_[2], bh_[3]);
+            cr_mma(o2[0], lo, bh_[0], bh_[1]);
+            cr_mma(o2[1], lo, bh_[2], bh_[3]);
+            cr_mma(o2[0], hi, bl_[0], bl_[1]);
+            cr_mma(o2[1], hi, bl_[2], bl_[3]);
+          }
+          uint32_t ph[4], pl[4];
+          const int arow = (((lane >> 4) & 1) * 8 + (lane & 7)) * PS + ((lane >> 3) & 1) * 8;
+          cr_ldm(ph, sm.a_hi[blk] + arow);
+          cr_ldm(pl, sm.a_lo[blk] + arow);
+          cr_mma(o[0], vf, ph[0], ph[1]);
+          cr_mma(o[1], vf, ph[2], ph[3]);
+          cr_mma(o2[0], vf, pl[0], pl[1]);
+          cr_mma(o2[1], vf, pl[2], pl[3]);
+          __syncwarp();
+          // over this warp's own columns of the V tile (nobody else reads them)
+#pragma unroll
+          for (int i = 0; i < 2; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+              v_s[(blk * 16 + i * 8 + 2 * gc + (e & 1)) * VS + p0 + gr + (e >> 1) * 8] = __float2bfloat16_rn(o[i][e] + o2[i][e]);
+        }
+        // ---- state
+        const int krow = (blk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * QS + ((lane >> 4) & 1) * 8;
+#pragma unroll
+        for (int n = 0; n < NP / 16; ++n) {
+          uint32_t bf[4];
+          cr_ldmt(bf, sm.k_hi + krow + n * 16);
+          cr_mma(s[2 * n], vf, bf[0], bf[1]);
+          cr_mma(s[2 * n + 1], vf, bf[2], bf[3]);
+          cr_ldmt(bf, sm.k_lo + krow + n * 16);
+          cr_mma(s[2 * n], vf, bf[0], bf[1]);
+          cr_mma(s[2 * n + 1], vf, bf[2], bf[3]);
+        }
+#pragma unroll
+        for (int nt = 0; nt < NP / 8; ++nt) {
+          const float2 d = *reinterpret_cast<const float2*>(&sm.end[blk][nt * 8 + 2 * gc]);
+          s[nt][0] *= d.x; s[nt][1] *= d.y; s[nt][2] *= d.x; s[nt][3] *= d.y;
+        }
+      }
+    } else {
+      // ---- token by token
+      const int live_tokens = min(kCrTokens, ntok - t0);
+      for (int r = 0; r < live_tokens; ++r) {
+        float (*g)[NP] = sm.gate[r & 1];
+        for (int c = tid; c < NP; c += kThreads) {
+          const bool ch = c < a.n;
+          gate(__bfloat162float(sm.zf[st][r * QS + c]) + (ch ? bias[c] : 0.f), ch ? lower[c] : 0.f, ch, &g[1][c], &g[2][c]);
+          if (!kStateOnly) g[0][c] = query(__bfloat162float(sm.zq[st][r * QS + c]));
+        }
+        __syncthreads();                                   // two buffers: one barrier per token
+        const float v0 = __bfloat162float(v_s[r * VS + p0 + gr]), v1 = __bfloat162float(v_s[r * VS + p0 + gr + 8]);
+        float o0 = 0.f, o1 = 0.f;
+#pragma unroll
+        for (int nt = 0; nt < NP / 8; ++nt)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int n = nt * 8 + 2 * gc + e;
+            const float f = g[1][n], k = g[2][n];
+            s[nt][e] = fmaf(f, s[nt][e], k * v0);
+            s[nt][2 + e] = fmaf(f, s[nt][2 + e], k * v1);
+            if (!kStateOnly) { o0 = fmaf(g[0][n], s[nt][e], o0); o1 = fmaf(g[0][n], s[nt][2 + e], o1); }
+          }
+        if (!kStateOnly) {
+#pragma unroll
+          for (int d = 1; d <= 2; d <<= 1) {
+            o0 += __shfl_xor_sync(0xffffffffu, o0, d);
+            o1 += __shfl_xor_sync(0xffffffffu, o1, d);
+          }
+          __syncwarp();
+          if (gc == 0) {
+            v_s[r * VS + p0 + gr] = __float2bfloat16_rn(o0);
+            v_s[r * VS + p0 + gr + 8] = __float2bfloat16_rn(o1);
+          }
+        }
+      }
+    }
+    if (!kStateOnly) {
+      __syncwarp();
+#pragma unroll
+      for (int i = 0; i < kCrTokens / 16; ++i) {
+        const int r = i * 16 + (lane >> 1), col = p0 + (lane & 1) * 8;
+        if (t0 + r < ntok && pbase + col < a.p)
+          st16((__nv_bfloat16*)a.out + ((int64_t)(tok0 + t0 + r) * a.heads + h) * a.p + pbase + col, ld16(v_s + r * VS + col));
+      }
+    }
+  }
+  float* dst = kStateOnly ? sg.start + ((int64_t)bh * sg.count + seg) * np : (c1 == nchunks ? final_state : nullptr);
+  if (dst != nullptr) {
+#pragma unroll
+    for (int nt = 0; nt < NP / 8; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int n = nt * 8 + 2 * gc + (e & 1), p = e < 2 ? pc0 : pc1;
+        if (n < a.n && p < a.p) dst[(int64_t)n * a.p + p] = s[nt][e];
+      }
+  }
+  if (kStateOnly && pt == 0) {
+#pragma unroll
+    for (int i = 0; i < kOwn; ++i) {
+      const int c = tid + i * kThreads;
+      if (c < a.n) sg.decay[((int64_t)bh * sg.count + seg) * a.n + c] = seg_decay[i];
+    }
+  }
+}
+
+// start[seg] <- state before the segment.  Thread per state element; on entry start[seg] holds the segment's own state.
+__global__ void __launch_bounds__(256) chanrec_chain_kernel(ChanrecParams a, ChanrecSegs sg) {
+  grid_dependency_wait();
+  grid_launch_dependents();
+  const int bh = blockIdx.y, b = bh / a.heads, h = bh - b * a.heads;
+  const int64_t np = (int64_t)a.n * a.p, i = (int64_t)blockIdx.x * 256 + threadIdx.x;
+  if (i >= np) return;
+  const int n = (int)(i / a.p);
+  const int used = (a.cu[b + 1] - a.cu[b] + sg.tokens - 1) / sg.tokens;
+  float run = a.pos0[b] == 0 ? 0.f : a.state[((int64_t)a.slots[b] * a.heads + h) * np + i];
+  float* at = sg.start + (int64_t)bh * sg.count * np + i;
+  const float* decay = sg.decay + (int64_t)bh * sg.count * a.n + n;
+  for (int k = 0; k < used; ++k) {
+    const float own = k + 1 < used ? at[(int64_t)k * np] : 0.f;
+    at[(int64_t)k * np] = run;
+    if (k + 1 < used) run = fmaf(decay[(int64_t)k * a.n], run, own);
+  }
+}
+
+static bool chanrec_chunk_shape(int n, int p) { return n % 8 == 0 && p % 8 == 0 && n <= 256; }
+static int chanrec_columns(int n, int p) { return (n <= 128 && p > 64) ? 128 : 64; }
+
+static ChanrecSegs plan_chanrec(int batch, int max_tokens, int heads, int n, int p) {
+  const int pt = chanrec_columns(n, p);
+  const int64_t ctas = (int64_t)batch * heads * ((p + pt - 1) / pt);
+  const int64_t room = 148 * (n > 128 ? 1 : 2);            // CTAs that run at the same time
+  const int chunks = (max_tokens + kCrTokens - 1) / kCrTokens;
+  int64_t segs = ctas > 0 ? room / ctas : 1;               // segments of at least eight chunks
+  if (segs > chunks / 8) segs = chunks / 8;
+  if (segs < 1) segs = 1;
+  ChanrecSegs s = {};
+  const int per = (int)((chunks + segs - 1) / segs);
+  s.tokens = per * kCrTokens;
+  s.count = per > 0 ? (chunks + per - 1) / per : 1;
+  return s;
+}
+
+template <int NP, int kWarps>
+static int launch_chanrec(const ChanrecParams& a, const ChanrecSegs& sg, cudaStream_t st) {
+  constexpr int kBytes = (int)sizeof(CrSmem<NP, kWarps>);
+  static bool configured = false;
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(chanrec_chunk_kernel<NP, kWarps, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kBytes);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(chanrec_chunk_kernel<NP, kWarps, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kBytes);
+    if (e != cudaSuccess) return fail(TKV_ERR_LAUNCH, "tkv_chanrec_chunk: %s", cudaGetErrorString(e));
+    configured = true;
+  }
+  const int64_t grid = (int64_t)a.batch * a.heads * ((a.p + kWarps * 16 - 1) / (kWarps * 16)) * sg.count;
+  if (grid > INT32_MAX) return fail(TKV_ERR_UNSUPPORTED, "tkv_chanrec_chunk: %lld blocks", (long long)grid);
+  cudaError_t e = cudaSuccess;
+  if (sg.count > 1) {
+    e = launch_pdl(chanrec_chunk_kernel<NP, kWarps, true>, dim3((unsigned)grid), dim3(kWarps * 32), (size_t)kBytes, st, a, sg);
+    if (e == cudaSuccess)
+      e = launch_pdl(chanrec_chain_kernel, dim3((unsigned)(((int64_t)a.n * a.p + 255) / 256), a.batch * a.heads), dim3(256), 0, st, a, sg);
+  }
+  if (e == cudaSuccess)
+    e = launch_pdl(chanrec_chunk_kernel<NP, kWarps, false>, dim3((unsigned)grid), dim3(kWarps * 32), (size_t)kBytes, st, a, sg);
+  if (e != cudaSuccess) return fail(TKV_ERR_LAUNCH, "tkv_chanrec_chunk: %s", cudaGetErrorString(e));
+  return check_launch("tkv_chanrec_chunk");
+}
+
+}  // namespace tkv
+
+using namespace tkv;
+
+extern "C" int64_t tkv_chanrec_chunk_workspace_bytes(int batch, int max_tokens, int heads, int n, int vdim, int dtype) {
+  if (dtype != TKV_BF16 || batch <= 0 || heads <= 0 || n <= 0 || vdim <= 0 || max_tokens <= 0 || !chanrec_chunk_shape(n, vdim)) return -1;
+  const ChanrecSegs s = plan_chanrec(batch, max_tokens, heads, n, vdim);
+  return s.count > 1 ? (int64_t)batch * heads * s.count * n * ((int64_t)vdim + 1) * (int64_t)sizeof(float) : 0;
+}
+
+extern "C" int tkv_chanrec_chunk(const void* q, const void* f, const void* v, int64_t row_stride, const float* f_bias,
+                                 const float* lower, void* out, float* state, const int32_t* slots, const int32_t* cu_tokens,
+                                 const int32_t* pos0, void* workspace, int64_t workspace_bytes, int batch, int max_tokens, int heads,
+                                 int n, int vdim, int dtype, tkv_stream_t stream) {
+  if (!q || !f || !v || !f_bias || !lower || !out || !state || !slots || !cu_tokens || !pos0)
+    return fail(TKV_ERR_ARG, "tkv_chanrec_chunk: NULL pointer argument");
+  if (batch < 0 || max_tokens < 0 || heads <= 0 || n <= 0 || vdim <= 0 || row_stride < (int64_t)heads * n || row_stride < (int64_t)heads * vdim)
+    return fail(TKV_ERR_ARG, "tkv_chanrec_chunk: bad sizes heads=%d n=%d vdim=%d", heads, n, vdim);
+  if (dtype != TKV_BF16 || !chanrec_chunk_shape(n, vdim))
+    return fail(TKV_ERR_UNSUPPORTED, "tkv_chanrec_chunk: dtype=%d n=%d vdim=%d (bf16, n <= 256, multiples of 8; others: tkv_chanrec_scan)", dtype, n, vdim);
+  if (row_stride % 8 || !aligned16(q) || !aligned16(f) || !aligned16(v) || !aligned16(out))
+    return fail(TKV_ERR_ARG, "tkv_chanrec_chunk: rows must start on 16-byte boundaries");
+  if (batch == 0 || max_tokens == 0) return TKV_OK;
+  if ((int64_t)batch * heads > 65535) return fail(TKV_ERR_UNSUPPORTED, "tkv_chanrec_chunk: batch * heads = %lld", (long long)batch * heads);
+  const int64_t need = tkv_chanrec_chunk_workspace_bytes(batch, max_tokens, heads, n, vdim, dtype);
+  if (need > 0 && (!workspace || workspace_bytes < need))
+    return fail(TKV_ERR_ARG, "tkv_chanrec_chunk: workspace of %lld bytes, %lld needed", (long long)workspace_bytes, (long long)need);
+  ChanrecParams a = {q, f, v, row_stride, f_bias, lower, out, state, slots, cu_tokens, pos0, batch, heads, n, vdim};
+  ChanrecSegs s = plan_chanrec(batch, max_tokens, heads, n, vdim);
+  s.start = (float*)workspace;
+  s.decay = s.start + (s.count > 1 ? (int64_t)batch * heads * s.count * n * vdim : 0);
+  cudaStream_t st = (cudaStream_t)stream;
+  const bool wide = chanrec_columns(n, vdim) == 128;
+  if (n <= 64) return wide ? launch_chanrec<64, 8>(a, s, st) : launch_chanrec<64, 4>(a, s, st);
+  if (n <= 128) return wide ? launch_chanrec<128, 8>(a, s, st) : launch_chanrec<128, 4>(a, s, st);
+  return launch_chanrec<256, 4>(a, s, st);
+}

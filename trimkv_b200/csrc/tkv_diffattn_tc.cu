@@ -9,15 +9,10 @@
 // goes to memory.  A row sees the columns [lo, hi) of the request's linear keys; tiles before the first row's window are
 // never loaded.  Waits are bounded; on expiry the CTA records TKV_DEV_TIMEOUT, drains its copies and frees its TMEM.
 #include <cuda.h>
+#include "tkv_attn_block.cuh"
 #include "tkv_diffattn.cuh"
-#include "tkv_tc.cuh"
 
 namespace tkv {
-
-constexpr int kDaSoftmaxThreads = 256, kDaThreads = kDaSoftmaxThreads + 32;
-constexpr int kDaTile = 128, kDaHalf = 16384;             // 128 rows x 64 elements
-constexpr int kDaTmemCols = 512;
-constexpr float kDaRescaleGap = 8.0f;
 
 struct DaSmem {
   uint64_t bar_k[2], bar_v[2], bar_s[2], bar_o, bar_p, bar_x;
@@ -26,46 +21,6 @@ struct DaSmem {
   float red[2][2][kDaTile];
 };
 template <int KH, int VH> constexpr int da_smem_bytes() { return (4 * KH + 2 * VH + 2) * kDaHalf + (int)sizeof(DaSmem); }
-
-__device__ __forceinline__ uint32_t da_idesc(int n, int b_mn_major) {   // kind::f16, bf16 operands, fp32 D, M = 128
-  return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)b_mn_major << 16) | ((uint32_t)(n >> 3) << 17) | ((128u >> 4) << 24);
-}
-__device__ __forceinline__ uint32_t da_swz(int r, int c) {              // 16-byte chunk c of row r, 64-element halves
-  return (uint32_t)((c >> 3) * kDaHalf + r * 128 + (((c & 7) ^ (r & 7)) << 4));
-}
-__device__ __forceinline__ void da_ld32_nowait(uint32_t taddr, uint32_t* r) {
-  asm volatile(
-      "tcgen05.ld.sync.aligned.32x32b.x32.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,"
-      "%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"
-      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]),
-        "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]),
-        "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]),
-        "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
-      : "r"(taddr));
-}
-__device__ __forceinline__ void da_st32(uint32_t taddr, const float* v) {
-  asm volatile(
-      "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,"
-      "%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31,%32};"
-      ::"r"(taddr), "r"(__float_as_uint(v[0])), "r"(__float_as_uint(v[1])), "r"(__float_as_uint(v[2])),
-        "r"(__float_as_uint(v[3])), "r"(__float_as_uint(v[4])), "r"(__float_as_uint(v[5])), "r"(__float_as_uint(v[6])),
-        "r"(__float_as_uint(v[7])), "r"(__float_as_uint(v[8])), "r"(__float_as_uint(v[9])), "r"(__float_as_uint(v[10])),
-        "r"(__float_as_uint(v[11])), "r"(__float_as_uint(v[12])), "r"(__float_as_uint(v[13])), "r"(__float_as_uint(v[14])),
-        "r"(__float_as_uint(v[15])), "r"(__float_as_uint(v[16])), "r"(__float_as_uint(v[17])), "r"(__float_as_uint(v[18])),
-        "r"(__float_as_uint(v[19])), "r"(__float_as_uint(v[20])), "r"(__float_as_uint(v[21])), "r"(__float_as_uint(v[22])),
-        "r"(__float_as_uint(v[23])), "r"(__float_as_uint(v[24])), "r"(__float_as_uint(v[25])), "r"(__float_as_uint(v[26])),
-        "r"(__float_as_uint(v[27])), "r"(__float_as_uint(v[28])), "r"(__float_as_uint(v[29])), "r"(__float_as_uint(v[30])),
-        "r"(__float_as_uint(v[31]))
-      : "memory");
-  asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
-}
-__device__ __forceinline__ void da_arrive(uint64_t* bar) {
-  asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(bar)) : "memory");
-}
-__device__ __forceinline__ uint32_t da_pack2(float a, float b) {
-  const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
-  return *reinterpret_cast<const uint32_t*>(&v);
-}
 
 // KH = dp / 64, VH = pp / 64.  Warps 0-7: softmax (row r is shared by threads r and 128 + r); warp 8 issues copies and MMAs.
 template <int KH, int VH>

@@ -285,7 +285,6 @@ extern "C" int tkv_moe_gemm(const void* a, int64_t a_stride, int64_t a_rows, con
   GroupedGemm p = {a, a_stride, a_rows, src, w, offsets, out, experts, n, k, act, max_rows, status};
   cudaStream_t st = (cudaStream_t)stream;
   if (moe_tc_shape(p, dtype)) return launch_moe_tc(p, st);
-  if (moe_stream_shape(p, dtype)) return launch_moe_stream(p, st);
   const int64_t tiles = max_rows / kAnyM + (experts < max_rows ? experts : max_rows);
   if (tiles > 65535) return fail(TKV_ERR_UNSUPPORTED, "tkv_moe_gemm: %lld row tiles", (long long)tiles);
   const dim3 grid((n + kAnyN - 1) / kAnyN, (unsigned)tiles);

@@ -35,9 +35,7 @@ __device__ __forceinline__ bool find_tile(const int32_t* offsets, int experts, i
   return false;
 }
 
-bool moe_stream_shape(const GroupedGemm& p, int dtype);   // few rows per expert: weights streamed once (tkv_moe_stream.cu)
-int launch_moe_stream(const GroupedGemm& p, cudaStream_t st);
-bool moe_tc_shape(const GroupedGemm& p, int dtype);       // many rows: tcgen05 (tkv_moe_tc.cu)
+bool moe_tc_shape(const GroupedGemm& p, int dtype);       // tcgen05 (tkv_moe_tc.cu)
 int launch_moe_tc(const GroupedGemm& p, cudaStream_t st);
 
 }  // namespace tkv

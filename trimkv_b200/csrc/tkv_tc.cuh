@@ -117,6 +117,8 @@ __device__ __forceinline__ void tmem_ld32(uint32_t taddr, float* v) {
 
 // Encodes a 2-D tiled tensor map over a row-major [rows, cols] matrix of 16-bit elements (128-byte swizzle).
 int make_map_2d(CUtensorMap* map, const void* base, int64_t cols, int64_t rows, int box_cols, int box_rows, int dtype);
+// The same over bf16 rows that are row_stride elements apart.
+int make_map_rows(CUtensorMap* map, const void* base, int64_t cols, int64_t rows, int64_t row_stride, int box_cols, int box_rows);
 // 3-D map over bf16 [outer][mid][inner] with element strides inner_len between mids and outer_stride between outers; the box
 // is one mid wide, so columns beyond inner_len read as zeros instead of the next mid's.
 int make_map_3d_bf16(CUtensorMap* map, const void* base, int64_t inner, int64_t mid, int64_t outer, int64_t outer_stride, int box_inner,

@@ -595,8 +595,19 @@ def chanrec_step(q, f, v, f_bias, lower, norm, state, batch, out, eps: float) ->
 
 
 def chanrec(q, f, v, f_bias, lower, state, batch, out, force_scan: bool = False) -> None:
-    """The recurrence over the packed tokens of ``batch`` (see tkv_chanrec_scan in the header)."""
+    """The recurrence over the packed tokens of ``batch`` (see tkv_chanrec_scan in the header): the chunked tensor-core kernel
+    where it covers the shape, the token-by-token scan otherwise."""
     _, heads, n, p = state.shape
+    dt = dtype_code(out.dtype)
+    need = lib().tkv_chanrec_chunk_workspace_bytes(batch.size, batch.max_tokens, heads, n, p, dt)
+    rows_ok = q.stride(0) % 8 == 0 and all(t.data_ptr() % 16 == 0 for t in (q, f, v, out))
+    if need >= 0 and rows_ok and batch.cu is not None and not force_scan and batch.size * heads <= 65535:
+        ws = torch.empty(need, dtype=torch.uint8, device=out.device) if need else None
+        check(lib().tkv_chanrec_chunk(q.data_ptr(), f.data_ptr(), v.data_ptr(), q.stride(0), f_bias.data_ptr(), lower.data_ptr(),
+                                      out.data_ptr(), state.data_ptr(), batch.slots.data_ptr(), batch.cu.data_ptr(), batch.pos0.data_ptr(),
+                                      _ptr(ws), need, batch.size, batch.max_tokens, heads, n, p, dt, _stream(out)), "tkv_chanrec_chunk")
+        _count(3 if need else 1)
+        return
     check(lib().tkv_chanrec_scan(q.data_ptr(), f.data_ptr(), v.data_ptr(), q.stride(0), f_bias.data_ptr(), lower.data_ptr(), out.data_ptr(),
                                  state.data_ptr(), batch.slots.data_ptr(), _ptr(batch.cu), batch.pos0.data_ptr(), batch.size, heads, n, p,
                                  dtype_code(out.dtype), _stream(out)), "tkv_chanrec_scan")
