@@ -354,13 +354,15 @@ def run_micro(args):
     generate: generate() of the model classes on --workload, HF loop against fused_decode=True (wall clock per token).
     hybrid: the hybrid decoder (Dafovik: retention, state-space and windowed differential-attention layers) beside the Qwen3
             model of equal width, depth and parameters: prompt pass, decoding, and every kernel against its roofline.
+    lonulix: the latent-attention / HGRN2 decoder with experts beside the other hybrid decoder (Dafovik) at equal width, depth
+            and head sizes, and every kernel beside the like kernel of that model.
     multi : --q-tokens new tokens per request against M cached ones (a piece of a chunked prefill, multi-token
             decoding): the multi-token kernels beside the library attention, causal and with a length mask.
     Each timed launch works on data that was not touched by the previous one (buffers rotate; each is > L2).
     """
-    if args.micro == "hybrid":
+    if args.micro in ("hybrid", "lonulix"):
         for size in sorted(HYBRID_SIZES) if args.hybrid_size == "all" else [args.hybrid_size]:
-            run_hybrid(args, size)
+            (run_hybrid if args.micro == "hybrid" else run_lonulix)(args, size)
         return
     from trimkv_b200 import ops
     dev = torch.device("cuda", 0)
@@ -627,12 +629,15 @@ def run_micro(args):
     print(json.dumps(res))
 
 
-# Layer sizes of the hybrid microbenchmark.  `attn` is the Qwen3 side (GLU of 3 x ff); the hybrid's dense feed-forward gets
+# Layer sizes of the hybrid microbenchmarks.  `attn` is the Qwen3 side (GLU of 3 x ff); the hybrid's dense feed-forward gets
 # 1.5 x ff (equal parameters), its mixers heads of the same size and twice the width as state-space channels.
 HYBRID_SIZES = {
-    "1.7b": dict(width=2048, heads=16, kv_heads=8, ff=6144, layers=8, window=4096, batch=32, prompt=8192),
-    "8b": dict(width=4096, heads=32, kv_heads=8, ff=12288, layers=4, window=4096, batch=32, prompt=4096),
-    "tiny": dict(width=256, heads=2, kv_heads=1, ff=512, layers=4, window=128, batch=4, prompt=384),
+    "1.7b": dict(width=2048, heads=16, kv_heads=8, ff=6144, layers=8, window=4096, batch=32, prompt=8192,
+                 latent=dict(q_rank=1536, kv_rank=512), experts=dict(count=32, identity=4, top=6)),
+    "8b": dict(width=4096, heads=32, kv_heads=8, ff=12288, layers=4, window=4096, batch=32, prompt=4096,
+               latent=dict(q_rank=1536, kv_rank=512), experts=dict(count=32, identity=4, top=6)),
+    "tiny": dict(width=256, heads=2, kv_heads=1, ff=512, layers=4, window=128, batch=4, prompt=384,
+                 latent=dict(q_rank=96, kv_rank=64), experts=dict(count=6, identity=2, top=4)),
 }
 
 
@@ -647,30 +652,21 @@ def hybrid_config(z, vocab=32768):
                         for i in range(z["layers"])], norm={"eps": 1e-6}, residual_mult=0.5, vocab=vocab, width=w)
 
 
-def run_hybrid(args, size):
-    """One JSON line: the hybrid decoder at one size beside the Qwen3 model of the framework (same width, depth, head size
-    and parameters per layer, M = window), and its kernels one by one beside the like kernel of that model.  Device times;
-    every kernel is timed as a CUDA graph of launches over rotating operands that together exceed L2."""
-    from trimkv_b200 import DafovikConfig, DafovikForCausalLM, TrimKVCache, ops
-    from trimkv_b200.attn import _dense_causal
-    from trimkv_b200.decoder import GreedyDecoder
-    from trimkv_b200.state_cache import HybridStateCache, RecurrentState, WindowState
-    z = HYBRID_SIZES[size]
-    dev = torch.device("cuda", 0)
-    torch.cuda.set_device(dev)
-    peak, peak_src = measured_peaks()
-    flops_peak = 1590.0
-    path = os.path.join(ROOT, "MEASURED_PEAKS.json")
-    if os.path.exists(path):
-        with open(path) as f:
-            flops_peak = json.load(f)["bf16_tflops"]
-    bf = torch.bfloat16
-    res = {"micro": "hybrid", "size": size, "config": z, "dtype": "bf16", "data": "synthetic", "peak_gbs": peak, "peak_tflops": flops_peak,
-           "peak_source": peak_src}
-    gen = torch.Generator(device=dev).manual_seed(0)
-    B, P = z["batch"], z["prompt"]
+class MicroTools:
+    """Device timing of the hybrid microbenchmarks: ``events`` times calls back to back, ``kernel`` a CUDA graph of launches
+    over rotating operands that together exceed L2 and files the result, against the roofline, under ``rows``."""
 
-    def events(fn, n):
+    def __init__(self, dev):
+        self.dev, self.rows = dev, {}
+        self.gen = torch.Generator(device=dev).manual_seed(0)
+        self.peak, self.peak_src = measured_peaks()
+        self.flops_peak = 1590.0
+        path = os.path.join(ROOT, "MEASURED_PEAKS.json")
+        if os.path.exists(path):
+            with open(path) as f:
+                self.flops_peak = json.load(f)["bf16_tflops"]
+
+    def events(self, fn, n):
         e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
         torch.cuda.synchronize(); e0.record()
         for _ in range(n):
@@ -678,62 +674,10 @@ def run_hybrid(args, size):
         e1.record(); torch.cuda.synchronize()
         return e0.elapsed_time(e1) / n
 
-    # ------------------------------------------------------------------------------------------------ whole models
-    if args.hybrid_part != "kernels":
-        torch.manual_seed(0)
-        with torch.device(dev):
-            hybrid = DafovikForCausalLM(DafovikConfig(**hybrid_config(z))).to(bf).eval()
-        wl = dict(hidden_size=z["width"], num_hidden_layers=z["layers"], num_attention_heads=z["heads"], num_key_value_heads=z["kv_heads"],
-                  head_dim=128, intermediate_size=z["ff"], vocab_size=32768, rope_theta=1e6, retention_gate_intermediate_size=128,
-                  retention_gate_bias_init=3.0, memory_size=z["window"], buffer_size=128)
-        qwen, _ = build_model(wl, dev)
-        with torch.inference_mode():
-            for name, model in (("hybrid", hybrid), ("qwen3", qwen)):
-                out = {"parameters": sum(p.numel() for p in model.parameters())}
-                for bsz, n in ((1, P), (max(1, B // 8), P)):
-                    ids = torch.randint(0, 32768, (bsz, n), generator=gen, device=dev)
+    def rnd(self, *shape, dtype=torch.bfloat16, scale=1.0):
+        return torch.randn(*shape, generator=self.gen, device=self.dev, dtype=dtype) * scale
 
-                    def prompt():
-                        cache = model.new_cache(dev, capacity_tokens=n) if name == "hybrid" else model.new_cache(dev)
-                        model(input_ids=ids, past_key_values=cache, logits_to_keep=1)
-                        return cache
-                    for _ in range(3):
-                        prompt()
-                    ms = events(prompt, 5)
-                    out[f"prefill_b{bsz}x{n}"] = {"ms": ms, "tok_per_s": bsz * n / (ms * 1e-3)}
-                for bsz in (B, 4 * B):
-                    cache = model.new_cache(dev, capacity_tokens=P + 512) if name == "hybrid" else TrimKVCache(
-                        device=dev, memory_size=z["window"], buffer_size=128, num_layers=z["layers"])
-                    n = min(P, z["window"] + 64)
-                    ids = torch.randint(0, 32768, (bsz, n), generator=gen, device=dev)
-                    if name == "hybrid":
-                        cache.open(bsz)
-                        for lo in range(0, bsz, 8):        # the prompt pass of a few requests at a time
-                            rows = list(range(lo, min(bsz, lo + 8)))
-                            model.forward_packed(ids[rows].reshape(-1), cache, [n] * len(rows), rows, [len(rows) * n - 1])
-                    elif bsz <= B:
-                        model(input_ids=ids, past_key_values=cache, logits_to_keep=1)
-                    else:
-                        continue
-                    dec = GreedyDecoder(model, cache)
-                    for _ in range(3):
-                        dec.step(eager=True)
-                    for _ in range(3):
-                        dec.step()
-                    ms = events(dec.step, 50)
-                    out[f"decode_b{bsz}_at_{n}"] = {"ms_per_step": ms, "tok_per_s": bsz / (ms * 1e-3)}
-                    cache.check_status()
-                    dec.close()
-                    del dec, cache
-                    torch.cuda.empty_cache()
-                res[name] = out
-        del hybrid, qwen, model
-        torch.cuda.empty_cache()
-
-    # ------------------------------------------------------------------------------------------------ single kernels
-    rows = {}
-
-    def kernel(name, calls, nbytes, flops=0.0, reps=8):
+    def kernel(self, name, calls, nbytes, flops=0.0, reps=8):
         """calls: closures over distinct operands, launched in turn inside one CUDA graph."""
         for c in calls:
             c()
@@ -745,17 +689,102 @@ def run_hybrid(args, size):
                 calls[i % len(calls)]()
         for _ in range(3):
             graph.replay()
-        ms = events(graph.replay, 5) / n
-        t_mem, t_math = nbytes / (peak * 1e9) * 1e3, flops / (flops_peak * 1e12) * 1e3
-        rows[name] = {"us": ms * 1e3, "gbs": nbytes / (ms * 1e-3) / 1e9, "tflops": flops / (ms * 1e-3) / 1e12,
-                      "bound": "tensor" if t_math > t_mem else "hbm", "frac_of_roofline": max(t_mem, t_math) / ms}
+        ms = self.events(graph.replay, 5) / n
+        t_mem, t_math = nbytes / (self.peak * 1e9) * 1e3, flops / (self.flops_peak * 1e12) * 1e3
+        self.rows[name] = {"us": ms * 1e3, "gbs": nbytes / (ms * 1e-3) / 1e9, "tflops": flops / (ms * 1e-3) / 1e12,
+                           "bound": "tensor" if t_math > t_mem else "hbm", "frac_of_roofline": max(t_mem, t_math) / ms}
         torch.cuda.synchronize()
         graph.reset()
         torch.cuda.empty_cache()
 
-    def rnd(*shape, dtype=bf, scale=1.0):
-        return torch.randn(*shape, generator=gen, device=dev, dtype=dtype) * scale
+    def batch_for(self, layer, bsz, n, start=0):
+        """A cache of one layer's state and a step of ``n`` tokens of ``bsz`` requests from position ``start``."""
+        from trimkv_b200.state_cache import HybridStateCache
+        cache = HybridStateCache([layer], self.dev, torch.bfloat16, capacity_tokens=start + n + 8)
+        cache.open(bsz)
+        if start:
+            cache._lens[cache._rows] = start
+            for s in cache._rows:
+                cache._len[s] = start
+        return cache, cache.begin([n] * bsz if n > 1 else None)
 
+    def model(self, model, z, hybrid):
+        """Prompt passes and decode steps of a whole model at the sizes of ``z``."""
+        from trimkv_b200 import TrimKVCache
+        from trimkv_b200.decoder import GreedyDecoder
+        dev, B, P = self.dev, z["batch"], z["prompt"]
+        out = {"parameters": sum(p.numel() for p in model.parameters())}
+        for bsz, n in ((1, P), (max(1, B // 8), P)):
+            ids = torch.randint(0, 32768, (bsz, n), generator=self.gen, device=dev)
+
+            def prompt():
+                cache = model.new_cache(dev, capacity_tokens=n) if hybrid else model.new_cache(dev)
+                model(input_ids=ids, past_key_values=cache, logits_to_keep=1)
+                return cache
+            for _ in range(3):
+                prompt()
+            ms = self.events(prompt, 5)
+            out[f"prefill_b{bsz}x{n}"] = {"ms": ms, "tok_per_s": bsz * n / (ms * 1e-3)}
+        for bsz in (B, 4 * B):
+            cache = model.new_cache(dev, capacity_tokens=P + 512) if hybrid else TrimKVCache(
+                device=dev, memory_size=z["window"], buffer_size=128, num_layers=z["layers"])
+            n = min(P, z["window"] + 64)
+            ids = torch.randint(0, 32768, (bsz, n), generator=self.gen, device=dev)
+            if hybrid:
+                cache.open(bsz)
+                for lo in range(0, bsz, 8):        # the prompt pass of a few requests at a time
+                    rows = list(range(lo, min(bsz, lo + 8)))
+                    model.forward_packed(ids[rows].reshape(-1), cache, [n] * len(rows), rows, [len(rows) * n - 1])
+            elif bsz <= B:
+                model(input_ids=ids, past_key_values=cache, logits_to_keep=1)
+            else:
+                continue
+            dec = GreedyDecoder(model, cache)
+            for _ in range(3):
+                dec.step(eager=True)
+            for _ in range(3):
+                dec.step()
+            ms = self.events(dec.step, 50)
+            out[f"decode_b{bsz}_at_{n}"] = {"ms_per_step": ms, "tok_per_s": bsz / (ms * 1e-3)}
+            cache.check_status()
+            dec.close()
+            del dec, cache
+            torch.cuda.empty_cache()
+        return out
+
+
+def run_hybrid(args, size):
+    """One JSON line: the hybrid decoder at one size beside the Qwen3 model of the framework (same width, depth, head size
+    and parameters per layer, M = window), and its kernels one by one beside the like kernel of that model.  Device times;
+    every kernel is timed as a CUDA graph of launches over rotating operands that together exceed L2."""
+    from trimkv_b200 import DafovikConfig, DafovikForCausalLM, ops
+    from trimkv_b200.attn import _dense_causal
+    from trimkv_b200.state_cache import RecurrentState, WindowState
+    z = HYBRID_SIZES[size]
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    bf = torch.bfloat16
+    tools = MicroTools(dev)
+    kernel, rnd, batch_for, rows, gen = tools.kernel, tools.rnd, tools.batch_for, tools.rows, tools.gen
+    res = {"micro": "hybrid", "size": size, "config": z, "dtype": "bf16", "data": "synthetic", "peak_gbs": tools.peak,
+           "peak_tflops": tools.flops_peak, "peak_source": tools.peak_src}
+    B, P = z["batch"], z["prompt"]
+    # ------------------------------------------------------------------------------------------------ whole models
+    if args.hybrid_part != "kernels":
+        torch.manual_seed(0)
+        with torch.device(dev):
+            hybrid = DafovikForCausalLM(DafovikConfig(**hybrid_config(z))).to(bf).eval()
+        wl = dict(hidden_size=z["width"], num_hidden_layers=z["layers"], num_attention_heads=z["heads"], num_key_value_heads=z["kv_heads"],
+                  head_dim=128, intermediate_size=z["ff"], vocab_size=32768, rope_theta=1e6, retention_gate_intermediate_size=128,
+                  retention_gate_bias_init=3.0, memory_size=z["window"], buffer_size=128)
+        qwen, _ = build_model(wl, dev)
+        with torch.inference_mode():
+            for name, model in (("hybrid", hybrid), ("qwen3", qwen)):
+                res[name] = tools.model(model, z, name == "hybrid")
+        del hybrid, qwen, model
+        torch.cuda.empty_cache()
+
+    # ------------------------------------------------------------------------------------------------ single kernels
     if args.hybrid_part != "models":
         w, H, G, ff, W = z["width"], z["heads"], z["kv_heads"], z["ff"], z["window"]
         bsz = max(1, B // 8)
@@ -777,14 +806,6 @@ def run_hybrid(args, size):
             kernel("prompt: silu_mul (qwen3)", [lambda: ops.silu_mul(gu, act)], T * ff * 6)
             del gu, act, x32, y, c16
 
-            def batch_for(layer, bsz, n, start=0):
-                cache = HybridStateCache([layer], dev, bf, capacity_tokens=start + n + 8)
-                cache.open(bsz)
-                if start:
-                    cache._lens[cache._rows] = start
-                    for s in cache._rows:
-                        cache._len[s] = start
-                return cache, cache.begin([n] * bsz if n > 1 else None)
             # retention
             D, V = 128, 128
             hd, hv = H * D, H * V
@@ -872,9 +893,165 @@ def run_hybrid(args, size):
     print(json.dumps(res))
 
 
+def lonulix_config(z, vocab=32768):
+    """Layers in turn latent attention, HGRN2, HGRN2; feed-forwards in turn dense and experts (as many active parameters)."""
+    w, h, lat = z["width"], z["heads"], z["latent"]
+    kinds = {"latent_attention": dict(heads=h, dim=128, rot_dim=64, vdim=128, q_rank=lat["q_rank"], kv_rank=lat["kv_rank"], mask=dict(size=z["window"]),
+                                      scale=192 ** -0.5, rot=dict(base=1e6, dims=64)),
+             "hgrn2": dict(heads=h, dim=128, vdim=128)}
+    e = z["experts"]
+    ffs = [{"kind": "dense", "ff": z["ff"]},
+           {"kind": "moe", "expert": {"ff": z["ff"] * 3 // 2 // e["top"]},
+            "router": {"experts": e["count"], "identity": e["identity"], "top": e["top"], "scale": 1.0, "groups": {"count": 4, "keep": 2}}}]
+    types = ["latent_attention", "hgrn2", "hgrn2"]
+    return dict(layers=[{"type": types[i % 3], "mixer": kinds[types[i % 3]], "mlp": ffs[i % 2]} for i in range(z["layers"])],
+                norm={"eps": 1e-6, "groups": 4}, embedding={"scale": 1.0}, postln_alpha=2.0, vocab=vocab, width=w)
+
+
+def run_lonulix(args, size):
+    """One JSON line: the latent-attention / HGRN2 decoder at one size beside the other hybrid decoder, and its kernels one by one
+    beside the like kernel (same sizes where the mechanism allows) of that model, or the library product of the same operands."""
+    from trimkv_b200 import DafovikConfig, DafovikForCausalLM, LonulixConfig, LonulixForCausalLM, ops
+    from trimkv_b200.mixers import rotary_frequencies
+    from trimkv_b200.state_cache import LatentState, RecurrentState, WindowState
+    z = HYBRID_SIZES[size]
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    bf = torch.bfloat16
+    tools = MicroTools(dev)
+    kernel, rnd, batch_for = tools.kernel, tools.rnd, tools.batch_for
+    res = {"micro": "lonulix", "size": size, "config": z, "dtype": "bf16", "data": "synthetic", "peak_gbs": tools.peak,
+           "peak_tflops": tools.flops_peak, "peak_source": tools.peak_src}
+    if args.hybrid_part != "kernels":
+        for name, cls, cfg in (("lonulix", LonulixForCausalLM, LonulixConfig(**lonulix_config(z))), ("dafovik", DafovikForCausalLM, DafovikConfig(**hybrid_config(z)))):
+            torch.manual_seed(0)
+            with torch.device(dev):
+                model = cls(cfg).to(bf).eval()
+            with torch.inference_mode():
+                res[name] = tools.model(model, z, True)
+            del model
+            torch.cuda.empty_cache()
+    if args.hybrid_part != "models":
+        w, H, G, ff, W, B, P = z["width"], z["heads"], z["kv_heads"], z["ff"], z["window"], z["batch"], z["prompt"]
+        q_rank, rank, D, R, V = z["latent"]["q_rank"], z["latent"]["kv_rank"], 128, 64, 128
+        E, same, top = (z["experts"][k] for k in ("count", "identity", "top"))
+        eff, bsz = ff * 3 // 2 // top, max(1, B // 8)
+        T = bsz * P
+        freq = rotary_frequencies(1e6, R).to(dev)
+        lw = -(-rank // 64) * 64 + 64
+        with torch.inference_mode():
+            # ---- the stream and the elementwise steps
+            wf, x32, y, u, c16 = torch.ones(w, device=dev), rnd(T, w, dtype=torch.float32), rnd(T, w), rnd(T, 2 * w), torch.empty(T, w, dtype=bf, device=dev)
+            kernel("prompt: gated_sum_norm", [lambda: ops.gated_sum_norm(x32, y, wf, c16, 4, 1e-6, 2.0, u[:, w:], wf)], T * w * 14)
+            kernel("prompt: postnorm_add (dafovik)", [lambda: ops.postnorm_add(x32, y, wf, c16, 1e-6, 0.5, 1.0)], T * w * 12)
+            z_ = rnd(T, E + same, dtype=torch.float32)
+            corr = torch.zeros(E + same, device=dev)
+            place, cw, src, off = ops.moe_route(z_, corr, same, top, 4, 2, 1.0)
+            rows_used = int(off[-1])
+            rows = rnd(T * top, w)
+            kernel("prompt: gated_sum_norm over expert rows", [lambda: ops.gated_sum_norm(x32, rows, wf, c16, 4, 1e-6, 2.0, u[:, w:], wf, place=place, choice_weight=cw)],
+                   T * w * 12 + rows_used * w * 2)
+            kernel("prompt: moe_route", [lambda: ops.moe_route(z_, corr, same, top, 4, 2, 1.0)], T * ((E + same) * 4 + top * 20))
+            del rows, y, u
+            gu, act = rnd(T, 2 * ff + w), torch.empty(T, ff, dtype=bf, device=dev)
+            kernel("prompt: swiglu", [lambda: ops.swiglu(gu, act)], T * ff * 6)
+            del gu, act
+            um = rnd(T, ff * 3 // 2)
+            kernel("prompt: gelu_tanh (dafovik)", [lambda: ops.gelu_tanh(um)], um.numel() * 4)
+            del um
+            # ---- expert products, and the library product of as many rows
+            up, down = rnd(E, eff, w, scale=w ** -0.5), rnd(E, w, eff, scale=eff ** -0.5)
+            hid, back = torch.empty(T * top, eff, dtype=bf, device=dev), torch.empty(T * top, w, dtype=bf, device=dev)
+            fl, wb = 2.0 * rows_used * w * eff, E * eff * w * 2
+            kernel("prompt: moe_gemm up + GELU", [lambda: ops.moe_gemm(c16, up, off, hid, src=src, act="gelu")], wb + T * w * 2 + rows_used * eff * 2, fl)
+            kernel("prompt: moe_gemm down", [lambda: ops.moe_gemm(hid, down, off, back)], wb + rows_used * (w + eff) * 2, fl)
+            a_, b_ = hid[:rows_used], back[:rows_used]
+            kernel("prompt: library product of the down shape (one weight)", [lambda: torch.mm(a_, down[0].t(), out=b_)], rows_used * (w + eff) * 2, fl)
+            del hid, back, a_, b_, x32, c16, z_, place, cw, src, off
+            # ---- recurrence
+            hd = H * D
+            cache, b = batch_for(RecurrentState(H, D, V), bsz, P)
+            proj, yy, oo = rnd(T, 3 * hd + w), torch.empty(T, H * V, dtype=bf, device=dev), torch.empty(T, H * V, dtype=bf, device=dev)
+            fb, lo, nw = 2 + rnd(hd, dtype=torch.float32), torch.rand(hd, device=dev) * 0.5, torch.ones(V, device=dev)
+            fl = T * H * (2.0 * 8 * (D + V) + 4.0 * D * V)          # blocks of 16: causal half of the block, state in and out
+            kernel("prompt: chanrec_chunk", [lambda: ops.chanrec(proj[:, :hd], proj[:, hd:2 * hd], proj[:, 2 * hd:3 * hd], fb, lo, cache.arrays(0)["state"], b, yy)],
+                   T * 4 * hd * 2, fl)
+            kernel("prompt: gated_norm (per head, no gate)", [lambda: ops.gated_norm(yy, None, nw, oo, H, 1e-6)], T * hd * 4)
+            dec_ = torch.linspace(0.9, 0.999, H, device=dev)
+            ldec = torch.log(dec_)
+            fl = T * H * (2.0 * 32 * (D + V) + 4.0 * D * V)
+            kernel("prompt: linrec (dafovik, retention)", [lambda: ops.linrec(proj[:, :hd], proj[:, hd:2 * hd], proj[:, 2 * hd:3 * hd], cache.arrays(0)["state"], b, yy, H, head_decay=dec_, head_log_decay=ldec)],
+                   T * 4 * hd * 2, fl)
+            kernel("prompt: gated_norm (dafovik, retention)", [lambda: ops.gated_norm(yy, proj[:, :hd], None, oo, H, 1e-6, False)], T * hd * 6)
+            del proj, yy, oo, cache
+            # ---- latent attention, prompt
+            cache, b = batch_for(LatentState(lw, W), bsz, P)
+            u, qn, kn = rnd(T, q_rank + rank + R + w), torch.ones(q_rank, device=dev), torch.ones(rank, device=dev)
+            kernel("prompt: latent_prep", [lambda: ops.latent_prep(u, qn, kn, 1e-6, R, R, freq, cache.arrays(0)["latent"], b, W)],
+                   T * (q_rank * 4 + (rank + R) * 2 + lw * 2) + bsz * min(W, P) * lw * 2)
+            lin = rnd(T, lw)
+            del u
+            q, kv, oo = rnd(T, H * (D + R)), rnd(T, H * (D + V)), torch.empty(T, H * V, dtype=bf, device=dev)
+            kernel("prompt: rotate_pairs", [lambda: ops.rotate_pairs(q, b, H, D + R, D, R, freq)], T * H * R * 4)
+            q = rnd(T, H * (D + R))
+            keys = sum(min(i + 1, W) for i in range(P)) * bsz
+            kernel("prompt: latent_prefill", [lambda: ops.latent_prefill(q, kv, lin, b, 192 ** -0.5, oo, H, D, R, V, rank, W)],
+                   T * (H * (2 * D + R + 2 * V) + lw) * 2, keys * H * 2.0 * (D + R + V))
+            del q, kv, lin, cache
+            dc = 64
+            cols = 2 * (H + G) * dc + G * V
+            lam, on = torch.full((1,), 0.4, device=dev), torch.ones(dc, device=dev)
+            cache, b = batch_for(WindowState(G, 64, 128, W), bsz, P)
+            proj, gate = rnd(T, cols + H), rnd(T, H)
+            kernel("prompt: diff_prep + diff_prefill (dafovik)", [lambda: ops.diff_attention(proj, gate, on, on, cache.arrays(0)["k"], cache.arrays(0)["v"], b, lam, 0.5, 0.125, 1e-6, oo, H, dc, V, W)],
+                   T * (2 * cols + 2 * H * V), keys * H * 2.0 * 2 * (dc + V))
+            del proj, gate, oo, cache
+            # ---- one token per request
+            for bsz in (B, 4 * B):
+                cache, b = batch_for(RecurrentState(H, D, V), bsz, 1, start=P)
+                state = cache.arrays(0)["state"]
+                n = max(1, -(-300_000_000 // (state.numel() * 4)))
+                states, proj, out = [torch.zeros_like(state) for _ in range(n)], rnd(bsz, 3 * hd + w), torch.empty(bsz, H * V, dtype=bf, device=dev)
+                kernel(f"decode b{bsz}: chanrec_step", [lambda s=s: ops.chanrec_step(proj[:, :hd], proj[:, hd:2 * hd], proj[:, 2 * hd:3 * hd], fb, lo, nw, s, b, out, 1e-6) for s in states],
+                       bsz * H * D * V * 8)
+                p4, f4 = rnd(bsz, 4 * hd), rotary_frequencies(1e6, D).to(dev)
+                kernel(f"decode b{bsz}: retention_step (dafovik)", [lambda s=s: ops.retention_step(p4, s, b, dec_, f4, out, D, D, D ** -0.5, 1e-6) for s in states],
+                       bsz * H * D * V * 8)
+                del states, state, cache
+                cache, b = batch_for(LatentState(lw, W), bsz, 1, start=W)
+                shape = cache.arrays(0)["latent"].shape
+                n = max(2, -(-300_000_000 // (shape[0] * shape[1] * shape[2] * 2)))
+                rings = [rnd(*shape) for _ in range(n)]
+                qa, q3, ol = rnd(H, bsz, rank), rnd(bsz, H, D + R), torch.empty(H, bsz, rank, dtype=bf, device=dev)
+                kernel(f"decode b{bsz}: latent_decode", [lambda r=r: ops.latent_decode(qa.transpose(0, 1), q3, R, freq, r, b, 192 ** -0.5, ol.transpose(0, 1), R) for r in rings],
+                       bsz * W * lw * 2, bsz * W * H * 2.0 * (lw + rank))
+                del rings, cache
+                cache, b = batch_for(WindowState(G, 64, 128, W), bsz, 1, start=W)
+                n = max(1, -(-300_000_000 // (cache.arrays(0)["k"].numel() * 4)))
+                rings = [(rnd(*cache.arrays(0)["k"].shape), rnd(*cache.arrays(0)["v"].shape)) for _ in range(n)]
+                proj, gate, out = rnd(bsz, cols + H), rnd(bsz, H), torch.empty(bsz, H * V, dtype=bf, device=dev)
+                kernel(f"decode b{bsz}: diff_prep + diff_decode (dafovik)", [lambda r=r: ops.diff_attention(proj, gate, on, on, r[0], r[1], b, lam, 0.5, 0.125, 1e-6, out, H, dc, V, W) for r in rings],
+                       bsz * G * W * (2 * dc + V) * 2)
+                del rings, cache, proj, gate
+                x16, z_ = rnd(bsz, w), rnd(bsz, E + same, dtype=torch.float32)
+                _, _, src, off = ops.moe_route(z_, corr, same, top, 4, 2, 1.0)
+                live, rows_used = int((off[1:] > off[:-1]).sum()), int(off[-1])
+                hid, back = torch.empty(bsz * top, eff, dtype=bf, device=dev), torch.empty(bsz * top, w, dtype=bf, device=dev)
+                n = max(1, -(-300_000_000 // (up.numel() * 2)))
+                ups, downs = [up] + [rnd(*up.shape, scale=w ** -0.5) for _ in range(n - 1)], [down] + [rnd(*down.shape, scale=eff ** -0.5) for _ in range(n - 1)]
+                kernel(f"decode b{bsz}: moe_route", [lambda: ops.moe_route(z_, corr, same, top, 4, 2, 1.0)], bsz * (E + same) * 4)
+                kernel(f"decode b{bsz}: moe_gemm up + GELU", [lambda a=a: ops.moe_gemm(x16, a, off, hid, src=src, act="gelu") for a in ups], live * eff * w * 2, 2.0 * rows_used * w * eff)
+                kernel(f"decode b{bsz}: moe_gemm down", [lambda a=a: ops.moe_gemm(hid, a, off, back) for a in downs], live * eff * w * 2, 2.0 * rows_used * w * eff)
+                dense = [rnd(2 * ff + w, w) for _ in range(max(2, -(-300_000_000 // ((2 * ff + w) * w * 2))))]
+                kernel(f"decode b{bsz}: library product (gate, up, residual gate)", [lambda a=a: torch.mm(x16, a.t()) for a in dense], dense[0].numel() * 2)
+                del ups, downs, dense
+        res["kernels"] = tools.rows
+    print(json.dumps(res))
+
+
 def parse_args(argv=None):
     ap = argparse.ArgumentParser()
-    ap.add_argument("--micro", default=None, choices=["evict", "attn", "append", "steady", "multi", "prefill", "generate", "hybrid"],
+    ap.add_argument("--micro", default=None, choices=["evict", "attn", "append", "steady", "multi", "prefill", "generate", "hybrid", "lonulix"],
                     help="run one kernel microbenchmark instead of the decode benchmark")
     ap.add_argument("--hybrid-size", default="1.7b", choices=sorted(HYBRID_SIZES) + ["all"], help="hybrid microbenchmark: layer sizes")
     ap.add_argument("--hybrid-part", default="all", choices=["all", "models", "kernels"],

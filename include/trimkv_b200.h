@@ -591,7 +591,7 @@ int tkv_rotate_pairs(void* x, int64_t row_stride, const int32_t* cu_tokens, cons
  * tkv_latent_decode: one token per request against the ring, in the latent space: q_abs [.., kv_rank] = W_uk^T q per head, q_rot
  * [.., rot_dim] not yet rotated (already rotated where the workspace size is -1), out [.., kv_rank] = softmax-weighted latents;
  * strides in elements between tokens and heads.  Workspace: tkv_latent_decode_workspace_bytes (-1: none, the form for every
- * size and dtype; the fast one takes bf16, kv_rank <= 512, rot_dim <= 128). */
+ * size and dtype; the fast one takes bf16, kv_rank <= 512, 0 < rot_dim <= 64). */
 int tkv_latent_prep(const void* u, int64_t u_stride, const float* q_norm, const float* kv_norm, float eps, int q_rank, int kv_rank,
                     int rot_dim, int rot_dims, const float* freq_hi_lo, void* cq, void* ring, int ring_rows, void* lin,
                     const int32_t* kv_start, const int32_t* cu_tokens, const int32_t* slots, const int32_t* pos0, int batch,

@@ -10,8 +10,8 @@
 //
 // One CTA walks chunks of 32 tokens (two blocks) of one (request, head, block of 16 * kWarps value columns, segment of the
 // sequence).  The state never leaves registers: a warp owns 16 columns of v and holds S^T [16 x n] as fp32 MMA accumulators, whose
-// layout is also the A-operand layout of the read-out.  Per chunk: gates and scaled vectors of all channels (a thread walks a
-// channel of a block), the two 16 x 16 blocks a, then every warp its own columns without further barriers.
+// layout is also the A-operand layout of the read-out.  Per chunk: gates and scaled vectors of all channels (a thread walks two
+// channels of half a block), the two 16 x 16 blocks a, then every warp its own columns without further barriers.
 // Where (request, head, column) blocks alone do not fill the GPU, the sequence is cut into segments: a first pass computes
 // every segment's own state, a small kernel chains them, and the main pass starts each segment from its true state.
 #include "tkv_chanrec.cuh"
@@ -55,11 +55,29 @@ __device__ __forceinline__ void cr_sigmoid(float x, float* pos, float* neg) {
   *neg = x >= 0.f ? small : r;
 }
 
+__device__ __forceinline__ float cr_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// f, 1 / f and k = 1 - f with one reciprocal: with e = exp(-|x|), sigmoid(|x|) = 1 / (1 + e), f = num / (1 + e).  Where f leaves
+// the range of fp32 the result is not a number, or zero; the caller looks at the product.
+__device__ __forceinline__ void cr_gate(float x, float lo, float* f, float* inv, float* k) {
+  const float e = exp2_weight(fabsf(x) * -1.4426950408889634f), den = 1.0f + e, rest = 1.0f - lo;
+  const float num = fmaf(rest, x >= 0.f ? 1.0f : e, lo * den);
+  const float t = cr_rcp(den * num), u = num * t;         // u = 1 / den
+  *f = num * u;
+  *inv = den * den * t;
+  *k = rest * (x >= 0.f ? e : 1.0f) * u;
+}
+__device__ __forceinline__ float cr_silu(float z) { return z * cr_rcp(1.0f + exp2_weight(z * -1.4426950408889634f)); }
+
 template <int NP, int kWarps> struct CrSmem {
   static constexpr int PT = kWarps * 16, QS = NP + 8, VS = PT + 8, PS = kCrBlock + 8;
   __nv_bfloat16 zq[2][kCrTokens * QS], zf[2][kCrTokens * QS], v[2][kCrTokens * VS];
   __nv_bfloat16 q_hi[kCrTokens * QS], q_lo[kCrTokens * QS], k_hi[kCrTokens * QS], k_lo[kCrTokens * QS];
   __nv_bfloat16 a_hi[2][kCrBlock * PS], a_lo[2][kCrBlock * PS];
+  float mid[2][2][NP];                                    // P and 1 / P in the middle of a block
   float end[2][NP];                                       // product of the gates of a block
   float gate[2][3][NP];                                   // q, f, k of one token (token-by-token path)
 };
@@ -104,18 +122,6 @@ __global__ void __launch_bounds__(kWarps * 32, NP == 256 ? 1 : kWarps == 8 ? 2 :
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  // f and k = 1 - f of a channel; a token or channel that does not exist leaves the state as it is
-  auto gate = [&](float z, float lo, bool live, float* f, float* k) {
-    float pos, neg;
-    cr_sigmoid(z, &pos, &neg);
-    *f = live ? fmaf(1.0f - lo, pos, lo) : 1.0f;
-    *k = live ? (1.0f - lo) * neg : 0.0f;
-  };
-  auto query = [&](float z) {
-    float pos, neg;
-    cr_sigmoid(z, &pos, &neg);
-    return z * pos;
-  };
 
   // ---- state: S^T rows p0 + gr (+ 8), columns 8 nt + 2 gc (+ 1)
   float s[NP / 8][4];
@@ -143,38 +149,70 @@ __global__ void __launch_bounds__(kWarps * 32, NP == 256 ? 1 : kWarps == 8 ? 2 :
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();                                       // this chunk is here; everyone is done with the last one
     if (chunk + 1 < c1) fetch(chunk + 1);
-    // ---- gates and scaled vectors: a thread walks one channel of one block
+    // ---- gates and scaled vectors: a thread walks two channels of half a block, four warps take 64 channels
     bool tiny = false;
-    for (int i = tid; i < 2 * NP; i += kThreads) {
-      const int blk = i / NP, c = i - blk * NP;
-      const bool ch = c < a.n;
-      const float bi = ch ? bias[c] : 0.f, lo = ch ? lower[c] : 0.f;
-      float P = 1.0f;
 #pragma unroll
-      for (int j = 0; j < kCrBlock; ++j) {
-        const int r = blk * kCrBlock + j;
-        float f, k;
-        gate(__bfloat162float(sm.zf[st][r * QS + c]) + bi, lo, ch && t0 + r < ntok, &f, &k);
-        P *= f;
-        const float ks = __fdividef(k, P);
-        const __nv_bfloat16 kh = __float2bfloat16_rn(ks);
-        sm.k_hi[r * QS + c] = kh;
-        sm.k_lo[r * QS + c] = __float2bfloat16_rn(ks - __bfloat162float(kh));
-        if (!kStateOnly) {
-          const float qs = query(__bfloat162float(sm.zq[st][r * QS + c])) * P;
-          const __nv_bfloat16 qh = __float2bfloat16_rn(qs);
-          sm.q_hi[r * QS + c] = qh;
-          sm.q_lo[r * QS + c] = __float2bfloat16_rn(qs - __bfloat162float(qh));
+    for (int c64 = 0; c64 < NP; c64 += kWarps * 16) {
+      const int blk = (warp >> 1) & 1, half = warp & 1, c = c64 + (warp >> 2) * 64 + 2 * lane, r0 = blk * kCrBlock + half * 8;
+      const bool on = c < NP;
+      float P[8][2], kp[8][2], inv[2] = {1.0f, 1.0f};      // product up to a token, k over it
+      if (on) {
+        // a channel that does not exist keeps its (zero) state: lower bound 1
+        const float2 bi = c < a.n ? *reinterpret_cast<const float2*>(bias + c) : make_float2(0.f, 0.f);
+        const float2 lo = c < a.n ? *reinterpret_cast<const float2*>(lower + c) : make_float2(1.f, 1.f);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          float f[2] = {1.0f, 1.0f}, fi[2] = {1.0f, 1.0f}, k[2] = {0.f, 0.f};
+          if (t0 + r0 + j < ntok) {
+            const uint32_t z = *reinterpret_cast<const uint32_t*>(&sm.zf[st][(r0 + j) * QS + c]);
+            cr_gate(__uint_as_float(z << 16) + bi.x, lo.x, &f[0], &fi[0], &k[0]);
+            cr_gate(__uint_as_float(z & 0xffff0000u) + bi.y, lo.y, &f[1], &fi[1], &k[1]);
+          }
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            P[j][e] = j > 0 ? P[j - 1][e] * f[e] : f[e];
+            inv[e] *= fi[e];
+            kp[j][e] = k[e] * inv[e];
+          }
+        }
+        if (half == 0) {
+          *reinterpret_cast<float2*>(&sm.mid[0][blk][c]) = make_float2(P[7][0], P[7][1]);
+          *reinterpret_cast<float2*>(&sm.mid[1][blk][c]) = make_float2(inv[0], inv[1]);
         }
       }
-      sm.end[blk][c] = P;
-      tiny |= P < kFloor;
+      __syncthreads();
+      if (on) {
+        float2 p0 = make_float2(1.0f, 1.0f), i0 = p0;
+        if (half == 1) {
+          p0 = *reinterpret_cast<const float2*>(&sm.mid[0][blk][c]);
+          i0 = *reinterpret_cast<const float2*>(&sm.mid[1][blk][c]);
+          const float2 end = make_float2(p0.x * P[7][0], p0.y * P[7][1]);
+          *reinterpret_cast<float2*>(&sm.end[blk][c]) = end;
+          tiny |= !(end.x >= kFloor && end.y >= kFloor);
+        }
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          const int at = (r0 + j) * QS + c;
+          uint32_t hi, lo_;
+          cr_split(kp[j][0] * i0.x, kp[j][1] * i0.y, &hi, &lo_);
+          *reinterpret_cast<uint32_t*>(&sm.k_hi[at]) = hi;
+          *reinterpret_cast<uint32_t*>(&sm.k_lo[at]) = lo_;
+          if (!kStateOnly) {
+            const uint32_t z = *reinterpret_cast<const uint32_t*>(&sm.zq[st][at]);
+            cr_split(cr_silu(__uint_as_float(z << 16)) * (P[j][0] * p0.x), cr_silu(__uint_as_float(z & 0xffff0000u)) * (P[j][1] * p0.y), &hi, &lo_);
+            *reinterpret_cast<uint32_t*>(&sm.q_hi[at]) = hi;
+            *reinterpret_cast<uint32_t*>(&sm.q_lo[at]) = lo_;
+          }
+        }
+      }
     }
     const bool walk = __syncthreads_or(tiny);
+    if (kStateOnly && !walk) {
 #pragma unroll
-    for (int i = 0; i < kOwn; ++i) {
-      const int c = tid + i * kThreads;
-      if (c < NP) seg_decay[i] *= sm.end[0][c] * sm.end[1][c];
+      for (int i = 0; i < kOwn; ++i) {
+        const int c = tid + i * kThreads;
+        if (c < NP) seg_decay[i] *= sm.end[0][c] * sm.end[1][c];
+      }
     }
     __nv_bfloat16* v_s = sm.v[st];
     if (!walk) {
@@ -269,10 +307,18 @@ __global__ void __launch_bounds__(kWarps * 32, NP == 256 ? 1 : kWarps == 8 ? 2 :
       const int live_tokens = min(kCrTokens, ntok - t0);
       for (int r = 0; r < live_tokens; ++r) {
         float (*g)[NP] = sm.gate[r & 1];
-        for (int c = tid; c < NP; c += kThreads) {
+#pragma unroll
+        for (int i = 0; i < kOwn; ++i) {
+          const int c = tid + i * kThreads;
+          if (c >= NP) continue;
           const bool ch = c < a.n;
-          gate(__bfloat162float(sm.zf[st][r * QS + c]) + (ch ? bias[c] : 0.f), ch ? lower[c] : 0.f, ch, &g[1][c], &g[2][c]);
-          if (!kStateOnly) g[0][c] = query(__bfloat162float(sm.zq[st][r * QS + c]));
+          float pos, neg;
+          cr_sigmoid(__bfloat162float(sm.zf[st][r * QS + c]) + (ch ? bias[c] : 0.f), &pos, &neg);
+          const float lo = ch ? lower[c] : 1.0f;
+          g[1][c] = fmaf(1.0f - lo, pos, lo);
+          g[2][c] = (1.0f - lo) * neg;
+          if (kStateOnly) seg_decay[i] *= g[1][c];
+          else g[0][c] = cr_silu(__bfloat162float(sm.zq[st][r * QS + c]));
         }
         __syncthreads();                                   // two buffers: one barrier per token
         const float v0 = __bfloat162float(v_s[r * VS + p0 + gr]), v1 = __bfloat162float(v_s[r * VS + p0 + gr + 8]);

@@ -214,10 +214,11 @@ int launch_two_part_any(const char* what, const TwoPartAttn& p, int dtype, cudaS
 }
 
 // ---------------------------------------------------------------------------------------------------- split-KV decode
-// CTA = (a chunk of ring rows, request, 16 * MT query heads), eight warps, tiles of 64 rows through shared memory (two stages,
-// 16-byte chunks XOR-swizzled by row).  Scores: warp w takes rows 8 w .. of the tile against all queries; softmax: a warp
-// takes 2 * MT heads; weighted sum: a warp takes cpad / 8 = 8 * NT value dims for all heads.
-constexpr int kLdThreads = 256, kLdTile = 64;
+// CTA = (a chunk of ring rows, request, 16 * MT query heads), eight warps, tiles of 32 rows through a ring of shared-memory
+// stages (16-byte pieces XOR-swizzled by row).  Scores: a warp takes 16 rows of the tile and a quarter of the contraction, its
+// part of the queries stays in registers; softmax: a warp adds the quarters up and takes 2 * MT heads; weighted sum: a warp takes
+// cpad / 8 = 8 * NT value dims for all heads.
+constexpr int kLdThreads = 256, kLdTile = 32;
 
 struct LatentDecode {
   const void* q_abs; int64_t qa_token, qa_head;           // queries in the latent space, [.., cdim]
@@ -246,21 +247,24 @@ __device__ __forceinline__ void ld_x4t(uint32_t* r, uint32_t addr) {
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
 }
 
-template <int NT, int MT>
-static size_t latent_decode_smem(int lw) {
-  return (size_t)2 * kLdTile * lw * 2 + (size_t)16 * MT * ((lw + 8) * 2 + (kLdTile + 4) * 4 + (kLdTile + 8) * 2 + 4);
-}
+template <int NT, int MT> struct LatentTile {
+  static constexpr int R = 16 * MT, LW = 64 * (NT + 1), QS = LW + 8, SS = kLdTile + 4, PS = kLdTile + 8;
+  static constexpr int kStages = NT <= 2 ? 8 : NT <= 5 ? 6 : 5, kStageBytes = kLdTile * LW * 2;
+  static constexpr int kQBytes = R * QS * 2, kSBytes = 4 * R * SS * 4;           // the queries' place is taken by the scores
+  static constexpr int kUnion = kQBytes > kSBytes ? kQBytes : kSBytes;
+  static constexpr int kBytes = kStages * kStageBytes + kUnion + R * PS * 2 + R * 4;
+};
 
 template <int NT, int MT>
 __global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(LatentDecode p) {
+  using L = LatentTile<NT, MT>;
+  constexpr int R = L::R, LW = L::LW, QS = L::QS, SS = L::SS, PS = L::PS, S = L::kStages, kPieces = LW / 8, KS = LW / 64;
   extern __shared__ __align__(128) uint8_t raw[];
-  constexpr int R = 16 * MT, kSs = kLdTile + 4, kPs = kLdTile + 8;
-  const int lw = p.lw, qs = lw + 8;
-  uint8_t* tiles = raw;                                                          // [2][64][lw] swizzled
-  __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(raw + (size_t)2 * kLdTile * lw * 2);   // [R][qs]
-  __nv_bfloat16* p_s = q_s + R * qs;                                             // [R][kPs]
-  float* s_s = reinterpret_cast<float*>(p_s + R * kPs);                          // [R][kSs]
-  float* fix_s = s_s + R * kSs;                                                  // [R]
+  uint8_t* tiles = raw;                                                          // [S][32][LW] swizzled
+  __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(raw + S * L::kStageBytes);   // [R][QS], then
+  float* s_s = reinterpret_cast<float*>(q_s);                                    // [4][R][SS]
+  __nv_bfloat16* p_s = reinterpret_cast<__nv_bfloat16*>(raw + S * L::kStageBytes + L::kUnion);   // [R][PS]
+  float* fix_s = reinterpret_cast<float*>(p_s + R * PS);                         // [R]
   grid_dependency_wait();
   grid_launch_dependents();
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gr = lane >> 2, gc = lane & 3;
@@ -268,93 +272,102 @@ __global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(LatentDecode 
   const int pos = p.pos0[b], len = min(pos + 1, p.ring_rows);
   const int t0 = blockIdx.x * p.chunk, t1 = min(len, t0 + p.chunk);
   if (t0 >= len) return;
-  const __nv_bfloat16* K = (const __nv_bfloat16*)p.ring + (int64_t)p.slots[b] * p.ring_rows * lw;
-  const int chunks = lw / 8;
-  auto fetch = [&](int t, int st) {
-    uint8_t* dst = tiles + (size_t)st * kLdTile * lw * 2;
-    for (int i = tid; i < kLdTile * chunks; i += kLdThreads) {
-      const int r = i / chunks, c = i - r * chunks;
-      const bool live = t + r < t1;                       // the rest reads as zeros
-      const int bytes = live ? 16 : 0;
-      const void* src = K + (live ? (int64_t)(t + r) * lw + c * 8 : 0);
-      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst + ((size_t)r * chunks + (c ^ (r & 7))) * 16)), "l"(src), "r"(bytes) : "memory");
-    }
+  const __nv_bfloat16* K = (const __nv_bfloat16*)p.ring + (int64_t)p.slots[b] * p.ring_rows * LW;
+  auto fetch = [&](int t, int st) {                       // a group per tile, empty beyond the end
+    const uint32_t dst = smem_u32(tiles) + st * L::kStageBytes;
+    if (t < t1)
+#pragma unroll
+      for (int j = 0; j < kLdTile * kPieces / kLdThreads; ++j) {
+        const int i = tid + j * kLdThreads, r = i / kPieces, c = i - r * kPieces;
+        const bool live = t + r < t1;                     // the rest reads as zeros
+        const int bytes = live ? 16 : 0;
+        const void* src = K + (live ? (int64_t)(t + r) * LW + c * 8 : 0);
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst + (r * kPieces + (c ^ (r & 7))) * 16), "l"(src), "r"(bytes) : "memory");
+      }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  fetch(t0, 0);
+#pragma unroll
+  for (int i = 0; i < S - 1; ++i) fetch(t0 + i * kLdTile, i);
   // ---- queries: absorbed part as it is, rotary part turned to this position
-  for (int i = tid; i < R * p.cpad; i += kLdThreads) {
-    const int r = i / p.cpad, c = i - r * p.cpad;
-    q_s[r * qs + c] = r < nh && c < p.cdim ? ((const __nv_bfloat16*)p.q_abs)[(int64_t)b * p.qa_token + (int64_t)(h0 + r) * p.qa_head + c]
+  for (int i = tid; i < R * NT * 64; i += kLdThreads) {
+    const int r = i / (NT * 64), c = i - r * (NT * 64);
+    q_s[r * QS + c] = r < nh && c < p.cdim ? ((const __nv_bfloat16*)p.q_abs)[(int64_t)b * p.qa_token + (int64_t)(h0 + r) * p.qa_head + c]
                                            : __float2bfloat16_rn(0.f);
   }
-  const int rpad = lw - p.cpad;
-  for (int i = tid; i < rpad / 2; i += kLdThreads) {
-    const int c = 2 * i;
+  {
+    const int i = tid & 31, c = 2 * i;                    // pair i of heads warp, warp + 8, ..
     float s = 0.f, co = 1.f;
     if (c < p.rot_dims) turn(pos, p.freq[i].x, p.freq[i].y, &s, &co);
-    for (int r = 0; r < R; ++r) {
+    for (int r = warp; r < R; r += kLdThreads / 32) {
       float x = 0.f, y = 0.f;
       if (r < nh && c < p.rot_dim) {
         const __nv_bfloat16* src = (const __nv_bfloat16*)p.q_rot + (int64_t)b * p.qr_token + (int64_t)(h0 + r) * p.qr_head + c;
         x = __bfloat162float(src[0]);
         if (c + 1 < p.rot_dim) y = __bfloat162float(src[1]);
       }
-      q_s[r * qs + p.cpad + c] = __float2bfloat16_rn(x * co - y * s);
-      q_s[r * qs + p.cpad + c + 1] = __float2bfloat16_rn(y * co + x * s);
+      q_s[r * QS + NT * 64 + c] = __float2bfloat16_rn(x * co - y * s);
+      q_s[r * QS + NT * 64 + c + 1] = __float2bfloat16_rn(y * co + x * s);
     }
   }
+  __syncthreads();
+  const int rg = warp & 1, kq = warp >> 1;                // 16 rows of a tile, quarter of the contraction
+  uint32_t qf[MT][KS][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int k = 0; k < KS; ++k)
+      ld_x4(qf[m][k], smem_u32(q_s) + (uint32_t)((m * 16 + (lane & 15)) * QS + (kq * KS + k) * 16 + (lane >> 4) * 8) * 2);
   float o[MT][NT][4] = {};
   float mx[2 * MT], l[2 * MT];
 #pragma unroll
   for (int i = 0; i < 2 * MT; ++i) { mx[i] = -INFINITY; l[i] = 0.f; }
-  const uint32_t q_addr = smem_u32(q_s), p_addr = smem_u32(p_s);
+  const uint32_t p_addr = smem_u32(p_s);
   int st = 0;
-  for (int t = t0; t < t1; t += kLdTile, st ^= 1) {
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();                                      // this tile is here; everyone is done with the other stage
-    if (t + kLdTile < t1) fetch(t + kLdTile, st ^ 1);
-    const uint32_t tile = smem_u32(tiles + (size_t)st * kLdTile * lw * 2);
-    // ---- scores: rows 8 * warp .. + 7, two accumulators per product to shorten the dependent chain
+  for (int t = t0; t < t1; t += kLdTile, st = st + 1 == S ? 0 : st + 1) {
+    asm volatile("cp.async.wait_group %0;" ::"n"(S - 2) : "memory");
+    __syncthreads();                                      // this tile is here; everyone is done with the last one
+    fetch(t + (S - 1) * kLdTile, st == 0 ? S - 1 : st - 1);
+    const uint32_t tile = smem_u32(tiles) + st * L::kStageBytes;
+    // ---- scores
     {
       float acc[MT][2][4] = {};
-      const int row = warp * 8 + (lane & 7);
-      const uint32_t krow = tile + (uint32_t)row * lw * 2;
-#pragma unroll 2
-      for (int kk = 0; kk < lw / 32; ++kk) {
+      const int row = rg * 16 + (lane & 7) + ((lane >> 4) & 1) * 8;
+      const uint32_t krow = tile + (uint32_t)row * LW * 2;
+#pragma unroll
+      for (int k = 0; k < KS; ++k) {
         uint32_t kf[4];
-        ld_x4(kf, krow + (uint32_t)(((kk * 4 + (lane >> 3)) ^ (row & 7)) * 16));
+        ld_x4(kf, krow + (uint32_t)((((kq * KS + k) * 2 + ((lane >> 3) & 1)) ^ (row & 7)) * 16));
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
-          uint32_t a0[4], a1[4];
-          const uint32_t at = q_addr + (uint32_t)((m * 16 + (lane & 15)) * qs + kk * 32 + (lane >> 4) * 8) * 2;
-          ld_x4(a0, at);
-          ld_x4(a1, at + 32);
-          ld_mma(acc[m][0], a0, kf[0], kf[1]);
-          ld_mma(acc[m][1], a1, kf[2], kf[3]);
+          ld_mma(acc[m][0], qf[m][k], kf[0], kf[1]);
+          ld_mma(acc[m][1], qf[m][k], kf[2], kf[3]);
         }
       }
 #pragma unroll
       for (int m = 0; m < MT; ++m)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) s_s[(m * 16 + gr + (e >> 1) * 8) * kSs + warp * 8 + 2 * gc + (e & 1)] = acc[m][0][e] + acc[m][1][e];
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+          for (int e = 0; e < 4; e += 2)
+            *reinterpret_cast<float2*>(s_s + (kq * R + m * 16 + gr + (e >> 1) * 8) * SS + rg * 16 + n * 8 + 2 * gc) = make_float2(acc[m][n][e], acc[m][n][e + 1]);
     }
     __syncthreads();
     // ---- softmax of heads warp * 2 MT ..
 #pragma unroll
     for (int i = 0; i < 2 * MT; ++i) {
       const int r = warp * 2 * MT + i;
-      const float s0 = t + lane < t1 ? s_s[r * kSs + lane] * p.scale_log2 : -INFINITY;
-      const float s1 = t + 32 + lane < t1 ? s_s[r * kSs + 32 + lane] * p.scale_log2 : -INFINITY;
-      float top = fmaxf(s0, s1);
+      float x = 0.f;
+#pragma unroll
+      for (int q = 0; q < 4; ++q) x += s_s[(q * R + r) * SS + lane];
+      x = t + lane < t1 ? x * p.scale_log2 : -INFINITY;
+      float top = x;
 #pragma unroll
       for (int d = 16; d >= 1; d >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, d));
       top = fmaxf(top, mx[i]);                            // finite: the first row of a tile is always in range
-      const float fix = exp2_weight(mx[i] - top), w0 = exp2_weight(s0 - top), w1 = exp2_weight(s1 - top);
+      const float fix = exp2_weight(mx[i] - top), w = exp2_weight(x - top);
       mx[i] = top;
-      l[i] = fmaf(l[i], fix, w0 + w1);                    // this lane's part of the sum
-      p_s[r * kPs + lane] = __float2bfloat16_rn(w0);
-      p_s[r * kPs + 32 + lane] = __float2bfloat16_rn(w1);
+      l[i] = fmaf(l[i], fix, w);                          // this lane's part of the sum
+      p_s[r * PS + lane] = __float2bfloat16_rn(w);
       if (lane == 0) fix_s[r] = fix;
     }
     __syncthreads();
@@ -369,13 +382,13 @@ __global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(LatentDecode 
     for (int k = 0; k < kLdTile / 16; ++k) {
       uint32_t pf[MT][4];
 #pragma unroll
-      for (int m = 0; m < MT; ++m) ld_x4(pf[m], p_addr + (uint32_t)((m * 16 + (lane & 15)) * kPs + k * 16 + (lane >> 4) * 8) * 2);
+      for (int m = 0; m < MT; ++m) ld_x4(pf[m], p_addr + (uint32_t)((m * 16 + (lane & 15)) * PS + k * 16 + (lane >> 4) * 8) * 2);
       const int row = k * 16 + (lane & 15);
 #pragma unroll
       for (int n = 0; n < NT; n += 2) {
         uint32_t vf[4];
         const int c = warp * NT + min(n + (lane >> 4), NT - 1);
-        ld_x4t(vf, tile + (uint32_t)row * lw * 2 + (uint32_t)((c ^ (row & 7)) * 16));
+        ld_x4t(vf, tile + (uint32_t)row * LW * 2 + (uint32_t)((c ^ (row & 7)) * 16));
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
           ld_mma(o[m][n], pf[m], vf[0], vf[1]);
@@ -427,13 +440,12 @@ __global__ void __launch_bounds__(kLpThreads) latent_merge_kernel(LatentDecode p
   }
 }
 
-static bool latent_decode_shape(int cdim, int rot_dim, int dtype) { return dtype == TKV_BF16 && cdim <= 512 && rot_dim <= 128; }
+static bool latent_decode_shape(int cdim, int rot_dim, int dtype) { return dtype == TKV_BF16 && cdim <= 512 && rot_dim >= 1 && rot_dim <= 64; }
 static int latent_row_tiles(int heads) { return heads > 16 ? 2 : 1; }
 
 // Rows of the ring per CTA: the smallest time under a simple cost (waves of CTAs, each its rows and a fixed start and merge).
-static int latent_chunk(int64_t segments, int ring_rows, int lw, int mt) {
-  const size_t smem = mt == 2 ? latent_decode_smem<8, 2>(lw) : latent_decode_smem<8, 1>(lw);
-  const int64_t width = 148 * (smem <= 112 * 1024 ? 2 : 1);
+static int latent_chunk(int64_t segments, int ring_rows, int cpad) {
+  const int64_t width = 148 * (cpad <= 128 ? 2 : 1);      // CTAs that run at the same time (shared memory)
   int best = 64;
   int64_t best_cost = -1;
   for (int c = 64; c < ring_rows + 64; c += 64) {
@@ -535,21 +547,22 @@ extern "C" int64_t tkv_latent_decode_workspace_bytes(int batch, int heads, int k
   if (batch <= 0 || heads <= 0 || kv_rank <= 0 || rot_dim < 0 || ring_rows <= 0) return 0;
   if (!latent_decode_shape(kv_rank, rot_dim, dtype)) return -1;
   const int mt = latent_row_tiles(heads), groups = (heads + 16 * mt - 1) / (16 * mt), cpad = pad64(kv_rank);
-  const int chunk = latent_chunk((int64_t)batch * groups, ring_rows, cpad + pad64(rot_dim), mt);
+  const int chunk = latent_chunk((int64_t)batch * groups, ring_rows, cpad);
   return (int64_t)batch * groups * ((ring_rows + chunk - 1) / chunk) * 16 * mt * (cpad + 2) * (int64_t)sizeof(float);
 }
 
 namespace tkv {
 template <int NT, int MT>
 static int launch_latent_decode(const LatentDecode& p, dim3 grid, cudaStream_t st) {
-  const size_t smem = latent_decode_smem<NT, MT>(p.lw);
-  static size_t allowed = 48 * 1024;
-  if (smem > allowed) {
-    cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<NT, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  constexpr int kBytes = LatentTile<NT, MT>::kBytes;
+  static_assert(kBytes <= 232448, "shared memory of the kernel");
+  static bool configured = false;
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<NT, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kBytes);
     if (e != cudaSuccess) return fail(TKV_ERR_LAUNCH, "tkv_latent_decode: %s", cudaGetErrorString(e));
-    allowed = smem;
+    configured = true;
   }
-  cudaError_t e = launch_pdl(latent_decode_kernel<NT, MT>, grid, dim3(kLdThreads), smem, st, p);
+  cudaError_t e = launch_pdl(latent_decode_kernel<NT, MT>, grid, dim3(kLdThreads), (size_t)kBytes, st, p);
   if (e == cudaSuccess) e = launch_pdl(latent_merge_kernel, dim3((unsigned)(p.batch * p.heads)), dim3(kLpThreads), 0, st, p, (int)grid.x, 16 * MT);
   if (e != cudaSuccess) return fail(TKV_ERR_LAUNCH, "tkv_latent_decode: %s", cudaGetErrorString(e));
   return check_launch("tkv_latent_decode");
@@ -599,7 +612,7 @@ extern "C" int tkv_latent_decode(const void* q_abs, int64_t qa_token, int64_t qa
   if (batch > 65535) return fail(TKV_ERR_UNSUPPORTED, "tkv_latent_decode: batch=%d", batch);
   const int mt = latent_row_tiles(heads), groups = (heads + 16 * mt - 1) / (16 * mt);
   LatentDecode p = {q_abs, qa_token, qa_head, q_rot, qr_token, qr_head, (const float2*)freq_hi_lo, rot_dim, rot_dims, ring, ring_rows, kv_rank,
-                    cpad, lw, slots, pos0, scale * 1.4426950408889634f, batch, heads, latent_chunk((int64_t)batch * groups, ring_rows, lw, mt),
+                    cpad, lw, slots, pos0, scale * 1.4426950408889634f, batch, heads, latent_chunk((int64_t)batch * groups, ring_rows, cpad),
                     nullptr, nullptr, out, out_token, out_head};
   const int chunks = (ring_rows + p.chunk - 1) / p.chunk;
   p.part_o = (float*)workspace;

@@ -25,16 +25,6 @@ struct MoeRoute {
   int32_t* offsets;                                       // [experts - identity + 1]
 };
 
-// Largest value and its lowest index over a warp.
-__device__ __forceinline__ void warp_argmax(float* v, int* i) {
-#pragma unroll
-  for (int o = 16; o >= 1; o >>= 1) {
-    const float ov = __shfl_xor_sync(0xffffffffu, *v, o);
-    const int oi = __shfl_xor_sync(0xffffffffu, *i, o);
-    if (ov > *v || (ov == *v && oi < *i)) { *v = ov; *i = oi; }
-  }
-}
-
 // Exclusive sums of the counts of the experts that own rows, by one warp; off[n] = total.
 __device__ __forceinline__ void warp_offsets(const int32_t* counts, int n, int32_t* off) {
   const int lane = threadIdx.x & 31;
@@ -53,12 +43,14 @@ __device__ __forceinline__ void warp_offsets(const int32_t* counts, int n, int32
   if (lane == 0) off[n] = base;
 }
 
-// One warp per token, kRoutePerWarp tokens in turn.
+// One warp per token, kRoutePerWarp tokens in turn; lane l holds experts l, l + 32, .. (kPer of them).  A choice is the largest
+// order-preserving integer image of the choice scores over the warp, the lowest expert on a tie.
+template <int kPer>
 __global__ void __launch_bounds__(kRouteThreads) moe_route_kernel(MoeRoute p) {
   extern __shared__ float sm[];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, E = p.experts, real = E - p.identity;
-  float* s = sm + (size_t)warp * (E + p.groups);          // scores of the warp's token, then the groups' best
-  float* gs = s + E;
+  float* cs = sm + (size_t)warp * (E + p.groups);         // choice scores of the warp's token, then the groups' best
+  float* gs = cs + E;
   int32_t* hist = reinterpret_cast<int32_t*>(sm + (size_t)kRouteWarps * (E + p.groups));   // [E]
   int32_t* base = hist + E;                               // [E + 1]
   grid_dependency_wait();
@@ -66,63 +58,87 @@ __global__ void __launch_bounds__(kRouteThreads) moe_route_kernel(MoeRoute p) {
   for (int e = threadIdx.x; e < E; e += kRouteThreads) hist[e] = 0;
   __syncthreads();
   const int size = E / p.groups;
+  const bool all_open = p.keep >= p.groups;
+  float corr[kPer];
+  int group[kPer];
+#pragma unroll
+  for (int i = 0; i < kPer; ++i) {
+    const int e = lane + 32 * i;
+    corr[i] = e < E ? p.correction[e] : 0.f;
+    group[i] = e < E ? e / size : 0;
+  }
   const int tok0 = blockIdx.x * kRouteTokens;
   for (int it = 0; it < kRoutePerWarp; ++it) {
     const int t = tok0 + it * kRouteWarps + warp;
     if (t >= p.tokens) break;
     const float* z = p.logits + (int64_t)t * p.stride;
-    float top = -INFINITY, sum = 0.f;
-    for (int e = lane; e < E; e += 32) top = fmaxf(top, z[e]);
+    float s[kPer], top = -INFINITY, sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < kPer; ++i) {
+      s[i] = lane + 32 * i < E ? z[lane + 32 * i] : -INFINITY;
+      top = fmaxf(top, s[i]);
+    }
 #pragma unroll
     for (int o = 16; o >= 1; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
-    for (int e = lane; e < E; e += 32) {
-      const float x = expf(z[e] - top);
-      s[e] = x;
-      sum += x;
+#pragma unroll
+    for (int i = 0; i < kPer; ++i) {
+      s[i] = lane + 32 * i < E ? expf(s[i] - top) : 0.f;
+      sum += s[i];
     }
-    sum = warp_add(sum);
-    const float inv = 1.0f / sum;
-    for (int e = lane; e < E; e += 32) s[e] *= inv;
-    __syncwarp();
-    const bool all_open = p.keep >= p.groups;
+    const float inv = 1.0f / warp_add(sum);
+    uint32_t key[kPer];                                   // 0: not open
+#pragma unroll
+    for (int i = 0; i < kPer; ++i) {
+      s[i] *= inv;
+      key[i] = lane + 32 * i < E ? max(score_key(s[i] + corr[i]), 1u) : 0u;
+    }
     if (!all_open) {
+#pragma unroll
+      for (int i = 0; i < kPer; ++i)
+        if (lane + 32 * i < E) cs[lane + 32 * i] = s[i] + corr[i];
+      __syncwarp();
       for (int g = lane; g < p.groups; g += 32) {
         float m = -INFINITY;
-        for (int e = g * size; e < (g + 1) * size; ++e) m = fmaxf(m, s[e] + p.correction[e]);
+        for (int e = g * size; e < (g + 1) * size; ++e) m = fmaxf(m, cs[e]);
         gs[g] = m;
       }
       __syncwarp();
-      // the kept groups are marked with +inf
-      for (int k = 0; k < p.keep; ++k) {
-        float m = -INFINITY;
-        int at = 0x7fffffff;
-        for (int g = lane; g < p.groups; g += 32)
-          if (gs[g] != INFINITY && (gs[g] > m || at == 0x7fffffff)) { m = gs[g]; at = g; }
-        warp_argmax(&m, &at);
-        __syncwarp();
-        if (lane == 0 && at < p.groups) gs[at] = INFINITY;
-        __syncwarp();
+      int last = -1;                                      // a group is kept if fewer than `keep` groups come before it
+      bool open = false;
+#pragma unroll
+      for (int i = 0; i < kPer; ++i) {
+        if (lane + 32 * i >= E) continue;
+        if (group[i] != last) {
+          last = group[i];
+          const float mine = gs[last];
+          int before = 0;
+          for (int g = 0; g < p.groups; ++g) before += gs[g] > mine || (gs[g] == mine && g < last);
+          open = before < p.keep;
+        }
+        if (!open) key[i] = 0u;
       }
+      __syncwarp();
     }
     float picked = 0.f;                                   // lane c (and c + 32): choice c
     int mine[2] = {-1, -1};
     float mine_w[2] = {0.f, 0.f};
     for (int c = 0; c < p.top; ++c) {
-      float m = -INFINITY;
-      int at = 0x7fffffff;
-      for (int e = lane; e < E; e += 32)
-        if (s[e] >= 0.f && (all_open || gs[e / size] == INFINITY)) {     // a chosen expert's score is stored negated below
-          const float v = s[e] + p.correction[e];
-          if (v > m || at == 0x7fffffff) { m = v; at = e; }
-        }
-      warp_argmax(&m, &at);
-      if (at >= E) at = 0;                                // fewer open experts than choices: the host refuses such sizes
-      const float w = fabsf(s[at]);
-      __syncwarp();
-      if (lane == 0) s[at] = -w - 1e-30f;
-      __syncwarp();
+      uint32_t best = 0u;
+      int at = 0;
+      float w = 0.f;
+#pragma unroll
+      for (int i = 0; i < kPer; ++i)
+        if (key[i] > best) { best = key[i]; at = lane + 32 * i; w = s[i]; }
+      const uint32_t top_key = __reduce_max_sync(0xffffffffu, best);
+      const int winner = (int)__reduce_min_sync(0xffffffffu, best == top_key && best != 0u ? (uint32_t)at : 0x7fffffffu);
+      // (fewer open experts than choices: the host refuses such sizes)
+      const int e = min(winner, E - 1);
+      w = __shfl_sync(0xffffffffu, w, e & 31);
+#pragma unroll
+      for (int i = 0; i < kPer; ++i)
+        if (lane + 32 * i == e) key[i] = 0u;
       picked += w;
-      if (lane == (c & 31)) { mine[c >> 5] = at; mine_w[c >> 5] = w; }
+      if (lane == (c & 31)) { mine[c >> 5] = e; mine_w[c >> 5] = w; }
     }
     const float norm = p.scale / (picked + 1e-20f);
 #pragma unroll
@@ -257,14 +273,11 @@ extern "C" int tkv_moe_route(const float* logits, int64_t logit_stride, const fl
   if (ctas > 1 && !counts) return fail(TKV_ERR_ARG, "tkv_moe_route: counts is needed for more than %d tokens", kRouteTokens);
   if (tokens == 0) return TKV_OK;
   const size_t smem = ((size_t)kRouteWarps * (experts + groups) + 2 * experts + 1) * sizeof(float);
-  static size_t allowed = 48 * 1024;
-  cudaError_t e = cudaSuccess;
-  if (smem > allowed) {
-    if (smem > 220 * 1024) return fail(TKV_ERR_UNSUPPORTED, "tkv_moe_route: experts=%d groups=%d", experts, groups);
-    e = cudaFuncSetAttribute(moe_route_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    allowed = smem;
-  }
-  if (e == cudaSuccess) e = launch_pdl(moe_route_kernel, dim3(ctas), dim3(kRouteThreads), smem, st, p);
+  if (smem > 220 * 1024) return fail(TKV_ERR_UNSUPPORTED, "tkv_moe_route: experts=%d groups=%d", experts, groups);
+  auto kern = experts <= 32 ? moe_route_kernel<1> : experts <= 64 ? moe_route_kernel<2> : experts <= 128 ? moe_route_kernel<4>
+              : experts <= 256 ? moe_route_kernel<8> : moe_route_kernel<32>;
+  cudaError_t e = smem > 48 * 1024 ? cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) : cudaSuccess;
+  if (e == cudaSuccess) e = launch_pdl(kern, dim3(ctas), dim3(kRouteThreads), smem, st, p);
   if (e == cudaSuccess && ctas > 1) {
     const int64_t blocks = ((int64_t)tokens * top + kPlaceThreads * 4 - 1) / (kPlaceThreads * 4);
     e = launch_pdl(moe_place_kernel, dim3((unsigned)blocks), dim3(kPlaceThreads), (size_t)(experts + 1) * sizeof(int32_t), st, p);

@@ -1,10 +1,11 @@
 // Grouped product of a mixture of experts on tcgen05 + TMEM, for prompts and for decoding:
 //   out[r, :] = act(a[src[r], :] . w[e]^T)   for the rows r of expert e.
 //
-// One persistent CTA per SM walks tiles of 128 rows x BN columns, expert by expert.  Per 64 columns of k: the rows of A are
-// gathered by TMA (tile::gather4, four rows per copy, one copy per lane of the producer warp; rows a tile does not have are not
-// fetched, so few rows per expert cost little more than the weights), the weight rows are one box.  A ring of stages feeds the
-// MMAs; two TMEM accumulators let the epilogue of a tile (activation, rounding, stores) overlap the next tile.
+// One persistent CTA per SM walks tiles of 128 rows x BN columns, expert by expert.  Per 64 columns of k the weight rows are one
+// TMA box; the rows of A are TMA boxes of 32 where they are consecutive, and are gathered by four warps with cp.async where they
+// are not (TMA's own gather moves four rows per instruction and was the limit).  Rows a tile does not have are not fetched, so
+// few rows per expert cost little more than the weights.  A ring of stages feeds the MMAs; two TMEM accumulators let the
+// epilogue of a tile (activation, rounding, stores) overlap the next tile.
 // A weight tile that reaches beyond an expert's n rows holds rows of the next expert: those columns are not stored.
 // Every wait is bounded; on expiry the CTA records TKV_DEV_TIMEOUT, drains its copies and frees its TMEM.
 #include <cuda.h>
@@ -13,8 +14,9 @@
 
 namespace tkv {
 
-constexpr int kMgThreads = 192;                           // warp 0: copies, warp 1: products, warps 2-5: epilogue
-constexpr int kMgM = 128, kMgK = 64;
+constexpr int kMgGather = 128, kMgLag = 2;                // gathering threads; stages they run ahead of what they hand over
+constexpr int kMgThreads = 192;                           // warp 0: copies, warp 1: products, warps 2-5: epilogue (6-9: gathering)
+constexpr int kMgM = 128, kMgK = 64, kMgBoxRows = 32;
 constexpr int kMgABytes = kMgM * kMgK * 2;
 template <int BN> struct MgRing {
   static constexpr int kStages = BN == 256 ? 4 : BN == 128 ? 6 : 8, kStageBytes = kMgABytes + BN * kMgK * 2;
@@ -22,18 +24,12 @@ template <int BN> struct MgRing {
 
 struct MgSmem {
   uint64_t full[8], empty[8], acc_full[2], acc_empty[2];
+  uint64_t full_a[8];                                     // gathered rows of a stage are there
   uint32_t tmem_base;
   int abort_flag;
 };
 template <int BN> constexpr int mg_smem_bytes(int experts) {
   return MgRing<BN>::kStages * MgRing<BN>::kStageBytes + (int)sizeof(MgSmem) + (2 * experts + 1) * 4;
-}
-
-// Four rows of a matrix (box: 64 columns, one row) into four consecutive 128-byte rows of shared memory.
-__device__ __forceinline__ void tma_gather4(void* smem_dst, const CUtensorMap* map, uint64_t* bar, int x, int r0, int r1, int r2, int r3) {
-  asm volatile(
-      "cp.async.bulk.tensor.2d.shared::cta.global.tile::gather4.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5, %6, %7}], [%2];"
-      ::"r"(smem_u32(smem_dst)), "l"(map), "r"(smem_u32(bar)), "r"(x), "r"(r0), "r"(r1), "r"(r2), "r"(r3) : "memory");
 }
 
 // Walks this CTA's tiles in order; every role keeps its own.
@@ -54,8 +50,8 @@ struct MgTiles {
   }
 };
 
-template <int BN>
-__global__ void __launch_bounds__(kMgThreads, 1)
+template <int BN, bool kGather>
+__global__ void __launch_bounds__(kMgThreads + (kGather ? kMgGather : 0), 1)
 moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w, GroupedGemm p) {
   extern __shared__ __align__(1024) uint8_t base[];
   constexpr int S = MgRing<BN>::kStages, kStage = MgRing<BN>::kStageBytes;
@@ -66,7 +62,7 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   volatile int* abort_flag = &sm->abort_flag;
   if (tid == 0) {
-    for (int s = 0; s < S; ++s) { mbar_init(&sm->full[s], 1); mbar_init(&sm->empty[s], 1); }
+    for (int s = 0; s < S; ++s) { mbar_init(&sm->full[s], 1); mbar_init(&sm->empty[s], 1); mbar_init(&sm->full_a[s], kMgGather); }
     for (int s = 0; s < 2; ++s) { mbar_init(&sm->acc_full[s], 1); mbar_init(&sm->acc_empty[s], 4); }
     sm->abort_flag = (smem_u32(base) & 1023u) != 0;       // the swizzled tiles need the alignment; the launch gives it
     if (sm->abort_flag) report(p.status, TKV_DEV_TIMEOUT);
@@ -78,7 +74,7 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__
   }
   grid_dependency_wait();
   grid_launch_dependents();
-  for (int e = tid; e <= p.experts; e += kMgThreads) off[e] = p.offsets[e];
+  for (int e = tid; e <= p.experts; e += blockDim.x) off[e] = p.offsets[e];
   __syncthreads();
   if (warp == 0) {                                        // running number of row tiles
     int sum = 0;
@@ -99,40 +95,70 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__
   tc_fence_after();
   const uint32_t tmem = sm->tmem_base;
   const int ksteps = (p.k + kMgK - 1) / kMgK, ncols = (p.n + BN - 1) / BN;
+  int mg_copies = 0;                                      // stages whose TMA copies thread 0 has started
   MgTiles t = {off, tile_end, p.experts, ncols, 0, (int)blockIdx.x - (int)gridDim.x, (int)gridDim.x, 0, 0, 0};
 
   if (warp == 0) {
-    // ---- producer: lane l fetches rows 4 l .. 4 l + 3 of a tile
+    // ---- weights, and consecutive rows
+    if (lane == 0) {
+      int it = 0;
+      bool ok = *abort_flag == 0;
+      while (ok && t.next()) {
+        const int boxes = kGather ? 0 : (t.rows + kMgBoxRows - 1) / kMgBoxRows;
+        const uint32_t bytes = (uint32_t)boxes * kMgBoxRows * 128 + BN * kMgK * 2;
+        const int wrow = t.e * p.n + t.col * BN;
+        for (int k = 0; k < ksteps; ++k, ++it) {
+          const int s = it % S;
+          ok = mbar_wait_or_abort(&sm->empty[s], ((it / S) & 1) ^ 1, abort_flag);
+          if (!ok) break;
+          uint8_t* st = base + s * kStage;
+          mbar_expect_tx(&sm->full[s], bytes);
+          tma_load_2d(st + kMgABytes, &map_w, &sm->full[s], k * kMgK, wrow);
+          for (int i = 0; i < boxes; ++i)
+            tma_load_2d(st + i * kMgBoxRows * 128, &map_a, &sm->full[s], k * kMgK, t.row0 + i * kMgBoxRows);
+        }
+      }
+      if (!ok && *abort_flag == 0) { *abort_flag = 1; report(p.status, TKV_DEV_TIMEOUT); }
+      mg_copies = it;
+    }
+    __syncwarp();
+  } else if (kGather && warp >= kMgThreads / 32) {
+    // ---- gathered rows: thread g fetches the 16-byte piece g % 8 of rows g / 8 + 16 i
+    const int g = tid - kMgThreads, piece = g & 7, r0 = g >> 3;
+    const uint32_t swz = (uint32_t)((piece ^ (r0 & 7)) << 4);        // rows 16 apart share it
+    auto hand_over = [&](int i) {
+      fence_async_smem();
+      asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(&sm->full_a[i % S])) : "memory");
+    };
     int it = 0;
     bool ok = *abort_flag == 0;
     while (ok && t.next()) {
-      int r[4];
+      const __nv_bfloat16* row[8];
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const int row = t.row0 + min(4 * lane + i, t.rows - 1);
-        r[i] = p.src != nullptr ? p.src[row] : row;
+      for (int i = 0; i < 8; ++i) {
+        const int r = r0 + 16 * i;
+        row[i] = r < t.rows ? (const __nv_bfloat16*)p.a + (int64_t)p.src[t.row0 + r] * p.a_stride + piece * 8 : nullptr;
       }
-      const bool mine = 4 * lane < t.rows;
-      const uint32_t bytes = (uint32_t)((t.rows + 3) / 4) * 512 + BN * kMgK * 2;
-      const int wrow = t.e * p.n + t.col * BN;
       for (int k = 0; k < ksteps; ++k, ++it) {
         const int s = it % S;
         ok = mbar_wait_or_abort(&sm->empty[s], ((it / S) & 1) ^ 1, abort_flag);
-        ok = __all_sync(0xffffffffu, ok);
         if (!ok) break;
-        uint8_t* st = base + s * kStage;
-        if (lane == 0) {
-          mbar_expect_tx(&sm->full[s], bytes);
-          tma_load_2d(st + kMgABytes, &map_w, &sm->full[s], k * kMgK, wrow);
+        const uint32_t dst = smem_u32(base + s * kStage) + (uint32_t)r0 * 128 + swz;
+        const int bytes = k * kMgK + piece * 8 < p.k ? 16 : 0;       // the rest of the last piece of k reads as zeros
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+          if (row[i] != nullptr)
+            asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst + i * 16 * 128), "l"(bytes ? row[i] + k * kMgK : row[i] - piece * 8), "r"(bytes) : "memory");
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        if (it >= kMgLag) {
+          asm volatile("cp.async.wait_group %0;" ::"n"(kMgLag) : "memory");
+          hand_over(it - kMgLag);
         }
-        __syncwarp();
-        if (mine) tma_gather4(st + lane * 512, &map_a, &sm->full[s], k * kMgK, r[0], r[1], r[2], r[3]);
       }
     }
-    if (!ok && lane == 0 && *abort_flag == 0) { *abort_flag = 1; report(p.status, TKV_DEV_TIMEOUT); }
-    __syncwarp();
-    if (lane == 0 && *abort_flag != 0)                    // copies in flight land before the shared memory is released
-      for (int i = max(0, it - S); i < it; ++i) mbar_wait(&sm->full[i % S], (i / S) & 1);
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    for (int i = max(0, it - kMgLag); i < it; ++i) hand_over(i);
+    if (!ok && *abort_flag == 0) { *abort_flag = 1; report(p.status, TKV_DEV_TIMEOUT); }
   } else if (warp == 1) {
     // ---- products
     if (lane == 0) {
@@ -146,6 +172,7 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__
         for (int k = 0; k < ksteps && ok; ++k, ++it) {
           const int s = it % S;
           ok = mbar_wait_or_abort(&sm->full[s], (it / S) & 1, abort_flag);
+          if (ok && kGather) ok = mbar_wait_or_abort(&sm->full_a[s], (it / S) & 1, abort_flag);
           if (!ok) break;
           tc_fence_after();
           const uint32_t a = smem_u32(base + s * kStage), w = a + kMgABytes;
@@ -198,6 +225,8 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__
   __syncwarp();
   tc_fence_before();
   __syncthreads();
+  if (tid == 0 && *abort_flag != 0)                       // copies in flight land before the shared memory is released
+    for (int i = max(0, mg_copies - S); i < mg_copies; ++i) mbar_wait(&sm->full[i % S], (i / S) & 1);
   if (warp == 1) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(kTmemCols));
 }
 
@@ -206,23 +235,28 @@ bool moe_tc_shape(const GroupedGemm& p, int dtype) {
          p.experts <= 1024 && (int64_t)p.experts * p.n + 256 <= INT32_MAX && p.a_rows > 0;
 }
 
-template <int BN>
+template <int BN, bool kGather>
 static int launch_mg(const GroupedGemm& p, int64_t tiles, cudaStream_t st) {
   CUtensorMap ma, mw;
-  int rc = make_map_rows(&ma, p.a, p.k, p.a_rows, p.a_stride, kMgK, 1);
+  int rc = make_map_rows(&ma, p.a, p.k, p.a_rows, p.a_stride, kMgK, kMgBoxRows);
   if (rc == TKV_OK) rc = make_map_2d(&mw, p.w, p.k, (int64_t)p.experts * p.n, kMgK, BN, TKV_BF16);
   if (rc != TKV_OK) return rc;
   const int bytes = mg_smem_bytes<BN>(p.experts);
   static int allowed = 0;
   if (bytes > allowed) {
     if (bytes > 232448) return fail(TKV_ERR_UNSUPPORTED, "tkv_moe_gemm: experts=%d", p.experts);
-    cudaError_t e = cudaFuncSetAttribute(moe_tc_kernel<BN>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+    cudaError_t e = cudaFuncSetAttribute(moe_tc_kernel<BN, kGather>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
     if (e != cudaSuccess) return fail(TKV_ERR_LAUNCH, "tkv_moe_gemm: %s", cudaGetErrorString(e));
     allowed = bytes;
   }
-  cudaError_t e = launch_pdl(moe_tc_kernel<BN>, dim3((unsigned)(tiles < 148 ? tiles : 148)), dim3(kMgThreads), (size_t)bytes, st, ma, mw, p);
+  cudaError_t e = launch_pdl(moe_tc_kernel<BN, kGather>, dim3((unsigned)(tiles < 148 ? tiles : 148)), dim3(kMgThreads + (kGather ? kMgGather : 0)),
+                             (size_t)bytes, st, ma, mw, p);
   if (e != cudaSuccess) return fail(TKV_ERR_LAUNCH, "tkv_moe_gemm: %s", cudaGetErrorString(e));
   return check_launch("tkv_moe_gemm");
+}
+template <int BN>
+static int launch_mg(const GroupedGemm& p, int64_t tiles, cudaStream_t st) {
+  return p.src != nullptr ? launch_mg<BN, true>(p, tiles, st) : launch_mg<BN, false>(p, tiles, st);
 }
 
 int launch_moe_tc(const GroupedGemm& p, cudaStream_t st) {

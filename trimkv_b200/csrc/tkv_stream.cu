@@ -126,7 +126,7 @@ struct GatedSumNorm {
 template <typename T, int V, int kKeep, bool kRouted>
 __global__ void __launch_bounds__(kRowThreads) gated_sum_norm_kernel(GatedSumNorm p) {
   extern __shared__ float dyn[];                          // red [groups][warps], then (kKeep = 0) the row
-  constexpr int kN = kKeep > 0 ? kKeep : 1;
+  constexpr int kN = kKeep > 0 ? kKeep : 1, kAhead = V == 8 ? 4 : 2;
   const int64_t row = blockIdx.x, off = row * p.width;
   const int nvec = p.width / V, glen = p.width / p.groups;
   float* held = dyn + p.groups * (kRowThreads / 32);
@@ -139,13 +139,21 @@ __global__ void __launch_bounds__(kRowThreads) gated_sum_norm_kernel(GatedSumNor
     if (kRouted) {
 #pragma unroll
       for (int e = 0; e < V; ++e) yv[e] = 0.f;
-      for (int c = 0; c < p.top; ++c) {
-        const int32_t at = p.place[row * p.top + c];
-        const float cw = p.choice_w[row * p.top + c];
-        float r[V];
-        if (at >= 0) load_vec<V>((const T*)p.y + (int64_t)at * p.width + (int64_t)i * V, r);
+      for (int c0 = 0; c0 < p.top; c0 += kAhead) {         // kAhead rows requested before the first is used
+        float r[kAhead][V], cw[kAhead];
+        int32_t at[kAhead];
 #pragma unroll
-        for (int e = 0; e < V; ++e) yv[e] = fmaf(cw, at >= 0 ? r[e] : xv[e], yv[e]);
+        for (int c = 0; c < kAhead; ++c) {
+          at[c] = c0 + c < p.top ? p.place[row * p.top + c0 + c] : -1;
+          cw[c] = c0 + c < p.top ? p.choice_w[row * p.top + c0 + c] : 0.f;
+        }
+#pragma unroll
+        for (int c = 0; c < kAhead; ++c)
+          if (at[c] >= 0) load_vec<V>((const T*)p.y + (int64_t)at[c] * p.width + (int64_t)i * V, r[c]);
+#pragma unroll
+        for (int c = 0; c < kAhead; ++c)
+#pragma unroll
+          for (int e = 0; e < V; ++e) yv[e] = fmaf(cw[c], at[c] >= 0 ? r[c][e] : xv[e], yv[e]);
       }
     } else {
       load_vec<V>((const T*)p.y + off + (int64_t)i * V, yv);
@@ -173,7 +181,20 @@ __global__ void __launch_bounds__(kRowThreads) gated_sum_norm_kernel(GatedSumNor
       for (int e = 0; e < V; ++e) held[i * V + e] = sv[0][e];
     }
   }
-  group_sums(p.groups, dyn, [&](int g) {                   // a vector lies in one group (the host chooses V so)
+  // Where a group is made of whole rounds of a warp, a round's sum belongs to one group: entry j * warps + warp, in order.
+  const bool whole = kKeep > 0 && glen % (32 * V) == 0;
+  if (whole) {
+#pragma unroll
+    for (int j = 0; j < kN; ++j) {
+      float ss = 0.f;
+      if (threadIdx.x + j * kRowThreads < nvec)
+#pragma unroll
+        for (int e = 0; e < V; ++e) ss += sv[j][e] * sv[j][e];
+      ss = warp_add(ss);
+      if ((threadIdx.x & 31) == 0) dyn[j * (kRowThreads / 32) + (threadIdx.x >> 5)] = ss;
+    }
+    __syncthreads();
+  } else group_sums(p.groups, dyn, [&](int g) {            // a vector lies in one group (the host chooses V so)
     float ss = 0.f;
     if (kKeep > 0) {
 #pragma unroll
@@ -192,7 +213,11 @@ __global__ void __launch_bounds__(kRowThreads) gated_sum_norm_kernel(GatedSumNor
     return ss;
   });
   auto finish = [&](int i, const float* s) {
-    const float rstd = 1.0f / sqrtf(group_total(dyn, i * V / glen) / (float)glen + p.eps);
+    const int g = p.groups == 1 ? 0 : i * V / glen;
+    float total = 0.f;
+    if (whole) for (int m = g * (glen / (32 * V)); m < (g + 1) * (glen / (32 * V)); ++m) total += dyn[m];
+    else total = group_total(dyn, g);
+    const float rstd = 1.0f / sqrtf(total / (float)glen + p.eps);
     float o[V];
     load_vec<V>(p.w + (int64_t)i * V, o);
 #pragma unroll
@@ -413,7 +438,7 @@ extern "C" int tkv_gated_sum_norm(float* x, const void* y, const int32_t* place,
                    (!gate || (aligned16(gate) && aligned16(gate_bias) && (gate_stride * elem_size(dtype)) % 16 == 0));
   const int per_thread = (width / (vec ? 8 : 1) + kRowThreads - 1) / kRowThreads;
   const int keep = !vec ? (per_thread <= 8 ? 8 : 0) : per_thread <= 1 ? 1 : per_thread <= 2 ? 2 : per_thread <= 4 ? 4 : 0;
-  const size_t smem = ((size_t)groups * (kRowThreads / 32) + (keep ? 0 : width)) * sizeof(float);
+  const size_t smem = ((size_t)(groups > keep ? groups : keep) * (kRowThreads / 32) + (keep ? 0 : width)) * sizeof(float);
   if (smem > 48 * 1024) return fail(TKV_ERR_UNSUPPORTED, "tkv_gated_sum_norm: width=%d groups=%d", width, groups);
   GatedSumNorm p = {x, y, gate, gate_stride, gate_bias, weight, copy_out, place, choice_w, top, width, groups, eps, alpha};
   TKV_WITH_TYPE(dtype, T, {
