@@ -1,26 +1,27 @@
 // Chunked form of the channel-decay recurrence (tkv_chanrec.cuh) for prompts, 16-bit operands with fp32 state.
 //
-// A block of 16 tokens, with P_i the product of the forget gates of its tokens up to i (per state row), S the state before it:
+// A block of tokens, with P_i the product of the forget gates of its tokens up to i (per state row), S the state before it:
 //   a_ij = (q_i P_i) . (k_j / P_j)           j <= i, k = 1 - f
 //   o_i  = S^T (q_i P_i) + sum_j a_ij v_j
-//   S   <- diag(P_16) (S + sum_j (k_j / P_j) v_j^T) .
-// The scaled vectors q P and k / P are fp32 and enter the 16-bit products as a high and a low part, as do the state and a; v is
-// 16-bit exactly.  Where the product of a row falls below kFloor within a block (gates near zero), 1 / P could leave the range of
-// fp32: such a chunk is walked token by token instead, in the same registers.
+//   S   <- diag(P_end) (S + sum_j (k_j / P_j) v_j^T) .
+// k / P is fp32 and enters the 16-bit products as a high and a low part, as do the state and a; v is 16-bit exactly, and q P is
+// rounded once, which is what rounding q itself to 16 bits does.  1 / P must stay in the range of fp32: a chunk of 32 tokens is one block where every channel's gates keep
+// kWide over eight tokens, two blocks of 16 where they keep kNarrow, and is walked token by token below that (gates near zero).
 //
-// One CTA walks chunks of 32 tokens (two blocks) of one (request, head, block of 16 * kWarps value columns, segment of the
-// sequence).  The state never leaves registers: a warp owns 16 columns of v and holds S^T [16 x n] as fp32 MMA accumulators, whose
-// layout is also the A-operand layout of the read-out.  Per chunk: gates and scaled vectors of all channels (a thread walks two
-// channels of half a block), the two 16 x 16 blocks a, then every warp its own columns without further barriers.
+// One CTA walks the chunks of one (request, head, block of 16 * kWarps value columns, segment of the sequence).  The state never
+// leaves registers: a warp owns 16 columns of v and holds S^T [16 x n] as fp32 MMA accumulators, whose layout is also the
+// A-operand layout of the read-out.  Per chunk: gates and scaled vectors of all channels (a thread walks two channels of eight
+// tokens), the 16 x 16 blocks of a, then every warp its own columns without further barriers.
 // Where (request, head, column) blocks alone do not fill the GPU, the sequence is cut into segments: a first pass computes
 // every segment's own state, a small kernel chains them, and the main pass starts each segment from its true state.
+#include <type_traits>
 #include "tkv_chanrec.cuh"
 #include "tkv_tc.cuh"
 
 namespace tkv {
 
-constexpr int kCrTokens = 32, kCrBlock = 16;
-constexpr float kFloor = 1e-24f;
+constexpr int kCrTokens = 32;
+constexpr float kWide = 3e-8f, kNarrow = 1e-15f;          // product of eight gates
 
 __device__ __forceinline__ void cr_mma(float* d, const uint32_t* a, uint32_t b0, uint32_t b1) {
   asm volatile(
@@ -40,11 +41,33 @@ __device__ __forceinline__ void cr_cp16(void* dst, const void* src, bool live) {
   const int bytes = live ? 16 : 0;                        // 0: the 16 bytes are zero-filled
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(bytes) : "memory");
 }
+// Two fp32 operations in one instruction.
+__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
+  float2 r;
+  asm("{\n\t.reg .b64 a, b, r;\n\tmov.b64 a, {%2, %3};\n\tmov.b64 b, {%4, %5};\n\tmul.rn.f32x2 r, a, b;\n\tmov.b64 {%0, %1}, r;\n\t}"
+      : "=f"(r.x), "=f"(r.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y));
+  return r;
+}
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+  float2 r;
+  asm("{\n\t.reg .b64 a, b, c, r;\n\tmov.b64 a, {%2, %3};\n\tmov.b64 b, {%4, %5};\n\tmov.b64 c, {%6, %7};\n\tfma.rn.f32x2 r, a, b, c;\n\t"
+      "mov.b64 {%0, %1}, r;\n\t}"
+      : "=f"(r.x), "=f"(r.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y), "f"(c.x), "f"(c.y));
+  return r;
+}
+__device__ __forceinline__ float2 add2(float2 a, float2 b) {
+  float2 r;
+  asm("{\n\t.reg .b64 a, b, r;\n\tmov.b64 a, {%2, %3};\n\tmov.b64 b, {%4, %5};\n\tadd.rn.f32x2 r, a, b;\n\tmov.b64 {%0, %1}, r;\n\t}"
+      : "=f"(r.x), "=f"(r.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y));
+  return r;
+}
+__device__ __forceinline__ float2 pair(float x) { return make_float2(x, x); }
 // x = hi + lo in bf16, two values at a time.
-__device__ __forceinline__ void cr_split(float a, float b, uint32_t* hi, uint32_t* lo) {
-  const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+__device__ __forceinline__ void cr_split(float2 x, uint32_t* hi, uint32_t* lo) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(x.x, x.y);
   *hi = *reinterpret_cast<const uint32_t*>(&h);
-  const __nv_bfloat162 l = __floats2bfloat162_rn(a - __uint_as_float(*hi << 16), b - __uint_as_float(*hi & 0xffff0000u));
+  const float2 r = add2(x, make_float2(-__uint_as_float(*hi << 16), -__uint_as_float(*hi & 0xffff0000u)));
+  const __nv_bfloat162 l = __floats2bfloat162_rn(r.x, r.y);
   *lo = *reinterpret_cast<const uint32_t*>(&l);
 }
 // sigmoid(x) and sigmoid(-x), each to a few units in the last place of fp32.
@@ -60,25 +83,32 @@ __device__ __forceinline__ float cr_rcp(float x) {
   asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-// f, 1 / f and k = 1 - f with one reciprocal: with e = exp(-|x|), sigmoid(|x|) = 1 / (1 + e), f = num / (1 + e).  Where f leaves
-// the range of fp32 the result is not a number, or zero; the caller looks at the product.
-__device__ __forceinline__ void cr_gate(float x, float lo, float* f, float* inv, float* k) {
-  const float e = exp2_weight(fabsf(x) * -1.4426950408889634f), den = 1.0f + e, rest = 1.0f - lo;
-  const float num = fmaf(rest, x >= 0.f ? 1.0f : e, lo * den);
-  const float t = cr_rcp(den * num), u = num * t;         // u = 1 / den
-  *f = num * u;
-  *inv = den * den * t;
-  *k = rest * (x >= 0.f ? e : 1.0f) * u;
+// f, 1 / f and k = 1 - f of two channels with one reciprocal each: with e = exp(-|x|), sigmoid(|x|) = 1 / (1 + e),
+// f = num / (1 + e).  Where f leaves the range of fp32 the result is not a number, or zero; the caller looks at the product.
+__device__ __forceinline__ void cr_gate(float2 x, float2 lo, float2 rest, float2* f, float2* inv, float2* k) {
+  const float2 e = make_float2(exp2_weight(fabsf(x.x) * -1.4426950408889634f), exp2_weight(fabsf(x.y) * -1.4426950408889634f));
+  const float2 den = add2(e, pair(1.0f));
+  const float2 pos = make_float2(x.x >= 0.f ? 1.0f : e.x, x.y >= 0.f ? 1.0f : e.y), neg = make_float2(x.x >= 0.f ? e.x : 1.0f, x.y >= 0.f ? e.y : 1.0f);
+  const float2 num = fma2(rest, pos, mul2(lo, den)), dn = mul2(den, num);
+  const float2 t = make_float2(cr_rcp(dn.x), cr_rcp(dn.y)), u = mul2(num, t);      // u = 1 / den
+  *f = mul2(num, u);
+  *inv = mul2(mul2(den, den), t);
+  *k = mul2(mul2(rest, neg), u);
 }
 __device__ __forceinline__ float cr_silu(float z) { return z * cr_rcp(1.0f + exp2_weight(z * -1.4426950408889634f)); }
+__device__ __forceinline__ float2 cr_silu2(float2 z) {
+  const float2 d = add2(make_float2(exp2_weight(z.x * -1.4426950408889634f), exp2_weight(z.y * -1.4426950408889634f)), pair(1.0f));
+  return mul2(z, make_float2(cr_rcp(d.x), cr_rcp(d.y)));
+}
 
 template <int NP, int kWarps> struct CrSmem {
-  static constexpr int PT = kWarps * 16, QS = NP + 8, VS = PT + 8, PS = kCrBlock + 8;
+  static constexpr int PT = kWarps * 16, QS = NP + 8, VS = PT + 8, PS = kCrTokens + 8;
   __nv_bfloat16 zq[2][kCrTokens * QS], zf[2][kCrTokens * QS], v[2][kCrTokens * VS];
-  __nv_bfloat16 q_hi[kCrTokens * QS], q_lo[kCrTokens * QS], k_hi[kCrTokens * QS], k_lo[kCrTokens * QS];
-  __nv_bfloat16 a_hi[2][kCrBlock * PS], a_lo[2][kCrBlock * PS];
-  float mid[2][2][NP];                                    // P and 1 / P in the middle of a block
-  float end[2][NP];                                       // product of the gates of a block
+  __nv_bfloat16 q[kCrTokens * QS], k_hi[kCrTokens * QS], k_lo[kCrTokens * QS];
+  __nv_bfloat16 a_hi[kCrTokens * PS], a_lo[kCrTokens * PS];
+  float oct[2][4][NP];                                    // product of eight tokens' gates, and of their reciprocals
+  float end[2][NP];                                       // product of the gates of a block (one block: the first)
+  int level[2];                                           // by chunk parity: 0 one block, 1 two blocks, 2 token by token
   float gate[2][3][NP];                                   // q, f, k of one token (token-by-token path)
 };
 
@@ -143,164 +173,187 @@ __global__ void __launch_bounds__(kWarps * 32, NP == 256 ? 1 : kWarps == 8 ? 2 :
 #pragma unroll
   for (int i = 0; i < kOwn; ++i) seg_decay[i] = 1.0f;
 
+  if (tid < 2) sm.level[tid] = 0;
   fetch(c0);
   for (int chunk = c0; chunk < c1; ++chunk) {
     const int st = chunk & 1, t0 = chunk * kCrTokens;
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();                                       // this chunk is here; everyone is done with the last one
     if (chunk + 1 < c1) fetch(chunk + 1);
-    // ---- gates and scaled vectors: a thread walks two channels of half a block, four warps take 64 channels
-    bool tiny = false;
+    // ---- gates and scaled vectors: a thread walks two channels of eight tokens, four warps take 64 channels
+    constexpr int kRounds = (NP + kWarps * 16 - 1) / (kWarps * 16);
+    float2 P[kRounds][8], kp[kRounds][8];                  // product up to a token, k over it
+    const int oct = warp & 3, r0 = oct * 8;
 #pragma unroll
-    for (int c64 = 0; c64 < NP; c64 += kWarps * 16) {
-      const int blk = (warp >> 1) & 1, half = warp & 1, c = c64 + (warp >> 2) * 64 + 2 * lane, r0 = blk * kCrBlock + half * 8;
-      const bool on = c < NP;
-      float P[8][2], kp[8][2], inv[2] = {1.0f, 1.0f};      // product up to a token, k over it
-      if (on) {
-        // a channel that does not exist keeps its (zero) state: lower bound 1
-        const float2 bi = c < a.n ? *reinterpret_cast<const float2*>(bias + c) : make_float2(0.f, 0.f);
-        const float2 lo = c < a.n ? *reinterpret_cast<const float2*>(lower + c) : make_float2(1.f, 1.f);
+    for (int rd = 0; rd < kRounds; ++rd) {
+      const int c = rd * kWarps * 16 + (warp >> 2) * 64 + 2 * lane;
+      if (c >= NP) continue;
+      // a channel that does not exist keeps its (zero) state: lower bound 1
+      const float2 bi = c < a.n ? *reinterpret_cast<const float2*>(bias + c) : pair(0.f);
+      const float2 lo = c < a.n ? *reinterpret_cast<const float2*>(lower + c) : pair(1.f);
+      const float2 rest = make_float2(1.0f - lo.x, 1.0f - lo.y);
+      float2 inv = pair(1.0f);
+      auto walk8 = [&](int live) {
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
-          float f[2] = {1.0f, 1.0f}, fi[2] = {1.0f, 1.0f}, k[2] = {0.f, 0.f};
-          if (t0 + r0 + j < ntok) {
-            const uint32_t z = *reinterpret_cast<const uint32_t*>(&sm.zf[st][(r0 + j) * QS + c]);
-            cr_gate(__uint_as_float(z << 16) + bi.x, lo.x, &f[0], &fi[0], &k[0]);
-            cr_gate(__uint_as_float(z & 0xffff0000u) + bi.y, lo.y, &f[1], &fi[1], &k[1]);
-          }
+          const uint32_t z = *reinterpret_cast<const uint32_t*>(&sm.zf[st][(r0 + j) * QS + c]);
+          float2 f, fi, k;
+          cr_gate(add2(make_float2(__uint_as_float(z << 16), __uint_as_float(z & 0xffff0000u)), bi), lo, rest, &f, &fi, &k);
+          if (j >= live) { f = pair(1.0f); fi = f; k = pair(0.0f); }
+          P[rd][j] = j > 0 ? mul2(P[rd][j - 1], f) : f;
+          inv = mul2(inv, fi);
+          kp[rd][j] = mul2(k, inv);
+        }
+      };
+      if (t0 + kCrTokens <= ntok) walk8(8);
+      else walk8(ntok - t0 - r0);
+      *reinterpret_cast<float2*>(&sm.oct[0][oct][c]) = P[rd][7];
+      *reinterpret_cast<float2*>(&sm.oct[1][oct][c]) = inv;
+      const float low = fminf(P[rd][7].x, P[rd][7].y);     // not a number counts as below
+      const bool nan = P[rd][7].x != P[rd][7].x || P[rd][7].y != P[rd][7].y;
+      if (nan || !(low >= kWide)) atomicMax(&sm.level[st], nan || !(low >= kNarrow) ? 2 : 1);
+    }
+    __syncthreads();
+    const int level = sm.level[st];
+    if (tid == 0) sm.level[st ^ 1] = 0;
+    if (level < 2) {
 #pragma unroll
-          for (int e = 0; e < 2; ++e) {
-            P[j][e] = j > 0 ? P[j - 1][e] * f[e] : f[e];
-            inv[e] *= fi[e];
-            kp[j][e] = k[e] * inv[e];
-          }
+      for (int rd = 0; rd < kRounds; ++rd) {
+        const int c = rd * kWarps * 16 + (warp >> 2) * 64 + 2 * lane;
+        if (c >= NP) continue;
+        float2 p0 = pair(1.0f), i0 = p0;                   // products of the block's tokens before this thread's
+        for (int q = level == 0 ? 0 : oct & 2; q < oct; ++q) {
+          p0 = mul2(p0, *reinterpret_cast<const float2*>(&sm.oct[0][q][c]));
+          i0 = mul2(i0, *reinterpret_cast<const float2*>(&sm.oct[1][q][c]));
         }
-        if (half == 0) {
-          *reinterpret_cast<float2*>(&sm.mid[0][blk][c]) = make_float2(P[7][0], P[7][1]);
-          *reinterpret_cast<float2*>(&sm.mid[1][blk][c]) = make_float2(inv[0], inv[1]);
-        }
-      }
-      __syncthreads();
-      if (on) {
-        float2 p0 = make_float2(1.0f, 1.0f), i0 = p0;
-        if (half == 1) {
-          p0 = *reinterpret_cast<const float2*>(&sm.mid[0][blk][c]);
-          i0 = *reinterpret_cast<const float2*>(&sm.mid[1][blk][c]);
-          const float2 end = make_float2(p0.x * P[7][0], p0.y * P[7][1]);
-          *reinterpret_cast<float2*>(&sm.end[blk][c]) = end;
-          tiny |= !(end.x >= kFloor && end.y >= kFloor);
-        }
+        if (oct == 3 || (level == 1 && oct == 1)) *reinterpret_cast<float2*>(&sm.end[level == 0 ? 0 : oct >> 1][c]) = mul2(p0, P[rd][7]);
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
           const int at = (r0 + j) * QS + c;
           uint32_t hi, lo_;
-          cr_split(kp[j][0] * i0.x, kp[j][1] * i0.y, &hi, &lo_);
+          cr_split(mul2(kp[rd][j], i0), &hi, &lo_);
           *reinterpret_cast<uint32_t*>(&sm.k_hi[at]) = hi;
           *reinterpret_cast<uint32_t*>(&sm.k_lo[at]) = lo_;
           if (!kStateOnly) {
             const uint32_t z = *reinterpret_cast<const uint32_t*>(&sm.zq[st][at]);
-            cr_split(cr_silu(__uint_as_float(z << 16)) * (P[j][0] * p0.x), cr_silu(__uint_as_float(z & 0xffff0000u)) * (P[j][1] * p0.y), &hi, &lo_);
-            *reinterpret_cast<uint32_t*>(&sm.q_hi[at]) = hi;
-            *reinterpret_cast<uint32_t*>(&sm.q_lo[at]) = lo_;
+            const float2 x = mul2(cr_silu2(make_float2(__uint_as_float(z << 16), __uint_as_float(z & 0xffff0000u))), mul2(P[rd][j], p0));
+            *reinterpret_cast<__nv_bfloat162*>(&sm.q[at]) = __floats2bfloat162_rn(x.x, x.y);
           }
         }
       }
+      __syncthreads();
     }
-    const bool walk = __syncthreads_or(tiny);
-    if (kStateOnly && !walk) {
+    if (kStateOnly && level < 2) {
 #pragma unroll
       for (int i = 0; i < kOwn; ++i) {
         const int c = tid + i * kThreads;
-        if (c < NP) seg_decay[i] *= sm.end[0][c] * sm.end[1][c];
+        if (c < NP) seg_decay[i] *= level == 0 ? sm.end[0][c] : sm.end[0][c] * sm.end[1][c];
       }
     }
     __nv_bfloat16* v_s = sm.v[st];
-    if (!walk) {
+    // ---- kTiles groups of 16 tokens from token `first` on, as one block
+    auto block = [&](auto tiles, int first, const float* end) {
+      constexpr int kTiles = decltype(tiles)::value;
+      uint32_t vf[kTiles][4];                              // V^T of this warp's columns, as A fragments
+#pragma unroll
+      for (int i = 0; i < kTiles; ++i)
+        cr_ldmt(vf[i], v_s + (first + i * 16 + ((lane >> 4) & 1) * 8 + (lane & 7)) * VS + p0 + ((lane >> 3) & 1) * 8);
       if (!kStateOnly) {
-        // ---- the blocks a: warps 0 .. 3 take (block, 8 columns)
-        if (warp < 4) {
-          const int blk = warp >> 1, jt = warp & 1;
-          float sc[3][4] = {};
-#pragma unroll 4
-          for (int kk = 0; kk < NP / 16; ++kk) {
-            uint32_t ah[4], al[4];
-            cr_ldm(ah, sm.q_hi + (blk * 16 + (lane & 15)) * QS + kk * 16 + (lane >> 4) * 8);
-            cr_ldm(al, sm.q_lo + (blk * 16 + (lane & 15)) * QS + kk * 16 + (lane >> 4) * 8);
-            const int at = (blk * 16 + jt * 8 + gr) * QS + kk * 16 + 2 * gc;
-            const uint32_t* kh = reinterpret_cast<const uint32_t*>(sm.k_hi + at);
-            const uint32_t* kl = reinterpret_cast<const uint32_t*>(sm.k_lo + at);
-            cr_mma(sc[0], ah, kh[0], kh[4]);
-            cr_mma(sc[1], ah, kl[0], kl[4]);
-            cr_mma(sc[2], al, kh[0], kh[4]);
-          }
-          const int j = jt * 8 + 2 * gc;
+        float o[2 * kTiles][4] = {};
+        const int qrow = (first + ((lane >> 4) & 1) * 8 + (lane & 7)) * QS + ((lane >> 3) & 1) * 8;
 #pragma unroll
-          for (int e = 0; e < 4; e += 2) {
-            const int i = gr + (e >> 1) * 8;
-            uint32_t hi, lo;
-            cr_split(j <= i ? sc[0][e] + sc[1][e] + sc[2][e] : 0.f, j + 1 <= i ? sc[0][e + 1] + sc[1][e + 1] + sc[2][e + 1] : 0.f, &hi, &lo);
-            *reinterpret_cast<uint32_t*>(sm.a_hi[blk] + i * PS + j) = hi;
-            *reinterpret_cast<uint32_t*>(sm.a_lo[blk] + i * PS + j) = lo;
+        for (int kk = 0; kk < NP / 16; ++kk) {
+          uint32_t hi[4], lo[4];
+          cr_split(make_float2(s[2 * kk][0], s[2 * kk][1]), &hi[0], &lo[0]);
+          cr_split(make_float2(s[2 * kk][2], s[2 * kk][3]), &hi[1], &lo[1]);
+          cr_split(make_float2(s[2 * kk + 1][0], s[2 * kk + 1][1]), &hi[2], &lo[2]);
+          cr_split(make_float2(s[2 * kk + 1][2], s[2 * kk + 1][3]), &hi[3], &lo[3]);
+#pragma unroll
+          for (int i = 0; i < kTiles; ++i) {
+            uint32_t bf[4];
+            cr_ldm(bf, sm.q + qrow + i * 16 * QS + kk * 16);
+            cr_mma(o[2 * i], hi, bf[0], bf[1]);
+            cr_mma(o[2 * i + 1], hi, bf[2], bf[3]);
+            cr_mma(o[2 * i], lo, bf[0], bf[1]);
+            cr_mma(o[2 * i + 1], lo, bf[2], bf[3]);
           }
         }
-        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < kTiles; ++i)
+#pragma unroll
+          for (int j = 0; j <= i; ++j) {
+            uint32_t bf[4];
+            const int at = (first + i * 16 + ((lane >> 4) & 1) * 8 + (lane & 7)) * PS + first + j * 16 + ((lane >> 3) & 1) * 8;
+            cr_ldm(bf, sm.a_hi + at);
+            cr_mma(o[2 * i], vf[j], bf[0], bf[1]);
+            cr_mma(o[2 * i + 1], vf[j], bf[2], bf[3]);
+            cr_ldm(bf, sm.a_lo + at);
+            cr_mma(o[2 * i], vf[j], bf[0], bf[1]);
+            cr_mma(o[2 * i + 1], vf[j], bf[2], bf[3]);
+          }
+        __syncwarp();
+        // over this warp's own columns of the V tile (nobody else reads them)
+#pragma unroll
+        for (int i = 0; i < 2 * kTiles; ++i)
+#pragma unroll
+          for (int e = 0; e < 4; ++e)
+            v_s[(first + i * 8 + 2 * gc + (e & 1)) * VS + p0 + gr + (e >> 1) * 8] = __float2bfloat16_rn(o[i][e]);
       }
+      // ---- state
 #pragma unroll
-      for (int blk = 0; blk < 2; ++blk) {
-        uint32_t vf[4];                                    // V^T of this warp's columns, as an A fragment
-        cr_ldmt(vf, v_s + (blk * 16 + ((lane >> 4) & 1) * 8 + (lane & 7)) * VS + p0 + ((lane >> 3) & 1) * 8);
-        if (!kStateOnly) {
-          float o[2][4] = {}, o2[2][4] = {};
-          const int qrow = (blk * 16 + ((lane >> 4) & 1) * 8 + (lane & 7)) * QS + ((lane >> 3) & 1) * 8;
-#pragma unroll
-          for (int kk = 0; kk < NP / 16; ++kk) {
-            uint32_t hi[4], lo[4], bh_[4], bl_[4];
-            cr_split(s[2 * kk][0], s[2 * kk][1], &hi[0], &lo[0]);
-            cr_split(s[2 * kk][2], s[2 * kk][3], &hi[1], &lo[1]);
-            cr_split(s[2 * kk + 1][0], s[2 * kk + 1][1], &hi[2], &lo[2]);
-            cr_split(s[2 * kk + 1][2], s[2 * kk + 1][3], &hi[3], &lo[3]);
-            cr_ldm(bh_, sm.q_hi + qrow + kk * 16);
-            cr_ldm(bl_, sm.q_lo + qrow + kk * 16);
-            cr_mma(o[0], hi, bh_[0], bh_[1]);
-            cr_mma(o[1], hi, bh_[2], bh_[3]);
-            cr_mma(o2[0], lo, bh_[0], bh_[1]);
-            cr_mma(o2[1], lo, bh_[2], bh_[3]);
-            cr_mma(o2[0], hi, bl_[0], bl_[1]);
-            cr_mma(o2[1], hi, bl_[2], bl_[3]);
-          }
-          uint32_t ph[4], pl[4];
-          const int arow = (((lane >> 4) & 1) * 8 + (lane & 7)) * PS + ((lane >> 3) & 1) * 8;
-          cr_ldm(ph, sm.a_hi[blk] + arow);
-          cr_ldm(pl, sm.a_lo[blk] + arow);
-          cr_mma(o[0], vf, ph[0], ph[1]);
-          cr_mma(o[1], vf, ph[2], ph[3]);
-          cr_mma(o2[0], vf, pl[0], pl[1]);
-          cr_mma(o2[1], vf, pl[2], pl[3]);
-          __syncwarp();
-          // over this warp's own columns of the V tile (nobody else reads them)
-#pragma unroll
-          for (int i = 0; i < 2; ++i)
-#pragma unroll
-            for (int e = 0; e < 4; ++e)
-              v_s[(blk * 16 + i * 8 + 2 * gc + (e & 1)) * VS + p0 + gr + (e >> 1) * 8] = __float2bfloat16_rn(o[i][e] + o2[i][e]);
-        }
-        // ---- state
-        const int krow = (blk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * QS + ((lane >> 4) & 1) * 8;
+      for (int i = 0; i < kTiles; ++i) {
+        const int krow = (first + i * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * QS + ((lane >> 4) & 1) * 8;
 #pragma unroll
         for (int n = 0; n < NP / 16; ++n) {
           uint32_t bf[4];
           cr_ldmt(bf, sm.k_hi + krow + n * 16);
-          cr_mma(s[2 * n], vf, bf[0], bf[1]);
-          cr_mma(s[2 * n + 1], vf, bf[2], bf[3]);
+          cr_mma(s[2 * n], vf[i], bf[0], bf[1]);
+          cr_mma(s[2 * n + 1], vf[i], bf[2], bf[3]);
           cr_ldmt(bf, sm.k_lo + krow + n * 16);
-          cr_mma(s[2 * n], vf, bf[0], bf[1]);
-          cr_mma(s[2 * n + 1], vf, bf[2], bf[3]);
+          cr_mma(s[2 * n], vf[i], bf[0], bf[1]);
+          cr_mma(s[2 * n + 1], vf[i], bf[2], bf[3]);
         }
+      }
 #pragma unroll
-        for (int nt = 0; nt < NP / 8; ++nt) {
-          const float2 d = *reinterpret_cast<const float2*>(&sm.end[blk][nt * 8 + 2 * gc]);
-          s[nt][0] *= d.x; s[nt][1] *= d.y; s[nt][2] *= d.x; s[nt][3] *= d.y;
+      for (int nt = 0; nt < NP / 8; ++nt) {
+        const float2 d = *reinterpret_cast<const float2*>(end + nt * 8 + 2 * gc);
+        const float2 x = mul2(make_float2(s[nt][0], s[nt][1]), d), y = mul2(make_float2(s[nt][2], s[nt][3]), d);
+        s[nt][0] = x.x; s[nt][1] = x.y; s[nt][2] = y.x; s[nt][3] = y.y;
+      }
+    };
+    if (level < 2) {
+      if (!kStateOnly) {
+        // ---- the blocks a: a task is 16 tokens against 8; the last two cross the middle (one block of 32 only)
+        for (int task = warp; task < (level == 0 ? 6 : 4); task += kWarps) {
+          const int ib = task < 4 ? task >> 1 : 1, jb = task < 4 ? ib : 0, j0 = jb * 16 + (task & 1) * 8;
+          float sc[2][4] = {};
+#pragma unroll 4
+          for (int kk = 0; kk < NP / 16; ++kk) {
+            uint32_t aq[4];
+            cr_ldm(aq, sm.q + (ib * 16 + (lane & 15)) * QS + kk * 16 + (lane >> 4) * 8);
+            const int at = (j0 + gr) * QS + kk * 16 + 2 * gc;
+            const uint32_t* kh = reinterpret_cast<const uint32_t*>(sm.k_hi + at);
+            const uint32_t* kl = reinterpret_cast<const uint32_t*>(sm.k_lo + at);
+            cr_mma(sc[0], aq, kh[0], kh[4]);
+            cr_mma(sc[1], aq, kl[0], kl[4]);
+          }
+          const int j = j0 + 2 * gc;
+#pragma unroll
+          for (int e = 0; e < 4; e += 2) {
+            const int i = ib * 16 + gr + (e >> 1) * 8;
+            uint32_t hi, lo;
+            cr_split(make_float2(j <= i ? sc[0][e] + sc[1][e] : 0.f, j + 1 <= i ? sc[0][e + 1] + sc[1][e + 1] : 0.f), &hi, &lo);
+            *reinterpret_cast<uint32_t*>(sm.a_hi + i * PS + j) = hi;
+            *reinterpret_cast<uint32_t*>(sm.a_lo + i * PS + j) = lo;
+          }
         }
+        __syncthreads();
+      }
+      if (level == 0) {
+        block(std::integral_constant<int, 2>{}, 0, sm.end[0]);
+      } else {
+        block(std::integral_constant<int, 1>{}, 0, sm.end[0]);
+        block(std::integral_constant<int, 1>{}, 16, sm.end[1]);
       }
     } else {
       // ---- token by token
@@ -388,10 +441,21 @@ __global__ void __launch_bounds__(256) chanrec_chain_kernel(ChanrecParams a, Cha
   float run = a.pos0[b] == 0 ? 0.f : a.state[((int64_t)a.slots[b] * a.heads + h) * np + i];
   float* at = sg.start + (int64_t)bh * sg.count * np + i;
   const float* decay = sg.decay + (int64_t)bh * sg.count * a.n + n;
-  for (int k = 0; k < used; ++k) {
-    const float own = k + 1 < used ? at[(int64_t)k * np] : 0.f;
-    at[(int64_t)k * np] = run;
-    if (k + 1 < used) run = fmaf(decay[(int64_t)k * a.n], run, own);
+  constexpr int kAhead = 8;                               // segments requested before the first is used
+  for (int k0 = 0; k0 < used; k0 += kAhead) {
+    float own[kAhead], f[kAhead];
+#pragma unroll
+    for (int k = 0; k < kAhead; ++k) {
+      const bool more = k0 + k + 1 < used;
+      own[k] = more ? at[(int64_t)(k0 + k) * np] : 0.f;
+      f[k] = more ? decay[(int64_t)(k0 + k) * a.n] : 0.f;
+    }
+#pragma unroll
+    for (int k = 0; k < kAhead; ++k)
+      if (k0 + k < used) {
+        at[(int64_t)(k0 + k) * np] = run;
+        run = fmaf(f[k], run, own[k]);
+      }
   }
 }
 
@@ -403,9 +467,15 @@ static ChanrecSegs plan_chanrec(int batch, int max_tokens, int heads, int n, int
   const int64_t ctas = (int64_t)batch * heads * ((p + pt - 1) / pt);
   const int64_t room = 148 * (n > 128 ? 1 : 2);            // CTAs that run at the same time
   const int chunks = (max_tokens + kCrTokens - 1) / kCrTokens;
-  int64_t segs = ctas > 0 ? room / ctas : 1;               // segments of at least eight chunks
-  if (segs > chunks / 8) segs = chunks / 8;
-  if (segs < 1) segs = 1;
+  // segments of at least eight chunks: the fewest steps of a CTA, counting the pass over states alone (all segments but one) half,
+  // and a little for every segment's state that goes through memory
+  int segs = 1;
+  double best = 0;
+  for (int k = 1; k <= chunks / 8 + 1 && ctas * (k - 1) < 2 * room; ++k) {
+    if (k > 1 && chunks / k < 8) break;
+    const double cost = (double)((ctas * k + room - 1) / room) / k * (k > 1 ? 1.0 + 0.5 * (k - 1) / k : 1.0) + 0.005 * k;
+    if (k == 1 || cost < best) { best = cost; segs = k; }
+  }
   ChanrecSegs s = {};
   const int per = (int)((chunks + segs - 1) / segs);
   s.tokens = per * kCrTokens;

@@ -214,11 +214,12 @@ int launch_two_part_any(const char* what, const TwoPartAttn& p, int dtype, cudaS
 }
 
 // ---------------------------------------------------------------------------------------------------- split-KV decode
-// CTA = (a chunk of ring rows, request, 16 * MT query heads), eight warps, tiles of 32 rows through a ring of shared-memory
-// stages (16-byte pieces XOR-swizzled by row).  Scores: a warp takes 16 rows of the tile and a quarter of the contraction, its
-// part of the queries stays in registers; softmax: a warp adds the quarters up and takes 2 * MT heads; weighted sum: a warp takes
-// cpad / 8 = 8 * NT value dims for all heads.
-constexpr int kLdThreads = 256, kLdTile = 32;
+// CTA = (a chunk of ring rows, request, 16 query heads), eight warps, two CTAs per SM, tiles of 32 rows through a ring of
+// shared-memory stages (16-byte pieces XOR-swizzled by row).  Scores: a warp takes 16 rows of the tile and a quarter of the
+// contraction, its part of the queries stays in registers; softmax: a warp adds the quarters up and takes two heads; weighted
+// sum: a warp takes cpad / 8 = 8 * NT value dims for all heads.  CTAs of the same rows and other heads are neighbours in the
+// grid, so that the rows come from HBM once.
+constexpr int kLdThreads = 256, kLdTile = 32, kLdHeads = 16;
 
 struct LatentDecode {
   const void* q_abs; int64_t qa_token, qa_head;           // queries in the latent space, [.., cdim]
@@ -227,8 +228,8 @@ struct LatentDecode {
   const void* ring; int ring_rows, cdim, cpad, lw;
   const int32_t* slots; const int32_t* pos0;
   float scale_log2;
-  int batch, heads, chunk;
-  float* part_o; float* part_ml;                          // [batch, groups, chunks, 16 * MT, cpad], [.., 2]
+  int batch, heads, groups, chunk;
+  float* part_o; float* part_ml;                          // [batch, groups, chunks, 16, cpad], [.., 2]
   void* out; int64_t out_token, out_head;
 };
 
@@ -247,17 +248,17 @@ __device__ __forceinline__ void ld_x4t(uint32_t* r, uint32_t addr) {
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
 }
 
-template <int NT, int MT> struct LatentTile {
-  static constexpr int R = 16 * MT, LW = 64 * (NT + 1), QS = LW + 8, SS = kLdTile + 4, PS = kLdTile + 8;
-  static constexpr int kStages = NT <= 2 ? 8 : NT <= 5 ? 6 : 5, kStageBytes = kLdTile * LW * 2;
+template <int NT> struct LatentTile {
+  static constexpr int R = kLdHeads, LW = 64 * (NT + 1), QS = LW + 8, SS = kLdTile + 4, PS = kLdTile + 8;
+  static constexpr int kStageBytes = kLdTile * LW * 2, kStages = NT >= 6 ? 2 : NT >= 4 ? 3 : NT >= 2 ? 5 : 8;
   static constexpr int kQBytes = R * QS * 2, kSBytes = 4 * R * SS * 4;           // the queries' place is taken by the scores
   static constexpr int kUnion = kQBytes > kSBytes ? kQBytes : kSBytes;
   static constexpr int kBytes = kStages * kStageBytes + kUnion + R * PS * 2 + R * 4;
 };
 
-template <int NT, int MT>
-__global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(LatentDecode p) {
-  using L = LatentTile<NT, MT>;
+template <int NT>
+__global__ void __launch_bounds__(kLdThreads, 2) latent_decode_kernel(LatentDecode p) {
+  using L = LatentTile<NT>;
   constexpr int R = L::R, LW = L::LW, QS = L::QS, SS = L::SS, PS = L::PS, S = L::kStages, kPieces = LW / 8, KS = LW / 64;
   extern __shared__ __align__(128) uint8_t raw[];
   uint8_t* tiles = raw;                                                          // [S][32][LW] swizzled
@@ -268,9 +269,9 @@ __global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(LatentDecode 
   grid_dependency_wait();
   grid_launch_dependents();
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gr = lane >> 2, gc = lane & 3;
-  const int b = blockIdx.y, grp = blockIdx.z, h0 = grp * R, nh = min(R, p.heads - h0);
+  const int b = blockIdx.y, chunk = blockIdx.x / p.groups, grp = blockIdx.x - chunk * p.groups, h0 = grp * R, nh = min(R, p.heads - h0);
   const int pos = p.pos0[b], len = min(pos + 1, p.ring_rows);
-  const int t0 = blockIdx.x * p.chunk, t1 = min(len, t0 + p.chunk);
+  const int t0 = chunk * p.chunk, t1 = min(len, t0 + p.chunk);
   if (t0 >= len) return;
   const __nv_bfloat16* K = (const __nv_bfloat16*)p.ring + (int64_t)p.slots[b] * p.ring_rows * LW;
   auto fetch = [&](int t, int st) {                       // a group per tile, empty beyond the end
@@ -311,16 +312,12 @@ __global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(LatentDecode 
   }
   __syncthreads();
   const int rg = warp & 1, kq = warp >> 1;                // 16 rows of a tile, quarter of the contraction
-  uint32_t qf[MT][KS][4];
+  uint32_t qf[KS][4];
 #pragma unroll
-  for (int m = 0; m < MT; ++m)
-#pragma unroll
-    for (int k = 0; k < KS; ++k)
-      ld_x4(qf[m][k], smem_u32(q_s) + (uint32_t)((m * 16 + (lane & 15)) * QS + (kq * KS + k) * 16 + (lane >> 4) * 8) * 2);
-  float o[MT][NT][4] = {};
-  float mx[2 * MT], l[2 * MT];
-#pragma unroll
-  for (int i = 0; i < 2 * MT; ++i) { mx[i] = -INFINITY; l[i] = 0.f; }
+  for (int k = 0; k < KS; ++k)
+    ld_x4(qf[k], smem_u32(q_s) + (uint32_t)((lane & 15) * QS + (kq * KS + k) * 16 + (lane >> 4) * 8) * 2);
+  float o[NT][4] = {};
+  float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   const uint32_t p_addr = smem_u32(p_s);
   int st = 0;
   for (int t = t0; t < t1; t += kLdTile, st = st + 1 == S ? 0 : st + 1) {
@@ -330,32 +327,27 @@ __global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(LatentDecode 
     const uint32_t tile = smem_u32(tiles) + st * L::kStageBytes;
     // ---- scores
     {
-      float acc[MT][2][4] = {};
+      float acc[2][4] = {};
       const int row = rg * 16 + (lane & 7) + ((lane >> 4) & 1) * 8;
       const uint32_t krow = tile + (uint32_t)row * LW * 2;
 #pragma unroll
       for (int k = 0; k < KS; ++k) {
         uint32_t kf[4];
         ld_x4(kf, krow + (uint32_t)((((kq * KS + k) * 2 + ((lane >> 3) & 1)) ^ (row & 7)) * 16));
-#pragma unroll
-        for (int m = 0; m < MT; ++m) {
-          ld_mma(acc[m][0], qf[m][k], kf[0], kf[1]);
-          ld_mma(acc[m][1], qf[m][k], kf[2], kf[3]);
-        }
+        ld_mma(acc[0], qf[k], kf[0], kf[1]);
+        ld_mma(acc[1], qf[k], kf[2], kf[3]);
       }
 #pragma unroll
-      for (int m = 0; m < MT; ++m)
+      for (int n = 0; n < 2; ++n)
 #pragma unroll
-        for (int n = 0; n < 2; ++n)
-#pragma unroll
-          for (int e = 0; e < 4; e += 2)
-            *reinterpret_cast<float2*>(s_s + (kq * R + m * 16 + gr + (e >> 1) * 8) * SS + rg * 16 + n * 8 + 2 * gc) = make_float2(acc[m][n][e], acc[m][n][e + 1]);
+        for (int e = 0; e < 4; e += 2)
+          *reinterpret_cast<float2*>(s_s + (kq * R + gr + (e >> 1) * 8) * SS + rg * 16 + n * 8 + 2 * gc) = make_float2(acc[n][e], acc[n][e + 1]);
     }
     __syncthreads();
-    // ---- softmax of heads warp * 2 MT ..
+    // ---- softmax of heads 2 warp, 2 warp + 1
 #pragma unroll
-    for (int i = 0; i < 2 * MT; ++i) {
-      const int r = warp * 2 * MT + i;
+    for (int i = 0; i < 2; ++i) {
+      const int r = warp * 2 + i;
       float x = 0.f;
 #pragma unroll
       for (int q = 0; q < 4; ++q) x += s_s[(q * R + r) * SS + lane];
@@ -372,68 +364,58 @@ __global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(LatentDecode 
     }
     __syncthreads();
     // ---- weighted sum of the latents
+    const float f0 = fix_s[gr], f1 = fix_s[gr + 8];
 #pragma unroll
-    for (int m = 0; m < MT; ++m) {
-      const float f0 = fix_s[m * 16 + gr], f1 = fix_s[m * 16 + gr + 8];
-#pragma unroll
-      for (int n = 0; n < NT; ++n) { o[m][n][0] *= f0; o[m][n][1] *= f0; o[m][n][2] *= f1; o[m][n][3] *= f1; }
-    }
+    for (int n = 0; n < NT; ++n) { o[n][0] *= f0; o[n][1] *= f0; o[n][2] *= f1; o[n][3] *= f1; }
 #pragma unroll
     for (int k = 0; k < kLdTile / 16; ++k) {
-      uint32_t pf[MT][4];
-#pragma unroll
-      for (int m = 0; m < MT; ++m) ld_x4(pf[m], p_addr + (uint32_t)((m * 16 + (lane & 15)) * PS + k * 16 + (lane >> 4) * 8) * 2);
+      uint32_t pf[4];
+      ld_x4(pf, p_addr + (uint32_t)((lane & 15) * PS + k * 16 + (lane >> 4) * 8) * 2);
       const int row = k * 16 + (lane & 15);
 #pragma unroll
       for (int n = 0; n < NT; n += 2) {
         uint32_t vf[4];
         const int c = warp * NT + min(n + (lane >> 4), NT - 1);
         ld_x4t(vf, tile + (uint32_t)row * LW * 2 + (uint32_t)((c ^ (row & 7)) * 16));
-#pragma unroll
-        for (int m = 0; m < MT; ++m) {
-          ld_mma(o[m][n], pf[m], vf[0], vf[1]);
-          if (n + 1 < NT) ld_mma(o[m][n + 1], pf[m], vf[2], vf[3]);
-        }
+        ld_mma(o[n], pf, vf[0], vf[1]);
+        if (n + 1 < NT) ld_mma(o[n + 1], pf, vf[2], vf[3]);
       }
     }
   }
-  const int64_t part = (((int64_t)b * gridDim.z + grp) * gridDim.x + blockIdx.x) * R;
+  const int64_t part = (((int64_t)b * p.groups + grp) * (gridDim.x / p.groups) + chunk) * R;
 #pragma unroll
-  for (int i = 0; i < 2 * MT; ++i) {
+  for (int i = 0; i < 2; ++i) {
     const float sum = warp_add(l[i]);
-    const int r = warp * 2 * MT + i;
+    const int r = warp * 2 + i;
     if (lane == 0) { p.part_ml[(part + r) * 2] = mx[i]; p.part_ml[(part + r) * 2 + 1] = sum; }
   }
 #pragma unroll
-  for (int m = 0; m < MT; ++m)
+  for (int n = 0; n < NT; ++n)
 #pragma unroll
-    for (int n = 0; n < NT; ++n)
-#pragma unroll
-      for (int e = 0; e < 4; e += 2) {
-        const int r = m * 16 + gr + (e >> 1) * 8;
-        if (r < nh) *reinterpret_cast<float2*>(p.part_o + (part + r) * p.cpad + (warp * NT + n) * 8 + 2 * gc) = make_float2(o[m][n][e], o[m][n][e + 1]);
-      }
+    for (int e = 0; e < 4; e += 2) {
+      const int r = gr + (e >> 1) * 8;
+      if (r < nh) *reinterpret_cast<float2*>(p.part_o + (part + r) * p.cpad + (warp * NT + n) * 8 + 2 * gc) = make_float2(o[n][e], o[n][e + 1]);
+    }
 }
 
 // Merge of the chunks.  One CTA per (request, head).
-__global__ void __launch_bounds__(kLpThreads) latent_merge_kernel(LatentDecode p, int nchunks, int rows_per_group) {
+__global__ void __launch_bounds__(kLpThreads) latent_merge_kernel(LatentDecode p, int nchunks) {
   grid_dependency_wait();
   grid_launch_dependents();
-  const int b = blockIdx.x / p.heads, h = blockIdx.x - b * p.heads, grp = h / rows_per_group, r = h - grp * rows_per_group;
-  const int groups = (p.heads + rows_per_group - 1) / rows_per_group;
+  const int b = blockIdx.x / p.heads, h = blockIdx.x - b * p.heads, grp = h / kLdHeads, r = h - grp * kLdHeads;
   const int len = min(p.pos0[b] + 1, p.ring_rows), used = (len + p.chunk - 1) / p.chunk;
-  const int64_t part = ((int64_t)b * groups + grp) * nchunks;
+  const int64_t part = ((int64_t)b * p.groups + grp) * nchunks;
   float top = -INFINITY, sum = 0.f;
-  for (int k = 0; k < used; ++k) top = fmaxf(top, p.part_ml[((part + k) * rows_per_group + r) * 2]);
+  for (int k = 0; k < used; ++k) top = fmaxf(top, p.part_ml[((part + k) * kLdHeads + r) * 2]);
   for (int k = 0; k < used; ++k) {
-    const float* ml = p.part_ml + ((part + k) * rows_per_group + r) * 2;
+    const float* ml = p.part_ml + ((part + k) * kLdHeads + r) * 2;
     sum = fmaf(exp2_weight(ml[0] - top), ml[1], sum);
   }
   __nv_bfloat16* dst = (__nv_bfloat16*)p.out + (int64_t)b * p.out_token + (int64_t)h * p.out_head;
   for (int c = threadIdx.x; c < p.cdim; c += kLpThreads) {
     float a = 0.f;
     for (int k = 0; k < used; ++k) {
-      const int64_t at = (part + k) * rows_per_group + r;
+      const int64_t at = (part + k) * kLdHeads + r;
       a = fmaf(exp2_weight(p.part_ml[at * 2] - top), p.part_o[at * p.cpad + c], a);
     }
     dst[c] = __float2bfloat16_rn(a / sum);
@@ -441,11 +423,10 @@ __global__ void __launch_bounds__(kLpThreads) latent_merge_kernel(LatentDecode p
 }
 
 static bool latent_decode_shape(int cdim, int rot_dim, int dtype) { return dtype == TKV_BF16 && cdim <= 512 && rot_dim >= 1 && rot_dim <= 64; }
-static int latent_row_tiles(int heads) { return heads > 16 ? 2 : 1; }
 
 // Rows of the ring per CTA: the smallest time under a simple cost (waves of CTAs, each its rows and a fixed start and merge).
-static int latent_chunk(int64_t segments, int ring_rows, int cpad) {
-  const int64_t width = 148 * (cpad <= 128 ? 2 : 1);      // CTAs that run at the same time (shared memory)
+static int latent_chunk(int64_t segments, int ring_rows) {
+  const int64_t width = 148 * 2;                          // CTAs that run at the same time
   int best = 64;
   int64_t best_cost = -1;
   for (int c = 64; c < ring_rows + 64; c += 64) {
@@ -546,38 +527,37 @@ extern "C" int tkv_latent_prefill(const void* q, int64_t q_stride, const void* k
 extern "C" int64_t tkv_latent_decode_workspace_bytes(int batch, int heads, int kv_rank, int rot_dim, int ring_rows, int dtype) {
   if (batch <= 0 || heads <= 0 || kv_rank <= 0 || rot_dim < 0 || ring_rows <= 0) return 0;
   if (!latent_decode_shape(kv_rank, rot_dim, dtype)) return -1;
-  const int mt = latent_row_tiles(heads), groups = (heads + 16 * mt - 1) / (16 * mt), cpad = pad64(kv_rank);
-  const int chunk = latent_chunk((int64_t)batch * groups, ring_rows, cpad);
-  return (int64_t)batch * groups * ((ring_rows + chunk - 1) / chunk) * 16 * mt * (cpad + 2) * (int64_t)sizeof(float);
+  const int groups = (heads + kLdHeads - 1) / kLdHeads, cpad = pad64(kv_rank);
+  const int chunk = latent_chunk((int64_t)batch * groups, ring_rows);
+  return (int64_t)batch * groups * ((ring_rows + chunk - 1) / chunk) * kLdHeads * (cpad + 2) * (int64_t)sizeof(float);
 }
 
 namespace tkv {
-template <int NT, int MT>
+template <int NT>
 static int launch_latent_decode(const LatentDecode& p, dim3 grid, cudaStream_t st) {
-  constexpr int kBytes = LatentTile<NT, MT>::kBytes;
+  constexpr int kBytes = LatentTile<NT>::kBytes;
   static_assert(kBytes <= 232448, "shared memory of the kernel");
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<NT, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kBytes);
+    cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kBytes);
     if (e != cudaSuccess) return fail(TKV_ERR_LAUNCH, "tkv_latent_decode: %s", cudaGetErrorString(e));
     configured = true;
   }
-  cudaError_t e = launch_pdl(latent_decode_kernel<NT, MT>, grid, dim3(kLdThreads), (size_t)kBytes, st, p);
-  if (e == cudaSuccess) e = launch_pdl(latent_merge_kernel, dim3((unsigned)(p.batch * p.heads)), dim3(kLpThreads), 0, st, p, (int)grid.x, 16 * MT);
+  cudaError_t e = launch_pdl(latent_decode_kernel<NT>, grid, dim3(kLdThreads), (size_t)kBytes, st, p);
+  if (e == cudaSuccess) e = launch_pdl(latent_merge_kernel, dim3((unsigned)(p.batch * p.heads)), dim3(kLpThreads), 0, st, p, (int)grid.x / p.groups);
   if (e != cudaSuccess) return fail(TKV_ERR_LAUNCH, "tkv_latent_decode: %s", cudaGetErrorString(e));
   return check_launch("tkv_latent_decode");
 }
-template <int MT>
 static int launch_latent_decode_nt(const LatentDecode& p, dim3 grid, cudaStream_t st) {
   switch (p.cpad / 64) {
-    case 1: return launch_latent_decode<1, MT>(p, grid, st);
-    case 2: return launch_latent_decode<2, MT>(p, grid, st);
-    case 3: return launch_latent_decode<3, MT>(p, grid, st);
-    case 4: return launch_latent_decode<4, MT>(p, grid, st);
-    case 5: return launch_latent_decode<5, MT>(p, grid, st);
-    case 6: return launch_latent_decode<6, MT>(p, grid, st);
-    case 7: return launch_latent_decode<7, MT>(p, grid, st);
-    default: return launch_latent_decode<8, MT>(p, grid, st);
+    case 1: return launch_latent_decode<1>(p, grid, st);
+    case 2: return launch_latent_decode<2>(p, grid, st);
+    case 3: return launch_latent_decode<3>(p, grid, st);
+    case 4: return launch_latent_decode<4>(p, grid, st);
+    case 5: return launch_latent_decode<5>(p, grid, st);
+    case 6: return launch_latent_decode<6>(p, grid, st);
+    case 7: return launch_latent_decode<7>(p, grid, st);
+    default: return launch_latent_decode<8>(p, grid, st);
   }
 }
 }  // namespace tkv
@@ -610,13 +590,12 @@ extern "C" int tkv_latent_decode(const void* q_abs, int64_t qa_token, int64_t qa
   if (!workspace || workspace_bytes < need)
     return fail(TKV_ERR_ARG, "tkv_latent_decode: workspace of %lld bytes, %lld needed", (long long)workspace_bytes, (long long)need);
   if (batch > 65535) return fail(TKV_ERR_UNSUPPORTED, "tkv_latent_decode: batch=%d", batch);
-  const int mt = latent_row_tiles(heads), groups = (heads + 16 * mt - 1) / (16 * mt);
+  const int groups = (heads + kLdHeads - 1) / kLdHeads;
   LatentDecode p = {q_abs, qa_token, qa_head, q_rot, qr_token, qr_head, (const float2*)freq_hi_lo, rot_dim, rot_dims, ring, ring_rows, kv_rank,
-                    cpad, lw, slots, pos0, scale * 1.4426950408889634f, batch, heads, latent_chunk((int64_t)batch * groups, ring_rows, cpad),
+                    cpad, lw, slots, pos0, scale * 1.4426950408889634f, batch, heads, groups, latent_chunk((int64_t)batch * groups, ring_rows),
                     nullptr, nullptr, out, out_token, out_head};
   const int chunks = (ring_rows + p.chunk - 1) / p.chunk;
   p.part_o = (float*)workspace;
-  p.part_ml = p.part_o + (int64_t)batch * groups * chunks * 16 * mt * cpad;
-  const dim3 grid(chunks, batch, groups);
-  return mt == 2 ? launch_latent_decode_nt<2>(p, grid, (cudaStream_t)stream) : launch_latent_decode_nt<1>(p, grid, (cudaStream_t)stream);
+  p.part_ml = p.part_o + (int64_t)batch * groups * chunks * kLdHeads * cpad;
+  return launch_latent_decode_nt(p, dim3(chunks * groups, batch), (cudaStream_t)stream);
 }
