@@ -107,13 +107,14 @@ def test_every_microbenchmark_runs_and_prints_a_line(argv, capsys):
 
 
 @pytest.mark.gpu
-def test_hybrid_microbenchmark_runs_and_prints_a_line(capsys):
+@pytest.mark.parametrize("micro,models", [("hybrid", ("hybrid", "qwen3")), ("lonulix", ("lonulix", "dafovik"))])
+def test_hybrid_microbenchmarks_run_and_print_a_line(micro, models, capsys):
     sys.path.insert(0, ROOT)
     import bench
-    bench.run_micro(bench.parse_args(["--micro", "hybrid", "--hybrid-size", "tiny"]))
+    bench.run_micro(bench.parse_args(["--micro", micro, "--hybrid-size", "tiny"]))
     lines = [l for l in capsys.readouterr().out.splitlines() if l.startswith("{")]
     assert len(lines) == 1
     d = json.loads(lines[0])
-    for model in ("hybrid", "qwen3"):
+    for model in models:
         assert any(k.startswith("prefill") for k in d[model]) and any(k.startswith("decode") for k in d[model])
     assert d["kernels"] and all(k["us"] > 0 for k in d["kernels"].values())

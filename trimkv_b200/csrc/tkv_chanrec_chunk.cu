@@ -61,12 +61,13 @@ __device__ __forceinline__ float2 add2(float2 a, float2 b) {
       : "=f"(r.x), "=f"(r.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y));
   return r;
 }
+constexpr float kMinusLog2e = -1.4426950408889634f;
 __device__ __forceinline__ float2 pair(float x) { return make_float2(x, x); }
 // x = hi + lo in bf16, two values at a time.
 __device__ __forceinline__ void cr_split(float2 x, uint32_t* hi, uint32_t* lo) {
   const __nv_bfloat162 h = __floats2bfloat162_rn(x.x, x.y);
   *hi = *reinterpret_cast<const uint32_t*>(&h);
-  const float2 r = add2(x, make_float2(-__uint_as_float(*hi << 16), -__uint_as_float(*hi & 0xffff0000u)));
+  const float2 r = fma2(make_float2(__uint_as_float(*hi << 16), __uint_as_float(*hi & 0xffff0000u)), pair(-1.0f), x);
   const __nv_bfloat162 l = __floats2bfloat162_rn(r.x, r.y);
   *lo = *reinterpret_cast<const uint32_t*>(&l);
 }
@@ -83,21 +84,21 @@ __device__ __forceinline__ float cr_rcp(float x) {
   asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-// f, 1 / f and k = 1 - f of two channels with one reciprocal each: with e = exp(-|x|), sigmoid(|x|) = 1 / (1 + e),
-// f = num / (1 + e).  Where f leaves the range of fp32 the result is not a number, or zero; the caller looks at the product.
-__device__ __forceinline__ void cr_gate(float2 x, float2 lo, float2 rest, float2* f, float2* inv, float2* k) {
-  const float2 e = make_float2(exp2_weight(fabsf(x.x) * -1.4426950408889634f), exp2_weight(fabsf(x.y) * -1.4426950408889634f));
-  const float2 den = add2(e, pair(1.0f));
-  const float2 pos = make_float2(x.x >= 0.f ? 1.0f : e.x, x.y >= 0.f ? 1.0f : e.y), neg = make_float2(x.x >= 0.f ? e.x : 1.0f, x.y >= 0.f ? e.y : 1.0f);
-  const float2 num = fma2(rest, pos, mul2(lo, den)), dn = mul2(den, num);
+// f, 1 / f and k = 1 - f of two channels with one reciprocal each, from -x / ln 2 of the gate's argument x: with e = exp(-x),
+// f = (lo (1 + e) + 1 - lo) / (1 + e) and k = (1 - lo) e / (1 + e).  e is held below 2^60 (sigmoid 1e-18), which only gates
+// that send the chunk to the token-by-token path ever reach.
+__device__ __forceinline__ void cr_gate(float2 y, float2 lo, float2 rest, float2* f, float2* inv, float2* k) {
+  const float2 e = make_float2(exp2_weight(fminf(y.x, 60.0f)), exp2_weight(fminf(y.y, 60.0f)));
+  const float2 den = add2(e, pair(1.0f)), num = fma2(lo, den, rest), dn = mul2(den, num);
   const float2 t = make_float2(cr_rcp(dn.x), cr_rcp(dn.y)), u = mul2(num, t);      // u = 1 / den
   *f = mul2(num, u);
-  *inv = mul2(mul2(den, den), t);
-  *k = mul2(mul2(rest, neg), u);
+  *inv = mul2(den, mul2(den, t));
+  *k = mul2(mul2(rest, e), u);
 }
 __device__ __forceinline__ float cr_silu(float z) { return z * cr_rcp(1.0f + exp2_weight(z * -1.4426950408889634f)); }
 __device__ __forceinline__ float2 cr_silu2(float2 z) {
-  const float2 d = add2(make_float2(exp2_weight(z.x * -1.4426950408889634f), exp2_weight(z.y * -1.4426950408889634f)), pair(1.0f));
+  const float2 y = mul2(z, pair(kMinusLog2e));
+  const float2 d = add2(make_float2(exp2_weight(y.x), exp2_weight(y.y)), pair(1.0f));
   return mul2(z, make_float2(cr_rcp(d.x), cr_rcp(d.y)));
 }
 
@@ -189,7 +190,7 @@ __global__ void __launch_bounds__(kWarps * 32, NP == 256 ? 1 : kWarps == 8 ? 2 :
       const int c = rd * kWarps * 16 + (warp >> 2) * 64 + 2 * lane;
       if (c >= NP) continue;
       // a channel that does not exist keeps its (zero) state: lower bound 1
-      const float2 bi = c < a.n ? *reinterpret_cast<const float2*>(bias + c) : pair(0.f);
+      const float2 bi = c < a.n ? mul2(*reinterpret_cast<const float2*>(bias + c), pair(kMinusLog2e)) : pair(0.f);
       const float2 lo = c < a.n ? *reinterpret_cast<const float2*>(lower + c) : pair(1.f);
       const float2 rest = make_float2(1.0f - lo.x, 1.0f - lo.y);
       float2 inv = pair(1.0f);
@@ -198,7 +199,7 @@ __global__ void __launch_bounds__(kWarps * 32, NP == 256 ? 1 : kWarps == 8 ? 2 :
         for (int j = 0; j < 8; ++j) {
           const uint32_t z = *reinterpret_cast<const uint32_t*>(&sm.zf[st][(r0 + j) * QS + c]);
           float2 f, fi, k;
-          cr_gate(add2(make_float2(__uint_as_float(z << 16), __uint_as_float(z & 0xffff0000u)), bi), lo, rest, &f, &fi, &k);
+          cr_gate(fma2(make_float2(__uint_as_float(z << 16), __uint_as_float(z & 0xffff0000u)), pair(kMinusLog2e), bi), lo, rest, &f, &fi, &k);
           if (j >= live) { f = pair(1.0f); fi = f; k = pair(0.0f); }
           P[rd][j] = j > 0 ? mul2(P[rd][j - 1], f) : f;
           inv = mul2(inv, fi);
@@ -209,9 +210,8 @@ __global__ void __launch_bounds__(kWarps * 32, NP == 256 ? 1 : kWarps == 8 ? 2 :
       else walk8(ntok - t0 - r0);
       *reinterpret_cast<float2*>(&sm.oct[0][oct][c]) = P[rd][7];
       *reinterpret_cast<float2*>(&sm.oct[1][oct][c]) = inv;
-      const float low = fminf(P[rd][7].x, P[rd][7].y);     // not a number counts as below
-      const bool nan = P[rd][7].x != P[rd][7].x || P[rd][7].y != P[rd][7].y;
-      if (nan || !(low >= kWide)) atomicMax(&sm.level[st], nan || !(low >= kNarrow) ? 2 : 1);
+      if (!(P[rd][7].x >= kWide && P[rd][7].y >= kWide))   // not a number counts as below
+        atomicMax(&sm.level[st], P[rd][7].x >= kNarrow && P[rd][7].y >= kNarrow ? 1 : 2);
     }
     __syncthreads();
     const int level = sm.level[st];

@@ -214,11 +214,11 @@ int launch_two_part_any(const char* what, const TwoPartAttn& p, int dtype, cudaS
 }
 
 // ---------------------------------------------------------------------------------------------------- split-KV decode
-// CTA = (a chunk of ring rows, request, 16 query heads), eight warps, two CTAs per SM, tiles of 32 rows through a ring of
-// shared-memory stages (16-byte pieces XOR-swizzled by row).  Scores: a warp takes 16 rows of the tile and a quarter of the
-// contraction, its part of the queries stays in registers; softmax: a warp adds the quarters up and takes two heads; weighted
-// sum: a warp takes cpad / 8 = 8 * NT value dims for all heads.  CTAs of the same rows and other heads are neighbours in the
-// grid, so that the rows come from HBM once.
+// CTA = (a chunk of ring rows, request, HG groups of 16 query heads), eight warps per group, 16 warps per SM, tiles of 32 rows
+// through a ring of shared-memory stages (16-byte pieces XOR-swizzled by row) that the groups share.  Scores: a warp takes 16
+// rows of the tile and a quarter of the contraction, its part of the queries stays in registers; softmax: a warp adds the
+// quarters up and takes two heads; weighted sum: a warp takes cpad / 8 = 8 * NT value dims for the group's heads.  CTAs of the
+// same rows and other heads are neighbours in the grid, so that the rows come from HBM once.
 constexpr int kLdThreads = 256, kLdTile = 32, kLdHeads = 16;
 
 struct LatentDecode {
@@ -248,28 +248,36 @@ __device__ __forceinline__ void ld_x4t(uint32_t* r, uint32_t addr) {
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
 }
 
-template <int NT> struct LatentTile {
-  static constexpr int R = kLdHeads, LW = 64 * (NT + 1), QS = LW + 8, SS = kLdTile + 4, PS = kLdTile + 8;
-  static constexpr int kStageBytes = kLdTile * LW * 2, kStages = NT >= 6 ? 2 : NT >= 4 ? 3 : NT >= 2 ? 5 : 8;
+template <int NT, int HG> struct LatentTile {
+  static constexpr int R = kLdHeads, LW = 64 * (NT + 1), QS = LW + 8, SS = kLdTile + 8, PS = kLdTile + 8;
+  static constexpr int kStageBytes = kLdTile * LW * 2, kStages = (NT >= 6 ? 2 : NT >= 4 ? 3 : NT >= 2 ? 4 : 6) * HG;
   static constexpr int kQBytes = R * QS * 2, kSBytes = 4 * R * SS * 4;           // the queries' place is taken by the scores
   static constexpr int kUnion = kQBytes > kSBytes ? kQBytes : kSBytes;
-  static constexpr int kBytes = kStages * kStageBytes + kUnion + R * PS * 2 + R * 4;
+  static constexpr int kGroupBytes = kUnion + R * PS * 2 + R * 4;
+  static constexpr int kBytes = kStages * kStageBytes + HG * kGroupBytes;
 };
 
-template <int NT>
-__global__ void __launch_bounds__(kLdThreads, 2) latent_decode_kernel(LatentDecode p) {
-  using L = LatentTile<NT>;
+template <int NT, int HG>
+__global__ void __launch_bounds__(kLdThreads * HG, 2 / HG) latent_decode_kernel(LatentDecode p) {
+  using L = LatentTile<NT, HG>;
   constexpr int R = L::R, LW = L::LW, QS = L::QS, SS = L::SS, PS = L::PS, S = L::kStages, kPieces = LW / 8, KS = LW / 64;
   extern __shared__ __align__(128) uint8_t raw[];
+  const int group = HG > 1 ? threadIdx.x / kLdThreads : 0, tid = threadIdx.x - group * kLdThreads;
   uint8_t* tiles = raw;                                                          // [S][32][LW] swizzled
-  __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(raw + S * L::kStageBytes);   // [R][QS], then
+  uint8_t* mine = raw + S * L::kStageBytes + group * L::kGroupBytes;
+  __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(mine);                   // [R][QS], then
   float* s_s = reinterpret_cast<float*>(q_s);                                    // [4][R][SS]
-  __nv_bfloat16* p_s = reinterpret_cast<__nv_bfloat16*>(raw + S * L::kStageBytes + L::kUnion);   // [R][PS]
+  __nv_bfloat16* p_s = reinterpret_cast<__nv_bfloat16*>(mine + L::kUnion);       // [R][PS]
   float* fix_s = reinterpret_cast<float*>(p_s + R * PS);                         // [R]
+  auto group_sync = [&]() {
+    if constexpr (HG == 1) __syncthreads();
+    else asm volatile("bar.sync %0, %1;" ::"r"(1 + group), "n"(kLdThreads) : "memory");
+  };
   grid_dependency_wait();
   grid_launch_dependents();
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gr = lane >> 2, gc = lane & 3;
-  const int b = blockIdx.y, chunk = blockIdx.x / p.groups, grp = blockIdx.x - chunk * p.groups, h0 = grp * R, nh = min(R, p.heads - h0);
+  const int lane = tid & 31, warp = tid >> 5, gr = lane >> 2, gc = lane & 3;
+  const int cgroups = (p.groups + HG - 1) / HG, chunk = blockIdx.x / cgroups, grp = (blockIdx.x - chunk * cgroups) * HG + group;
+  const int b = blockIdx.y, h0 = grp * R, nh = max(0, min(R, p.heads - h0));      // a last CTA may have a group without heads
   const int pos = p.pos0[b], len = min(pos + 1, p.ring_rows);
   const int t0 = chunk * p.chunk, t1 = min(len, t0 + p.chunk);
   if (t0 >= len) return;
@@ -278,8 +286,9 @@ __global__ void __launch_bounds__(kLdThreads, 2) latent_decode_kernel(LatentDeco
     const uint32_t dst = smem_u32(tiles) + st * L::kStageBytes;
     if (t < t1)
 #pragma unroll
-      for (int j = 0; j < kLdTile * kPieces / kLdThreads; ++j) {
-        const int i = tid + j * kLdThreads, r = i / kPieces, c = i - r * kPieces;
+      for (int j = 0; j < (kLdTile * kPieces + kLdThreads * HG - 1) / (kLdThreads * HG); ++j) {
+        const int i = threadIdx.x + j * kLdThreads * HG, r = i / kPieces, c = i - r * kPieces;
+        if (kLdTile * kPieces % (kLdThreads * HG) != 0 && r >= kLdTile) break;
         const bool live = t + r < t1;                     // the rest reads as zeros
         const int bytes = live ? 16 : 0;
         const void* src = K + (live ? (int64_t)(t + r) * LW + c * 8 : 0);
@@ -310,7 +319,7 @@ __global__ void __launch_bounds__(kLdThreads, 2) latent_decode_kernel(LatentDeco
       q_s[r * QS + NT * 64 + c + 1] = __float2bfloat16_rn(y * co + x * s);
     }
   }
-  __syncthreads();
+  group_sync();
   const int rg = warp & 1, kq = warp >> 1;                // 16 rows of a tile, quarter of the contraction
   uint32_t qf[KS][4];
 #pragma unroll
@@ -343,7 +352,7 @@ __global__ void __launch_bounds__(kLdThreads, 2) latent_decode_kernel(LatentDeco
         for (int e = 0; e < 4; e += 2)
           *reinterpret_cast<float2*>(s_s + (kq * R + gr + (e >> 1) * 8) * SS + rg * 16 + n * 8 + 2 * gc) = make_float2(acc[n][e], acc[n][e + 1]);
     }
-    __syncthreads();
+    group_sync();
     // ---- softmax of heads 2 warp, 2 warp + 1
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
@@ -362,7 +371,7 @@ __global__ void __launch_bounds__(kLdThreads, 2) latent_decode_kernel(LatentDeco
       p_s[r * PS + lane] = __float2bfloat16_rn(w);
       if (lane == 0) fix_s[r] = fix;
     }
-    __syncthreads();
+    group_sync();
     // ---- weighted sum of the latents
     const float f0 = fix_s[gr], f1 = fix_s[gr + 8];
 #pragma unroll
@@ -382,7 +391,8 @@ __global__ void __launch_bounds__(kLdThreads, 2) latent_decode_kernel(LatentDeco
       }
     }
   }
-  const int64_t part = (((int64_t)b * p.groups + grp) * (gridDim.x / p.groups) + chunk) * R;
+  if (nh == 0) return;
+  const int64_t part = (((int64_t)b * p.groups + grp) * (gridDim.x / cgroups) + chunk) * R;
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     const float sum = warp_add(l[i]);
@@ -425,11 +435,11 @@ __global__ void __launch_bounds__(kLpThreads) latent_merge_kernel(LatentDecode p
 static bool latent_decode_shape(int cdim, int rot_dim, int dtype) { return dtype == TKV_BF16 && cdim <= 512 && rot_dim >= 1 && rot_dim <= 64; }
 
 // Rows of the ring per CTA: the smallest time under a simple cost (waves of CTAs, each its rows and a fixed start and merge).
-static int latent_chunk(int64_t segments, int ring_rows) {
-  const int64_t width = 148 * 2;                          // CTAs that run at the same time
-  int best = 64;
+static int latent_chunk(int batch, int groups, int ring_rows) {
+  const int64_t segments = (int64_t)batch * (groups > 1 ? (groups + 1) / 2 : 1), width = 148 * (groups > 1 ? 1 : 2);
+  int best = kLdTile;
   int64_t best_cost = -1;
-  for (int c = 64; c < ring_rows + 64; c += 64) {
+  for (int c = kLdTile; c < ring_rows + kLdTile; c += kLdTile) {
     const int64_t ctas = segments * ((ring_rows + c - 1) / c), waves = (ctas + width - 1) / width;
     const int64_t cost = waves * (c + 128);
     if (best_cost < 0 || cost < best_cost) { best = c; best_cost = cost; }
@@ -528,36 +538,38 @@ extern "C" int64_t tkv_latent_decode_workspace_bytes(int batch, int heads, int k
   if (batch <= 0 || heads <= 0 || kv_rank <= 0 || rot_dim < 0 || ring_rows <= 0) return 0;
   if (!latent_decode_shape(kv_rank, rot_dim, dtype)) return -1;
   const int groups = (heads + kLdHeads - 1) / kLdHeads, cpad = pad64(kv_rank);
-  const int chunk = latent_chunk((int64_t)batch * groups, ring_rows);
+  const int chunk = latent_chunk(batch, groups, ring_rows);
   return (int64_t)batch * groups * ((ring_rows + chunk - 1) / chunk) * kLdHeads * (cpad + 2) * (int64_t)sizeof(float);
 }
 
 namespace tkv {
-template <int NT>
-static int launch_latent_decode(const LatentDecode& p, dim3 grid, cudaStream_t st) {
-  constexpr int kBytes = LatentTile<NT>::kBytes;
+template <int NT, int HG>
+static int launch_latent_decode(const LatentDecode& p, int chunks, cudaStream_t st) {
+  constexpr int kBytes = LatentTile<NT, HG>::kBytes;
+  const dim3 grid(chunks * ((p.groups + HG - 1) / HG), p.batch);
   static_assert(kBytes <= 232448, "shared memory of the kernel");
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kBytes);
+    cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<NT, HG>, cudaFuncAttributeMaxDynamicSharedMemorySize, kBytes);
     if (e != cudaSuccess) return fail(TKV_ERR_LAUNCH, "tkv_latent_decode: %s", cudaGetErrorString(e));
     configured = true;
   }
-  cudaError_t e = launch_pdl(latent_decode_kernel<NT>, grid, dim3(kLdThreads), (size_t)kBytes, st, p);
-  if (e == cudaSuccess) e = launch_pdl(latent_merge_kernel, dim3((unsigned)(p.batch * p.heads)), dim3(kLpThreads), 0, st, p, (int)grid.x / p.groups);
+  cudaError_t e = launch_pdl(latent_decode_kernel<NT, HG>, grid, dim3(kLdThreads * HG), (size_t)kBytes, st, p);
+  if (e == cudaSuccess) e = launch_pdl(latent_merge_kernel, dim3((unsigned)(p.batch * p.heads)), dim3(kLpThreads), 0, st, p, chunks);
   if (e != cudaSuccess) return fail(TKV_ERR_LAUNCH, "tkv_latent_decode: %s", cudaGetErrorString(e));
   return check_launch("tkv_latent_decode");
 }
-static int launch_latent_decode_nt(const LatentDecode& p, dim3 grid, cudaStream_t st) {
+template <int HG>
+static int launch_latent_decode_nt(const LatentDecode& p, int chunks, cudaStream_t st) {
   switch (p.cpad / 64) {
-    case 1: return launch_latent_decode<1>(p, grid, st);
-    case 2: return launch_latent_decode<2>(p, grid, st);
-    case 3: return launch_latent_decode<3>(p, grid, st);
-    case 4: return launch_latent_decode<4>(p, grid, st);
-    case 5: return launch_latent_decode<5>(p, grid, st);
-    case 6: return launch_latent_decode<6>(p, grid, st);
-    case 7: return launch_latent_decode<7>(p, grid, st);
-    default: return launch_latent_decode<8>(p, grid, st);
+    case 1: return launch_latent_decode<1, HG>(p, chunks, st);
+    case 2: return launch_latent_decode<2, HG>(p, chunks, st);
+    case 3: return launch_latent_decode<3, HG>(p, chunks, st);
+    case 4: return launch_latent_decode<4, HG>(p, chunks, st);
+    case 5: return launch_latent_decode<5, HG>(p, chunks, st);
+    case 6: return launch_latent_decode<6, HG>(p, chunks, st);
+    case 7: return launch_latent_decode<7, HG>(p, chunks, st);
+    default: return launch_latent_decode<8, HG>(p, chunks, st);
   }
 }
 }  // namespace tkv
@@ -592,10 +604,10 @@ extern "C" int tkv_latent_decode(const void* q_abs, int64_t qa_token, int64_t qa
   if (batch > 65535) return fail(TKV_ERR_UNSUPPORTED, "tkv_latent_decode: batch=%d", batch);
   const int groups = (heads + kLdHeads - 1) / kLdHeads;
   LatentDecode p = {q_abs, qa_token, qa_head, q_rot, qr_token, qr_head, (const float2*)freq_hi_lo, rot_dim, rot_dims, ring, ring_rows, kv_rank,
-                    cpad, lw, slots, pos0, scale * 1.4426950408889634f, batch, heads, groups, latent_chunk((int64_t)batch * groups, ring_rows),
+                    cpad, lw, slots, pos0, scale * 1.4426950408889634f, batch, heads, groups, latent_chunk(batch, groups, ring_rows),
                     nullptr, nullptr, out, out_token, out_head};
   const int chunks = (ring_rows + p.chunk - 1) / p.chunk;
   p.part_o = (float*)workspace;
   p.part_ml = p.part_o + (int64_t)batch * groups * chunks * kLdHeads * cpad;
-  return launch_latent_decode_nt(p, dim3(chunks * groups, batch), (cudaStream_t)stream);
+  return groups > 1 ? launch_latent_decode_nt<2>(p, chunks, (cudaStream_t)stream) : launch_latent_decode_nt<1>(p, chunks, (cudaStream_t)stream);
 }
