@@ -13,7 +13,8 @@
 // A-operand layout of the read-out.  Per chunk: gates and scaled vectors of all channels (a thread walks two channels of eight
 // tokens), the 16 x 16 blocks of a, then every warp its own columns without further barriers.
 // Where (request, head, column) blocks alone do not fill the GPU, the sequence is cut into segments: a first pass computes
-// every segment's own state, a small kernel chains them, and the main pass starts each segment from its true state.
+// every segment's own state (with the products of the gates AFTER a token, which need no quotient and hold for all gates), a
+// small kernel chains them, and the main pass starts each segment from its true state.
 #include <type_traits>
 #include "tkv_chanrec.cuh"
 #include "tkv_tc.cuh"
@@ -36,6 +37,10 @@ __device__ __forceinline__ void cr_ldm(uint32_t* r, const __nv_bfloat16* p) {
 __device__ __forceinline__ void cr_ldmt(uint32_t* r, const __nv_bfloat16* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)) : "memory");
+}
+__device__ __forceinline__ void cr_stmt(__nv_bfloat16* p, const uint32_t* r) {
+  asm volatile("stmatrix.sync.aligned.m8n8.x4.trans.shared.b16 [%0], {%1,%2,%3,%4};"
+               ::"r"(smem_u32(p)), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]) : "memory");
 }
 __device__ __forceinline__ void cr_cp16(void* dst, const void* src, bool live) {
   const int bytes = live ? 16 : 0;                        // 0: the 16 bytes are zero-filled
@@ -95,6 +100,13 @@ __device__ __forceinline__ void cr_gate(float2 y, float2 lo, float2 rest, float2
   *inv = mul2(den, mul2(den, t));
   *k = mul2(mul2(rest, e), u);
 }
+// The same without 1 / f.
+__device__ __forceinline__ void cr_gate(float2 y, float2 lo, float2 rest, float2* f, float2* k) {
+  const float2 e = make_float2(exp2_weight(fminf(y.x, 60.0f)), exp2_weight(fminf(y.y, 60.0f)));
+  const float2 den = add2(e, pair(1.0f)), t = make_float2(cr_rcp(den.x), cr_rcp(den.y));
+  *f = mul2(fma2(lo, den, rest), t);
+  *k = mul2(mul2(rest, e), t);
+}
 __device__ __forceinline__ float cr_silu(float z) { return z * cr_rcp(1.0f + exp2_weight(z * -1.4426950408889634f)); }
 __device__ __forceinline__ float2 cr_silu2(float2 z) {
   const float2 y = mul2(z, pair(kMinusLog2e));
@@ -137,19 +149,27 @@ __global__ void __launch_bounds__(kWarps * 32, NP == 256 ? 1 : kWarps == 8 ? 2 :
   const __nv_bfloat16* V = (const __nv_bfloat16*)a.v + (int64_t)tok0 * a.row_stride + (int64_t)h * a.p + pbase;
   const float *bias = a.f_bias + (int64_t)h * a.n, *lower = a.lower + (int64_t)h * a.n;
 
+  // This thread's pieces of a chunk: rows fr0 + i * (kThreads / pieces of a row), one column.
+  constexpr int kQPieces = NP / 8, kVPieces = PT / 8, kQStep = kThreads / kQPieces, kVStep = kThreads / kVPieces;
+  const int qr = tid / kQPieces, qc = (tid - qr * kQPieces) * 8, vr = tid / kVPieces, vc = (tid - vr * kVPieces) * 8;
+  const bool q_in = qc < a.n, v_in = pbase + vc < a.p;
   auto fetch = [&](int chunk) {
     const int st = chunk & 1, t0 = chunk * kCrTokens;
-    for (int i = tid; i < kCrTokens * (NP / 8); i += kThreads) {
-      const int r = i / (NP / 8), c = (i - r * (NP / 8)) * 8;
-      const bool live = t0 + r < ntok && c < a.n;
-      const int64_t at = live ? (int64_t)(t0 + r) * a.row_stride + c : 0;
-      if (!kStateOnly) cr_cp16(&sm.zq[st][r * QS + c], Q + at, live);
-      cr_cp16(&sm.zf[st][r * QS + c], F + at, live);
+    const int64_t at = (int64_t)(t0 + qr) * a.row_stride + qc;
+#pragma unroll
+    for (int i = 0; i < kCrTokens / kQStep; ++i) {
+      const int r = qr + i * kQStep;
+      const bool live = q_in && t0 + r < ntok;
+      const int64_t from = live ? at + (int64_t)(i * kQStep) * a.row_stride : 0;
+      if (!kStateOnly) cr_cp16(&sm.zq[st][r * QS + qc], Q + from, live);
+      cr_cp16(&sm.zf[st][r * QS + qc], F + from, live);
     }
-    for (int i = tid; i < kCrTokens * (PT / 8); i += kThreads) {
-      const int r = i / (PT / 8), c = (i - r * (PT / 8)) * 8;
-      const bool live = t0 + r < ntok && pbase + c < a.p;
-      cr_cp16(&sm.v[st][r * VS + c], V + (live ? (int64_t)(t0 + r) * a.row_stride + c : 0), live);
+    const __nv_bfloat16* from_v = V + (int64_t)(t0 + vr) * a.row_stride + vc;
+#pragma unroll
+    for (int i = 0; i < kCrTokens / kVStep; ++i) {
+      const int r = vr + i * kVStep;
+      const bool live = v_in && t0 + r < ntok;
+      cr_cp16(&sm.v[st][r * VS + vc], live ? from_v + (int64_t)(i * kVStep) * a.row_stride : V, live);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -174,6 +194,28 @@ __global__ void __launch_bounds__(kWarps * 32, NP == 256 ? 1 : kWarps == 8 ? 2 :
 #pragma unroll
   for (int i = 0; i < kOwn; ++i) seg_decay[i] = 1.0f;
 
+  // S += V^T k of 16 tokens, both parts of k
+  auto add_keys = [&](const uint32_t* vf, int first) {
+    const int krow = (first + ((lane >> 3) & 1) * 8 + (lane & 7)) * QS + ((lane >> 4) & 1) * 8;
+#pragma unroll
+    for (int n = 0; n < NP / 16; ++n) {
+      uint32_t bf[4];
+      cr_ldmt(bf, sm.k_hi + krow + n * 16);
+      cr_mma(s[2 * n], vf, bf[0], bf[1]);
+      cr_mma(s[2 * n + 1], vf, bf[2], bf[3]);
+      cr_ldmt(bf, sm.k_lo + krow + n * 16);
+      cr_mma(s[2 * n], vf, bf[0], bf[1]);
+      cr_mma(s[2 * n + 1], vf, bf[2], bf[3]);
+    }
+  };
+  auto rescale = [&](const float* by) {
+#pragma unroll
+    for (int nt = 0; nt < NP / 8; ++nt) {
+      const float2 d = *reinterpret_cast<const float2*>(by + nt * 8 + 2 * gc);
+      const float2 x = mul2(make_float2(s[nt][0], s[nt][1]), d), y = mul2(make_float2(s[nt][2], s[nt][3]), d);
+      s[nt][0] = x.x; s[nt][1] = x.y; s[nt][2] = y.x; s[nt][3] = y.y;
+    }
+  };
   if (tid < 2) sm.level[tid] = 0;
   fetch(c0);
   for (int chunk = c0; chunk < c1; ++chunk) {
@@ -198,22 +240,67 @@ __global__ void __launch_bounds__(kWarps * 32, NP == 256 ? 1 : kWarps == 8 ? 2 :
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
           const uint32_t z = *reinterpret_cast<const uint32_t*>(&sm.zf[st][(r0 + j) * QS + c]);
+          const float2 y = fma2(make_float2(__uint_as_float(z << 16), __uint_as_float(z & 0xffff0000u)), pair(kMinusLog2e), bi);
           float2 f, fi, k;
-          cr_gate(fma2(make_float2(__uint_as_float(z << 16), __uint_as_float(z & 0xffff0000u)), pair(kMinusLog2e), bi), lo, rest, &f, &fi, &k);
+          if (kStateOnly) cr_gate(y, lo, rest, &f, &k);
+          else cr_gate(y, lo, rest, &f, &fi, &k);
           if (j >= live) { f = pair(1.0f); fi = f; k = pair(0.0f); }
-          P[rd][j] = j > 0 ? mul2(P[rd][j - 1], f) : f;
-          inv = mul2(inv, fi);
-          kp[rd][j] = mul2(k, inv);
+          if (kStateOnly) {
+            P[rd][j] = f;
+            kp[rd][j] = k;
+            inv = mul2(inv, f);
+          } else {
+            P[rd][j] = j > 0 ? mul2(P[rd][j - 1], f) : f;
+            inv = mul2(inv, fi);
+            kp[rd][j] = mul2(k, inv);
+          }
         }
       };
       if (t0 + kCrTokens <= ntok) walk8(8);
       else walk8(ntok - t0 - r0);
-      *reinterpret_cast<float2*>(&sm.oct[0][oct][c]) = P[rd][7];
-      *reinterpret_cast<float2*>(&sm.oct[1][oct][c]) = inv;
-      if (!(P[rd][7].x >= kWide && P[rd][7].y >= kWide))   // not a number counts as below
-        atomicMax(&sm.level[st], P[rd][7].x >= kNarrow && P[rd][7].y >= kNarrow ? 1 : 2);
+      if (kStateOnly) {
+        *reinterpret_cast<float2*>(&sm.oct[0][oct][c]) = inv;
+      } else {
+        *reinterpret_cast<float2*>(&sm.oct[0][oct][c]) = P[rd][7];
+        *reinterpret_cast<float2*>(&sm.oct[1][oct][c]) = inv;
+        if (!(P[rd][7].x >= kWide && P[rd][7].y >= kWide)) // not a number counts as below
+          atomicMax(&sm.level[st], P[rd][7].x >= kNarrow && P[rd][7].y >= kNarrow ? 1 : 2);
+      }
     }
     __syncthreads();
+    if constexpr (kStateOnly) {
+      // ---- k_j times the gates after it; the state moves on by the whole chunk
+#pragma unroll
+      for (int rd = 0; rd < kRounds; ++rd) {
+        const int c = rd * kWarps * 16 + (warp >> 2) * 64 + 2 * lane;
+        if (c >= NP) continue;
+        float2 after = pair(1.0f);
+        for (int q = oct + 1; q < 4; ++q) after = mul2(after, *reinterpret_cast<const float2*>(&sm.oct[0][q][c]));
+#pragma unroll
+        for (int j = 7; j >= 0; --j) {
+          uint32_t hi, lo_;
+          cr_split(mul2(kp[rd][j], after), &hi, &lo_);
+          *reinterpret_cast<uint32_t*>(&sm.k_hi[(r0 + j) * QS + c]) = hi;
+          *reinterpret_cast<uint32_t*>(&sm.k_lo[(r0 + j) * QS + c]) = lo_;
+          after = mul2(after, P[rd][j]);
+        }
+        if (oct == 0) *reinterpret_cast<float2*>(&sm.end[0][c]) = after;
+      }
+      __syncthreads();
+#pragma unroll
+      for (int i = 0; i < kOwn; ++i) {
+        const int c = tid + i * kThreads;
+        if (c < NP) seg_decay[i] *= sm.end[0][c];
+      }
+      rescale(sm.end[0]);
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        uint32_t vf[4];
+        cr_ldmt(vf, sm.v[st] + (i * 16 + ((lane >> 4) & 1) * 8 + (lane & 7)) * VS + p0 + ((lane >> 3) & 1) * 8);
+        add_keys(vf, i * 16);
+      }
+      continue;
+    }
     const int level = sm.level[st];
     if (tid == 0) sm.level[st ^ 1] = 0;
     if (level < 2) {
@@ -234,21 +321,12 @@ __global__ void __launch_bounds__(kWarps * 32, NP == 256 ? 1 : kWarps == 8 ? 2 :
           cr_split(mul2(kp[rd][j], i0), &hi, &lo_);
           *reinterpret_cast<uint32_t*>(&sm.k_hi[at]) = hi;
           *reinterpret_cast<uint32_t*>(&sm.k_lo[at]) = lo_;
-          if (!kStateOnly) {
-            const uint32_t z = *reinterpret_cast<const uint32_t*>(&sm.zq[st][at]);
-            const float2 x = mul2(cr_silu2(make_float2(__uint_as_float(z << 16), __uint_as_float(z & 0xffff0000u))), mul2(P[rd][j], p0));
-            *reinterpret_cast<__nv_bfloat162*>(&sm.q[at]) = __floats2bfloat162_rn(x.x, x.y);
-          }
+          const uint32_t z = *reinterpret_cast<const uint32_t*>(&sm.zq[st][at]);
+          const float2 x = mul2(cr_silu2(make_float2(__uint_as_float(z << 16), __uint_as_float(z & 0xffff0000u))), mul2(P[rd][j], p0));
+          *reinterpret_cast<__nv_bfloat162*>(&sm.q[at]) = __floats2bfloat162_rn(x.x, x.y);
         }
       }
       __syncthreads();
-    }
-    if (kStateOnly && level < 2) {
-#pragma unroll
-      for (int i = 0; i < kOwn; ++i) {
-        const int c = tid + i * kThreads;
-        if (c < NP) seg_decay[i] *= level == 0 ? sm.end[0][c] : sm.end[0][c] * sm.end[1][c];
-      }
     }
     __nv_bfloat16* v_s = sm.v[st];
     // ---- kTiles groups of 16 tokens from token `first` on, as one block
@@ -258,97 +336,81 @@ __global__ void __launch_bounds__(kWarps * 32, NP == 256 ? 1 : kWarps == 8 ? 2 :
 #pragma unroll
       for (int i = 0; i < kTiles; ++i)
         cr_ldmt(vf[i], v_s + (first + i * 16 + ((lane >> 4) & 1) * 8 + (lane & 7)) * VS + p0 + ((lane >> 3) & 1) * 8);
-      if (!kStateOnly) {
-        float o[2 * kTiles][4] = {};
-        const int qrow = (first + ((lane >> 4) & 1) * 8 + (lane & 7)) * QS + ((lane >> 3) & 1) * 8;
+      float o[2 * kTiles][4] = {};
+      const int qrow = (first + ((lane >> 4) & 1) * 8 + (lane & 7)) * QS + ((lane >> 3) & 1) * 8;
 #pragma unroll
-        for (int kk = 0; kk < NP / 16; ++kk) {
-          uint32_t hi[4], lo[4];
-          cr_split(make_float2(s[2 * kk][0], s[2 * kk][1]), &hi[0], &lo[0]);
-          cr_split(make_float2(s[2 * kk][2], s[2 * kk][3]), &hi[1], &lo[1]);
-          cr_split(make_float2(s[2 * kk + 1][0], s[2 * kk + 1][1]), &hi[2], &lo[2]);
-          cr_split(make_float2(s[2 * kk + 1][2], s[2 * kk + 1][3]), &hi[3], &lo[3]);
+      for (int kk = 0; kk < NP / 16; ++kk) {
+        uint32_t hi[4], lo[4];
+        cr_split(make_float2(s[2 * kk][0], s[2 * kk][1]), &hi[0], &lo[0]);
+        cr_split(make_float2(s[2 * kk][2], s[2 * kk][3]), &hi[1], &lo[1]);
+        cr_split(make_float2(s[2 * kk + 1][0], s[2 * kk + 1][1]), &hi[2], &lo[2]);
+        cr_split(make_float2(s[2 * kk + 1][2], s[2 * kk + 1][3]), &hi[3], &lo[3]);
 #pragma unroll
-          for (int i = 0; i < kTiles; ++i) {
-            uint32_t bf[4];
-            cr_ldm(bf, sm.q + qrow + i * 16 * QS + kk * 16);
-            cr_mma(o[2 * i], hi, bf[0], bf[1]);
-            cr_mma(o[2 * i + 1], hi, bf[2], bf[3]);
-            cr_mma(o[2 * i], lo, bf[0], bf[1]);
-            cr_mma(o[2 * i + 1], lo, bf[2], bf[3]);
-          }
+        for (int i = 0; i < kTiles; ++i) {
+          uint32_t bf[4];
+          cr_ldm(bf, sm.q + qrow + i * 16 * QS + kk * 16);
+          cr_mma(o[2 * i], hi, bf[0], bf[1]);
+          cr_mma(o[2 * i + 1], hi, bf[2], bf[3]);
+          cr_mma(o[2 * i], lo, bf[0], bf[1]);
+          cr_mma(o[2 * i + 1], lo, bf[2], bf[3]);
         }
-#pragma unroll
-        for (int i = 0; i < kTiles; ++i)
-#pragma unroll
-          for (int j = 0; j <= i; ++j) {
-            uint32_t bf[4];
-            const int at = (first + i * 16 + ((lane >> 4) & 1) * 8 + (lane & 7)) * PS + first + j * 16 + ((lane >> 3) & 1) * 8;
-            cr_ldm(bf, sm.a_hi + at);
-            cr_mma(o[2 * i], vf[j], bf[0], bf[1]);
-            cr_mma(o[2 * i + 1], vf[j], bf[2], bf[3]);
-            cr_ldm(bf, sm.a_lo + at);
-            cr_mma(o[2 * i], vf[j], bf[0], bf[1]);
-            cr_mma(o[2 * i + 1], vf[j], bf[2], bf[3]);
-          }
-        __syncwarp();
-        // over this warp's own columns of the V tile (nobody else reads them)
-#pragma unroll
-        for (int i = 0; i < 2 * kTiles; ++i)
-#pragma unroll
-          for (int e = 0; e < 4; ++e)
-            v_s[(first + i * 8 + 2 * gc + (e & 1)) * VS + p0 + gr + (e >> 1) * 8] = __float2bfloat16_rn(o[i][e]);
       }
-      // ---- state
+#pragma unroll
+      for (int i = 0; i < kTiles; ++i)
+#pragma unroll
+        for (int j = 0; j <= i; ++j) {
+          uint32_t bf[4];
+          const int at = (first + i * 16 + ((lane >> 4) & 1) * 8 + (lane & 7)) * PS + first + j * 16 + ((lane >> 3) & 1) * 8;
+          cr_ldm(bf, sm.a_hi + at);
+          cr_mma(o[2 * i], vf[j], bf[0], bf[1]);
+          cr_mma(o[2 * i + 1], vf[j], bf[2], bf[3]);
+          cr_ldm(bf, sm.a_lo + at);
+          cr_mma(o[2 * i], vf[j], bf[0], bf[1]);
+          cr_mma(o[2 * i + 1], vf[j], bf[2], bf[3]);
+        }
+      __syncwarp();
+      // over this warp's own columns of the V tile (nobody else reads them), 16 tokens x 16 columns at a time
 #pragma unroll
       for (int i = 0; i < kTiles; ++i) {
-        const int krow = (first + i * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * QS + ((lane >> 4) & 1) * 8;
+        uint32_t w[4];
 #pragma unroll
-        for (int n = 0; n < NP / 16; ++n) {
-          uint32_t bf[4];
-          cr_ldmt(bf, sm.k_hi + krow + n * 16);
-          cr_mma(s[2 * n], vf[i], bf[0], bf[1]);
-          cr_mma(s[2 * n + 1], vf[i], bf[2], bf[3]);
-          cr_ldmt(bf, sm.k_lo + krow + n * 16);
-          cr_mma(s[2 * n], vf[i], bf[0], bf[1]);
-          cr_mma(s[2 * n + 1], vf[i], bf[2], bf[3]);
+        for (int e = 0; e < 4; ++e) {
+          const __nv_bfloat162 x = __floats2bfloat162_rn(o[2 * i + (e >> 1)][2 * (e & 1)], o[2 * i + (e >> 1)][2 * (e & 1) + 1]);
+          w[e] = *reinterpret_cast<const uint32_t*>(&x);
         }
+        // fragments: tokens 0 .. 7 of columns 0 .. 7 and 8 .. 15, then tokens 8 .. 15
+        cr_stmt(v_s + (first + i * 16 + ((lane >> 4) & 1) * 8 + (lane & 7)) * VS + p0 + ((lane >> 3) & 1) * 8, w);
       }
 #pragma unroll
-      for (int nt = 0; nt < NP / 8; ++nt) {
-        const float2 d = *reinterpret_cast<const float2*>(end + nt * 8 + 2 * gc);
-        const float2 x = mul2(make_float2(s[nt][0], s[nt][1]), d), y = mul2(make_float2(s[nt][2], s[nt][3]), d);
-        s[nt][0] = x.x; s[nt][1] = x.y; s[nt][2] = y.x; s[nt][3] = y.y;
-      }
+      for (int i = 0; i < kTiles; ++i) add_keys(vf[i], first + i * 16);
+      rescale(end);
     };
     if (level < 2) {
-      if (!kStateOnly) {
-        // ---- the blocks a: a task is 16 tokens against 8; the last two cross the middle (one block of 32 only)
-        for (int task = warp; task < (level == 0 ? 6 : 4); task += kWarps) {
-          const int ib = task < 4 ? task >> 1 : 1, jb = task < 4 ? ib : 0, j0 = jb * 16 + (task & 1) * 8;
-          float sc[2][4] = {};
+      // ---- the blocks a: a task is 16 tokens against 8; the last two cross the middle (one block of 32 only)
+      for (int task = warp; task < (level == 0 ? 6 : 4); task += kWarps) {
+        const int ib = task < 4 ? task >> 1 : 1, jb = task < 4 ? ib : 0, j0 = jb * 16 + (task & 1) * 8;
+        float sc[2][4] = {};
 #pragma unroll 4
-          for (int kk = 0; kk < NP / 16; ++kk) {
-            uint32_t aq[4];
-            cr_ldm(aq, sm.q + (ib * 16 + (lane & 15)) * QS + kk * 16 + (lane >> 4) * 8);
-            const int at = (j0 + gr) * QS + kk * 16 + 2 * gc;
-            const uint32_t* kh = reinterpret_cast<const uint32_t*>(sm.k_hi + at);
-            const uint32_t* kl = reinterpret_cast<const uint32_t*>(sm.k_lo + at);
-            cr_mma(sc[0], aq, kh[0], kh[4]);
-            cr_mma(sc[1], aq, kl[0], kl[4]);
-          }
-          const int j = j0 + 2 * gc;
-#pragma unroll
-          for (int e = 0; e < 4; e += 2) {
-            const int i = ib * 16 + gr + (e >> 1) * 8;
-            uint32_t hi, lo;
-            cr_split(make_float2(j <= i ? sc[0][e] + sc[1][e] : 0.f, j + 1 <= i ? sc[0][e + 1] + sc[1][e + 1] : 0.f), &hi, &lo);
-            *reinterpret_cast<uint32_t*>(sm.a_hi + i * PS + j) = hi;
-            *reinterpret_cast<uint32_t*>(sm.a_lo + i * PS + j) = lo;
-          }
+        for (int kk = 0; kk < NP / 16; ++kk) {
+          uint32_t aq[4];
+          cr_ldm(aq, sm.q + (ib * 16 + (lane & 15)) * QS + kk * 16 + (lane >> 4) * 8);
+          const int at = (j0 + gr) * QS + kk * 16 + 2 * gc;
+          const uint32_t* kh = reinterpret_cast<const uint32_t*>(sm.k_hi + at);
+          const uint32_t* kl = reinterpret_cast<const uint32_t*>(sm.k_lo + at);
+          cr_mma(sc[0], aq, kh[0], kh[4]);
+          cr_mma(sc[1], aq, kl[0], kl[4]);
         }
-        __syncthreads();
+        const int j = j0 + 2 * gc;
+#pragma unroll
+        for (int e = 0; e < 4; e += 2) {
+          const int i = ib * 16 + gr + (e >> 1) * 8;
+          uint32_t hi, lo;
+          cr_split(make_float2(j <= i ? sc[0][e] + sc[1][e] : 0.f, j + 1 <= i ? sc[0][e + 1] + sc[1][e + 1] : 0.f), &hi, &lo);
+          *reinterpret_cast<uint32_t*>(sm.a_hi + i * PS + j) = hi;
+          *reinterpret_cast<uint32_t*>(sm.a_lo + i * PS + j) = lo;
+        }
       }
+      __syncthreads();
       if (level == 0) {
         block(std::integral_constant<int, 2>{}, 0, sm.end[0]);
       } else {
@@ -370,8 +432,7 @@ __global__ void __launch_bounds__(kWarps * 32, NP == 256 ? 1 : kWarps == 8 ? 2 :
           const float lo = ch ? lower[c] : 1.0f;
           g[1][c] = fmaf(1.0f - lo, pos, lo);
           g[2][c] = (1.0f - lo) * neg;
-          if (kStateOnly) seg_decay[i] *= g[1][c];
-          else g[0][c] = cr_silu(__bfloat162float(sm.zq[st][r * QS + c]));
+          g[0][c] = cr_silu(__bfloat162float(sm.zq[st][r * QS + c]));
         }
         __syncthreads();                                   // two buffers: one barrier per token
         const float v0 = __bfloat162float(v_s[r * VS + p0 + gr]), v1 = __bfloat162float(v_s[r * VS + p0 + gr + 8]);
@@ -384,30 +445,27 @@ __global__ void __launch_bounds__(kWarps * 32, NP == 256 ? 1 : kWarps == 8 ? 2 :
             const float f = g[1][n], k = g[2][n];
             s[nt][e] = fmaf(f, s[nt][e], k * v0);
             s[nt][2 + e] = fmaf(f, s[nt][2 + e], k * v1);
-            if (!kStateOnly) { o0 = fmaf(g[0][n], s[nt][e], o0); o1 = fmaf(g[0][n], s[nt][2 + e], o1); }
+            o0 = fmaf(g[0][n], s[nt][e], o0);
+            o1 = fmaf(g[0][n], s[nt][2 + e], o1);
           }
-        if (!kStateOnly) {
 #pragma unroll
-          for (int d = 1; d <= 2; d <<= 1) {
-            o0 += __shfl_xor_sync(0xffffffffu, o0, d);
-            o1 += __shfl_xor_sync(0xffffffffu, o1, d);
-          }
-          __syncwarp();
-          if (gc == 0) {
-            v_s[r * VS + p0 + gr] = __float2bfloat16_rn(o0);
-            v_s[r * VS + p0 + gr + 8] = __float2bfloat16_rn(o1);
-          }
+        for (int d = 1; d <= 2; d <<= 1) {
+          o0 += __shfl_xor_sync(0xffffffffu, o0, d);
+          o1 += __shfl_xor_sync(0xffffffffu, o1, d);
+        }
+        __syncwarp();
+        if (gc == 0) {
+          v_s[r * VS + p0 + gr] = __float2bfloat16_rn(o0);
+          v_s[r * VS + p0 + gr + 8] = __float2bfloat16_rn(o1);
         }
       }
     }
-    if (!kStateOnly) {
-      __syncwarp();
+    __syncwarp();
 #pragma unroll
-      for (int i = 0; i < kCrTokens / 16; ++i) {
-        const int r = i * 16 + (lane >> 1), col = p0 + (lane & 1) * 8;
-        if (t0 + r < ntok && pbase + col < a.p)
-          st16((__nv_bfloat16*)a.out + ((int64_t)(tok0 + t0 + r) * a.heads + h) * a.p + pbase + col, ld16(v_s + r * VS + col));
-      }
+    for (int i = 0; i < kCrTokens / 16; ++i) {
+      const int r = i * 16 + (lane >> 1), col = p0 + (lane & 1) * 8;
+      if (t0 + r < ntok && pbase + col < a.p)
+        st16((__nv_bfloat16*)a.out + ((int64_t)(tok0 + t0 + r) * a.heads + h) * a.p + pbase + col, ld16(v_s + r * VS + col));
     }
   }
   float* dst = kStateOnly ? sg.start + ((int64_t)bh * sg.count + seg) * np : (c1 == nchunks ? final_state : nullptr);
@@ -473,7 +531,7 @@ static ChanrecSegs plan_chanrec(int batch, int max_tokens, int heads, int n, int
   double best = 0;
   for (int k = 1; k <= chunks / 8 + 1 && ctas * (k - 1) < 2 * room; ++k) {
     if (k > 1 && chunks / k < 8) break;
-    const double cost = (double)((ctas * k + room - 1) / room) / k * (k > 1 ? 1.0 + 0.5 * (k - 1) / k : 1.0) + 0.005 * k;
+    const double cost = (double)((ctas * k + room - 1) / room) / k * (k > 1 ? 1.0 + 0.5 * (k - 1) / k : 1.0) + 0.003 * k;
     if (k == 1 || cost < best) { best = cost; segs = k; }
   }
   ChanrecSegs s = {};
