@@ -559,7 +559,8 @@ int tkv_diff_prefill(const void* q, const void* k_lin, const void* v_lin, const 
  * with f_bias, lower [heads * n] and state [slots, heads, n, vdim] fp32, read and written.
  * tkv_chanrec_step: one token per request, writes RMS(o) * norm_w [vdim] per head.  tkv_chanrec_scan: token by token, every size
  * (n <= 1400) and dtype, writes o; cu_tokens may be NULL.  tkv_chanrec_chunk: the tensor-core form for prompts, writes o: bf16,
- * n <= 256, n, vdim and row_stride multiples of 8, 16-byte aligned rows.  Its workspace (tkv_chanrec_chunk_workspace_bytes; -1 =
+ * n <= 256, n, vdim and row_stride multiples of 8, 16-byte aligned rows (64 < n <= 128, vdim > 64 and prompts of at least 64
+ * tokens: tcgen05; else mma.sync).  Its workspace (tkv_chanrec_chunk_workspace_bytes; -1 =
  * shape not supported, 0 = none) holds the states between the segments of long sequences. */
 int tkv_chanrec_step(const void* q, const void* f, const void* v, int64_t row_stride, const float* f_bias, const float* lower,
                      const float* norm_w, float eps, void* out, float* state, const int32_t* slots, const int32_t* pos0, int batch,
@@ -571,7 +572,8 @@ int tkv_chanrec_scan(const void* q, const void* f, const void* v, int64_t row_st
 int64_t tkv_chanrec_chunk_workspace_bytes(int batch, int max_tokens, int heads, int n, int vdim, int dtype);
 int tkv_chanrec_chunk(const void* q, const void* f, const void* v, int64_t row_stride, const float* f_bias, const float* lower,
                       void* out, float* state, const int32_t* slots, const int32_t* cu_tokens, const int32_t* pos0, void* workspace,
-                      int64_t workspace_bytes, int batch, int max_tokens, int heads, int n, int vdim, int dtype, tkv_stream_t stream);
+                      int64_t workspace_bytes, int batch, int max_tokens, int heads, int n, int vdim, int dtype, int32_t* status,
+                      tkv_stream_t stream);
 
 /* Rotary positions in place on elements offset .. offset + rot_dims of every head of head_len elements: the pair (2i, 2i + 1)
  * turns by position * f_i, freq_hi_lo[i] = {f_i rounded to fp32, the rest}. */

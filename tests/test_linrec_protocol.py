@@ -66,7 +66,8 @@ class Sim:
             for r in reads:
                 self.busy[r] -= 1
             self.buf[out] = chunk
-        self.bar[bar].arrive()
+        if bar is not None:
+            self.bar[bar].arrive()
 
     # ---- roles
     def load_qk(self, i):
@@ -159,8 +160,11 @@ class Sim:
         yield from self.wait("st", self.n - 1)
         self.read("ST", self.n - 1)
 
+    def agents(self):
+        return [self.control(), self.scan(), self.rows(), self.rows()]
+
     def run(self):
-        agents = [self.control(), self.scan(), self.rows(), self.rows()]
+        agents = self.agents()
         speed = [self.rng.choice([1, 1, 4, 30]) for _ in agents]
         blocked = {}
         while agents:

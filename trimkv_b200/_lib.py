@@ -74,7 +74,7 @@ SIGNATURES = {
     "tkv_chanrec_step": (I, [P, P, P, L, P, P, P, F, P, P, P, P, I, I, I, I, I, P]),
     "tkv_chanrec_scan": (I, [P, P, P, L, P, P, P, P, P, P, P, I, I, I, I, I, P]),
     "tkv_chanrec_chunk_workspace_bytes": (L, [I, I, I, I, I, I]),
-    "tkv_chanrec_chunk": (I, [P, P, P, L, P, P, P, P, P, P, P, P, L, I, I, I, I, I, I, P]),
+    "tkv_chanrec_chunk": (I, [P, P, P, L, P, P, P, P, P, P, P, P, L, I, I, I, I, I, I, P, P]),
     "tkv_rotate_pairs": (I, [P, L, P, P, I, I, I, I, I, I, P, I, P]),
     "tkv_latent_prep": (I, [P, L, P, P, F, I, I, I, I, P, P, P, I, P, P, P, P, P, I, I, I, I, I, P]),
     "tkv_latent_prefill": (I, [P, L, P, L, P, P, L, P, P, F, P, I, I, I, I, I, I, I, I, I, I, P, P]),

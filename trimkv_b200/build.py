@@ -10,7 +10,7 @@ CSRC = os.path.join(HERE, "csrc")
 LIB = os.path.join(HERE, "libtrimkv_b200.so")
 SOURCES = ["tkv_abi.cu", "tkv_append.cu", "tkv_evict.cu", "tkv_attn.cu", "tkv_attn_tc.cu", "tkv_attn_multi.cu", "tkv_attn_prefill.cu", "tkv_gemm_tc.cu", "tkv_fused.cu",
            "tkv_stream.cu", "tkv_linrec.cu", "tkv_linrec_chunk.cu", "tkv_linrec_tc.cu", "tkv_diffattn.cu", "tkv_diffattn_tc.cu",
-           "tkv_chanrec.cu", "tkv_chanrec_chunk.cu", "tkv_latent.cu", "tkv_latent_tc.cu", "tkv_moe.cu", "tkv_moe_tc.cu"]
+           "tkv_chanrec.cu", "tkv_chanrec_chunk.cu", "tkv_chanrec_tc.cu", "tkv_latent.cu", "tkv_latent_tc.cu", "tkv_moe.cu", "tkv_moe_tc.cu"]
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     "-Xcompiler", "-fPIC", "--use_fast_math=false",

@@ -31,4 +31,10 @@ struct ChanrecSegs {
   float* decay;                                       // [batch, heads, count, n]: product of f over the segment
 };
 
+int launch_chanrec_chain(const ChanrecParams& a, const ChanrecSegs& sg, cudaStream_t st);
+// The tcgen05 form (tkv_chanrec_tc.cu): shapes it takes, value columns of a CTA.
+bool chanrec_tc_shape(int n, int p, int max_tokens);
+int chanrec_tc_columns();
+int launch_chanrec_tc(const ChanrecParams& a, const ChanrecSegs& sg, int32_t* status, cudaStream_t st);
+
 }  // namespace tkv

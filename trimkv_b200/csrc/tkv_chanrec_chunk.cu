@@ -16,103 +16,12 @@
 // every segment's own state (with the products of the gates AFTER a token, which need no quotient and hold for all gates), a
 // small kernel chains them, and the main pass starts each segment from its true state.
 #include <type_traits>
-#include "tkv_chanrec.cuh"
-#include "tkv_tc.cuh"
+#include "tkv_chanrec_math.cuh"
 
 namespace tkv {
 
 constexpr int kCrTokens = 32;
 constexpr float kWide = 3e-8f, kNarrow = 1e-15f;          // product of eight gates
-
-__device__ __forceinline__ void cr_mma(float* d, const uint32_t* a, uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void cr_ldm(uint32_t* r, const __nv_bfloat16* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)) : "memory");
-}
-__device__ __forceinline__ void cr_ldmt(uint32_t* r, const __nv_bfloat16* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)) : "memory");
-}
-__device__ __forceinline__ void cr_stmt(__nv_bfloat16* p, const uint32_t* r) {
-  asm volatile("stmatrix.sync.aligned.m8n8.x4.trans.shared.b16 [%0], {%1,%2,%3,%4};"
-               ::"r"(smem_u32(p)), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]) : "memory");
-}
-__device__ __forceinline__ void cr_cp16(void* dst, const void* src, bool live) {
-  const int bytes = live ? 16 : 0;                        // 0: the 16 bytes are zero-filled
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(bytes) : "memory");
-}
-// Two fp32 operations in one instruction.
-__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
-  float2 r;
-  asm("{\n\t.reg .b64 a, b, r;\n\tmov.b64 a, {%2, %3};\n\tmov.b64 b, {%4, %5};\n\tmul.rn.f32x2 r, a, b;\n\tmov.b64 {%0, %1}, r;\n\t}"
-      : "=f"(r.x), "=f"(r.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y));
-  return r;
-}
-__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
-  float2 r;
-  asm("{\n\t.reg .b64 a, b, c, r;\n\tmov.b64 a, {%2, %3};\n\tmov.b64 b, {%4, %5};\n\tmov.b64 c, {%6, %7};\n\tfma.rn.f32x2 r, a, b, c;\n\t"
-      "mov.b64 {%0, %1}, r;\n\t}"
-      : "=f"(r.x), "=f"(r.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y), "f"(c.x), "f"(c.y));
-  return r;
-}
-__device__ __forceinline__ float2 add2(float2 a, float2 b) {
-  float2 r;
-  asm("{\n\t.reg .b64 a, b, r;\n\tmov.b64 a, {%2, %3};\n\tmov.b64 b, {%4, %5};\n\tadd.rn.f32x2 r, a, b;\n\tmov.b64 {%0, %1}, r;\n\t}"
-      : "=f"(r.x), "=f"(r.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y));
-  return r;
-}
-constexpr float kMinusLog2e = -1.4426950408889634f;
-__device__ __forceinline__ float2 pair(float x) { return make_float2(x, x); }
-// x = hi + lo in bf16, two values at a time.
-__device__ __forceinline__ void cr_split(float2 x, uint32_t* hi, uint32_t* lo) {
-  const __nv_bfloat162 h = __floats2bfloat162_rn(x.x, x.y);
-  *hi = *reinterpret_cast<const uint32_t*>(&h);
-  const float2 r = fma2(make_float2(__uint_as_float(*hi << 16), __uint_as_float(*hi & 0xffff0000u)), pair(-1.0f), x);
-  const __nv_bfloat162 l = __floats2bfloat162_rn(r.x, r.y);
-  *lo = *reinterpret_cast<const uint32_t*>(&l);
-}
-// sigmoid(x) and sigmoid(-x), each to a few units in the last place of fp32.
-__device__ __forceinline__ void cr_sigmoid(float x, float* pos, float* neg) {
-  const float e = exp2_weight(fabsf(x) * -1.4426950408889634f), r = __frcp_rn(1.0f + e);
-  const float small = e * r;
-  *pos = x >= 0.f ? r : small;
-  *neg = x >= 0.f ? small : r;
-}
-
-__device__ __forceinline__ float cr_rcp(float x) {
-  float y;
-  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-// f, 1 / f and k = 1 - f of two channels with one reciprocal each, from -x / ln 2 of the gate's argument x: with e = exp(-x),
-// f = (lo (1 + e) + 1 - lo) / (1 + e) and k = (1 - lo) e / (1 + e).  e is held below 2^60 (sigmoid 1e-18), which only gates
-// that send the chunk to the token-by-token path ever reach.
-__device__ __forceinline__ void cr_gate(float2 y, float2 lo, float2 rest, float2* f, float2* inv, float2* k) {
-  const float2 e = make_float2(exp2_weight(fminf(y.x, 60.0f)), exp2_weight(fminf(y.y, 60.0f)));
-  const float2 den = add2(e, pair(1.0f)), num = fma2(lo, den, rest), dn = mul2(den, num);
-  const float2 t = make_float2(cr_rcp(dn.x), cr_rcp(dn.y)), u = mul2(num, t);      // u = 1 / den
-  *f = mul2(num, u);
-  *inv = mul2(den, mul2(den, t));
-  *k = mul2(mul2(rest, e), u);
-}
-// The same without 1 / f.
-__device__ __forceinline__ void cr_gate(float2 y, float2 lo, float2 rest, float2* f, float2* k) {
-  const float2 e = make_float2(exp2_weight(fminf(y.x, 60.0f)), exp2_weight(fminf(y.y, 60.0f)));
-  const float2 den = add2(e, pair(1.0f)), t = make_float2(cr_rcp(den.x), cr_rcp(den.y));
-  *f = mul2(fma2(lo, den, rest), t);
-  *k = mul2(mul2(rest, e), t);
-}
-__device__ __forceinline__ float cr_silu(float z) { return z * cr_rcp(1.0f + exp2_weight(z * -1.4426950408889634f)); }
-__device__ __forceinline__ float2 cr_silu2(float2 z) {
-  const float2 y = mul2(z, pair(kMinusLog2e));
-  const float2 d = add2(make_float2(exp2_weight(y.x), exp2_weight(y.y)), pair(1.0f));
-  return mul2(z, make_float2(cr_rcp(d.x), cr_rcp(d.y)));
-}
 
 template <int NP, int kWarps> struct CrSmem {
   static constexpr int PT = kWarps * 16, QS = NP + 8, VS = PT + 8, PS = kCrTokens + 8;
@@ -517,13 +426,20 @@ __global__ void __launch_bounds__(256) chanrec_chain_kernel(ChanrecParams a, Cha
   }
 }
 
+int launch_chanrec_chain(const ChanrecParams& a, const ChanrecSegs& sg, cudaStream_t st) {
+  cudaError_t e = launch_pdl(chanrec_chain_kernel, dim3((unsigned)(((int64_t)a.n * a.p + 255) / 256), a.batch * a.heads), dim3(256), 0, st, a, sg);
+  if (e != cudaSuccess) return fail(TKV_ERR_LAUNCH, "tkv_chanrec_chunk: %s", cudaGetErrorString(e));
+  return TKV_OK;
+}
+
 static bool chanrec_chunk_shape(int n, int p) { return n % 8 == 0 && p % 8 == 0 && n <= 256; }
 static int chanrec_columns(int n, int p) { return (n <= 128 && p > 64) ? 128 : 64; }
 
 static ChanrecSegs plan_chanrec(int batch, int max_tokens, int heads, int n, int p) {
-  const int pt = chanrec_columns(n, p);
+  const bool tc = chanrec_tc_shape(n, p, max_tokens);
+  const int pt = tc ? chanrec_tc_columns() : chanrec_columns(n, p);
   const int64_t ctas = (int64_t)batch * heads * ((p + pt - 1) / pt);
-  const int64_t room = 148 * (n > 128 ? 1 : 2);            // CTAs that run at the same time
+  const int64_t room = 148 * (tc || n > 128 ? 1 : 2);      // CTAs that run at the same time
   const int chunks = (max_tokens + kCrTokens - 1) / kCrTokens;
   // segments of at least eight chunks: the fewest steps of a CTA, counting the pass over states alone (all segments but one) half,
   // and a little for every segment's state that goes through memory
@@ -556,8 +472,10 @@ static int launch_chanrec(const ChanrecParams& a, const ChanrecSegs& sg, cudaStr
   cudaError_t e = cudaSuccess;
   if (sg.count > 1) {
     e = launch_pdl(chanrec_chunk_kernel<NP, kWarps, true>, dim3((unsigned)grid), dim3(kWarps * 32), (size_t)kBytes, st, a, sg);
-    if (e == cudaSuccess)
-      e = launch_pdl(chanrec_chain_kernel, dim3((unsigned)(((int64_t)a.n * a.p + 255) / 256), a.batch * a.heads), dim3(256), 0, st, a, sg);
+    if (e == cudaSuccess) {
+      int rc = launch_chanrec_chain(a, sg, st);
+      if (rc != TKV_OK) return rc;
+    }
   }
   if (e == cudaSuccess)
     e = launch_pdl(chanrec_chunk_kernel<NP, kWarps, false>, dim3((unsigned)grid), dim3(kWarps * 32), (size_t)kBytes, st, a, sg);
@@ -578,7 +496,7 @@ extern "C" int64_t tkv_chanrec_chunk_workspace_bytes(int batch, int max_tokens, 
 extern "C" int tkv_chanrec_chunk(const void* q, const void* f, const void* v, int64_t row_stride, const float* f_bias,
                                  const float* lower, void* out, float* state, const int32_t* slots, const int32_t* cu_tokens,
                                  const int32_t* pos0, void* workspace, int64_t workspace_bytes, int batch, int max_tokens, int heads,
-                                 int n, int vdim, int dtype, tkv_stream_t stream) {
+                                 int n, int vdim, int dtype, int32_t* status, tkv_stream_t stream) {
   if (!q || !f || !v || !f_bias || !lower || !out || !state || !slots || !cu_tokens || !pos0)
     return fail(TKV_ERR_ARG, "tkv_chanrec_chunk: NULL pointer argument");
   if (batch < 0 || max_tokens < 0 || heads <= 0 || n <= 0 || vdim <= 0 || row_stride < (int64_t)heads * n || row_stride < (int64_t)heads * vdim)
@@ -597,6 +515,7 @@ extern "C" int tkv_chanrec_chunk(const void* q, const void* f, const void* v, in
   s.start = (float*)workspace;
   s.decay = s.start + (s.count > 1 ? (int64_t)batch * heads * s.count * n * vdim : 0);
   cudaStream_t st = (cudaStream_t)stream;
+  if (chanrec_tc_shape(n, vdim, max_tokens)) return launch_chanrec_tc(a, s, status, st);
   const bool wide = chanrec_columns(n, vdim) == 128;
   if (n <= 64) return wide ? launch_chanrec<64, 8>(a, s, st) : launch_chanrec<64, 4>(a, s, st);
   if (n <= 128) return wide ? launch_chanrec<128, 8>(a, s, st) : launch_chanrec<128, 4>(a, s, st);

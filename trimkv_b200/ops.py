@@ -605,7 +605,7 @@ def chanrec(q, f, v, f_bias, lower, state, batch, out, force_scan: bool = False)
         ws = torch.empty(need, dtype=torch.uint8, device=out.device) if need else None
         check(lib().tkv_chanrec_chunk(q.data_ptr(), f.data_ptr(), v.data_ptr(), q.stride(0), f_bias.data_ptr(), lower.data_ptr(),
                                       out.data_ptr(), state.data_ptr(), batch.slots.data_ptr(), batch.cu.data_ptr(), batch.pos0.data_ptr(),
-                                      _ptr(ws), need, batch.size, batch.max_tokens, heads, n, p, dt, _stream(out)), "tkv_chanrec_chunk")
+                                      _ptr(ws), need, batch.size, batch.max_tokens, heads, n, p, dt, _ptr(batch.status), _stream(out)), "tkv_chanrec_chunk")
         _count(3 if need else 1)
         return
     check(lib().tkv_chanrec_scan(q.data_ptr(), f.data_ptr(), v.data_ptr(), q.stride(0), f_bias.data_ptr(), lower.data_ptr(), out.data_ptr(),
