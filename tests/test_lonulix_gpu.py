@@ -101,7 +101,8 @@ def test_rotation_of_neighbours_far_from_the_start(heads, head_len, offset, dims
 def _gates_case(rng, T, heads, n, p, dtype, kind):
     """Projections of q, f, v side by side, bias, lower bound.  ``far``: one early value that one late query asks for, in a
     channel that forgets nothing in between.  ``shut``: gates near zero in some channels and places (decays far below what a
-    product over a block can hold), beside channels that keep everything."""
+    product over a block can hold), beside channels that keep everything.  ``low``: gates around a tenth for a while, which a
+    product over 32 tokens cannot hold and one over 16 can."""
     zq, zf, v = (as_held(rng.standard_normal(s), dtype) for s in ((T, heads, n), (T, heads, n), (T, heads, p)))
     bias, lower = rng.standard_normal((heads, n)) + 1.5, np.clip(rng.uniform(-0.3, 0.9, (heads, n)), 0.0, 1.0)
     if kind == "far":
@@ -117,6 +118,9 @@ def _gates_case(rng, T, heads, n, p, dtype, kind):
         zf[:, :, 1] = 40.0
         zf[T // 3, :, 1] = -6.0
         zf[5:9, :, 2 % n] = -90.0
+    if kind == "low":
+        lower[:, 1::2] = 0.0
+        zf[T // 5:T // 2, :, 1::2] = -2.5 - bias[:, 1::2]
     return zq, as_held(zf, dtype), v, as_held(bias, F32), as_held(lower, F32)
 
 
@@ -141,7 +145,7 @@ def _run_recurrence(c, b, sel, zq, zf, v, bias, lower, dtype, scan=False):
     return out.double().cpu().numpy().reshape(n, heads, p)
 
 
-@pytest.mark.parametrize("kind", ["far", "shut"])
+@pytest.mark.parametrize("kind", ["far", "shut", "low"])
 @pytest.mark.parametrize("dtype,scan", [(F32, True), (BF16, True), (BF16, False)])
 @pytest.mark.parametrize("heads,n,p", [(2, 64, 64), (4, 56, 24), (1, 128, 128), (1, 8, 136), (2, 200, 72), (6, 16, 8), (2, 72, 80)])
 def test_recurrence_ragged_and_in_portions(heads, n, p, dtype, scan, kind):
@@ -171,7 +175,7 @@ def test_recurrence_ragged_and_in_portions(heads, n, p, dtype, scan, kind):
             assert rel_rms(c.arrays(0)["state"][c._rows[r]], S) < 3e-5, (sizes, r)
 
 
-@pytest.mark.parametrize("kind", ["far", "shut"])
+@pytest.mark.parametrize("kind", ["far", "shut", "low"])
 @pytest.mark.parametrize("n,p", [(32, 40), (128, 64), (96, 136), (200, 64)])
 def test_recurrence_cut_into_segments(n, p, kind):
     """Few heads and a long sequence: segments run side by side and start from the chained states."""

@@ -24,11 +24,12 @@ __device__ __forceinline__ void forget_gate(float x, float lower, float* f, floa
   *k = (1.0f - lower) * (x >= 0.f ? small : big);
 }
 
-// A long sequence cut into segments that run side by side (see LinrecSegs), with a decay per state row.
+// A long sequence cut into segments that run side by side (see LinrecSegs), with a decay per state row.  The pass over states
+// alone, which leaves the last segment out, cuts each segment into pieces of its own, so that it too fills the GPU.
 struct ChanrecSegs {
-  int count, tokens;                                  // segments per request, tokens per segment
-  float* start;                                       // [batch, heads, count, n, p]
-  float* decay;                                       // [batch, heads, count, n]: product of f over the segment
+  int count, tokens, pieces;                          // segments per request, tokens per segment, pieces per segment
+  float* start;                                       // [batch, heads, count * pieces, n, p]
+  float* decay;                                       // [batch, heads, count * pieces, n]: product of f over the piece
 };
 
 int launch_chanrec_chain(const ChanrecParams& a, const ChanrecSegs& sg, cudaStream_t st);

@@ -49,9 +49,9 @@ __global__ void __launch_bounds__(kWarps * 32, NP == 256 ? 1 : kWarps == 8 ? 2 :
   const int pt = item % ptiles, bh = item / ptiles, b = bh / a.heads, h = bh - b * a.heads;
   const int tok0 = a.cu[b], ntok = a.cu[b + 1] - tok0;
   const int nchunks = (ntok + kCrTokens - 1) / kCrTokens;
-  const int per = sg.tokens / kCrTokens, c0 = seg * per, c1 = min(nchunks, c0 + per);
+  const int per = (kStateOnly ? sg.tokens / sg.pieces : sg.tokens) / kCrTokens, c0 = seg * per, c1 = min(nchunks, c0 + per);
   if (c0 >= c1) return;
-  if (kStateOnly && c1 == nchunks) return;                // nobody starts from the end of the last segment
+  if (kStateOnly && (seg / sg.pieces + 1) * sg.tokens >= ntok) return;           // nobody starts from the end of the last segment
   const int pbase = pt * PT, p0 = warp * 16;              // this CTA's columns, this warp's columns within them
   const __nv_bfloat16* Q = (const __nv_bfloat16*)a.q + (int64_t)tok0 * a.row_stride + (int64_t)h * a.n;
   const __nv_bfloat16* F = (const __nv_bfloat16*)a.f + (int64_t)tok0 * a.row_stride + (int64_t)h * a.n;
@@ -89,7 +89,7 @@ __global__ void __launch_bounds__(kWarps * 32, NP == 256 ? 1 : kWarps == 8 ? 2 :
   const int64_t np = (int64_t)a.n * a.p;
   float* const final_state = a.state + ((int64_t)a.slots[b] * a.heads + h) * np;
   {
-    const float* S = kStateOnly ? nullptr : sg.count > 1 ? sg.start + ((int64_t)bh * sg.count + seg) * np : a.pos0[b] == 0 ? nullptr : final_state;
+    const float* S = kStateOnly ? nullptr : sg.count > 1 ? sg.start + ((int64_t)bh * sg.count + seg) * sg.pieces * np : a.pos0[b] == 0 ? nullptr : final_state;
 #pragma unroll
     for (int nt = 0; nt < NP / 8; ++nt)
 #pragma unroll
@@ -377,7 +377,7 @@ __global__ void __launch_bounds__(kWarps * 32, NP == 256 ? 1 : kWarps == 8 ? 2 :
         st16((__nv_bfloat16*)a.out + ((int64_t)(tok0 + t0 + r) * a.heads + h) * a.p + pbase + col, ld16(v_s + r * VS + col));
     }
   }
-  float* dst = kStateOnly ? sg.start + ((int64_t)bh * sg.count + seg) * np : (c1 == nchunks ? final_state : nullptr);
+  float* dst = kStateOnly ? sg.start + ((int64_t)bh * sg.count * sg.pieces + seg) * np : (c1 == nchunks ? final_state : nullptr);
   if (dst != nullptr) {
 #pragma unroll
     for (int nt = 0; nt < NP / 8; ++nt)
@@ -391,12 +391,13 @@ __global__ void __launch_bounds__(kWarps * 32, NP == 256 ? 1 : kWarps == 8 ? 2 :
 #pragma unroll
     for (int i = 0; i < kOwn; ++i) {
       const int c = tid + i * kThreads;
-      if (c < a.n) sg.decay[((int64_t)bh * sg.count + seg) * a.n + c] = seg_decay[i];
+      if (c < a.n) sg.decay[((int64_t)bh * sg.count * sg.pieces + seg) * a.n + c] = seg_decay[i];
     }
   }
 }
 
-// start[seg] <- state before the segment.  Thread per state element; on entry start[seg] holds the segment's own state.
+// start[first piece of a segment] <- state before the segment.  Thread per state element; on entry every piece of the segments
+// before the last holds its own state.
 __global__ void __launch_bounds__(256) chanrec_chain_kernel(ChanrecParams a, ChanrecSegs sg) {
   grid_dependency_wait();
   grid_launch_dependents();
@@ -404,11 +405,11 @@ __global__ void __launch_bounds__(256) chanrec_chain_kernel(ChanrecParams a, Cha
   const int64_t np = (int64_t)a.n * a.p, i = (int64_t)blockIdx.x * 256 + threadIdx.x;
   if (i >= np) return;
   const int n = (int)(i / a.p);
-  const int used = (a.cu[b + 1] - a.cu[b] + sg.tokens - 1) / sg.tokens;
+  const int used = (a.cu[b + 1] - a.cu[b] - 1) / sg.tokens * sg.pieces + 1, all = sg.count * sg.pieces;
   float run = a.pos0[b] == 0 ? 0.f : a.state[((int64_t)a.slots[b] * a.heads + h) * np + i];
-  float* at = sg.start + (int64_t)bh * sg.count * np + i;
-  const float* decay = sg.decay + (int64_t)bh * sg.count * a.n + n;
-  constexpr int kAhead = 8;                               // segments requested before the first is used
+  float* at = sg.start + (int64_t)bh * all * np + i;
+  const float* decay = sg.decay + (int64_t)bh * all * a.n + n;
+  constexpr int kAhead = 8;                               // pieces requested before the first is used
   for (int k0 = 0; k0 < used; k0 += kAhead) {
     float own[kAhead], f[kAhead];
 #pragma unroll
@@ -420,7 +421,7 @@ __global__ void __launch_bounds__(256) chanrec_chain_kernel(ChanrecParams a, Cha
 #pragma unroll
     for (int k = 0; k < kAhead; ++k)
       if (k0 + k < used) {
-        at[(int64_t)(k0 + k) * np] = run;
+        if ((k0 + k) % sg.pieces == 0) at[(int64_t)(k0 + k) * np] = run;
         run = fmaf(f[k], run, own[k]);
       }
   }
@@ -441,18 +442,21 @@ static ChanrecSegs plan_chanrec(int batch, int max_tokens, int heads, int n, int
   const int64_t ctas = (int64_t)batch * heads * ((p + pt - 1) / pt);
   const int64_t room = 148 * (tc || n > 128 ? 1 : 2);      // CTAs that run at the same time
   const int chunks = (max_tokens + kCrTokens - 1) / kCrTokens;
-  // segments of at least eight chunks: the fewest steps of a CTA, counting the pass over states alone (all segments but one) half,
-  // and a little for every segment's state that goes through memory
-  int segs = 1;
-  double best = 0;
-  for (int k = 1; k <= chunks / 8 + 1 && ctas * (k - 1) < 2 * room; ++k) {
-    if (k > 1 && chunks / k < 8) break;
-    const double cost = (double)((ctas * k + room - 1) / room) / k * (k > 1 ? 1.0 + 0.5 * (k - 1) / k : 1.0) + 0.003 * k;
-    if (k == 1 || cost < best) { best = cost; segs = k; }
-  }
+  // segments of at least eight chunks, pieces of at least four: the fewest steps of a CTA, a step of the pass over states alone
+  // (all segments but one) counting half, and a little for every piece's state that goes through memory
+  auto waves = [&](int64_t n_ctas) { return (double)((n_ctas + room - 1) / room); };
+  int segs = 1, pieces = 1;
+  double best = waves(ctas);
+  for (int k = 2; k <= chunks / 8 && ctas * (k - 1) < 2 * room; ++k)
+    for (int m = 1; m <= 4 && chunks / (k * m) >= 4; ++m) {
+      const double cost = waves(ctas * k) / k + 0.5 * waves(ctas * (k - 1) * m) / (k * m) + 0.003 * k * m;
+      if (cost < best) { best = cost; segs = k; pieces = m; }
+    }
   ChanrecSegs s = {};
-  const int per = (int)((chunks + segs - 1) / segs);
+  int per = (chunks + segs - 1) / segs;
+  per = (per + pieces - 1) / pieces * pieces;
   s.tokens = per * kCrTokens;
+  s.pieces = pieces;
   s.count = per > 0 ? (chunks + per - 1) / per : 1;
   return s;
 }
@@ -467,11 +471,11 @@ static int launch_chanrec(const ChanrecParams& a, const ChanrecSegs& sg, cudaStr
     if (e != cudaSuccess) return fail(TKV_ERR_LAUNCH, "tkv_chanrec_chunk: %s", cudaGetErrorString(e));
     configured = true;
   }
-  const int64_t grid = (int64_t)a.batch * a.heads * ((a.p + kWarps * 16 - 1) / (kWarps * 16)) * sg.count;
-  if (grid > INT32_MAX) return fail(TKV_ERR_UNSUPPORTED, "tkv_chanrec_chunk: %lld blocks", (long long)grid);
+  const int64_t grid = (int64_t)a.batch * a.heads * ((a.p + kWarps * 16 - 1) / (kWarps * 16)) * sg.count, pieces = grid * sg.pieces;
+  if (pieces > INT32_MAX) return fail(TKV_ERR_UNSUPPORTED, "tkv_chanrec_chunk: %lld blocks", (long long)grid);
   cudaError_t e = cudaSuccess;
   if (sg.count > 1) {
-    e = launch_pdl(chanrec_chunk_kernel<NP, kWarps, true>, dim3((unsigned)grid), dim3(kWarps * 32), (size_t)kBytes, st, a, sg);
+    e = launch_pdl(chanrec_chunk_kernel<NP, kWarps, true>, dim3((unsigned)pieces), dim3(kWarps * 32), (size_t)kBytes, st, a, sg);
     if (e == cudaSuccess) {
       int rc = launch_chanrec_chain(a, sg, st);
       if (rc != TKV_OK) return rc;
@@ -490,7 +494,7 @@ using namespace tkv;
 extern "C" int64_t tkv_chanrec_chunk_workspace_bytes(int batch, int max_tokens, int heads, int n, int vdim, int dtype) {
   if (dtype != TKV_BF16 || batch <= 0 || heads <= 0 || n <= 0 || vdim <= 0 || max_tokens <= 0 || !chanrec_chunk_shape(n, vdim)) return -1;
   const ChanrecSegs s = plan_chanrec(batch, max_tokens, heads, n, vdim);
-  return s.count > 1 ? (int64_t)batch * heads * s.count * n * ((int64_t)vdim + 1) * (int64_t)sizeof(float) : 0;
+  return s.count > 1 ? (int64_t)batch * heads * s.count * s.pieces * n * ((int64_t)vdim + 1) * (int64_t)sizeof(float) : 0;
 }
 
 extern "C" int tkv_chanrec_chunk(const void* q, const void* f, const void* v, int64_t row_stride, const float* f_bias,
@@ -513,7 +517,7 @@ extern "C" int tkv_chanrec_chunk(const void* q, const void* f, const void* v, in
   ChanrecParams a = {q, f, v, row_stride, f_bias, lower, out, state, slots, cu_tokens, pos0, batch, heads, n, vdim};
   ChanrecSegs s = plan_chanrec(batch, max_tokens, heads, n, vdim);
   s.start = (float*)workspace;
-  s.decay = s.start + (s.count > 1 ? (int64_t)batch * heads * s.count * n * vdim : 0);
+  s.decay = s.start + (s.count > 1 ? (int64_t)batch * heads * s.count * s.pieces * n * vdim : 0);
   cudaStream_t st = (cudaStream_t)stream;
   if (chanrec_tc_shape(n, vdim, max_tokens)) return launch_chanrec_tc(a, s, status, st);
   const bool wide = chanrec_columns(n, vdim) == 128;

@@ -6,8 +6,9 @@
 // The state stays in TMEM as the accumulator of its own update (lane = value column, column = state row); once per chunk it
 // passes through registers to be written as the operand of the read-out, a high and a low bf16 part, and to be scaled by E.  k R
 // and a enter their products as two parts as well, v is 16-bit exactly, q P and q / R are rounded once, which is what rounding
-// q to 16 bits does.  k R and q P exist for all gates; q / R is used where every channel's gates keep kWide over eight tokens,
-// and a is summed up pair by pair in fp32 otherwise.
+// q to 16 bits does.  k R and q P exist for all gates; q / R is used where every channel's gates keep kCtWide over eight tokens.
+// Where they keep kCtNarrow, products and quotients of a reach over 16 tokens only (between the halves of the chunk: the gates
+// before the one and after the other); below that a is summed up pair by pair in fp32.
 //
 // Roles, each ahead of the next by up to one chunk:
 //   warps 0-7   gates and scaled vectors (a thread walks two channels of eight tokens), the blocks of a (mma.sync), the
@@ -25,18 +26,18 @@ constexpr int kCtTile = 8192, kCtHalf = 4096;              // 32 rows x 128 colu
 constexpr int kCtSop = 65536;                              // state operand: [part][64-column half][128 rows x 128 bytes]
 constexpr int kCtStage = 3 * kCtTile + 4096;               // q P | k R high | k R low | a
 constexpr int kCtSt = 0, kCtO = 128, kCtCols = 256;        // TMEM columns: state, two output buffers of 32
-constexpr float kCtWide = 3e-8f;
+constexpr float kCtWide = 3e-8f, kCtNarrow = 1e-15f;        // product of eight gates
 
 struct CtSmem {
   float oct[2][4][kCtN];                                   // product of eight tokens' gates, and of their reciprocals
   float end[2][kCtN];                                      // E, by chunk parity
   uint64_t full[2], done[2], sop, sync[3];
-  int level[2];                                            // by chunk parity: 1 = a pair by pair
+  int level[2];                                            // by chunk parity: 0 wide, 1 narrow, 2 pair by pair
   uint32_t tmem_base;
   int abort_flag;
 };
 constexpr int kCtRaw = 2 * kCtTile;                        // z_q | z_f of a chunk, rows of 256 bytes
-constexpr int kCtBytes = kCtSop + 2 * kCtStage + 3 * kCtTile + kCtTile + 2 * kCtRaw + (int)sizeof(CtSmem);
+constexpr int kCtBytes = kCtSop + 2 * kCtStage + 3 * kCtTile + 3 * kCtTile + 2 * kCtRaw + (int)sizeof(CtSmem);
 static_assert(kCtBytes <= 232448, "shared memory of the kernel");
 
 __device__ __forceinline__ uint32_t ct_idesc(int n, int a_mn, int b_mn) {   // bf16 operands, fp32 D, M = 128
@@ -50,6 +51,12 @@ __device__ __forceinline__ uint32_t ct_a(int i, int j, int part) {
   return (uint32_t)(i * 128 + (((col >> 3) ^ (i & 7)) << 4) + (col & 7) * 2);
 }
 
+// One arrival per warp, after what all its lanes have written.
+__device__ __forceinline__ void ct_arrive(uint64_t* bar) {
+  __syncwarp();
+  if ((threadIdx.x & 31) == 0) da_arrive(bar);
+}
+
 template <bool kStateOnly>
 __global__ void __launch_bounds__(kCtThreads, 1) chanrec_tc_kernel(ChanrecParams a, ChanrecSegs sg, int32_t* status) {
   extern __shared__ __align__(1024) uint8_t base[];
@@ -57,12 +64,13 @@ __global__ void __launch_bounds__(kCtThreads, 1) chanrec_tc_kernel(ChanrecParams
   grid_launch_dependents();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int ptiles = (a.p + kCtP - 1) / kCtP, per_seg = a.batch * a.heads * ptiles;
-  const int seg = blockIdx.x / per_seg, item = blockIdx.x - seg * per_seg;
+  const int seg = blockIdx.x / per_seg, item = blockIdx.x - seg * per_seg;      // kStateOnly: a piece of a segment
   const int pt = item % ptiles, bh = item / ptiles, b = bh / a.heads, h = bh - b * a.heads;
   const int tok0 = a.cu[b], ntok = a.cu[b + 1] - tok0;
-  const int t_first = seg * sg.tokens, t_end = min(ntok, t_first + sg.tokens);
+  const int seg_tokens = kStateOnly ? sg.tokens / sg.pieces : sg.tokens;
+  const int t_first = seg * seg_tokens, t_end = min(ntok, t_first + seg_tokens);
   if (t_first >= t_end) return;
-  if (kStateOnly && t_end == ntok) return;                 // nobody starts from the end of the last segment
+  if (kStateOnly && (seg / sg.pieces + 1) * sg.tokens >= ntok) return;          // nobody starts from the end of the last segment
   if ((smem_u32(base) & 1023u) != 0) {                     // the swizzled tiles need it; the launch gives it
     if (tid == 0) report(status, TKV_DEV_TIMEOUT);
     return;
@@ -72,14 +80,16 @@ __global__ void __launch_bounds__(kCtThreads, 1) chanrec_tc_kernel(ChanrecParams
   uint8_t* op_s = sop_s + kCtSop;                          // two stages
   uint8_t* v_s = op_s + 2 * kCtStage;                      // three stages
   uint8_t* qh_s = v_s + 3 * kCtTile;                       // q / R
-  uint8_t* raw_s = qh_s + kCtTile;                         // two stages
+  uint8_t* k16_s = qh_s + kCtTile;                         // narrow: k times the gates after it in its half, high | low (rows 0-15); q
+                                                           // times those before it in its half (rows 16-31 of the first tile)
+  uint8_t* raw_s = k16_s + 2 * kCtTile;                    // two stages
   CtSmem* sm = reinterpret_cast<CtSmem*>(raw_s + 2 * kCtRaw);
   volatile int* abort_flag = &sm->abort_flag;
 
   if (tid == 0) {
-    for (int i = 0; i < 2; ++i) { mbar_init(&sm->full[i], kCtGroup); mbar_init(&sm->done[i], 1); sm->level[i] = 0; }
-    mbar_init(&sm->sop, kCtGroup);
-    for (int i = 0; i < 3; ++i) mbar_init(&sm->sync[i], kCtGroup);
+    for (int i = 0; i < 2; ++i) { mbar_init(&sm->full[i], kCtGroup / 32); mbar_init(&sm->done[i], 1); sm->level[i] = 0; }
+    mbar_init(&sm->sop, kCtGroup / 32);
+    for (int i = 0; i < 3; ++i) mbar_init(&sm->sync[i], kCtGroup / 32);
     sm->abort_flag = 0;
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
@@ -106,22 +116,28 @@ __global__ void __launch_bounds__(kCtThreads, 1) chanrec_tc_kernel(ChanrecParams
     const int tokens = t_end - t_first;
     // copies: this thread's 16-byte piece of rows cr, cr + 16
     const int cr = tid >> 4, cc = tid & 15;
-    auto load = [&](int i) {
-      uint8_t* raw = raw_s + (i & 1) * kCtRaw;
-      uint8_t* vt = v_s + (i % 3) * kCtTile;
+    const bool q_in = cc * 8 < a.n, v_in = pbase + cc * 8 < a.p;
+    const int64_t step16 = 16 * a.row_stride;
+    const __nv_bfloat16 *Qt = Q + (int64_t)cr * a.row_stride + cc * 8, *Ft = F + (int64_t)cr * a.row_stride + cc * 8, *Vt = V + (int64_t)cr * a.row_stride + cc * 8;
+    const uint32_t raw_to = smem_u32(raw_s) + cr * 256 + cc * 16, v_to = smem_u32(v_s) + ct_at(cr, cc);   // rows 16 apart: + 4096, + 2048
+    auto copy = [&](uint32_t to, const __nv_bfloat16* from, const __nv_bfloat16* any, bool live) {
+      const int bytes = live ? 16 : 0;                     // 0: the 16 bytes are zero-filled
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(to), "l"(live ? from : any), "r"(bytes) : "memory");
+    };
+    auto load = [&](int i, int vst) {
+      const uint32_t raw = raw_to + (i & 1) * kCtRaw, vt = v_to + vst * kCtTile;
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        const int r = cr + 16 * e, t = i * kCtTok + r;
-        const bool in = t < tokens, qf = in && cc * 8 < a.n, vv = in && pbase + cc * 8 < a.p;
-        const int64_t at = (int64_t)t * a.row_stride + cc * 8;
-        if (!kStateOnly) cr_cp16(raw + r * 256 + cc * 16, qf ? Q + at : Q, qf);
-        cr_cp16(raw + kCtTile + r * 256 + cc * 16, qf ? F + at : F, qf);
-        cr_cp16(vt + ct_at(r, cc), vv ? V + at : V, vv);
+        const bool in = i * kCtTok + cr + 16 * e < tokens;
+        if (!kStateOnly) copy(raw + e * 4096, Qt + e * step16, Q, in && q_in);
+        copy(raw + kCtTile + e * 4096, Ft + e * step16, F, in && q_in);
+        copy(vt + e * 2048, Vt + e * step16, V, in && v_in);
       }
+      Qt += 2 * step16; Ft += 2 * step16; Vt += 2 * step16;
       asm volatile("cp.async.commit_group;" ::: "memory");
     };
     auto meet = [&](int which, int i) {
-      da_arrive(&sm->sync[which]);
+      ct_arrive(&sm->sync[which]);
       const bool ok = mbar_wait_or_abort(&sm->sync[which], i & 1, abort_flag);
       return (bool)__all_sync(0xffffffffu, ok);
     };
@@ -130,10 +146,14 @@ __global__ void __launch_bounds__(kCtThreads, 1) chanrec_tc_kernel(ChanrecParams
     const float2 bi = c < a.n ? mul2(*reinterpret_cast<const float2*>(bias + c), pair(kMinusLog2e)) : pair(0.f);
     const float2 lo = c < a.n ? *reinterpret_cast<const float2*>(lower + c) : pair(1.f);
     const float2 rest = make_float2(1.0f - lo.x, 1.0f - lo.y);
+    uint32_t at8[8];                                       // byte of this thread's channels in its eight rows of a tile
+#pragma unroll
+    for (int j = 0; j < 8; ++j) at8[j] = ct_at(r0 + j, c >> 3) + (c & 7) * 2;
     float2 seg_decay = pair(1.0f);
     bool alive = true;
-    load(0);
-    for (int i = 0; i < nchunks; ++i) {
+    int vnext = 1;                                         // (i + 1) mod 3
+    load(0, 0);
+    for (int i = 0; i < nchunks; ++i, vnext = vnext == 2 ? 0 : vnext + 1) {
       const int st = i & 1;
       uint8_t* op = op_s + st * kCtStage;
       const uint8_t* raw = raw_s + st * kCtRaw;
@@ -145,7 +165,7 @@ __global__ void __launch_bounds__(kCtThreads, 1) chanrec_tc_kernel(ChanrecParams
       asm volatile("cp.async.wait_group 0;" ::: "memory");
       alive = meet(0, i);                                  // this chunk is here; everyone is done with the last one
       if (!alive) break;
-      if (i + 1 < nchunks) load(i + 1);
+      if (i + 1 < nchunks) load(i + 1, vnext);
       float2 f[8], fi[8], k[8], fp = pair(1.0f), ip = fp;
       auto walk8 = [&](int live) {
 #pragma unroll
@@ -164,11 +184,11 @@ __global__ void __launch_bounds__(kCtThreads, 1) chanrec_tc_kernel(ChanrecParams
       *reinterpret_cast<float2*>(&sm->oct[0][oct][c]) = fp;
       if (!kStateOnly) {
         *reinterpret_cast<float2*>(&sm->oct[1][oct][c]) = ip;
-        if (!(fp.x >= kCtWide && fp.y >= kCtWide)) sm->level[st] = 1;
+        if (!(fp.x >= kCtWide && fp.y >= kCtWide)) atomicMax(&sm->level[st], fp.x >= kCtNarrow && fp.y >= kCtNarrow ? 1 : 2);
       }
       alive = meet(1, i);
       if (!alive) break;
-      const bool wide = kStateOnly || *(volatile int*)&sm->level[st] == 0;
+      const int level = kStateOnly ? 0 : *(volatile int*)&sm->level[st];
       if (tid == 0) sm->level[st ^ 1] = 0;
       // ---- q P forward, k R and q / R backward
       float2 before = pair(1.0f), after = before, iafter = before;
@@ -186,7 +206,6 @@ __global__ void __launch_bounds__(kCtThreads, 1) chanrec_tc_kernel(ChanrecParams
         *reinterpret_cast<float2*>(&sm->end[st][c]) = end;
         seg_decay = mul2(seg_decay, end);
       }
-      const uint32_t piece = (uint32_t)(c >> 3), sub = (c & 7) * 2;
       float2 qv[8];
       if (!kStateOnly) {
         float2 P = before;
@@ -196,33 +215,58 @@ __global__ void __launch_bounds__(kCtThreads, 1) chanrec_tc_kernel(ChanrecParams
           qv[j] = cr_silu2(make_float2(__uint_as_float(z << 16), __uint_as_float(z & 0xffff0000u)));
           P = mul2(P, f[j]);
           const float2 x = mul2(qv[j], P);
-          *reinterpret_cast<__nv_bfloat162*>(op + ct_at(r0 + j, piece) + sub) = __floats2bfloat162_rn(x.x, x.y);
+          *reinterpret_cast<__nv_bfloat162*>(op + at8[j]) = __floats2bfloat162_rn(x.x, x.y);
         }
       }
 #pragma unroll
       for (int j = 7; j >= 0; --j) {
-        const uint32_t at = ct_at(r0 + j, piece) + sub;
         uint32_t hi, lo_;
         cr_split(mul2(k[j], after), &hi, &lo_);
-        *reinterpret_cast<uint32_t*>(op + kCtTile + at) = hi;
-        *reinterpret_cast<uint32_t*>(op + 2 * kCtTile + at) = lo_;
+        *reinterpret_cast<uint32_t*>(op + kCtTile + at8[j]) = hi;
+        *reinterpret_cast<uint32_t*>(op + 2 * kCtTile + at8[j]) = lo_;
         after = mul2(after, f[j]);
         if (!kStateOnly) {
           const float2 x = mul2(qv[j], iafter);
-          *reinterpret_cast<__nv_bfloat162*>(qh_s + at) = __floats2bfloat162_rn(x.x, x.y);
+          *reinterpret_cast<__nv_bfloat162*>(qh_s + at8[j]) = __floats2bfloat162_rn(x.x, x.y);
           iafter = mul2(iafter, fi[j]);
         }
       }
       if (!kStateOnly) {
         uint8_t* at = op + 3 * kCtTile;
-        if (wide) {
+        if (level == 1) {
+          if (oct < 2) {
+            float2 a16 = pair(1.0f), i16 = a16;
+            if (oct == 0) { a16 = *reinterpret_cast<const float2*>(&sm->oct[0][1][c]); i16 = *reinterpret_cast<const float2*>(&sm->oct[1][1][c]); }
+#pragma unroll
+            for (int j = 7; j >= 0; --j) {
+              uint32_t hi, lo_;
+              cr_split(mul2(k[j], a16), &hi, &lo_);
+              *reinterpret_cast<uint32_t*>(k16_s + at8[j]) = hi;
+              *reinterpret_cast<uint32_t*>(k16_s + kCtTile + at8[j]) = lo_;
+              const float2 x = mul2(qv[j], i16);
+              *reinterpret_cast<__nv_bfloat162*>(qh_s + at8[j]) = __floats2bfloat162_rn(x.x, x.y);
+              a16 = mul2(a16, f[j]);
+              i16 = mul2(i16, fi[j]);
+            }
+          } else {
+            float2 p16 = oct == 3 ? *reinterpret_cast<const float2*>(&sm->oct[0][2][c]) : pair(1.0f);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+              p16 = mul2(p16, f[j]);
+              const float2 x = mul2(qv[j], p16);
+              *reinterpret_cast<__nv_bfloat162*>(k16_s + at8[j]) = __floats2bfloat162_rn(x.x, x.y);
+            }
+          }
+        }
+        if (level < 2) {
           alive = meet(2, i);
           if (!alive) break;
           if (warp < 6) {
             // ---- a task is 16 tokens against 8; the last two cross the middle of the chunk
             const int gr = lane >> 2, gc = lane & 3;
             const int ib = warp < 4 ? warp >> 1 : 1, jb = warp < 4 ? ib : 0, j0 = jb * 16 + (warp & 1) * 8;
-            const uint32_t qa = smem_u32(qh_s), ka = smem_u32(op + kCtTile) + (lane >> 4) * kCtTile;
+            const uint32_t qa = smem_u32(level == 1 && warp >= 4 ? k16_s : qh_s);
+            const uint32_t ka = smem_u32(level == 1 && jb == 0 ? k16_s : op + kCtTile) + (lane >> 4) * kCtTile;
             const int qrow = ib * 16 + (lane & 15), krow = j0 + (lane & 7);
             float sc[2][4] = {};
 #pragma unroll
@@ -287,12 +331,12 @@ __global__ void __launch_bounds__(kCtThreads, 1) chanrec_tc_kernel(ChanrecParams
         }
       }
       fence_async_smem();
-      da_arrive(&sm->full[st]);
+      ct_arrive(&sm->full[st]);
     }
     asm volatile("cp.async.wait_all;" ::: "memory");
     if (!alive && lane == 0 && *abort_flag == 0) { *abort_flag = 1; report(status, TKV_DEV_TIMEOUT); }
     if (kStateOnly && alive && oct == 3 && pt == 0 && c < a.n)
-      *reinterpret_cast<float2*>(sg.decay + ((int64_t)bh * sg.count + seg) * a.n + c) = seg_decay;
+      *reinterpret_cast<float2*>(sg.decay + ((int64_t)bh * sg.count * sg.pieces + seg) * a.n + c) = seg_decay;
   } else {
     // ------------------------------------------------------------------------------------ state and outputs: lane = value column
     const int quarter = warp & 3, half = (warp - 8) >> 2, row = quarter * 32 + lane, pc = pbase + row;
@@ -303,7 +347,7 @@ __global__ void __launch_bounds__(kCtThreads, 1) chanrec_tc_kernel(ChanrecParams
       return (bool)__all_sync(0xffffffffu, ok);
     };
     {
-      const float* S = kStateOnly ? nullptr : sg.count > 1 ? sg.start + ((int64_t)bh * sg.count + seg) * np : a.pos0[b] == 0 ? nullptr : final_state;
+      const float* S = kStateOnly ? nullptr : sg.count > 1 ? sg.start + ((int64_t)bh * sg.count + seg) * sg.pieces * np : a.pos0[b] == 0 ? nullptr : final_state;
 #pragma unroll
       for (int c2 = 0; c2 < 2; ++c2) {
         float s[32];
@@ -316,41 +360,44 @@ __global__ void __launch_bounds__(kCtThreads, 1) chanrec_tc_kernel(ChanrecParams
       }
     }
     // outputs of chunk i: 16 tokens of this column; neighbouring lanes exchange, so that a store holds two columns
+    const bool odd = lane & 1;
+    const int64_t out_row = (int64_t)a.heads * a.p;        // elements between tokens
+    __nv_bfloat16* const out0 = (__nv_bfloat16*)a.out + (int64_t)(tok0 + t_first + half * 16 + (odd ? 1 : 0)) * out_row + (int64_t)h * a.p + (pc & ~1);
     auto outputs = [&](int i) {
       float v[16];
       tmem_ld16(lanes + kCtO + (i & 1) * kCtTok + half * 16, v);
-      const bool odd = lane & 1;
+      const int live = pc < a.p ? t_end - (t_first + i * kCtTok + half * 16 + (odd ? 1 : 0)) : 0;
+      __nv_bfloat16* dst = out0 + (int64_t)i * kCtTok * out_row;
 #pragma unroll
       for (int c = 0; c < 16; c += 2) {
-        const float y = __shfl_xor_sync(0xffffffffu, odd ? v[c] : v[c + 1], 1);
-        const int t = t_first + i * kCtTok + half * 16 + c + (odd ? 1 : 0);
-        const uint32_t w = odd ? da_pack2(y, v[c + 1]) : da_pack2(v[c], y);
-        if (t < t_end && pc < a.p)
-          *reinterpret_cast<uint32_t*>((__nv_bfloat16*)a.out + ((int64_t)(tok0 + t) * a.heads + h) * a.p + (pc & ~1)) = w;
+        const float mine = odd ? v[c + 1] : v[c], y = __shfl_xor_sync(0xffffffffu, odd ? v[c] : v[c + 1], 1);
+        if (c < live) *reinterpret_cast<uint32_t*>(dst) = odd ? da_pack2(y, mine) : da_pack2(mine, y);
+        dst += 2 * out_row;
       }
     };
     const uint32_t id_o = ct_idesc(kCtTok, 0, 0), id_a = ct_idesc(kCtTok, 1, 0), id_s = ct_idesc(kCtN, 1, 1);
-    auto products = [&](int i) {                           // one thread, once the chunk's operands and the state's are there
+    // descriptors of the first stage; another place is the address field (16-byte units) moved on
+    const uint64_t d_sop = make_desc(smem_u32(sop_s), 16, 1024, 2), d_q = make_desc(smem_u32(op_s), 16, 1024, 2);
+    const uint64_t d_k = make_desc(smem_u32(op_s) + kCtTile, kCtHalf, 1024, 2), d_v = make_desc(smem_u32(v_s), kCtHalf, 1024, 2);
+    auto products = [&](int i, int vst) {                  // one thread, once the chunk's operands and the state's are there
       tc_fence_after();
-      const uint32_t sop = smem_u32(sop_s), q = smem_u32(op_s + (i & 1) * kCtStage), kh = q + kCtTile, at = q + 3 * kCtTile;
-      const uint32_t v = smem_u32(v_s + (i % 3) * kCtTile);
+      const uint64_t q = d_q + (i & 1) * (kCtStage >> 4), k = d_k + (i & 1) * (kCtStage >> 4), v = d_v + vst * (kCtTile >> 4), at = q + (3 * kCtTile >> 4);
+      const uint32_t o = tmem + kCtO + (i & 1) * kCtTok;
 #pragma unroll
-      for (int k = 0; k < 4; ++k)                          // high and low part of k R, 16 tokens each
-        umma(tmem + kCtSt, make_desc(v + (k & 1) * 2048, kCtHalf, 1024, 2), make_desc(kh + (k >> 1) * kCtTile + (k & 1) * 2048, kCtHalf, 1024, 2), id_s, 1);
+      for (int e = 0; e < 4; ++e)                          // high and low part of k R, 16 tokens each
+        umma(tmem + kCtSt, v + (e & 1) * 128, k + (e >> 1) * (kCtTile >> 4) + (e & 1) * 128, id_s, 1);
       if (!kStateOnly) {
-        const uint32_t o = tmem + kCtO + (i & 1) * kCtTok;
 #pragma unroll
-        for (int k = 0; k < 16; ++k)
-          umma(o, make_desc(sop + (k >> 3) * 32768 + ((k >> 2) & 1) * 16384 + (k & 3) * 32, 16, 1024, 2),
-               make_desc(q + ((k >> 2) & 1) * kCtHalf + (k & 3) * 32, 16, 1024, 2), id_o, k > 0);
+        for (int e = 0; e < 16; ++e)
+          umma(o, d_sop + (e >> 3) * 2048 + ((e >> 2) & 1) * 1024 + (e & 3) * 2, q + ((e >> 2) & 1) * (kCtHalf >> 4) + (e & 3) * 2, id_o, e > 0);
 #pragma unroll
-        for (int k = 0; k < 4; ++k)
-          umma(o, make_desc(v + (k & 1) * 2048, kCtHalf, 1024, 2), make_desc(at + k * 32, 16, 1024, 2), id_a, 1);
+        for (int e = 0; e < 4; ++e) umma(o, v + (e & 1) * 128, at + e * 2, id_a, 1);
       }
       umma_commit(&sm->done[i & 1]);
     };
     bool alive = true;
-    for (int i = 0; i < nchunks; ++i) {
+    int vst = 0;                                           // i mod 3
+    for (int i = 0; i < nchunks; ++i, vst = vst == 2 ? 0 : vst + 1) {
       if (i > 0) alive = sync_on(&sm->done[(i - 1) & 1], (i - 1) >> 1);
       if (alive) alive = sync_on(&sm->full[i & 1], i >> 1);
       if (!alive) break;
@@ -387,11 +434,11 @@ __global__ void __launch_bounds__(kCtThreads, 1) chanrec_tc_kernel(ChanrecParams
       }
       if (!kStateOnly) fence_async_smem();
       tc_fence_before();
-      da_arrive(&sm->sop);
+      ct_arrive(&sm->sop);
       if (warp == 8) {
         alive = sync_on(&sm->sop, i);
         if (!alive) break;
-        if (lane == 0) products(i);
+        if (lane == 0) products(i, vst);
         __syncwarp();
       }
       if (!kStateOnly && i > 0) outputs(i - 1);
@@ -400,7 +447,7 @@ __global__ void __launch_bounds__(kCtThreads, 1) chanrec_tc_kernel(ChanrecParams
     if (alive) {
       tc_fence_after();
       if (!kStateOnly) outputs(nchunks - 1);
-      float* dst = kStateOnly ? sg.start + ((int64_t)bh * sg.count + seg) * np : (t_end == ntok ? final_state : nullptr);
+      float* dst = kStateOnly ? sg.start + ((int64_t)bh * sg.count * sg.pieces + seg) * np : (t_end == ntok ? final_state : nullptr);
 #pragma unroll
       for (int c2 = 0; c2 < 2; ++c2) {
         float s[32];
@@ -432,11 +479,11 @@ int launch_chanrec_tc(const ChanrecParams& a, const ChanrecSegs& sg, int32_t* st
     if (e != cudaSuccess) return fail(TKV_ERR_LAUNCH, "tkv_chanrec_chunk(tc): %s", cudaGetErrorString(e));
     configured = true;
   }
-  const int64_t grid = (int64_t)a.batch * a.heads * ((a.p + kCtP - 1) / kCtP) * sg.count;
-  if (grid > INT32_MAX) return fail(TKV_ERR_UNSUPPORTED, "tkv_chanrec_chunk: %lld blocks", (long long)grid);
+  const int64_t grid = (int64_t)a.batch * a.heads * ((a.p + kCtP - 1) / kCtP) * sg.count, pieces = grid * sg.pieces;
+  if (pieces > INT32_MAX) return fail(TKV_ERR_UNSUPPORTED, "tkv_chanrec_chunk: %lld blocks", (long long)grid);
   cudaError_t e = cudaSuccess;
   if (sg.count > 1) {
-    e = launch_pdl(chanrec_tc_kernel<true>, dim3((unsigned)grid), dim3(kCtThreads), (size_t)kCtBytes, st, a, sg, status);
+    e = launch_pdl(chanrec_tc_kernel<true>, dim3((unsigned)pieces), dim3(kCtThreads), (size_t)kCtBytes, st, a, sg, status);
     if (e == cudaSuccess) {
       int rc = launch_chanrec_chain(a, sg, st);
       if (rc != TKV_OK) return rc;
