@@ -5,8 +5,9 @@
 //   o_i  = S^T (q_i P_i) + sum_j a_ij v_j
 //   S   <- diag(P_end) (S + sum_j (k_j / P_j) v_j^T) .
 // k / P is fp32 and enters the 16-bit products as a high and a low part, as do the state and a; v is 16-bit exactly, and q P is
-// rounded once, which is what rounding q itself to 16 bits does.  1 / P must stay in the range of fp32: a chunk of 32 tokens is one block where every channel's gates keep
-// kWide over eight tokens, two blocks of 16 where they keep kNarrow, and is walked token by token below that (gates near zero).
+// rounded once, which is what rounding q itself to 16 bits does.  1 / P must stay in the range of fp32: a chunk of 32 tokens is
+// one block where every channel's gates keep kWide over eight tokens, two blocks of 16 where they keep kNarrow, and is walked
+// token by token below that (gates near zero).
 //
 // One CTA walks the chunks of one (request, head, block of 16 * kWarps value columns, segment of the sequence).  The state never
 // leaves registers: a warp owns 16 columns of v and holds S^T [16 x n] as fp32 MMA accumulators, whose layout is also the
