@@ -682,6 +682,7 @@ class MicroTools:
         for c in calls:
             c()
         torch.cuda.synchronize()
+        time.sleep(0.3)                            # the power cap that a long run of products before left behind is lifted by then
         graph = torch.cuda.CUDAGraph()
         n = max(reps, len(calls))
         with torch.cuda.graph(graph):
